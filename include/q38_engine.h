@@ -37,7 +37,7 @@ typedef struct q38e_sampling {
 typedef struct q38e_runner_options {
   int max_batch;
   int prefill_chunk;
-  int kv_dtype;        /* 0 int8, 1 bf16 */
+  int kv_dtype;        /* -1 the architecture's own, 0 int8, 1 bf16, 2 fp32 */
   int64_t kv_tokens;   /* 0 = everything that fits */
   int max_context;
   size_t reserve_mib;
@@ -45,6 +45,7 @@ typedef struct q38e_runner_options {
   int cuda_graphs;
   int history_cap;
   int verbose;
+  int compute_dtype;   /* 0 bf16, 1 fp32 (dense-weight architectures only) */
 } q38e_runner_options;
 void q38e_default_runner_options(q38e_runner_options* o);
 
@@ -82,13 +83,15 @@ typedef struct q38e_prefill_row {
 int q38e_tuning_load(const char* path);
 int q38e_tuning_lookup(int bits, int n, int k, int m);
 
-/* ModelFile */
+/* ModelFile: a .q38 file, or a folder with config.json and model.safetensors */
 int q38e_model_open(const char* path, q38e_model** out);
 void q38e_model_close(q38e_model* m);
 int q38e_model_vocab(const q38e_model* m);
 int q38e_model_hidden(const q38e_model* m);
 int q38e_model_layers(const q38e_model* m);
 const char* q38e_model_summary(const q38e_model* m);
+const char* q38e_model_architecture(const q38e_model* m);
+int q38e_model_max_positions(const q38e_model* m);
 /* Host spec decoder (qwen38::BQView::dequant_all): out = float[n * k] of tensor `name`. */
 int q38e_model_dequant(const q38e_model* m, const char* name, float* out, size_t out_floats);
 
@@ -102,6 +105,10 @@ int q38e_runner_kv_pages(q38e_runner* r, int slot, int* pages_out, int capacity,
 int q38e_runner_kv_free_pages(q38e_runner* r, int* count);
 int q38e_runner_prefill(q38e_runner* r, const q38e_prefill_row* rows, int num_rows, int32_t* tokens_out,
                         float* logprobs_out, int* num_out);
+/* One ragged step as q38e_runner_prefill runs it, returning the logits of the places (want_row[i], want_index[i]): token
+ * want_index of row want_row. logits_out holds [num_want][vocab] floats. */
+int q38e_runner_step_logits(q38e_runner* r, const q38e_prefill_row* rows, int num_rows, const int32_t* want_row,
+                            const int32_t* want_index, int num_want, float* logits_out);
 int q38e_runner_decode(q38e_runner* r, const q38e_decode_row* rows, int num_rows, int32_t* tokens_out,
                        float* logprobs_out);
 int q38e_runner_prefill_logits(q38e_runner* r, int slot, int pos0, const int32_t* tokens, int n, float* logits_out);

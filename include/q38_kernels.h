@@ -52,6 +52,7 @@ typedef struct q38_batch_desc {
  * K [kv_head][64][4], V same. */
 #define Q38_KV_INT8 0
 #define Q38_KV_BF16 1
+#define Q38_KV_F32 2 /* q38_kv_layer_desc only */
 typedef struct q38_kv_cache_desc {
   uint8_t* pool;
   int dtype; /* Q38_KV_INT8 | Q38_KV_BF16 */
@@ -302,6 +303,146 @@ int q38_target_logprobs(const float* logits, int ld, int vocab, const int32_t* t
  * entries; outputs are the arrays a q38_batch_desc points at. num_tokens must equal sum(count). */
 int q38_pack_ragged(const int* seq_count, const int* seq_pos0, int num_seqs, int num_tokens, int* seq_start,
                     int* tok_pos, int* tok_seq, void* stream);
+
+/* ---------------------------------------------------------------------------------------------------------------
+ * Layer-list architectures with dense (bf16) weights: decoders whose configuration lists a mixer and an optional gated
+ * feed-forward per layer. No counterpart in the reference. Activations are bf16 or fp32 (`act`); with Q38_ACT_F32 every
+ * product is computed in 32-bit. Rows of activation matrices start every `ld` elements; the elements between a row's
+ * length and `ld` must be finite (they meet zero weights).
+ * ------------------------------------------------------------------------------------------------------------- */
+#define Q38_ACT_BF16 0
+#define Q38_ACT_F32 1
+
+/* One attention layer's pages: page p at pages + p * page_bytes, first K [kv_head][64 tokens][k_dim], then V transposed,
+ * [kv_head][v_dim][64 tokens]; k_dim is a multiple of 32, v_dim of 8 (heads are padded with zeros). */
+typedef struct q38_kv_layer_desc {
+  uint8_t* pages;
+  int dtype; /* Q38_KV_BF16 | Q38_KV_F32, equal to the activations' precision */
+  int kv_heads, k_dim, v_dim;
+  int num_pages;
+  size_t page_bytes;
+  const int* block_table; /* [slots][max_pages_per_seq] */
+  int max_pages_per_seq;
+} q38_kv_layer_desc;
+
+/* One recurrent layer's state: slot s at byte offset s * slot_bytes of both pointers. `state` is fp32 [width]; `conv` is
+ * a ring [taps][channels] in activation precision, the input of position p in row p % taps. Positions before the
+ * sequence's start are zero and are never read, so a fresh sequence needs no clearing: at position 0 the recurrence
+ * starts from zero by itself. */
+typedef struct q38_recurrent_state_desc {
+  uint8_t* state;
+  uint8_t* conv;
+  size_t slot_bytes;
+} q38_recurrent_state_desc;
+
+/* y[m][n] = x[m][k] W^T + bias. W bf16 [n][k], rows `ld` elements apart (a multiple of 64, zero beyond k), with zero
+ * rows up to a multiple of 16. */
+typedef struct q38_dense_weight {
+  const q38_bf16* w;
+  const float* bias; /* [n] or NULL */
+  int n, k, ld;
+} q38_dense_weight;
+#define Q38_DENSE_STORE 0     /* out[m][n] in activation precision */
+#define Q38_DENSE_STORE_F32 1 /* out[m][n] fp32 */
+#define Q38_DENSE_GLU_GELU 2  /* rows of W alternate gate, up: out[m][n / 2] = gelu_tanh(gate) * up, activation precision */
+#define Q38_DENSE_GLU_SILU 3  /* the same with silu */
+typedef struct q38_dense_epilogue {
+  int kind;
+  void* out;
+  int ldo;
+} q38_dense_epilogue;
+#define Q38_DENSE_AUTO (-1)
+int q38_dense_gemm_num_configs(void);
+const char* q38_dense_gemm_config_name(int config);
+int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_dense_weight* w, const q38_dense_epilogue* ep,
+                   const q38_gemm_workspace* ws, void* stream, int config);
+
+/* RMS norm with a gain per coordinate (gain_stride 1) or one gain for all (gain_stride 0); `out` in activation precision. */
+typedef struct q38_norm {
+  const float* gain;
+  int gain_stride;
+  float eps;
+} q38_norm;
+/* residual = table[token] (+ positions[position] if not NULL); out = norm(residual) */
+int q38_embed_norm(const q38_bf16* table, const q38_bf16* positions, const int32_t* tokens, const int* tok_pos, int m,
+                   int width, float* residual, const q38_norm* norm, void* out, int ld_out, int act, void* stream);
+/* residual += post(y); out = next(residual) unless next is NULL. Post-norm, residual sum and the following sublayer's
+ * pre-norm in one pass over the row. */
+int q38_residual_norm(const float* y, int ldy, int m, int width, const q38_norm* post, float* residual,
+                      const q38_norm* next, void* out, int ld_out, int act, void* stream);
+/* out[i] = norm(residual[rows ? rows[i] : first + i]), i < n (rows is a device array) */
+int q38_gather_norm(const float* residual, const int* rows, int first, int n, int width, const q38_norm* norm, void* out,
+                    int ld_out, int act, void* stream);
+
+/* Rotary positions on the leading rot_dims of every query and key head (dimension i turns with i + rot_dims / 2 by
+ * position * base^(-2 i / rot_dims)), optional blending of the values with a first layer's, and the append to the cache.
+ * proj rows: [q: heads x dim | k: kv_heads x dim | v: kv_heads x vdim]. */
+typedef struct q38_rope_append_params {
+  const void* proj;
+  int ld_proj;
+  int act;
+  int heads, kv_heads, dim, vdim;
+  int rot_dims;
+  double rot_base;
+  void* q_out;            /* [M][heads][k_dim of the cache], zero beyond dim */
+  void* v_first_out;      /* [M][kv_heads * vdim]: where to keep this layer's values, or NULL */
+  const void* v_first_in; /* values to blend with, or NULL: v = (1 - *v_mix) v + *v_mix v_first */
+  const float* v_mix;
+} q38_rope_append_params;
+int q38_rope_append(const q38_rope_append_params* p, const q38_batch_desc* batch, const q38_kv_layer_desc* kv, void* stream);
+
+/* Causal attention over the cache whose heads' softmax weights are mixed before they meet the values:
+ * w_h(i, j) = sum_g head_mix[h][g] softmax_g(i, j); head_mix NULL = no mixing. Query head h reads kv head
+ * h / (heads / kv_heads). */
+typedef struct q38_mixed_attention_params {
+  const void* q; /* [M][heads][k_dim] */
+  int act;
+  int heads, vdim;
+  float scale;
+  const float* head_mix; /* [heads][heads] or NULL */
+  void* out;             /* [M][ld_out]: heads x vdim */
+  int ld_out;
+  float* stats;          /* [M][heads][2] */
+  float* scores;         /* decode: [num_pages][heads][64] (NULL: the decode call uses the prefill kernels) */
+  float* partials;       /* decode: [num_seqs][max_splits][heads][v_dim of the cache + 2] */
+  int max_splits;
+} q38_mixed_attention_params;
+int q38_mixed_attention_prefill(const q38_mixed_attention_params* p, const q38_batch_desc* batch,
+                                const q38_kv_layer_desc* kv, void* stream);
+int q38_mixed_attention_decode(const q38_mixed_attention_params* p, const q38_batch_desc* batch,
+                               const q38_kv_layer_desc* kv, void* stream);
+
+/* minGRU: proj rows [z | x | g], each `width`; z = sigmoid(z), candidate x + 1/2 (x >= 0) or sigmoid(x),
+ * S = (1 - z) S + z candidate, out = S silu(g). */
+typedef struct q38_mingru_params {
+  const void* proj;
+  int ld_proj;
+  int act;
+  int width;
+  void* out;
+  int ld_out;
+} q38_mingru_params;
+int q38_mingru(const q38_mingru_params* p, const q38_batch_desc* batch, const q38_recurrent_state_desc* st, void* stream);
+
+/* Real-gated linear recurrent unit behind a causal convolution: proj rows [y | x], each `width`; u = conv(x) + conv_b;
+ * r, i = sigmoid(block-diagonal products of u); log a = log_decay * r * softplus(lam); S = a S + sqrt(1 - a^2) i u;
+ * out = S gelu_tanh(y). gate_w [blocks][2 (r, i)][block_ld][block_ld] bf16 with block_ld a multiple of 32, zero padded. */
+typedef struct q38_rglru_params {
+  const void* proj;
+  int ld_proj;
+  int act;
+  int width, blocks, block_ld, taps;
+  const float* conv_w; /* [taps][width], the last row meets the current token */
+  const float* conv_b; /* [width] */
+  const q38_bf16* gate_w;
+  const float* gate_b; /* [2][width] */
+  const float* lam;    /* [width] */
+  float log_decay;     /* negative */
+  float* scratch;      /* [2][num_tokens][width]; batches of one token per sequence do not use it */
+  void* out;
+  int ld_out;
+} q38_rglru_params;
+int q38_rglru(const q38_rglru_params* p, const q38_batch_desc* batch, const q38_recurrent_state_desc* st, void* stream);
 
 /* Diagnostics. */
 const char* q38_last_error(void);           /* message of the last failed launcher call on this thread */

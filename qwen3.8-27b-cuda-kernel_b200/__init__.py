@@ -12,7 +12,16 @@ import ctypes as C
 from pathlib import Path
 
 HERE = Path(__file__).resolve().parent
-LIB_DIR = HERE / "lib"
+LIB_DIR = HERE / "lib"  # use_libraries() selects another build
+
+
+def use_libraries(folder) -> None:
+    """Loads the native libraries from `folder` (a build of some model families only) instead of lib/. Must come before
+    the first use of a library."""
+    global LIB_DIR
+    if _kernels is not None:
+        raise RuntimeError("the native libraries are already loaded")
+    LIB_DIR = Path(folder)
 
 
 class NativeLibraryMissing(RuntimeError):
@@ -96,6 +105,52 @@ class GdnRecurrenceParams(C.Structure):
                 ("out", C.c_void_p), ("gdn_layer", C.c_int)]
 
 
+class KvLayerDesc(C.Structure):
+    _fields_ = [("pages", C.c_void_p), ("dtype", C.c_int), ("kv_heads", C.c_int), ("k_dim", C.c_int), ("v_dim", C.c_int),
+                ("num_pages", C.c_int), ("page_bytes", C.c_size_t), ("block_table", C.c_void_p),
+                ("max_pages_per_seq", C.c_int)]
+
+
+class RecurrentStateDesc(C.Structure):
+    _fields_ = [("state", C.c_void_p), ("conv", C.c_void_p), ("slot_bytes", C.c_size_t)]
+
+
+class DenseWeight(C.Structure):
+    _fields_ = [("w", C.c_void_p), ("bias", C.c_void_p), ("n", C.c_int), ("k", C.c_int), ("ld", C.c_int)]
+
+
+class DenseEpilogue(C.Structure):
+    _fields_ = [("kind", C.c_int), ("out", C.c_void_p), ("ldo", C.c_int)]
+
+
+class Norm(C.Structure):
+    _fields_ = [("gain", C.c_void_p), ("gain_stride", C.c_int), ("eps", C.c_float)]
+
+
+class RopeAppendParams(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int),
+                ("dim", C.c_int), ("vdim", C.c_int), ("rot_dims", C.c_int), ("rot_base", C.c_double),
+                ("q_out", C.c_void_p), ("v_first_out", C.c_void_p), ("v_first_in", C.c_void_p), ("v_mix", C.c_void_p)]
+
+
+class MixedAttentionParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("act", C.c_int), ("heads", C.c_int), ("vdim", C.c_int), ("scale", C.c_float),
+                ("head_mix", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int), ("stats", C.c_void_p),
+                ("scores", C.c_void_p), ("partials", C.c_void_p), ("max_splits", C.c_int)]
+
+
+class MinGruParams(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("width", C.c_int), ("out", C.c_void_p),
+                ("ld_out", C.c_int)]
+
+
+class RgLruParams(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("width", C.c_int), ("blocks", C.c_int),
+                ("block_ld", C.c_int), ("taps", C.c_int), ("conv_w", C.c_void_p), ("conv_b", C.c_void_p),
+                ("gate_w", C.c_void_p), ("gate_b", C.c_void_p), ("lam", C.c_void_p), ("log_decay", C.c_float),
+                ("scratch", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int)]
+
+
 class SamplingParamsDev(C.Structure):
     _fields_ = [("temperature", C.c_float), ("top_k", C.c_int), ("top_p", C.c_float), ("min_p", C.c_float),
                 ("presence_penalty", C.c_float), ("repetition_penalty", C.c_float), ("seed", C.c_uint64)]
@@ -109,7 +164,9 @@ class SamplingArgs(C.Structure):
 
 
 EPI_STORE_BF16, EPI_SWIGLU, EPI_RESIDUAL, EPI_STORE_F32, EPI_ALLREDUCE_RESIDUAL = 0, 1, 2, 3, 4
-KV_INT8, KV_BF16 = 0, 1
+KV_INT8, KV_BF16, KV_F32 = 0, 1, 2
+ACT_BF16, ACT_F32 = 0, 1
+DENSE_STORE, DENSE_STORE_F32, DENSE_GLU_GELU, DENSE_GLU_SILU = 0, 1, 2, 3
 
 # every entry point include/q38_kernels.h declares, with its ctypes signature
 KERNEL_API = {
@@ -152,6 +209,23 @@ KERNEL_API = {
     "q38_target_logprobs": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p]),
     "q38_pack_ragged": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_void_p, C.c_void_p,
                                   C.c_void_p]),
+    "q38_dense_gemm_num_configs": (C.c_int, []),
+    "q38_dense_gemm_config_name": (C.c_char_p, [C.c_int]),
+    "q38_dense_gemm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(DenseWeight), C.POINTER(DenseEpilogue),
+                                 C.POINTER(GemmWorkspace), C.c_void_p, C.c_int]),
+    "q38_embed_norm": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p,
+                                 C.POINTER(Norm), C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
+    "q38_residual_norm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(Norm), C.c_void_p, C.POINTER(Norm),
+                                    C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
+    "q38_gather_norm": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(Norm), C.c_void_p, C.c_int,
+                                  C.c_int, C.c_void_p]),
+    "q38_rope_append": (C.c_int, [C.POINTER(RopeAppendParams), C.POINTER(BatchDesc), C.POINTER(KvLayerDesc), C.c_void_p]),
+    "q38_mixed_attention_prefill": (C.c_int, [C.POINTER(MixedAttentionParams), C.POINTER(BatchDesc),
+                                              C.POINTER(KvLayerDesc), C.c_void_p]),
+    "q38_mixed_attention_decode": (C.c_int, [C.POINTER(MixedAttentionParams), C.POINTER(BatchDesc),
+                                             C.POINTER(KvLayerDesc), C.c_void_p]),
+    "q38_mingru": (C.c_int, [C.POINTER(MinGruParams), C.POINTER(BatchDesc), C.POINTER(RecurrentStateDesc), C.c_void_p]),
+    "q38_rglru": (C.c_int, [C.POINTER(RgLruParams), C.POINTER(BatchDesc), C.POINTER(RecurrentStateDesc), C.c_void_p]),
     "q38_last_error": (C.c_char_p, []),
     "q38_set_dependent_launch": (None, [C.c_int]),
     "q38_device_error": (C.c_uint, [C.c_int]),
@@ -169,6 +243,8 @@ def kernels() -> C.CDLL:
     if _kernels is None:
         lib = _load("libq38_kernels.so")
         for name, (res, args) in KERNEL_API.items():
+            if LIB_DIR != HERE / "lib" and not hasattr(lib, name):
+                continue  # a build of some families only
             fn = getattr(lib, name)
             fn.restype = res
             fn.argtypes = args

@@ -1,10 +1,14 @@
 """In-tree build of the native libraries (no GPU needed: nvcc cross-compiles for sm_100a).
 
-    python qwen3.8-27b-cuda-kernel_b200/build.py [--force] [--verbose]
+    python qwen3.8-27b-cuda-kernel_b200/build.py [--force] [--verbose] [--family NAME]
 
 Outputs, next to this file:
     lib/libq38_kernels.so   every CUDA kernel + the C ABI declared in include/q38_kernels.h
     lib/libq38_engine.so    the C++20 host engine (ModelFile, KvCache, ModelRunner, Engine) + its C ABI
+
+The sources belong to model families (FAMILIES) or are shared. A build of one family only (`build(family=...)`) compiles
+its own and the shared sources and puts the same two libraries into lib/<family>/: an engine that serves that family's
+architectures and nothing else.
 """
 
 from __future__ import annotations
@@ -31,6 +35,15 @@ HOST_FLAGS = ["-std=c++20", "-O2", "-fPIC", "-I", str(ROOT / "include"), "-I", s
               "-I", "/usr/local/cuda/include"]
 
 
+# sources of one model family; everything else is shared
+FAMILIES = {
+    "bq": {"cu": {"attention", "gdn", "qgemm", "qgemm_stream", "qgemm_umma"}, "host": {"bq_model"}},
+    "layer_list": {"cu": {"dense_gemm", "dense_umma", "mixed_attention", "mixed_attention_mma", "recurrent", "row_norm"},
+                   "host": {"layer_list_model", "fegenex"}},
+}
+ARCHITECTURE_FAMILY = {"Qwen3.8": "bq", "Fegenex": "layer_list"}
+
+
 def _stale(target: Path, deps: list[Path]) -> bool:
     if not target.exists():
         return True
@@ -49,28 +62,36 @@ def _run(cmd: list[str], verbose: bool) -> None:
         print(r.stdout + r.stderr)
 
 
-def build(force: bool = False, verbose: bool = False, ptxas_verbose: bool = False) -> dict[str, Path]:
+def _sources(folder: Path, pattern: str, kind: str, family: str | None) -> list[Path]:
+    skip = set().union(*(f[kind] for name, f in FAMILIES.items() if family is not None and name != family))
+    return [p for p in sorted(folder.glob(pattern)) if p.stem not in skip]
+
+
+def build(force: bool = False, verbose: bool = False, ptxas_verbose: bool = False,
+          family: str | None = None) -> dict[str, Path]:
+    lib_dir = LIB if family is None else LIB / family
     OBJ.mkdir(exist_ok=True)
-    LIB.mkdir(exist_ok=True)
+    lib_dir.mkdir(parents=True, exist_ok=True)
     cu_headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h")) + [ROOT / "include" / "q38_kernels.h"]
     jobs = []
     cu_objs = []
-    for src in sorted(CSRC.glob("*.cu")):
+    for src in _sources(CSRC, "*.cu", "cu", family):
         obj = OBJ / (src.stem + ".o")
         cu_objs.append(obj)
         if force or _stale(obj, [src] + cu_headers):
             extra = ["-Xptxas", "-v"] if ptxas_verbose else []
             jobs.append([NVCC, *CUDA_FLAGS, *extra, "-c", str(src), "-o", str(obj)])
-    host_headers = sorted((HOST / "include").rglob("*.h")) + sorted((ROOT / "include").glob("*.h"))
+    host_headers = sorted((HOST / "include").rglob("*.h")) + sorted((HOST / "src").glob("*.h")) + sorted((ROOT / "include").glob("*.h"))
     host_objs = []
-    for src in sorted((HOST / "src").glob("*.cpp")):
+    for src in _sources(HOST / "src", "*.cpp", "host", family):
         obj = OBJ / ("host_" + src.stem + ".o")
         host_objs.append(obj)
         if force or _stale(obj, [src] + host_headers):
             jobs.append(["g++", *HOST_FLAGS, "-c", str(src), "-o", str(obj)])
+    jobs.sort(key=lambda c: c[0] != NVCC)  # the long ones first
     with ThreadPoolExecutor(max_workers=os.cpu_count() or 4) as pool:
         list(pool.map(lambda c: _run(c, verbose or ptxas_verbose), jobs))
-    kernels_so = LIB / "libq38_kernels.so"
+    kernels_so = lib_dir / "libq38_kernels.so"
     if force or _stale(kernels_so, cu_objs):
         # both libraries use the one shared CUDA runtime of the process (a host application's, or torch's in the
         # tests and benchmarks): same soname, so whichever copy is loaded first serves everybody
@@ -78,13 +99,22 @@ def build(force: bool = False, verbose: bool = False, ptxas_verbose: bool = Fals
               "-Xlinker", f"-rpath,{CUDA_LIB}"], verbose)
     out = {"kernels": kernels_so}
     if host_objs:
-        engine_so = LIB / "libq38_engine.so"
+        engine_so = lib_dir / "libq38_engine.so"
         if force or _stale(engine_so, host_objs + [kernels_so]):
-            _run(["g++", "-shared", "-o", str(engine_so), *map(str, host_objs), "-L", str(LIB), "-lq38_kernels",
+            _run(["g++", "-shared", "-o", str(engine_so), *map(str, host_objs), "-L", str(lib_dir), "-lq38_kernels",
                   f"-L{CUDA_LIB}", "-lcudart", "-ldl", "-lrt", "-lpthread",
                   f"-Wl,-rpath,$ORIGIN:{CUDA_LIB}"], verbose)
         out["engine"] = engine_so
     return out
+
+
+def up_to_date(family: str | None) -> bool:
+    """Whether the libraries of this build exist and are newer than all their sources."""
+    lib_dir = LIB if family is None else LIB / family
+    deps = (_sources(CSRC, "*.cu", "cu", family) + list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h")) +
+            _sources(HOST / "src", "*.cpp", "host", family) + list((HOST / "src").glob("*.h")) +
+            list((HOST / "include").rglob("*.h")) + list((ROOT / "include").glob("*.h")))
+    return not any(_stale(lib_dir / n, deps) for n in ("libq38_kernels.so", "libq38_engine.so"))
 
 
 if __name__ == "__main__":
@@ -92,6 +122,7 @@ if __name__ == "__main__":
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
     ap.add_argument("--ptxas", action="store_true", help="print registers / spills / shared memory per kernel")
+    ap.add_argument("--family", choices=sorted(FAMILIES), help="this model family only, into lib/<family>/")
     a = ap.parse_args()
-    for name, path in build(a.force, a.verbose, a.ptxas).items():
+    for name, path in build(a.force, a.verbose, a.ptxas, a.family).items():
         print(f"{name}: {path}")

@@ -1,6 +1,7 @@
 // Library-wide pieces of the C ABI: error reporting, device properties, layout helpers.
 #include <cstdarg>
 #include <cstdio>
+#include <cstdlib>
 #include <cstring>
 #include <mutex>
 
@@ -42,28 +43,43 @@ bool g_dependent_launch = true;
 }
 bool dependent_launch_allowed() { return g_dependent_launch; }
 
+namespace {
+q38_gemm_tuning_lookup g_tuning = nullptr;
+}
+q38_gemm_tuning_lookup gemm_tuning() { return g_tuning; }
+
 int num_sms() { return props().sms > 0 ? props().sms : 1; }
 int max_optin_smem() { return props().smem_optin; }
 
-// per-translation-unit device error words
-unsigned int qgemm_stream_error(bool clear);
-unsigned int qgemm_dispatch_error(bool clear);
-unsigned int qgemm_umma_error(bool clear);
-unsigned int attention_error(bool clear);
-unsigned int gdn_error(bool clear);
-unsigned int misc_error(bool clear);
-
-unsigned int* qgemm_stream_error_address();
-unsigned int* qgemm_dispatch_error_address();
-unsigned int* qgemm_umma_error_address();
-unsigned int* attention_error_address();
-unsigned int* gdn_error_address();
+// per-translation-unit device error words: every .cu that reports errors registers its own when the library is loaded
+namespace {
+constexpr int kMaxErrorWords = 24;
+struct ErrorWordList {
+  unsigned int (*read[kMaxErrorWords])(bool);
+  unsigned int* (*address[kMaxErrorWords])();
+  int count = 0;
+};
+ErrorWordList& error_word_list() {
+  static ErrorWordList list;
+  return list;
+}
+}  // namespace
+void register_error_word(unsigned int (*read)(bool clear), unsigned int* (*address)()) {
+  ErrorWordList& l = error_word_list();
+  if (l.count == kMaxErrorWords) {
+    std::fprintf(stderr, "q38: more than %d translation units report errors\n", kMaxErrorWords);
+    std::abort();
+  }
+  l.read[l.count] = read;
+  l.address[l.count] = address;
+  ++l.count;
+}
 unsigned int* misc_error_address();
 
 namespace {
-constexpr int kErrorWords = 6;
 struct ErrorWords {
-  unsigned int* word[kErrorWords];
+  unsigned int* word[kMaxErrorWords];
+  int count;
 };
 
 // Moves the first non-zero error word of the library into *dst and clears the words; *dst is left alone when no
@@ -72,7 +88,7 @@ __global__ void collect_errors_kernel(ErrorWords w, unsigned int* dst) {
   pdl_wait();
   pdl_launch_dependents();
   unsigned int first = 0;
-  for (int i = 0; i < kErrorWords; ++i) {
+  for (int i = 0; i < w.count; ++i) {
     const unsigned int v = atomicExch(w.word[i], 0u);
     if (first == 0) first = v;
   }
@@ -103,13 +119,12 @@ extern "C" int q38_device_error_collect(unsigned int* dst, void* stream) {
   Q38_REQUIRE(dev >= 0 && dev < kMaxErrorDevices, "device_error_collect: device index %d out of range", dev);
   ErrorWordCache& c = g_error_words[dev];
   std::call_once(c.once, [&c] {  // with this device current; the first call must come before any stream capture
-    unsigned int* p[kErrorWords] = {qgemm_stream_error_address(), qgemm_dispatch_error_address(),
-                                    qgemm_umma_error_address(),   attention_error_address(),
-                                    gdn_error_address(),          misc_error_address()};
+    const ErrorWordList& l = error_word_list();
+    c.words.count = l.count;
     c.ok = true;
-    for (int i = 0; i < kErrorWords; ++i) {
-      c.words.word[i] = p[i];
-      c.ok = c.ok && p[i] != nullptr;
+    for (int i = 0; i < l.count; ++i) {
+      c.words.word[i] = l.address[i]();
+      c.ok = c.ok && c.words.word[i] != nullptr;
     }
   });
   Q38_REQUIRE(c.ok, "device_error_collect: the error words of the library could not be located");
@@ -126,17 +141,15 @@ extern "C" int q38_device_error_inject(unsigned int code) {
   return Q38_OK;
 }
 
+extern "C" void q38_set_qgemm_tuning(q38_gemm_tuning_lookup lookup) { q38::g_tuning = lookup; }
+
 extern "C" void q38_set_dependent_launch(int allowed) { q38::g_dependent_launch = allowed != 0; }
 
 extern "C" unsigned int q38_device_error(int clear) {
   cudaDeviceSynchronize();
   unsigned int e = 0;
-  e |= q38::qgemm_stream_error(clear != 0);
-  e |= q38::qgemm_dispatch_error(clear != 0);
-  e |= q38::qgemm_umma_error(clear != 0);
-  e |= q38::attention_error(clear != 0);
-  e |= q38::gdn_error(clear != 0);
-  e |= q38::misc_error(clear != 0);
+  const q38::ErrorWordList& l = q38::error_word_list();
+  for (int i = 0; i < l.count; ++i) e |= l.read[i](clear != 0);
   return e;
 }
 

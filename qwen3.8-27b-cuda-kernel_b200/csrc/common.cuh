@@ -38,6 +38,14 @@ static inline unsigned int* tu_error_address() {
   return cudaGetSymbolAddress(&p, g_tu_error) == cudaSuccess ? static_cast<unsigned int*>(p) : nullptr;
 }
 
+// Makes this translation unit's error word known to the readers in c_abi.cu (one line per .cu that reports errors).
+void register_error_word(unsigned int (*read)(bool clear), unsigned int* (*address)());
+struct ErrorWordRegistration {
+  ErrorWordRegistration(unsigned int (*read)(bool), unsigned int* (*address)()) { register_error_word(read, address); }
+};
+#define Q38_REGISTER_ERROR_WORD() \
+  namespace { const ::q38::ErrorWordRegistration error_word_registration(&::q38::read_tu_error, &::q38::tu_error_address); }
+
 // Programmatic dependent launch: let the next kernel of the stream be scheduled / wait until everything the
 // previous kernels of the stream wrote is visible. Both are no-ops for a kernel launched without the attribute.
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }

@@ -1178,8 +1178,7 @@ __global__ void __launch_bounds__(kDv) gdn_norm_gate_kernel(const float* __restr
 
 int g_chunk_scan_tensor_cores = 1;
 
-unsigned int gdn_error(bool clear) { return read_tu_error(clear); }
-unsigned int* gdn_error_address() { return tu_error_address(); }
+Q38_REGISTER_ERROR_WORD();
 
 }  // namespace q38
 

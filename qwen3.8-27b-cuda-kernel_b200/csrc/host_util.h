@@ -14,6 +14,7 @@ namespace q38 {
 void set_error(const char* fmt, ...);  // defined in c_abi.cu
 int num_sms();                         // SM count of the device current at first use (one device per process)
 int max_optin_smem();
+q38_gemm_tuning_lookup gemm_tuning();  // the installed tile-configuration lookup of the BQ GEMM, or null
 
 #define Q38_REQUIRE(cond, ...)            \
   do {                                    \

@@ -27,8 +27,6 @@ constexpr ConfigInfo kConfigs[] = {
 };
 constexpr int kNumConfigs = int(sizeof(kConfigs) / sizeof(kConfigs[0]));
 
-q38_gemm_tuning_lookup g_tuning = nullptr;
-
 // Small batches stream the weights through mma.sync (tokens are the 8-wide operand); from 17 tokens on the
 // tcgen05 kernel keeps the accumulators in TMEM and, in the tmem_* configurations, also hands the decoded weights
 // to the MMA through TMEM (no shared-memory round trip of the bf16 tile: faster at every token count measured, so
@@ -85,10 +83,9 @@ using namespace q38;
 extern "C" int q38_qgemm_num_configs(void) { return kNumConfigs; }
 extern "C" const char* q38_qgemm_config_name(int c) { return c >= 0 && c < kNumConfigs ? kConfigs[c].name : "?"; }
 extern "C" int q38_qgemm_config_tile_m(int c) { return c >= 0 && c < kNumConfigs ? kConfigs[c].tile_m : 0; }
-extern "C" void q38_set_qgemm_tuning(q38_gemm_tuning_lookup lookup) { g_tuning = lookup; }
 extern "C" int q38_qgemm_auto_config(int bits, int n, int k, int m) {
-  if (g_tuning) {
-    const int t = g_tuning(bits, n, k, m);
+  if (gemm_tuning()) {
+    const int t = gemm_tuning()(bits, n, k, m);
     if (t >= 0 && t < kNumConfigs) return t;
   }
   q38_bq_weight w{};
@@ -123,8 +120,8 @@ extern "C" int q38_qgemm(const q38_bf16* a, int m, const q38_bq_weight* w, const
     Q38_REQUIRE(ep->kind >= 0 && ep->kind <= 3 && ep->out && ep->ldo > 0, "qgemm: epilogue output");
   }
   if (ep->partials_in) Q38_REQUIRE(ep->hidden > 0 && ep->hidden % 128 == 0, "qgemm: hidden %d", ep->hidden);
-  if (config < 0 && g_tuning) {
-    const int t = g_tuning(w->bits, w->n, w->k, m);
+  if (config < 0 && gemm_tuning()) {
+    const int t = gemm_tuning()(w->bits, w->n, w->k, m);
     if (t >= 0 && t < kNumConfigs) config = t;
   }
   if (config < 0) config = auto_config(m, *w, ws);
@@ -245,6 +242,5 @@ extern "C" int q38_qgemm_static(const q38_bf16* a, int m, const q38_bq_weight* w
 }
 
 namespace q38 {
-unsigned int qgemm_dispatch_error(bool clear) { return read_tu_error(clear); }
-unsigned int* qgemm_dispatch_error_address() { return tu_error_address(); }
+Q38_REGISTER_ERROR_WORD();
 }

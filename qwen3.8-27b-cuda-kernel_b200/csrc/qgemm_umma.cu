@@ -1112,7 +1112,6 @@ int qgemm_umma_launch(int tok, int mblocks, bool a_in_tmem, const __nv_bfloat16*
   }
 }
 
-unsigned int qgemm_umma_error(bool clear) { return read_tu_error(clear); }
-unsigned int* qgemm_umma_error_address() { return tu_error_address(); }
+Q38_REGISTER_ERROR_WORD();
 
 }  // namespace q38

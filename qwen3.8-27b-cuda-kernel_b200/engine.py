@@ -26,7 +26,8 @@ def greedy() -> Sampling:
 class RunnerOptions(C.Structure):
     _fields_ = [("max_batch", C.c_int), ("prefill_chunk", C.c_int), ("kv_dtype", C.c_int), ("kv_tokens", C.c_int64),
                 ("max_context", C.c_int), ("reserve_mib", C.c_size_t), ("embedding_on_host", C.c_int),
-                ("cuda_graphs", C.c_int), ("history_cap", C.c_int), ("verbose", C.c_int)]
+                ("cuda_graphs", C.c_int), ("history_cap", C.c_int), ("verbose", C.c_int),
+                ("compute_dtype", C.c_int)]
 
 
 class DecodeRow(C.Structure):
@@ -54,12 +55,16 @@ _lib = None
 def lib() -> C.CDLL:
     global _lib
     if _lib is None:
-        kernels()  # dependency, loaded RTLD_GLOBAL
+        kernels()  # dependency, loaded RTLD_GLOBAL (from the same folder)
         L = _load("libq38_engine.so")
         L.q38e_last_error.restype = C.c_char_p
         L.q38e_model_summary.restype = C.c_char_p
+        L.q38e_model_architecture.restype = C.c_char_p
         _lib = L
     return _lib
+
+
+COMPUTE_BF16, COMPUTE_F32 = 0, 1
 
 
 class EngineError(RuntimeError):
@@ -96,6 +101,8 @@ class Model:
         self.vocab = lib().q38e_model_vocab(self.h)
         self.hidden = lib().q38e_model_hidden(self.h)
         self.layers = lib().q38e_model_layers(self.h)
+        self.architecture = lib().q38e_model_architecture(self.h).decode()
+        self.max_positions = lib().q38e_model_max_positions(self.h)
 
     def summary(self) -> str:
         return lib().q38e_model_summary(self.h).decode()
@@ -152,9 +159,8 @@ class Runner:
         _ok(lib().q38e_runner_kv_free_pages(self.h, C.byref(n)))
         return n.value
 
-    def prefill(self, rows) -> tuple[np.ndarray, np.ndarray]:
-        """rows: iterable of (slot, pos0, tokens, sampling_or_None, step)."""
-        rows = list(rows)
+    @staticmethod
+    def _prefill_rows(rows):
         arr = (PrefillRow * len(rows))()
         keep = []
         for i, (slot, pos0, tokens, sampling, step) in enumerate(rows):
@@ -162,6 +168,22 @@ class Runner:
             keep.append(t)
             arr[i] = PrefillRow(slot, pos0, t.ctypes.data_as(C.POINTER(C.c_int32)), len(t), int(sampling is not None),
                                 sampling if sampling is not None else greedy(), step)
+        return arr, keep
+
+    def step_logits(self, rows, want) -> np.ndarray:
+        """One ragged step; rows as in prefill(), want: iterable of (row, token index) -> logits [len(want), vocab]."""
+        rows, want = list(rows), list(want)
+        arr, keep = self._prefill_rows(rows)
+        at = _i32([w[0] for w in want]), _i32([w[1] for w in want])
+        out = np.empty((len(want), self.model.vocab), dtype=np.float32)
+        _ok(lib().q38e_runner_step_logits(self.h, arr, len(rows), at[0].ctypes.data_as(C.c_void_p),
+                                          at[1].ctypes.data_as(C.c_void_p), len(want), out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def prefill(self, rows) -> tuple[np.ndarray, np.ndarray]:
+        """rows: iterable of (slot, pos0, tokens, sampling_or_None, step)."""
+        rows = list(rows)
+        arr, keep = self._prefill_rows(rows)
         toks = np.zeros(len(rows), dtype=np.int32)
         lps = np.zeros(len(rows), dtype=np.float32)
         n = C.c_int()

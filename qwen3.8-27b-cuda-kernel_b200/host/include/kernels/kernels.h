@@ -42,7 +42,7 @@ struct BatchDesc {
   }
 };
 
-enum class KvDtype : int { Int8 = Q38_KV_INT8, BF16 = Q38_KV_BF16 };
+enum class KvDtype : int { Auto = -1, Int8 = Q38_KV_INT8, BF16 = Q38_KV_BF16, F32 = Q38_KV_F32 };
 constexpr int kPageTokens = Q38_PAGE_TOKENS;
 constexpr int kHeadDim = Q38_HEAD_DIM;
 
@@ -284,6 +284,57 @@ inline void gather_rows(const __nv_bfloat16* x, const float* partials, const int
 // Extension: the library's device error status as a node of the step (see q38_device_error_collect).
 inline void collect_device_errors(unsigned int* dst, cudaStream_t stream) {
   detail::ok(q38_device_error_collect(dst, stream));
+}
+
+// ---- layer-list architectures with dense weights (extension): the C structs are used as they are -------------------
+using KvLayerDesc = q38_kv_layer_desc;
+using RecurrentStateDesc = q38_recurrent_state_desc;
+using DenseWeight = q38_dense_weight;
+using DenseEpilogue = q38_dense_epilogue;
+using Norm = q38_norm;
+using RopeAppendParams = q38_rope_append_params;
+using MixedAttentionParams = q38_mixed_attention_params;
+using MinGruParams = q38_mingru_params;
+using RgLruParams = q38_rglru_params;
+
+inline void dense_gemm(const void* x, int ldx, int act, int m, const DenseWeight& w, const DenseEpilogue& ep,
+                       const GemmWorkspace& ws, cudaStream_t stream) {
+  const q38_gemm_workspace cws{ws.partials, ws.partial_floats, ws.counters, ws.num_counters};
+  detail::ok(q38_dense_gemm(x, ldx, act, m, &w, &ep, &cws, stream, Q38_DENSE_AUTO));
+}
+inline void embed_norm(const q38_bf16* table, const q38_bf16* positions, const int32_t* tokens, const int* tok_pos, int m,
+                       int width, float* residual, const Norm& norm, void* out, int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_embed_norm(table, positions, tokens, tok_pos, m, width, residual, &norm, out, ld_out, act, stream));
+}
+inline void residual_norm(const float* y, int ldy, int m, int width, const Norm& post, float* residual, const Norm* next,
+                          void* out, int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_residual_norm(y, ldy, m, width, &post, residual, next, out, ld_out, act, stream));
+}
+inline void gather_norm(const float* residual, const int* rows, int first, int n, int width, const Norm& norm, void* out,
+                        int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_gather_norm(residual, rows, first, n, width, &norm, out, ld_out, act, stream));
+}
+inline void rope_append(const RopeAppendParams& p, const BatchDesc& batch, const KvLayerDesc& kv, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_rope_append(&p, &b, &kv, stream));
+}
+inline void mixed_attention_prefill(const MixedAttentionParams& p, const BatchDesc& batch, const KvLayerDesc& kv,
+                                    cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_mixed_attention_prefill(&p, &b, &kv, stream));
+}
+inline void mixed_attention_decode(const MixedAttentionParams& p, const BatchDesc& batch, const KvLayerDesc& kv,
+                                   cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_mixed_attention_decode(&p, &b, &kv, stream));
+}
+inline void mingru(const MinGruParams& p, const BatchDesc& batch, const RecurrentStateDesc& st, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_mingru(&p, &b, &st, stream));
+}
+inline void rglru(const RgLruParams& p, const BatchDesc& batch, const RecurrentStateDesc& st, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_rglru(&p, &b, &st, stream));
 }
 
 }  // namespace qwen38::kernels

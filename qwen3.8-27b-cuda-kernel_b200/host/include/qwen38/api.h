@@ -84,7 +84,32 @@ inline int64_t align_up(int64_t a, int64_t b) { return ceil_div(a, b) * b; }
 // ===================================================================================================
 // model configuration (reference include/qwen38/config.h; header block of docs/FORMAT.md 1.1)
 // ===================================================================================================
+// Extension: one layer of a decoder whose configuration lists its layers one by one (layer-list architectures): a
+// sequence mixer with its own sizes and an optional gated feed-forward.
+enum class MixerKind : uint8_t { Attention, MinGru, RgLru };
+struct AttentionSpec {
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+  int rot_dims = 0;          // leading dimensions of a query / key head that turn, dimension i with i + rot_dims / 2
+  double rot_base = 10000.0;
+  float scale = 1.0f;
+  bool value_mix = false;    // values are blended with those of the first value-mixing layer
+  bool head_mix = false;     // the heads' softmax weights are mixed by a [heads][heads] matrix
+  int group() const { return heads / kv_heads; }
+};
+struct RecurrentSpec {
+  int width = 0;
+  int blocks = 1;            // RG-LRU: block-diagonal gates
+  int taps = 0;              // RG-LRU: causal convolution, current token included
+};
+struct LayerSpec {
+  MixerKind mixer = MixerKind::Attention;
+  AttentionSpec attn;
+  RecurrentSpec rec;
+  int ff = 0;                // feed-forward width, 0 = the layer has none
+};
+
 struct ModelConfig {
+  std::string architecture = "Qwen3.8";
   int hidden_size = 0, num_layers = 0, vocab_size = 0, intermediate_size = 0;
   int num_attention_heads = 0, num_key_value_heads = 0, head_dim = 0, rotary_dim = 0;
   double rope_theta = 0;
@@ -95,6 +120,8 @@ struct ModelConfig {
   bool norm_folded = true;
   std::vector<uint8_t> is_attention;   // per layer: 1 full attention, 0 Gated DeltaNet
   std::vector<int32_t> eos_token_ids;
+  bool learned_positions = false;      // a learned position table bounds the context
+  std::vector<LayerSpec> layers;       // layer-list architectures; empty for the BQ family
 
   int num_attention_layers() const;
   int num_gdn_layers() const;
@@ -117,11 +144,11 @@ struct ModelConfig {
 // ===================================================================================================
 // .q38 model file (reference include/qwen38/model_file.h, docs/FORMAT.md 1)
 // ===================================================================================================
-enum class DType : uint8_t { BQ4, BQ5, BQ6, BQ8, BF16, F32 };
+enum class DType : uint8_t { BQ4, BQ5, BQ6, BQ8, BF16, F32, I32 };
 const char* dtype_name(DType dtype);
 inline bool is_bq(DType d) { return d <= DType::BQ8; }
 inline int bq_bits(DType d) {
-  constexpr int kBits[] = {4, 5, 6, 8, 0, 0};
+  constexpr int kBits[] = {4, 5, 6, 8, 0, 0, 0};
   return kBits[int(d)];
 }
 
@@ -140,6 +167,7 @@ struct TensorInfo {
 
 class ModelFile {
  public:
+  // A .q38 file, or (extension) a folder with config.json and model.safetensors.
   static std::unique_ptr<ModelFile> open(const std::string& path);
   ~ModelFile();
   ModelFile(const ModelFile&) = delete;
@@ -165,6 +193,8 @@ class ModelFile {
 
  private:
   ModelFile() = default;
+  void open_folder(const std::string& path);
+  void map(const std::string& path);
   std::string path_, header_, recipe_;
   ModelConfig config_;
   std::map<std::string, TensorInfo> tensors_;
@@ -249,6 +279,7 @@ class DeviceArena {
   T* allocate_array(size_t count, size_t align = 256) {
     return static_cast<T*>(allocate(count * sizeof(T), align));
   }
+  void* base() const { return block_.get(); }
   size_t used() const { return used_; }
   size_t capacity() const { return block_.bytes(); }
 
@@ -356,11 +387,22 @@ class ModelWeights {
 // ===================================================================================================
 // paged KV cache + GDN state pool (reference include/qwen38/kv_cache.h)
 // ===================================================================================================
+// Extension: what one attention layer keeps per token. The fixed-geometry layers of the BQ family (head dimension 256,
+// int8 with scales or bf16) are described by their head count alone (k_dim == 0).
+struct KvLayerGeometry {
+  int kv_heads = 0;
+  int k_dim = 0, v_dim = 0;  // stored head sizes
+  size_t page_bytes(kernels::KvDtype dtype) const;
+};
+
 class KvCache {
  public:
   KvCache(const ModelConfig& cfg, kernels::KvDtype dtype, int num_pages, int num_slots, int max_pages_per_seq);
+  KvCache(std::vector<KvLayerGeometry> layers, kernels::KvDtype dtype, int num_pages, int num_slots, int max_pages_per_seq);
   static size_t page_bytes_all_layers(const ModelConfig& cfg, kernels::KvDtype dtype);
-  kernels::KvCacheDesc desc() const;
+  static size_t page_bytes_all_layers(const std::vector<KvLayerGeometry>& layers, kernels::KvDtype dtype);
+  kernels::KvCacheDesc desc() const;                    // fixed-geometry layers
+  kernels::KvLayerDesc layer_desc(int attn_layer) const;  // one layer of any geometry
   int num_pages() const { return num_pages_; }
   int free_pages() const { return int(free_.size()); }
   int pages_of(int slot) const { return int(owned_[size_t(slot)].size()); }
@@ -374,8 +416,8 @@ class KvCache {
  private:
   int num_pages_, num_slots_, max_pages_per_seq_;
   kernels::KvDtype dtype_;
-  int kv_heads_;
-  size_t page_bytes_ = 0, layer_stride_ = 0;
+  std::vector<KvLayerGeometry> layers_;
+  std::vector<size_t> layer_offset_;  // byte offset of each layer's pages in the pool
   DeviceBuffer pool_, table_dev_;
   PinnedBuffer table_host_;
   std::vector<int> free_;
@@ -396,6 +438,26 @@ class GdnStatePool {
   DeviceBuffer recurrent_, conv_;
 };
 
+// Extension: per-slot state of elementwise recurrent layers: one fp32 vector per layer, and for layers with a causal
+// convolution a ring of the last `taps` inputs indexed by position (activation precision).
+struct RecurrentLayerGeometry {
+  int width = 0;
+  int taps = 0, channels = 0;
+};
+class RecurrentStatePool {
+ public:
+  RecurrentStatePool(std::vector<RecurrentLayerGeometry> layers, size_t conv_elem_bytes, int num_slots);
+  static size_t bytes_per_slot(const std::vector<RecurrentLayerGeometry>& layers, size_t conv_elem_bytes);
+  kernels::RecurrentStateDesc layer_desc(int recurrent_layer) const;
+  void reset(int slot, cudaStream_t stream);
+
+ private:
+  std::vector<RecurrentLayerGeometry> layers_;
+  std::vector<size_t> state_offset_, conv_offset_;  // within a slot's block
+  size_t slot_bytes_ = 0, elem_bytes_ = 2;
+  DeviceBuffer pool_;
+};
+
 // ===================================================================================================
 // step executor (reference include/qwen38/model_runner.h)
 // ===================================================================================================
@@ -409,10 +471,12 @@ struct SamplingParams {
   uint64_t seed = 0;
 };
 
+enum class ComputeDtype : int { BF16 = 0, F32 = 1 };
+
 struct RunnerOptions {
   int max_batch = 8;
   int prefill_chunk = 1024;
-  kernels::KvDtype kv_dtype = kernels::KvDtype::Int8;
+  kernels::KvDtype kv_dtype = kernels::KvDtype::Auto;  // the architecture's own: int8 for BQ models
   int64_t kv_tokens = 0;        // 0 = everything that fits
   int max_context = 262144;
   size_t reserve_mib = 640;
@@ -420,6 +484,9 @@ struct RunnerOptions {
   bool cuda_graphs = true;
   int history_cap = 1024;
   bool verbose = true;
+  // Extension: precision of the matrix products, activations and cache of dense-weight architectures. F32 computes
+  // everything in 32-bit (no reduced-precision matrix mode). BQ models run in BF16 only.
+  ComputeDtype compute = ComputeDtype::BF16;
 };
 
 struct DecodeRow {
@@ -439,9 +506,15 @@ struct PrefillRow {
   int step = 0;
 };
 
+// A place whose logits a prefill step returns: token `index` of the step's row `row` (extension).
+struct LogitsAt {
+  int row = 0, index = 0;
+};
+
 struct StepResult {
   std::vector<int32_t> tokens;
   std::vector<float> logprobs;
+  std::vector<float> logits;  // [wanted places][vocab], in the order they were asked for (extension)
 };
 
 struct MemoryPlan {
@@ -481,7 +554,7 @@ class ModelRunner {
 
   // Ragged prefill: chunks of several sequences in one step (sum of lengths <= prefill_chunk). The result
   // holds one token per row that asked for a sample, in row order.
-  StepResult prefill_batch(std::span<const PrefillRow> rows);
+  StepResult prefill_batch(std::span<const PrefillRow> rows, std::span<const LogitsAt> want = {});
 
   void set_profiling(bool on);
   const OpProfile& profile() const;

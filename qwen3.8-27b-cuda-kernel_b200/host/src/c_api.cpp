@@ -54,7 +54,8 @@ RunnerOptions from_c(const q38e_runner_options& o) {
   RunnerOptions r;
   r.max_batch = o.max_batch;
   r.prefill_chunk = o.prefill_chunk;
-  r.kv_dtype = o.kv_dtype == 0 ? kernels::KvDtype::Int8 : kernels::KvDtype::BF16;
+  QWEN38_CHECK(o.kv_dtype >= -1 && o.kv_dtype <= 2, "kv_dtype ", o.kv_dtype);
+  r.kv_dtype = kernels::KvDtype(o.kv_dtype);
   r.kv_tokens = o.kv_tokens;
   r.max_context = o.max_context;
   r.reserve_mib = o.reserve_mib;
@@ -62,6 +63,8 @@ RunnerOptions from_c(const q38e_runner_options& o) {
   r.cuda_graphs = o.cuda_graphs != 0;
   r.history_cap = o.history_cap;
   r.verbose = o.verbose != 0;
+  QWEN38_CHECK(o.compute_dtype == 0 || o.compute_dtype == 1, "compute_dtype ", o.compute_dtype);
+  r.compute = ComputeDtype(o.compute_dtype);
   return r;
 }
 }  // namespace
@@ -82,6 +85,7 @@ void q38e_default_runner_options(q38e_runner_options* o) {
   o->cuda_graphs = d.cuda_graphs;
   o->history_cap = d.history_cap;
   o->verbose = d.verbose;
+  o->compute_dtype = int(d.compute);
 }
 
 int q38e_step_status(unsigned int device_error_word, const char* where) {
@@ -110,6 +114,8 @@ void q38e_model_close(q38e_model* m) { delete m; }
 int q38e_model_vocab(const q38e_model* m) { return m->file->config().vocab_size; }
 int q38e_model_hidden(const q38e_model* m) { return m->file->config().hidden_size; }
 int q38e_model_layers(const q38e_model* m) { return m->file->config().num_layers; }
+const char* q38e_model_architecture(const q38e_model* m) { return m->file->config().architecture.c_str(); }
+int q38e_model_max_positions(const q38e_model* m) { return m->file->config().max_position_embeddings; }
 const char* q38e_model_summary(const q38e_model* m) { return m->summary.c_str(); }
 int q38e_model_dequant(const q38e_model* m, const char* name, float* out, size_t out_floats) {
   return guard([&] {
@@ -142,25 +148,44 @@ int q38e_runner_kv_pages(q38e_runner* r, int slot, int* pages_out, int capacity,
 }
 int q38e_runner_kv_free_pages(q38e_runner* r, int* count) { return guard([&] { *count = r->r->kv().free_pages(); }); }
 
+namespace {
+// the C rows as the runner's; `sp` keeps the sampling parameters the rows point at
+std::vector<PrefillRow> prefill_rows(const q38e_prefill_row* rows, int num_rows, std::vector<SamplingParams>& sp) {
+  std::vector<PrefillRow> pr(static_cast<size_t>(num_rows));
+  sp.resize(size_t(num_rows));
+  for (int i = 0; i < num_rows; ++i) {
+    pr[size_t(i)].slot = rows[i].slot;
+    pr[size_t(i)].pos0 = rows[i].pos0;
+    pr[size_t(i)].tokens = std::span<const int32_t>(rows[i].tokens, size_t(rows[i].num_tokens));
+    sp[size_t(i)] = from_c(rows[i].sampling);
+    pr[size_t(i)].sample = rows[i].sample ? &sp[size_t(i)] : nullptr;
+    pr[size_t(i)].step = rows[i].step;
+  }
+  return pr;
+}
+}  // namespace
+
 int q38e_runner_prefill(q38e_runner* r, const q38e_prefill_row* rows, int num_rows, int32_t* tokens_out,
                         float* logprobs_out, int* num_out) {
   return guard([&] {
-    std::vector<PrefillRow> pr(static_cast<size_t>(num_rows));
-    std::vector<SamplingParams> sp(static_cast<size_t>(num_rows));
-    for (int i = 0; i < num_rows; ++i) {
-      pr[size_t(i)].slot = rows[i].slot;
-      pr[size_t(i)].pos0 = rows[i].pos0;
-      pr[size_t(i)].tokens = std::span<const int32_t>(rows[i].tokens, size_t(rows[i].num_tokens));
-      sp[size_t(i)] = from_c(rows[i].sampling);
-      pr[size_t(i)].sample = rows[i].sample ? &sp[size_t(i)] : nullptr;
-      pr[size_t(i)].step = rows[i].step;
-    }
-    const StepResult res = r->r->prefill_batch(pr);
+    std::vector<SamplingParams> sp;
+    const StepResult res = r->r->prefill_batch(prefill_rows(rows, num_rows, sp));
     if (num_out) *num_out = int(res.tokens.size());
     for (size_t i = 0; i < res.tokens.size(); ++i) {
       if (tokens_out) tokens_out[i] = res.tokens[i];
       if (logprobs_out) logprobs_out[i] = res.logprobs[i];
     }
+  });
+}
+
+int q38e_runner_step_logits(q38e_runner* r, const q38e_prefill_row* rows, int num_rows, const int32_t* want_row,
+                            const int32_t* want_index, int num_want, float* logits_out) {
+  return guard([&] {
+    std::vector<SamplingParams> sp;
+    std::vector<LogitsAt> want(static_cast<size_t>(num_want));
+    for (int i = 0; i < num_want; ++i) want[size_t(i)] = {want_row[i], want_index[i]};
+    const StepResult res = r->r->prefill_batch(prefill_rows(rows, num_rows, sp), want);
+    std::memcpy(logits_out, res.logits.data(), res.logits.size() * sizeof(float));
   });
 }
 

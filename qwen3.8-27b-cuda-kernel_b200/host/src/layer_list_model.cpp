@@ -1,0 +1,534 @@
+// Weights, cache, state and step of the layer-list architectures (see layer_list_model.h).
+#include "layer_list_model.h"
+
+#include <algorithm>
+
+namespace qwen38 {
+
+namespace {
+
+constexpr int kMaxSplits = 64;
+int up(int x, int to) { return int(align_up(x, to)); }
+
+// The tensors of one design by name and expected shape; `at` reads one as fp32.
+class TensorReader {
+ public:
+  explicit TensorReader(const ModelFile& f) : file_(f) {}
+  void require(const std::string& name, std::vector<int64_t> shape) const {
+    const TensorInfo& t = file_.tensor(name);
+    QWEN38_CHECK(t.dtype == DType::BF16 || t.dtype == DType::F32, name, ": dtype ", dtype_name(t.dtype));
+    auto text = [](const std::vector<int64_t>& s) {
+      std::string o = "[";
+      for (size_t i = 0; i < s.size(); ++i) o += (i ? ", " : "") + std::to_string(s[i]);
+      return o + "]";
+    };
+    QWEN38_CHECK(t.shape == shape, name, ": shape ", text(t.shape), ", expected ", text(shape));
+  }
+  float at(const TensorInfo& t, int64_t i) const {
+    const uint8_t* p = file_.data(t.offset, t.bytes).data();
+    if (t.dtype == DType::F32) {
+      float v;
+      std::memcpy(&v, p + 4 * i, 4);
+      return v;
+    }
+    uint16_t b;
+    std::memcpy(&b, p + 2 * i, 2);
+    return bf16_to_f32(b);
+  }
+  // `count` consecutive elements from element i as bf16
+  void copy_bf16(const TensorInfo& t, int64_t i, int64_t count, q38_bf16* dst) const {
+    const uint8_t* p = file_.data(t.offset, t.bytes).data();
+    if (t.dtype == DType::BF16) std::memcpy(dst, p + 2 * i, size_t(2 * count));
+    else
+      for (int64_t k = 0; k < count; ++k) dst[k] = f32_to_bf16(at(t, i + k));
+  }
+  const ModelFile& file() const { return file_; }
+
+ private:
+  const ModelFile& file_;
+};
+
+struct Linear {
+  std::vector<std::string> weights;             // stacked along the output
+  std::vector<std::string> biases;              // one per weight, "" = none
+  bool interleave = false;                      // two weights whose rows alternate
+};
+
+struct LayerTensors {
+  Linear in, out, glu, down;
+};
+
+std::string mix(int i, const char* name) { return "l" + std::to_string(i) + ".mix." + name; }
+std::string at_layer(int i, const char* name) { return "l" + std::to_string(i) + "." + name; }
+
+LayerTensors names_of(const LayerSpec& l, int i) {
+  LayerTensors t;
+  auto w = [&](const char* n) { return mix(i, n); };
+  switch (l.mixer) {
+    case MixerKind::Attention:
+      t.in = {{w("q"), w("k"), w("v")}, {w("q.b"), w("k.b"), w("v.b")}};
+      t.out = {{w("o")}, {w("o.b")}};
+      break;
+    case MixerKind::MinGru:
+      t.in = {{w("z"), w("x"), w("g")}, {w("z.b"), w("x.b"), ""}};
+      t.out = {{w("o")}, {""}};
+      break;
+    case MixerKind::RgLru:
+      t.in = {{w("y"), w("x")}, {w("y.b"), w("x.b")}};
+      t.out = {{w("o")}, {""}};
+      break;
+  }
+  if (l.ff) {
+    t.glu = {{at_layer(i, "mlp.gate"), at_layer(i, "mlp.up")}, {"", ""}, true};
+    t.down = {{at_layer(i, "mlp.down")}, {""}};
+  }
+  return t;
+}
+
+struct LayerWeightsDev {
+  kernels::DenseWeight in{}, out{}, glu{}, down{};
+  const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
+  const float *v_mix = nullptr, *head_mix = nullptr;
+  const float *conv_w = nullptr, *conv_b = nullptr, *gate_b = nullptr, *lam = nullptr;
+  const q38_bf16* gate_w = nullptr;
+  int block_ld = 0;
+};
+
+class LayerListModel final : public StepModel {
+ public:
+  LayerListModel(const ModelFile& f, const RunnerOptions& o, const LayerListDesign& d);
+
+  size_t weight_bytes() const override { return weight_bytes_; }
+  kernels::KvDtype resolve_kv_dtype(kernels::KvDtype d) const override {
+    const kernels::KvDtype own = f32_ ? kernels::KvDtype::F32 : kernels::KvDtype::BF16;
+    QWEN38_CHECK(d == kernels::KvDtype::Auto || d == own, cfg_.architecture, ": the KV cache has the activations' precision");
+    return own;
+  }
+  size_t kv_page_bytes(kernels::KvDtype d) const override {
+    size_t scores = 0;  // the decode kernels keep one page's scores of every head beside the pool
+    if (score_heads_ > 0) scores = size_t(score_heads_) * kernels::kPageTokens * 4;
+    return KvCache::page_bytes_all_layers(kv_layers_, d) + scores;
+  }
+  size_t state_bytes_per_slot() const override { return RecurrentStatePool::bytes_per_slot(rec_layers_, elem_); }
+  void load_weights() override;
+  std::unique_ptr<KvCache> make_kv(kernels::KvDtype d, int pages, int slots, int max_pages) const override {
+    return std::make_unique<KvCache>(kv_layers_, d, pages, slots, max_pages);
+  }
+  void make_state(int slots) override { state_ = std::make_unique<RecurrentStatePool>(rec_layers_, elem_, slots); }
+  void reset_slot(int slot, cudaStream_t s) override { state_->reset(slot, s); }
+  void carve(Workspace& w, const StepContext& ctx) override;
+  void prepare(const StepContext& ctx) override;
+  void forward(const StepContext& ctx, const StepBatch& b) override;
+  void head(const StepContext& ctx, const HeadRows& rows, float* logits) override;
+  const kernels::GemmWorkspace* gemm_workspace() const override { return &gemm_ws_; }
+
+ private:
+  // weight upload; without an arena the sizes are only added up
+  void visit_weights(DeviceArena* arena);
+  template <typename T>
+  const T* put(DeviceArena* arena, const std::vector<T>& v);
+  kernels::DenseWeight put_linear(DeviceArena* arena, const Linear& l);
+  const float* put_f32(DeviceArena* arena, const std::string& name);
+  const q38_bf16* put_bf16(DeviceArena* arena, const std::string& name);
+
+  void gemm(const StepContext& ctx, const void* x, int ldx, int m, const kernels::DenseWeight& w, int kind, void* out, int ldo) {
+    kernels::dense_gemm(x, ldx, act_, m, w, {kind, out, ldo}, gemm_ws_, ctx.stream);
+  }
+  kernels::Norm norm(const float* gain) const { return {gain, design_.norm_gain_is_scalar ? 0 : 1, cfg_.rms_norm_eps}; }
+  void attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i, bool first_values, bool blend);
+  void recurrent(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int rec_i);
+
+  TensorReader reader_;
+  ModelConfig cfg_;
+  LayerListDesign design_;
+  bool f32_ = false;
+  int act_ = Q38_ACT_BF16;
+  size_t elem_ = 2;
+  std::vector<KvLayerGeometry> kv_layers_;
+  std::vector<RecurrentLayerGeometry> rec_layers_;
+  int score_heads_ = 0;
+  size_t weight_bytes_ = 0;
+
+  DeviceArena arena_;
+  std::vector<LayerWeightsDev> layers_;
+  const q38_bf16 *embed_ = nullptr, *pos_ = nullptr;
+  const float* final_norm_ = nullptr;
+  kernels::DenseWeight head_{};
+  std::unique_ptr<RecurrentStatePool> state_;
+  DeviceBuffer scores_;
+
+  // activations; leading dimensions are multiples of 64 elements
+  int ld_x_ = 0, ld_proj_ = 0, ld_mixer_ = 0, ld_ff_ = 0, max_q_ = 0, max_v_ = 0, max_heads_ = 0, max_rec_ = 0, max_attn_out_ = 0;
+  float* residual_ = nullptr;
+  uint8_t* x_ = nullptr;       // normed input of the sublayer
+  uint8_t* proj_ = nullptr;    // the mixer's input projections
+  uint8_t* mixer_ = nullptr;   // what enters the output projection
+  uint8_t* ff_ = nullptr;
+  float* y_ = nullptr;         // sublayer output before its post-norm
+  uint8_t* q_ = nullptr;
+  uint8_t* v_first_ = nullptr;
+  float* stats_ = nullptr;
+  float* partials_ = nullptr;
+  float* rec_scratch_ = nullptr;
+  uint8_t* head_x_ = nullptr;
+  kernels::GemmWorkspace gemm_ws_;
+};
+
+LayerListModel::LayerListModel(const ModelFile& f, const RunnerOptions& o, const LayerListDesign& d)
+    : reader_(f), cfg_(f.config()), design_(d), f32_(o.compute == ComputeDtype::F32) {
+  act_ = f32_ ? Q38_ACT_F32 : Q38_ACT_BF16;
+  elem_ = f32_ ? 4 : 2;
+  ld_x_ = up(cfg_.hidden_size, 64);
+  int v_first = 0;
+  for (const LayerSpec& l : cfg_.layers) {
+    if (l.mixer == MixerKind::Attention) {
+      const AttentionSpec& a = l.attn;
+      const KvLayerGeometry g{a.kv_heads, up(a.dim, 32), up(a.vdim, 8)};
+      kv_layers_.push_back(g);
+      if (!f32_) score_heads_ = std::max(score_heads_, a.heads);
+      max_heads_ = std::max(max_heads_, a.heads);
+      max_q_ = std::max(max_q_, a.heads * g.k_dim);
+      max_attn_out_ = std::max(max_attn_out_, a.heads * g.v_dim);
+      ld_proj_ = std::max(ld_proj_, up(a.heads * a.dim + a.kv_heads * (a.dim + a.vdim), 64));
+      ld_mixer_ = std::max(ld_mixer_, up(a.heads * a.vdim, 64));
+      if (a.value_mix) {
+        QWEN38_CHECK(v_first == 0 || v_first == a.kv_heads * a.vdim, "layers that blend values need value heads of one total size");
+        v_first = a.kv_heads * a.vdim;
+      }
+    } else {
+      RecurrentLayerGeometry g;
+      g.width = l.rec.width;
+      g.taps = l.mixer == MixerKind::RgLru ? l.rec.taps : 0;
+      g.channels = g.taps ? l.rec.width : 0;
+      rec_layers_.push_back(g);
+      const int parts = l.mixer == MixerKind::MinGru ? 3 : 2;
+      ld_proj_ = std::max(ld_proj_, up(parts * l.rec.width, 64));
+      ld_mixer_ = std::max(ld_mixer_, up(l.rec.width, 64));
+      if (l.mixer == MixerKind::RgLru) max_rec_ = std::max(max_rec_, l.rec.width);
+    }
+    if (l.ff) ld_ff_ = std::max(ld_ff_, up(l.ff, 64));
+  }
+  max_v_ = v_first;
+  visit_weights(nullptr);
+}
+
+// ---- weights ----------------------------------------------------------------------------------------------
+template <typename T>
+const T* LayerListModel::put(DeviceArena* arena, const std::vector<T>& v) {
+  const size_t bytes = up256(std::max<size_t>(v.size() * sizeof(T), 1));
+  if (!arena) {
+    weight_bytes_ += bytes;
+    return nullptr;
+  }
+  void* dst = arena->allocate(bytes);
+  QWEN38_CUDA(cudaMemcpy(dst, v.data(), v.size() * sizeof(T), cudaMemcpyHostToDevice));
+  return static_cast<const T*>(dst);
+}
+
+const float* LayerListModel::put_f32(DeviceArena* arena, const std::string& name) {
+  const TensorInfo& t = reader_.file().tensor(name);
+  std::vector<float> v(size_t(t.numel()));
+  if (arena)
+    for (size_t i = 0; i < v.size(); ++i) v[i] = reader_.at(t, int64_t(i));
+  return put(arena, v);
+}
+
+const q38_bf16* LayerListModel::put_bf16(DeviceArena* arena, const std::string& name) {
+  const TensorInfo& t = reader_.file().tensor(name);
+  std::vector<q38_bf16> v(size_t(t.numel()));
+  if (arena) reader_.copy_bf16(t, 0, t.numel(), v.data());
+  return put(arena, v);
+}
+
+// Stacks matrices [n_i][k] along n (or alternates the rows of two), rows padded with zeros to a multiple of 64 columns
+// and the stack to a multiple of 16 rows.
+kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear& l) {
+  kernels::DenseWeight d{};
+  bool bias = false;
+  for (size_t i = 0; i < l.weights.size(); ++i) {
+    const TensorInfo& t = reader_.file().tensor(l.weights[i]);
+    QWEN38_CHECK(t.shape.size() == 2 && (i == 0 || int(t.shape[1]) == d.k), l.weights[i], ": shape");
+    d.n += int(t.shape[0]);
+    d.k = int(t.shape[1]);
+    bias = bias || !l.biases[i].empty();
+  }
+  d.ld = up(d.k, 64);
+  std::vector<q38_bf16> w(size_t(up(d.n, 16)) * size_t(d.ld), 0);
+  std::vector<float> b(bias ? size_t(up(d.n, 16)) : 0, 0.0f);
+  if (arena) {
+    int row0 = 0;
+    for (size_t i = 0; i < l.weights.size(); ++i) {
+      const TensorInfo& t = reader_.file().tensor(l.weights[i]);
+      for (int64_t r = 0; r < t.shape[0]; ++r) {
+        const int64_t to = l.interleave ? 2 * r + int64_t(i) : row0 + r;
+        reader_.copy_bf16(t, r * t.shape[1], t.shape[1], w.data() + to * d.ld);
+        if (!l.biases[i].empty()) b[size_t(to)] = reader_.at(reader_.file().tensor(l.biases[i]), r);
+      }
+      row0 += int(t.shape[0]);
+    }
+  }
+  d.w = put(arena, w);
+  d.bias = bias ? put(arena, b) : nullptr;
+  return d;
+}
+
+void LayerListModel::visit_weights(DeviceArena* arena) {
+  weight_bytes_ = arena ? weight_bytes_ : 0;
+  layers_.assign(cfg_.layers.size(), {});
+  embed_ = put_bf16(arena, "embed");
+  if (cfg_.learned_positions) pos_ = put_bf16(arena, "pos");
+  for (int i = 0; i < cfg_.num_layers; ++i) {
+    const LayerSpec& l = cfg_.layers[size_t(i)];
+    LayerWeightsDev& W = layers_[size_t(i)];
+    const LayerTensors names = names_of(l, i);
+    W.in = put_linear(arena, names.in);
+    W.out = put_linear(arena, names.out);
+    W.norm1 = put_f32(arena, at_layer(i, "norm1"));
+    W.norm1b = put_f32(arena, at_layer(i, "norm1b"));
+    if (l.ff) {
+      W.norm2 = put_f32(arena, at_layer(i, "norm2"));
+      W.norm2b = put_f32(arena, at_layer(i, "norm2b"));
+      W.glu = put_linear(arena, names.glu);
+      W.down = put_linear(arena, names.down);
+    }
+    if (l.mixer == MixerKind::Attention) {
+      if (l.attn.value_mix) W.v_mix = put_f32(arena, mix(i, "vmix"));
+      if (l.attn.head_mix) W.head_mix = put_f32(arena, mix(i, "talk"));
+    }
+    if (l.mixer == MixerKind::RgLru) {
+      const int width = l.rec.width, blocks = l.rec.blocks, bs = width / blocks, taps = l.rec.taps;
+      W.block_ld = up(bs, 32);
+      std::vector<float> conv(size_t(taps) * size_t(width)), gate_b(size_t(2) * size_t(width));
+      std::vector<q38_bf16> gates(size_t(blocks) * 2 * size_t(W.block_ld) * size_t(W.block_ld), 0);
+      if (arena) {
+        const TensorInfo& ct = reader_.file().tensor(mix(i, "conv"));
+        for (int c = 0; c < width; ++c)
+          for (int j = 0; j < taps; ++j) conv[size_t(j) * width + c] = reader_.at(ct, int64_t(c) * taps + j);
+        for (int g = 0; g < 2; ++g) {
+          const TensorInfo& gt = reader_.file().tensor(mix(i, g ? "ri" : "ra"));
+          const TensorInfo& bt = reader_.file().tensor(mix(i, g ? "ri.b" : "ra.b"));
+          for (int c = 0; c < width; ++c) gate_b[size_t(g) * width + c] = reader_.at(bt, c);
+          for (int b = 0; b < blocks; ++b)
+            for (int o = 0; o < bs; ++o)
+              reader_.copy_bf16(gt, (int64_t(b) * bs + o) * bs, bs, gates.data() + ((size_t(b) * 2 + g) * W.block_ld + o) * W.block_ld);
+        }
+      }
+      W.conv_w = put(arena, conv);
+      W.conv_b = put_f32(arena, mix(i, "conv.b"));
+      W.gate_w = put(arena, gates);
+      W.gate_b = put(arena, gate_b);
+      W.lam = put_f32(arena, mix(i, "lam"));
+    }
+  }
+  final_norm_ = put_f32(arena, "final.norm");
+  head_ = put_linear(arena, {{"head"}, {""}});
+}
+
+void LayerListModel::load_weights() {
+  arena_ = DeviceArena(weight_bytes_ + 256);
+  visit_weights(&arena_);
+}
+
+// ---- activations -------------------------------------------------------------------------------------------
+void LayerListModel::carve(Workspace& w, const StepContext& ctx) {
+  const size_t T = size_t(ctx.max_tokens), R = size_t(ctx.max_rows);
+  const size_t gemm_partials = f32_ ? 0 : size_t(2) * size_t(ctx.num_sms) * 128 * 256;
+  residual_ = w.take<float>(T * size_t(cfg_.hidden_size));
+  x_ = w.take<uint8_t>(T * size_t(ld_x_) * elem_);
+  proj_ = w.take<uint8_t>(T * size_t(ld_proj_) * elem_);
+  mixer_ = w.take<uint8_t>(T * size_t(ld_mixer_) * elem_);
+  ff_ = w.take<uint8_t>(T * size_t(ld_ff_) * elem_);
+  y_ = w.take<float>(T * size_t(ld_x_));
+  q_ = w.take<uint8_t>(T * size_t(max_q_) * elem_);
+  v_first_ = w.take<uint8_t>(T * size_t(max_v_) * elem_);
+  stats_ = w.take<float>(T * size_t(max_heads_) * 2);
+  if (!f32_) partials_ = w.take<float>(R * kMaxSplits * (size_t(max_attn_out_) + 2 * size_t(max_heads_)));
+  rec_scratch_ = w.take<float>(2 * T * size_t(max_rec_));
+  head_x_ = w.take<uint8_t>(R * size_t(ld_x_) * elem_);
+  gemm_ws_.partials = w.take<float>(gemm_partials);
+  gemm_ws_.partial_floats = gemm_partials;
+  gemm_ws_.counters = w.take<int>(4096);
+  gemm_ws_.num_counters = 4096;
+}
+
+void LayerListModel::prepare(const StepContext& ctx) {
+  if (score_heads_ > 0)
+    scores_ = DeviceBuffer(size_t(ctx.kv->num_pages()) * size_t(score_heads_) * kernels::kPageTokens * 4);
+}
+
+// ---- the step ------------------------------------------------------------------------------------------------
+void LayerListModel::attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W,
+                               int attn_i, bool first_values, bool blend) {
+  const AttentionSpec& a = l.attn;
+  const kernels::KvLayerDesc kv = ctx.kv->layer_desc(attn_i);
+  kernels::RopeAppendParams rp{};
+  rp.proj = proj_;
+  rp.ld_proj = ld_proj_;
+  rp.act = act_;
+  rp.heads = a.heads;
+  rp.kv_heads = a.kv_heads;
+  rp.dim = a.dim;
+  rp.vdim = a.vdim;
+  rp.rot_dims = a.rot_dims;
+  rp.rot_base = a.rot_base;
+  rp.q_out = q_;
+  rp.v_first_out = first_values ? v_first_ : nullptr;
+  rp.v_first_in = blend ? v_first_ : nullptr;
+  rp.v_mix = W.v_mix;
+  kernels::rope_append(rp, b.all, kv, ctx.stream);
+  ctx.mark("mix.rope_append");
+  kernels::MixedAttentionParams ap{};
+  ap.q = q_;
+  ap.act = act_;
+  ap.heads = a.heads;
+  ap.vdim = a.vdim;
+  ap.scale = a.scale;
+  ap.head_mix = W.head_mix;
+  ap.out = mixer_;
+  ap.ld_out = ld_mixer_;
+  ap.stats = stats_;
+  ap.scores = scores_.as<float>();
+  ap.partials = partials_;
+  ap.max_splits = kMaxSplits;
+  if (b.decode || b.mixed) kernels::mixed_attention_decode(ap, b.single_part, kv, ctx.stream);
+  if (!b.decode) kernels::mixed_attention_prefill(ap, b.chunk_part, kv, ctx.stream);
+  ctx.mark(b.decode ? "mix.attn_decode" : "mix.attn_prefill");
+}
+
+void LayerListModel::recurrent(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int rec_i) {
+  const kernels::RecurrentStateDesc st = state_->layer_desc(rec_i);
+  if (l.mixer == MixerKind::MinGru) {
+    const kernels::MinGruParams p{proj_, ld_proj_, act_, l.rec.width, mixer_, ld_mixer_};
+    if (b.decode || b.mixed) kernels::mingru(p, b.single_part, st, ctx.stream);
+    if (!b.decode) kernels::mingru(p, b.chunk_part, st, ctx.stream);
+    ctx.mark("mix.mingru");
+    return;
+  }
+  kernels::RgLruParams p{};
+  p.proj = proj_;
+  p.ld_proj = ld_proj_;
+  p.act = act_;
+  p.width = l.rec.width;
+  p.blocks = l.rec.blocks;
+  p.block_ld = W.block_ld;
+  p.taps = l.rec.taps;
+  p.conv_w = W.conv_w;
+  p.conv_b = W.conv_b;
+  p.gate_w = W.gate_w;
+  p.gate_b = W.gate_b;
+  p.lam = W.lam;
+  p.log_decay = design_.rglru_log_decay;
+  p.scratch = rec_scratch_;
+  p.out = mixer_;
+  p.ld_out = ld_mixer_;
+  if (b.decode || b.mixed) kernels::rglru(p, b.single_part, st, ctx.stream);
+  if (!b.decode) kernels::rglru(p, b.chunk_part, st, ctx.stream);
+  ctx.mark("mix.rglru");
+}
+
+void LayerListModel::forward(const StepContext& ctx, const StepBatch& b) {
+  const int m = b.m, H = cfg_.hidden_size, n = cfg_.num_layers;
+  cudaStream_t s = ctx.stream;
+  const int glu = design_.glu == LayerListDesign::Glu::Gelu ? Q38_DENSE_GLU_GELU : Q38_DENSE_GLU_SILU;
+  kernels::embed_norm(embed_, pos_, b.tokens, b.all.tok_pos, m, H, residual_, norm(n ? layers_[0].norm1 : final_norm_), x_, ld_x_,
+                      act_, s);
+  ctx.mark("embed");
+  int attn_i = 0, rec_i = 0;
+  bool have_values = false;
+  for (int i = 0; i < n; ++i) {
+    const LayerSpec& l = cfg_.layers[size_t(i)];
+    const LayerWeightsDev& W = layers_[size_t(i)];
+    // the pre-norm that follows this layer; the last layer's successor is the final norm, taken over the sampled rows only
+    const kernels::Norm next_layer = norm(i + 1 < n ? layers_[size_t(i + 1)].norm1 : nullptr);
+    const kernels::Norm* after = i + 1 < n ? &next_layer : nullptr;
+    gemm(ctx, x_, ld_x_, m, W.in, Q38_DENSE_STORE, proj_, ld_proj_);
+    ctx.mark(l.mixer == MixerKind::Attention ? "gemm.attn_qkv" : l.mixer == MixerKind::MinGru ? "gemm.mingru_in" : "gemm.rglru_in");
+    if (l.mixer == MixerKind::Attention) {
+      attention(ctx, b, l, W, attn_i++, l.attn.value_mix && !have_values, l.attn.value_mix && have_values);
+      have_values = have_values || l.attn.value_mix;
+    } else {
+      recurrent(ctx, b, l, W, rec_i++);
+    }
+    gemm(ctx, mixer_, ld_mixer_, m, W.out, Q38_DENSE_STORE_F32, y_, ld_x_);
+    ctx.mark(l.mixer == MixerKind::Attention ? "gemm.attn_o" : l.mixer == MixerKind::MinGru ? "gemm.mingru_out" : "gemm.rglru_out");
+    const kernels::Norm norm2 = norm(W.norm2);
+    kernels::residual_norm(y_, ld_x_, m, H, norm(W.norm1b), residual_, l.ff ? &norm2 : after, x_, ld_x_, act_, s);
+    ctx.mark("residual_norm");
+    if (!l.ff) continue;
+    gemm(ctx, x_, ld_x_, m, W.glu, glu, ff_, ld_ff_);
+    ctx.mark("gemm.mlp_gate_up");
+    gemm(ctx, ff_, ld_ff_, m, W.down, Q38_DENSE_STORE_F32, y_, ld_x_);
+    ctx.mark("gemm.mlp_down");
+    kernels::residual_norm(y_, ld_x_, m, H, norm(W.norm2b), residual_, after, x_, ld_x_, act_, s);
+    ctx.mark("residual_norm");
+  }
+}
+
+void LayerListModel::head(const StepContext& ctx, const HeadRows& rows, float* logits) {
+  kernels::gather_norm(residual_, rows.rows, rows.first, rows.count, cfg_.hidden_size, norm(final_norm_), head_x_, ld_x_, act_,
+                       ctx.stream);
+  gemm(ctx, head_x_, ld_x_, rows.count, head_, Q38_DENSE_STORE_F32, logits, cfg_.vocab_size);
+  ctx.mark("gemm.lm_head");
+}
+
+}  // namespace
+
+std::unique_ptr<StepModel> make_layer_list_model(const ModelFile& file, const RunnerOptions& options,
+                                                 const LayerListDesign& design) {
+  return std::make_unique<LayerListModel>(file, options, design);
+}
+
+void check_layer_list_tensors(const ModelFile& file, const LayerListDesign& design) {
+  const ModelConfig& c = file.config();
+  const TensorReader r(file);
+  const int64_t W = c.hidden_size, V = c.vocab_size;
+  const std::vector<int64_t> gain = design.norm_gain_is_scalar ? std::vector<int64_t>{} : std::vector<int64_t>{W};
+  r.require("embed", {V, W});
+  if (c.learned_positions) r.require("pos", {c.max_position_embeddings, W});
+  r.require("final.norm", gain);
+  r.require("head", {V, W});
+  for (int i = 0; i < c.num_layers; ++i) {
+    const LayerSpec& l = c.layers[size_t(i)];
+    auto linear = [&](const char* name, int64_t n, int64_t k, bool bias) {
+      r.require(mix(i, name), {n, k});
+      if (bias) r.require(mix(i, (std::string(name) + ".b").c_str()), {n});
+    };
+    r.require(at_layer(i, "norm1"), gain);
+    r.require(at_layer(i, "norm1b"), gain);
+    if (l.ff) {
+      r.require(at_layer(i, "norm2"), gain);
+      r.require(at_layer(i, "norm2b"), gain);
+      r.require(at_layer(i, "mlp.gate"), {l.ff, W});
+      r.require(at_layer(i, "mlp.up"), {l.ff, W});
+      r.require(at_layer(i, "mlp.down"), {W, l.ff});
+    }
+    if (l.mixer == MixerKind::Attention) {
+      const AttentionSpec& a = l.attn;
+      linear("q", int64_t(a.heads) * a.dim, W, true);
+      linear("k", int64_t(a.kv_heads) * a.dim, W, true);
+      linear("v", int64_t(a.kv_heads) * a.vdim, W, true);
+      linear("o", W, int64_t(a.heads) * a.vdim, true);
+      if (a.head_mix) r.require(mix(i, "talk"), {a.heads, a.heads});
+      if (a.value_mix) r.require(mix(i, "vmix"), {});
+    } else if (l.mixer == MixerKind::MinGru) {
+      linear("z", l.rec.width, W, true);
+      linear("x", l.rec.width, W, true);
+      linear("g", l.rec.width, W, false);
+      linear("o", W, l.rec.width, false);
+    } else {
+      const int64_t w = l.rec.width, nb = l.rec.blocks, bs = w / nb;
+      linear("y", w, W, true);
+      linear("x", w, W, true);
+      r.require(mix(i, "conv"), {w, l.rec.taps});
+      r.require(mix(i, "conv.b"), {w});
+      for (const char* g : {"ra", "ri"}) {
+        r.require(mix(i, g), {nb, bs, bs});
+        r.require(mix(i, (std::string(g) + ".b").c_str()), {nb, bs});
+      }
+      r.require(mix(i, "lam"), {w});
+      linear("o", W, w, false);
+    }
+  }
+}
+
+}  // namespace qwen38

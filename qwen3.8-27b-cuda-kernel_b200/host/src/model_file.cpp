@@ -8,9 +8,9 @@
 
 #include <cstdio>
 #include <fstream>
+#include <iterator>
 
-#include "json_min.h"
-#include "qwen38/api.h"
+#include "step_model.h"
 
 namespace qwen38 {
 
@@ -69,6 +69,10 @@ int ModelConfig::gdn_index(int layer) const {
 }
 
 void ModelConfig::validate() const {
+  if (!layers.empty()) {  // a layer-list architecture: its reader has checked the sizes of every layer
+    QWEN38_CHECK(int(layers.size()) == num_layers && hidden_size > 0 && vocab_size > 0, "layer list");
+    return;
+  }
   QWEN38_CHECK(num_layers > 0 && int(is_attention.size()) == num_layers, "layer_types size");
   QWEN38_CHECK(hidden_size > 0 && hidden_size % 128 == 0, "hidden_size must be a multiple of 128, got ", hidden_size);
   QWEN38_CHECK(vocab_size > 0 && vocab_size % 128 == 0, "vocab_size must be a multiple of 128, got ", vocab_size);
@@ -90,6 +94,13 @@ void ModelConfig::validate() const {
 
 std::string ModelConfig::summary() const {
   std::ostringstream os;
+  if (!layers.empty()) {
+    int kinds[3] = {0, 0, 0};
+    for (const LayerSpec& l : layers) ++kinds[int(l.mixer)];
+    os << architecture << ": hidden " << hidden_size << ", layers " << num_layers << " (" << kinds[0] << " attention / "
+       << kinds[1] << " minGRU / " << kinds[2] << " RG-LRU), vocab " << vocab_size;
+    return os.str();
+  }
   os << "hidden " << hidden_size << ", layers " << num_layers << " (" << num_attention_layers() << " attention / "
      << num_gdn_layers() << " GDN), vocab " << vocab_size << ", ffn " << intermediate_size << ", attn "
      << num_attention_heads << "q/" << num_key_value_heads << "kv x" << head_dim << ", gdn " << linear_num_key_heads
@@ -99,7 +110,7 @@ std::string ModelConfig::summary() const {
 
 // ---- model file -----------------------------------------------------------------------------------
 const char* dtype_name(DType dtype) {
-  constexpr const char* kNames[] = {"bq4", "bq5", "bq6", "bq8", "bf16", "f32"};
+  constexpr const char* kNames[] = {"bq4", "bq5", "bq6", "bq8", "bf16", "f32", "i32"};
   return kNames[int(dtype)];
 }
 
@@ -152,6 +163,11 @@ int64_t TensorInfo::numel() const {
 std::unique_ptr<ModelFile> ModelFile::open(const std::string& path) {
   std::unique_ptr<ModelFile> mf(new ModelFile());
   mf->path_ = path;
+  struct stat st{};
+  if (::stat(path.c_str(), &st) == 0 && S_ISDIR(st.st_mode)) {
+    mf->open_folder(path);
+    return mf;
+  }
   {
     std::ifstream in(path, std::ios::binary);
     QWEN38_CHECK(in.good(), "cannot open ", path);
@@ -214,12 +230,7 @@ std::unique_ptr<ModelFile> ModelFile::open(const std::string& path) {
     fail(path + ": malformed header: " + e.what());
   }
 
-  mf->fd_ = ::open(path.c_str(), O_RDONLY);
-  QWEN38_CHECK(mf->fd_ >= 0, "cannot open ", path);
-  void* p = ::mmap(nullptr, mf->file_size_, PROT_READ, MAP_PRIVATE, mf->fd_, 0);
-  QWEN38_CHECK(p != MAP_FAILED, "mmap failed for ", path);
-  mf->base_ = static_cast<const uint8_t*>(p);
-  mf->mapped_size_ = mf->file_size_;
+  mf->map(path);
 
   // every object must lie inside the file (catches truncated copies)
   for (const auto& [name, t] : mf->tensors_) {
@@ -237,6 +248,76 @@ std::unique_ptr<ModelFile> ModelFile::open(const std::string& path) {
   }
   mf->config_.validate();
   return mf;
+}
+
+void ModelFile::map(const std::string& path) {
+  fd_ = ::open(path.c_str(), O_RDONLY);
+  QWEN38_CHECK(fd_ >= 0, "cannot open ", path);
+  void* p = ::mmap(nullptr, file_size_, PROT_READ, MAP_PRIVATE, fd_, 0);
+  QWEN38_CHECK(p != MAP_FAILED, "mmap failed for ", path);
+  base_ = static_cast<const uint8_t*>(p);
+  mapped_size_ = file_size_;
+}
+
+// A model folder: config.json, whose "architecture" names the registered reader of the rest, and model.safetensors
+// (8-byte little-endian header length, JSON header name -> {dtype, shape, data_offsets}, tensor data).
+void ModelFile::open_folder(const std::string& path) {
+  const std::string config_path = path + "/config.json", data_path = path + "/model.safetensors";
+  std::ifstream cin(config_path, std::ios::binary);
+  QWEN38_CHECK(cin.good(), "cannot open ", config_path);
+  header_.assign(std::istreambuf_iterator<char>(cin), std::istreambuf_iterator<char>());
+  const Architecture* arch = nullptr;
+  try {
+    const jsonmin::Value j = jsonmin::parse(header_);
+    arch = &find_architecture(j.at("architecture").as_string());
+    QWEN38_CHECK(arch->read_config != nullptr, "architecture ", arch->name, " is read from .q38 files, not from a folder");
+    config_ = arch->read_config(j);
+    config_.architecture = arch->name;
+  } catch (const Error&) {
+    throw;
+  } catch (const std::exception& e) {
+    fail(config_path + ": malformed configuration: " + e.what());
+  }
+  std::ifstream in(data_path, std::ios::binary);
+  QWEN38_CHECK(in.good(), "cannot open ", data_path);
+  uint64_t header_len = 0;
+  in.read(reinterpret_cast<char*>(&header_len), 8);
+  QWEN38_CHECK(in.good() && header_len > 0 && header_len < (1ull << 30), data_path, ": bad header length");
+  std::string head(header_len, '\0');
+  in.read(head.data(), std::streamsize(header_len));
+  QWEN38_CHECK(in.good(), data_path, ": truncated header");
+  in.seekg(0, std::ios::end);
+  file_size_ = uint64_t(in.tellg());
+  data_start_ = 8 + header_len;
+  try {
+    const jsonmin::Value j = jsonmin::parse(head);
+    for (const auto& [name, rec] : j.obj) {
+      if (name == "__metadata__") continue;
+      TensorInfo t;
+      t.name = name;
+      const std::string& dtype = rec.at("dtype").as_string();
+      if (dtype == "BF16") t.dtype = DType::BF16;
+      else if (dtype == "F32") t.dtype = DType::F32;
+      else if (dtype == "I32") t.dtype = DType::I32;
+      else fail(data_path + ": tensor '" + name + "' has dtype " + dtype + " (BF16, F32 and I32 are read)");
+      for (const auto& d : rec.at("shape").arr) t.shape.push_back(d.as_int());
+      t.rows = t.shape.empty() ? 1 : t.shape[0];
+      const auto& span = rec.at("data_offsets").arr;
+      t.offset = span.at(0).as_int();
+      t.bytes = span.at(1).as_int() - t.offset;
+      QWEN38_CHECK(t.bytes == t.numel() * (t.dtype == DType::BF16 ? 2 : 4), name, ": size mismatch");
+      QWEN38_CHECK(t.offset >= 0 && data_start_ + uint64_t(t.offset + t.bytes) <= file_size_, name,
+                   ": object outside the file (truncated download?)");
+      tensors_.emplace(name, std::move(t));
+    }
+  } catch (const Error&) {
+    throw;
+  } catch (const std::exception& e) {
+    fail(data_path + ": malformed header: " + e.what());
+  }
+  map(data_path);
+  config_.validate();
+  if (arch->check_tensors) arch->check_tensors(*this);
 }
 
 ModelFile::~ModelFile() {

@@ -9,20 +9,14 @@
 #include <algorithm>
 #include <iostream>
 
-#include "qwen38/api.h"
+#include "step_model.h"
 
 namespace qwen38 {
 
 namespace {
 
 constexpr size_t kMiB = 1024 * 1024;
-constexpr int kMaxSplits = 64;
-// From this run length on, a step's GDN layers use the chunked recurrence: a 64-token chunk costs about as much as
-// a dozen sequential token updates.
-constexpr int kGdnChunkedMinRun = 16;
 constexpr int kBuckets[] = {1, 2, 4, 8, 12, 16, 24, 32, 48, 64, 96, 128, 192, 256};
-
-size_t up256(size_t x) { return (x + 255) / 256 * 256; }
 
 std::string mib(size_t bytes) { return std::to_string((bytes + kMiB / 2) / kMiB) + " MiB"; }
 
@@ -96,40 +90,20 @@ struct ModelRunner::Impl {
   RunnerOptions opt;
   DeviceInfo dev;
   MemoryPlan plan;
-  std::unique_ptr<ModelWeights> weights;
+  std::unique_ptr<StepModel> model;
   std::unique_ptr<KvCache> kv;
-  std::unique_ptr<GdnStatePool> state;
-  Stream stream;
-  // side branch of the step: the a/b gate projection of a GDN layer needs only the layer's input, so it runs beside
-  // the layer's (much larger) in-projection GEMM; fork / join events make it a parallel branch of the captured graph
-  Stream side;
-  Event fork_ev, join_ev;
+  Stream stream, side;
+  StepContext ctx;
   DeviceArena ws;
-  int max_tokens = 0, max_rows = 0, dummy_slot = 0, proj_ld = 0;
+  int max_tokens = 0, max_rows = 0, dummy_slot = 0;
 
-  // activations
-  float* residual = nullptr;
-  __nv_bfloat16* xbf = nullptr;
-  float* partials = nullptr;
-  __nv_bfloat16* proj = nullptr;
-  float* ab = nullptr;
-  float* qkv = nullptr;
-  __nv_bfloat16* mixer = nullptr;
-  __nv_bfloat16* act = nullptr;
-  __half* q16 = nullptr;
   float* logits = nullptr;
-  float* split = nullptr;
   float* logprob_rows = nullptr;
-  __nv_bfloat16* lm_x = nullptr;   // gathered rows for the LM head of ragged prefill steps
-  float* lm_partials = nullptr;
-  kernels::GemmWorkspace gemm_ws;
-  float* gdn_scratch = nullptr;    // chunked GDN recurrence (prefill): per-chunk U0 / W / P
-  size_t gdn_scratch_floats = 0;
   int32_t* history = nullptr;
   int* history_len = nullptr;
   int32_t* tokens_out = nullptr;
   float* logprob_out = nullptr;
-  int32_t* targets = nullptr;
+  int32_t* targets = nullptr;   // per token row: scoring targets, or the rows whose logits are wanted
 
   MetaMap meta;
   uint8_t* meta_dev = nullptr;
@@ -221,7 +195,10 @@ struct ModelRunner::Impl {
   // the rest of the batch are single-token rows (a pure decode step has multi_seqs == 0, a pure prefill step none of
   // the latter)
   void forward(int m, const kernels::BatchDesc& batch, bool decode, int multi_seqs = -1, int multi_tokens = 0);
-  void lm_head(const __nv_bfloat16* x, const float* part, int rows);
+  void head(const HeadRows& rows) {
+    if (rows.count > 0) model->head(ctx, rows, logits);
+  }
+  void carve(Workspace& w);
   void run_sampler(int rows);
   void download(int rows) {
     QWEN38_CUDA(cudaMemcpyAsync(out_host.get(), tokens_out, size_t(rows) * 4, cudaMemcpyDeviceToHost, stream.get()));
@@ -250,7 +227,7 @@ struct ModelRunner::Impl {
     const auto batch = batch_desc(bucket, bucket, 1);
     pack(bucket, bucket);
     forward(bucket, batch, true);
-    lm_head(xbf, partials, bucket);
+    head({nullptr, 0, bucket});
     run_sampler(bucket);
     collect_status();
   }
@@ -264,90 +241,59 @@ void ModelRunner::Impl::setup() {
               << dev.sm_major << dev.sm_minor << ")\n";
   }
   if (opt.embedding == EmbeddingPlacement::Host && !dev.can_map_host) opt.embedding = EmbeddingPlacement::Device;
-  const int H = cfg.hidden_size, V = cfg.vocab_size;
   QWEN38_CHECK(opt.max_batch > 0, "max_batch must be positive");
   QWEN38_CHECK(opt.prefill_chunk >= 64 && opt.prefill_chunk % 64 == 0, "prefill chunk must be a multiple of 64");
+  if (cfg.learned_positions) opt.max_context = std::min(opt.max_context, cfg.max_position_embeddings);
   max_rows = opt.max_batch + 1;
   dummy_slot = opt.max_batch;
   max_tokens = std::max(opt.prefill_chunk, max_rows);
+  model = find_architecture(cfg.architecture).make(file, opt);
+  opt.kv_dtype = model->resolve_kv_dtype(opt.kv_dtype);
+  ctx.stream = stream.get();
+  ctx.side = side.get();
+  ctx.num_sms = dev.num_sms;
+  ctx.max_tokens = max_tokens;
+  ctx.max_rows = max_rows;
+  ctx.mark = [this](const char* name) { mark(name); };
 
   plan.free_at_start = dev.free_mem;
-  plan.weights = ModelWeights::required_device_bytes(file, opt.embedding);
-  if (opt.embedding == EmbeddingPlacement::Host) plan.embedding_host = size_t(file.tensor("embed").bytes);
-  proj_ld = 0;
-  for (int i = 0; i < cfg.num_layers; ++i) {
-    const std::string name = std::to_string(i) + (cfg.is_attention[size_t(i)] ? ".attn.qkvg" : ".gdn.qkvz");
-    proj_ld = std::max(proj_ld, int(file.tensor(name).shape[0]));
-  }
-  const size_t T = size_t(max_tokens), R = size_t(max_rows);
-  const size_t mixer_w = size_t(std::max(cfg.q_dim(), cfg.gdn_value_dim()));
-  const size_t nv2 = 2 * size_t(std::max(1, cfg.linear_num_value_heads));
-  const size_t gemm_partials = size_t(2) * size_t(dev.num_sms) * 128 * 512;  // stream-K partial tiles of a 512-token pass
+  plan.weights = model->weight_bytes();
+  plan.embedding_host = model->host_weight_bytes();
   meta = MetaMap(max_tokens, max_rows);
-  gdn_scratch_floats = cfg.linear_num_value_heads > 0 && max_tokens >= kGdnChunkedMinRun
-                           ? kernels::gdn_chunk_scratch_floats(max_tokens, max_rows, cfg.linear_num_value_heads)
-                           : 0;
-  const size_t sizes[] = {
-      T * H * 4, T * H * 2, T * size_t(cfg.norm_blocks()) * 4, T * size_t(proj_ld) * 2, T * nv2 * 4,
-      T * size_t(std::max(128, cfg.gdn_conv_dim())) * 4, T * mixer_w * 2, T * size_t(cfg.intermediate_size) * 2,
-      T * size_t(std::max(256, cfg.q_dim())) * 2, R * size_t(V) * 4,
-      R * size_t(std::max(1, cfg.num_attention_heads)) * kMaxSplits * (kernels::kHeadDim + 2) * 4, T * 4,
-      R * size_t(H) * 2, R * size_t(cfg.norm_blocks()) * 4, gemm_partials * 4, 65536 * 4,
-      R * size_t(opt.history_cap) * 4, R * 4, R * 4, R * 4, T * 4, meta.bytes, gdn_scratch_floats * 4};
-  size_t w = 4096;
-  for (size_t s : sizes) w += up256(s);
-  plan.workspace = w;
-  plan.state = GdnStatePool::bytes_per_slot(cfg) * R;
+  Workspace count;
+  carve(count);
+  plan.workspace = count.bytes + 4096;
+  plan.state = model->state_bytes_per_slot() * size_t(max_rows);
   plan.reserve = opt.reserve_mib * kMiB;
-  const size_t page_bytes = std::max<size_t>(KvCache::page_bytes_all_layers(cfg, opt.kv_dtype), 1);
+  const size_t page_bytes = std::max<size_t>(model->kv_page_bytes(opt.kv_dtype), 1);
   const size_t fixed = plan.weights + plan.workspace + plan.state + plan.reserve;
   QWEN38_CHECK(plan.free_at_start > fixed + 2 * page_bytes, "not enough GPU memory: need ", (fixed + 2 * page_bytes) / kMiB,
                " MiB before any KV cache, ", plan.free_at_start / kMiB, " MiB free");
   int64_t pages = int64_t((plan.free_at_start - fixed) / page_bytes);
+  const int max_pages_per_seq = int(ceil_div(opt.max_context, kernels::kPageTokens));
   if (opt.kv_tokens > 0) pages = std::min<int64_t>(pages, ceil_div(opt.kv_tokens, kernels::kPageTokens) + 1);
+  // more pages than every slot can hold at its longest context are of no use
+  pages = std::min<int64_t>(pages, int64_t(opt.max_batch) * max_pages_per_seq + 1);
   pages = std::min<int64_t>(pages, 1 << 22);
   plan.kv_pages = int(pages);
   plan.kv = size_t(pages) * page_bytes;
   plan.kv_tokens = (pages - 1) * kernels::kPageTokens;  // one page belongs to the dummy sequence
 
-  weights = std::make_unique<ModelWeights>(file, opt.embedding);
-  const int max_pages_per_seq = int(ceil_div(opt.max_context, kernels::kPageTokens));
-  kv = std::make_unique<KvCache>(cfg, opt.kv_dtype, plan.kv_pages, max_rows, max_pages_per_seq);
+  model->load_weights();
+  kv = model->make_kv(opt.kv_dtype, plan.kv_pages, max_rows, max_pages_per_seq);
+  ctx.kv = kv.get();
   QWEN38_CHECK(kv->ensure(dummy_slot, 1), "KV cache too small");
-  state = std::make_unique<GdnStatePool>(cfg, max_rows);
+  model->make_state(max_rows);
 
   ws = DeviceArena(plan.workspace);
-  residual = ws.allocate_array<float>(T * H);
-  xbf = ws.allocate_array<__nv_bfloat16>(T * H);
-  partials = ws.allocate_array<float>(T * size_t(cfg.norm_blocks()));
-  proj = ws.allocate_array<__nv_bfloat16>(T * size_t(proj_ld));
-  ab = ws.allocate_array<float>(T * nv2);
-  qkv = ws.allocate_array<float>(T * size_t(std::max(128, cfg.gdn_conv_dim())));
-  mixer = ws.allocate_array<__nv_bfloat16>(T * mixer_w);
-  act = ws.allocate_array<__nv_bfloat16>(T * size_t(cfg.intermediate_size));
-  q16 = ws.allocate_array<__half>(T * size_t(std::max(256, cfg.q_dim())));
-  logits = ws.allocate_array<float>(R * size_t(V));
-  split = ws.allocate_array<float>(R * size_t(std::max(1, cfg.num_attention_heads)) * kMaxSplits * (kernels::kHeadDim + 2));
-  logprob_rows = ws.allocate_array<float>(T);
-  lm_x = ws.allocate_array<__nv_bfloat16>(R * size_t(H));
-  lm_partials = ws.allocate_array<float>(R * size_t(cfg.norm_blocks()));
-  gemm_ws.partials = ws.allocate_array<float>(gemm_partials);
-  gemm_ws.partial_floats = gemm_partials;
-  gemm_ws.counters = ws.allocate_array<int>(65536);
-  if (gdn_scratch_floats) gdn_scratch = ws.allocate_array<float>(gdn_scratch_floats);
-  gemm_ws.num_counters = 65536;
-  history = ws.allocate_array<int32_t>(R * size_t(opt.history_cap));
-  history_len = ws.allocate_array<int>(R);
-  tokens_out = ws.allocate_array<int32_t>(R);
-  logprob_out = ws.allocate_array<float>(R);
-  targets = ws.allocate_array<int32_t>(T);
-  meta_dev = static_cast<uint8_t*>(ws.allocate(meta.bytes));
-  QWEN38_CUDA(cudaMemset(gemm_ws.counters, 0, 65536 * 4));
-  QWEN38_CUDA(cudaMemset(history_len, 0, R * 4));
-  QWEN38_CUDA(cudaMemset(meta_dev, 0, meta.bytes));
+  QWEN38_CUDA(cudaMemset(ws.base(), 0, ws.capacity()));  // counters, metadata, row padding
+  Workspace hand_out;
+  hand_out.arena = &ws;
+  carve(hand_out);
+  model->prepare(ctx);
   meta_host = PinnedBuffer(meta.host_bytes, false);
   std::memset(meta_host.get(), 0, meta.host_bytes);
-  out_host = PinnedBuffer(R * 8, false);
+  out_host = PinnedBuffer(size_t(max_rows) * 8, false);
   status_host = PinnedBuffer(64, true);
   std::memset(status_host.get(), 0, 64);
   status_dev = static_cast<unsigned int*>(status_host.device_ptr());
@@ -358,155 +304,37 @@ void ModelRunner::Impl::setup() {
   if (opt.verbose) std::cerr << "qwen38: " << plan.describe() << "\n";
 }
 
-// The kernel sequence of one step over m tokens (reference src/model_runner.cpp:292-410).
+// The step's activation memory: the model's, then the sampler's and the metadata block.
+void ModelRunner::Impl::carve(Workspace& w) {
+  const size_t T = size_t(max_tokens), R = size_t(max_rows);
+  model->carve(w, ctx);
+  logits = w.take<float>(R * size_t(cfg.vocab_size));
+  logprob_rows = w.take<float>(T);
+  history = w.take<int32_t>(R * size_t(opt.history_cap));
+  history_len = w.take<int>(R);
+  tokens_out = w.take<int32_t>(R);
+  logprob_out = w.take<float>(R);
+  targets = w.take<int32_t>(T);
+  meta_dev = w.take<uint8_t>(meta.bytes);
+}
+
 void ModelRunner::Impl::forward(int m, const kernels::BatchDesc& batch, bool decode, int multi_seqs, int multi_tokens) {
-  cudaStream_t s = stream.get();
   if (multi_seqs < 0 || multi_seqs >= batch.num_seqs) {  // not a mixed step
     multi_seqs = decode ? 0 : batch.num_seqs;
     multi_tokens = decode ? 0 : m;
   }
   const int single_seqs = batch.num_seqs - multi_seqs;  // rows of one token each, placed after the chunk rows
-  const bool mixed = multi_seqs > 0 && single_seqs > 0;
-  const kernels::BatchDesc chunk_part = mixed ? sub_batch(0, 0, multi_seqs, multi_tokens, batch.max_tokens_per_seq) : batch;
-  const kernels::BatchDesc single_part =
-      mixed ? sub_batch(multi_seqs, multi_tokens, single_seqs, single_seqs, 1) : batch;
-  const int H = cfg.hidden_size;
-  const float eps = cfg.rms_norm_eps;
-  const kernels::KvCacheDesc kvd = kv->desc();
-  const kernels::GdnStateDesc sd = state->desc();
-  kernels::GdnDims gd;
-  gd.num_k_heads = cfg.linear_num_key_heads;
-  gd.num_v_heads = cfg.linear_num_value_heads;
-  gd.conv_dim = cfg.gdn_conv_dim();
-  gd.ld_proj = proj_ld;
-
+  StepBatch b;
+  b.tokens = dmeta<int32_t>(meta.tokens);
+  b.m = m;
+  b.decode = decode;
+  b.mixed = multi_seqs > 0 && single_seqs > 0;
+  b.all = batch;
+  b.chunk_part = b.mixed ? sub_batch(0, 0, multi_seqs, multi_tokens, batch.max_tokens_per_seq) : batch;
+  b.single_part = b.mixed ? sub_batch(multi_seqs, multi_tokens, single_seqs, single_seqs, 1) : batch;
+  ctx.profiling = profiling;
   mark("start");
-  kernels::embed(weights->embedding(), dmeta<int32_t>(meta.tokens), m, H, residual, xbf, partials, s);
-  mark("embed");
-
-  kernels::GemmEpilogue into_residual;
-  into_residual.kind = kernels::Epilogue::Residual;
-  into_residual.residual = residual;
-  into_residual.xbf = xbf;
-  into_residual.partials_out = partials;
-
-  int attn_i = 0, gdn_i = 0;
-  for (const LayerWeights& W : weights->layers()) {
-    kernels::GemmEpilogue in;
-    in.kind = kernels::Epilogue::StoreBF16;
-    in.out = proj;
-    in.ldo = proj_ld;
-    in.n_store = W.in_proj.rows;
-    in.partials_in = partials;
-    in.hidden = H;
-    in.eps = eps;
-    const bool side_ab = !W.attention && !profiling;  // the per-op profile keeps everything on one stream
-    if (side_ab) {
-      fork_ev.record(s);
-      QWEN38_CUDA(cudaStreamWaitEvent(side.get(), fork_ev.get(), 0));
-      kernels::gdn_ab(xbf, m, H, W.ab, W.ab_rows, partials, eps, ab, side.get());
-      join_ev.record(side.get());
-    }
-    kernels::qgemm(xbf, m, W.in_proj, in, gemm_ws, s);
-    mark(W.attention ? "gemm.attn_qkvg" : "gemm.gdn_qkvz");
-    if (W.attention) {
-      kernels::QkNormRopeParams qp;
-      qp.proj = proj;
-      qp.ld_proj = proj_ld;
-      qp.q_norm = W.q_norm;
-      qp.k_norm = W.k_norm;
-      qp.eps = eps;
-      qp.rope_theta = float(cfg.rope_theta);
-      qp.num_q_heads = cfg.num_attention_heads;
-      qp.num_kv_heads = cfg.num_key_value_heads;
-      qp.q_out = q16;
-      qp.attn_layer = attn_i;
-      kernels::qk_norm_rope_append(qp, batch, kvd, s);
-      mark("attn.qk_norm_rope_kv");
-      kernels::AttentionParams ap;
-      ap.q = q16;
-      ap.gate = proj + cfg.q_dim();
-      ap.ld_gate = proj_ld;
-      ap.out = mixer;
-      ap.num_q_heads = cfg.num_attention_heads;
-      ap.num_kv_heads = cfg.num_key_value_heads;
-      ap.attn_layer = attn_i;
-      ap.split_scratch = split;
-      ap.max_splits = kMaxSplits;
-      if (decode) {
-        kernels::attention_decode(ap, batch, kvd, s);
-      } else if (mixed) {
-        // chunk rows through the query-tiled kernel (no key split: the scratch serves the single-token rows), the
-        // single-token rows through split-KV flash decoding
-        kernels::attention_decode(ap, single_part, kvd, s);
-        ap.split_scratch = nullptr;
-        kernels::attention_prefill(ap, chunk_part, kvd, s);
-      } else {  // the scratch of max_rows x kMaxSplits states seen as one row per prompt token of this step
-        ap.max_splits = std::min(kMaxSplits, int(size_t(max_rows) * kMaxSplits / size_t(std::max(1, m))));
-        ap.scratch_rows = ap.max_splits > 1 ? m : 0;
-        kernels::attention_prefill(ap, batch, kvd, s);
-      }
-      mark(decode ? "attn.decode" : "attn.prefill");
-      ++attn_i;
-    } else {
-      if (side_ab) QWEN38_CUDA(cudaStreamWaitEvent(s, join_ev.get(), 0));
-      else kernels::gdn_ab(xbf, m, H, W.ab, W.ab_rows, partials, eps, ab, s);
-      mark("gdn.ab");
-      kernels::GdnConvParams cp;
-      cp.proj = proj;
-      cp.conv_w = W.conv;
-      cp.qkv = qkv;
-      cp.gdn_layer = gdn_i;
-      kernels::gdn_conv(cp, gd, batch, sd, s);
-      mark("gdn.conv");
-      kernels::GdnRecurrenceParams rp;
-      rp.qkv = qkv;
-      rp.ab = ab;
-      rp.A = W.A;
-      rp.dt_bias = W.dt_bias;
-      rp.z = proj + cfg.gdn_conv_dim();
-      rp.ld_z = proj_ld;
-      rp.norm_w = W.gdn_norm;
-      rp.eps = eps;
-      rp.out = mixer;
-      rp.gdn_layer = gdn_i;
-      // runs of prefill length take the chunked form (token-parallel preparation + per-chunk state scan)
-      if (gdn_scratch && chunk_part.max_tokens_per_seq >= kGdnChunkedMinRun)
-        kernels::gdn_recurrence_chunked(rp, gd, chunk_part, sd, gdn_scratch, gdn_scratch_floats, s);
-      else
-        kernels::gdn_recurrence(rp, gd, chunk_part, sd, s);
-      if (mixed) kernels::gdn_recurrence(rp, gd, single_part, sd, s);  // the state-streaming decode kernel
-      mark("gdn.recurrence");
-      ++gdn_i;
-    }
-    kernels::qgemm(mixer, m, W.out_proj, into_residual, gemm_ws, s);
-    mark(W.attention ? "gemm.attn_o" : "gemm.gdn_out");
-
-    kernels::GemmEpilogue mlp;
-    mlp.kind = kernels::Epilogue::SwiGLU;
-    mlp.out = act;
-    mlp.ldo = cfg.intermediate_size;
-    mlp.partials_in = partials;
-    mlp.hidden = H;
-    mlp.eps = eps;
-    kernels::qgemm(xbf, m, W.gate_up, mlp, gemm_ws, s);
-    mark("gemm.mlp_gate_up");
-    kernels::qgemm(act, m, W.down, into_residual, gemm_ws, s);
-    mark("gemm.mlp_down");
-  }
-}
-
-void ModelRunner::Impl::lm_head(const __nv_bfloat16* x, const float* part, int rows) {
-  if (rows <= 0) return;
-  kernels::GemmEpilogue head;
-  head.kind = kernels::Epilogue::StoreF32;
-  head.out = logits;
-  head.ldo = cfg.vocab_size;
-  head.partials_in = part;
-  head.hidden = cfg.hidden_size;
-  head.eps = cfg.rms_norm_eps;
-  kernels::qgemm(x, rows, weights->lm_head(), head, gemm_ws, stream.get());
-  mark("gemm.lm_head");
+  model->forward(ctx, b);
 }
 
 void ModelRunner::Impl::run_sampler(int rows) {
@@ -538,9 +366,17 @@ const MemoryPlan& ModelRunner::memory() const { return impl_->plan; }
 const DeviceInfo& ModelRunner::device() const { return impl_->dev; }
 int ModelRunner::num_slots() const { return impl_->opt.max_batch; }
 KvCache& ModelRunner::kv() { return *impl_->kv; }
-const ModelWeights& ModelRunner::weights() const { return *impl_->weights; }
+const ModelWeights& ModelRunner::weights() const {
+  const ModelWeights* w = impl_->model->bq_weights();
+  QWEN38_CHECK(w != nullptr, impl_->cfg.architecture, " has no BQ weights");
+  return *w;
+}
 cudaStream_t ModelRunner::stream() const { return impl_->stream.get(); }
-const kernels::GemmWorkspace& ModelRunner::gemm_workspace() const { return impl_->gemm_ws; }
+const kernels::GemmWorkspace& ModelRunner::gemm_workspace() const {
+  const kernels::GemmWorkspace* w = impl_->model->gemm_workspace();
+  QWEN38_CHECK(w != nullptr, impl_->cfg.architecture, " has no GEMM workspace");
+  return *w;
+}
 void ModelRunner::set_profiling(bool on) { impl_->profiling = on; }
 const OpProfile& ModelRunner::profile() const { return impl_->prof; }
 void ModelRunner::clear_profile() { impl_->prof = OpProfile{}; }
@@ -554,7 +390,7 @@ float ModelRunner::last_step_device_ms() const {
 
 void ModelRunner::reset_slot(int slot) {
   QWEN38_CHECK(slot >= 0 && slot < impl_->opt.max_batch, "reset_slot: slot out of range");
-  impl_->state->reset(slot, impl_->stream.get());
+  impl_->model->reset_slot(slot, impl_->stream.get());
   QWEN38_CUDA(cudaMemsetAsync(impl_->history_len + slot, 0, sizeof(int), impl_->stream.get()));
 }
 
@@ -575,7 +411,7 @@ StepResult ModelRunner::prefill(int slot, int pos0, std::span<const int32_t> tok
   return prefill_batch(std::span<const PrefillRow>(&row, 1));
 }
 
-StepResult ModelRunner::prefill_batch(std::span<const PrefillRow> rows) {
+StepResult ModelRunner::prefill_batch(std::span<const PrefillRow> rows, std::span<const LogitsAt> want) {
   Impl& I = *impl_;
   const int nseq = int(rows.size());
   QWEN38_CHECK(nseq > 0 && nseq <= I.opt.max_batch, "prefill: ", nseq, " sequences in one step (max ", I.opt.max_batch, ")");
@@ -630,24 +466,38 @@ StepResult ModelRunner::prefill_batch(std::span<const PrefillRow> rows) {
   I.forward(total, I.batch_desc(nseq, total, longest), false, multi_seqs, multi_tokens);
   StepResult result;
   if (samples > 0) {
-    const int H = I.cfg.hidden_size, nb = I.cfg.norm_blocks();
-    if (samples == 1) {
-      const int row = I.hmeta<int>(I.meta.sample_row)[0];
-      I.lm_head(I.xbf + size_t(row) * H, I.partials + size_t(row) * nb, 1);
-    } else {
-      kernels::gather_rows(I.xbf, I.partials, I.dmeta<int>(I.meta.sample_row), samples, H, I.lm_x, I.lm_partials, s);
-      I.lm_head(I.lm_x, I.lm_partials, samples);
-    }
+    if (samples == 1) I.head({nullptr, I.hmeta<int>(I.meta.sample_row)[0], 1});
+    else I.head({I.dmeta<int>(I.meta.sample_row), 0, samples});
     I.run_sampler(samples);
   }
-  I.collect_status();
   I.t_end.record(s);
   I.timed = true;
   if (samples > 0) I.download(samples);
+  std::vector<float> wanted;
+  if (!want.empty()) {  // after the sampler, which may rewrite its logits: each block of rows through the head again
+    const size_t V = size_t(I.cfg.vocab_size);
+    std::vector<int32_t> at;
+    for (const LogitsAt& w : want) {
+      QWEN38_CHECK(w.row >= 0 && w.row < nseq, "prefill: logits of row ", w.row);
+      const int n = int(rows[size_t(w.row)].tokens.size());
+      QWEN38_CHECK(w.index >= 0 && w.index < n, "prefill: logits at token ", w.index, " of ", n);
+      at.push_back(last_token_row[size_t(w.row)] - (n - 1) + w.index);
+    }
+    wanted.resize(at.size() * V);
+    for (size_t r0 = 0; r0 < at.size(); r0 += size_t(I.max_rows)) {
+      const int n = int(std::min<size_t>(size_t(I.max_rows), at.size() - r0));
+      QWEN38_CUDA(cudaMemcpyAsync(I.targets, at.data() + r0, size_t(n) * 4, cudaMemcpyHostToDevice, s));
+      I.head({I.targets, 0, n});
+      QWEN38_CUDA(cudaMemcpyAsync(wanted.data() + r0 * V, I.logits, size_t(n) * V * 4, cudaMemcpyDeviceToHost, s));
+      I.stream.sync();
+    }
+  }
+  I.collect_status();
   I.stream.sync();
   I.collect_marks();
   I.check_status("prefill step");
   if (samples > 0) result = I.results(samples);
+  result.logits = std::move(wanted);
   return result;
 }
 
@@ -725,7 +575,7 @@ std::vector<float> ModelRunner::score(int slot, int pos0, std::span<const int32_
   QWEN38_CHECK(tokens.size() == targets.size(), "score: tokens/targets size");
   std::vector<float> out;
   out.reserve(tokens.size());
-  const int H = I.cfg.hidden_size, nb = I.cfg.norm_blocks(), V = I.cfg.vocab_size;
+  const int V = I.cfg.vocab_size;
   cudaStream_t s = I.stream.get();
   int pos = pos0;
   for (size_t off = 0; off < tokens.size(); off += size_t(I.opt.prefill_chunk)) {
@@ -739,7 +589,7 @@ std::vector<float> ModelRunner::score(int slot, int pos0, std::span<const int32_
     I.forward(n, I.batch_desc(1, n, n), false);
     for (int r0 = 0; r0 < n; r0 += I.max_rows) {
       const int rows = std::min(I.max_rows, n - r0);
-      I.lm_head(I.xbf + size_t(r0) * H, I.partials + size_t(r0) * nb, rows);
+      I.head({nullptr, r0, rows});
       kernels::target_logprobs(I.logits, V, V, I.targets + r0, rows, I.logprob_rows + r0, s);
     }
     std::vector<float> chunk(static_cast<size_t>(n));
@@ -759,7 +609,7 @@ std::vector<float> ModelRunner::prefill_logits(int slot, int pos0, std::span<con
   const int n = int(tokens.size());
   QWEN38_CHECK(n > 0 && n <= I.opt.prefill_chunk, "prefill_logits: chunk size");
   QWEN38_CHECK(I.kv->ensure(slot, pos0 + n), "prefill_logits: KV cache full");
-  const int H = I.cfg.hidden_size, nb = I.cfg.norm_blocks(), V = I.cfg.vocab_size;
+  const int V = I.cfg.vocab_size;
   cudaStream_t s = I.stream.get();
   I.single_chunk_meta(slot, pos0, tokens, nullptr, 0);
   I.kv->sync(s);
@@ -769,7 +619,7 @@ std::vector<float> ModelRunner::prefill_logits(int slot, int pos0, std::span<con
   std::vector<float> out(size_t(n) * size_t(V));
   for (int r0 = 0; r0 < n; r0 += I.max_rows) {
     const int rows = std::min(I.max_rows, n - r0);
-    I.lm_head(I.xbf + size_t(r0) * H, I.partials + size_t(r0) * nb, rows);
+    I.head({nullptr, r0, rows});
     QWEN38_CUDA(cudaMemcpyAsync(out.data() + size_t(r0) * V, I.logits, size_t(rows) * V * 4, cudaMemcpyDeviceToHost, s));
     I.collect_status();
     I.stream.sync();

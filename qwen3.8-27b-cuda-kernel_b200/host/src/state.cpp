@@ -86,18 +86,44 @@ ModelWeights::ModelWeights(const ModelFile& file, EmbeddingPlacement placement)
 }
 
 // ---- KV cache -------------------------------------------------------------------------------------
+size_t KvLayerGeometry::page_bytes(kernels::KvDtype dtype) const {
+  if (k_dim == 0) return kernels::KvCacheDesc::page_bytes_for(dtype, kv_heads);
+  QWEN38_CHECK(dtype == kernels::KvDtype::BF16 || dtype == kernels::KvDtype::F32, "KV cache: int8 pages need head_dim 256");
+  return size_t(kv_heads) * size_t(kernels::kPageTokens) * size_t(k_dim + v_dim) * (dtype == kernels::KvDtype::F32 ? 4 : 2);
+}
+
+namespace {
+std::vector<KvLayerGeometry> fixed_geometry(const ModelConfig& cfg) {
+  return std::vector<KvLayerGeometry>(size_t(cfg.num_attention_layers()), KvLayerGeometry{cfg.num_key_value_heads, 0, 0});
+}
+}  // namespace
+
+size_t KvCache::page_bytes_all_layers(const std::vector<KvLayerGeometry>& layers, kernels::KvDtype dtype) {
+  size_t total = 0;
+  for (const KvLayerGeometry& l : layers) total += l.page_bytes(dtype);
+  return total;
+}
+
 size_t KvCache::page_bytes_all_layers(const ModelConfig& cfg, kernels::KvDtype dtype) {
-  return kernels::KvCacheDesc::page_bytes_for(dtype, cfg.num_key_value_heads) * size_t(cfg.num_attention_layers());
+  return page_bytes_all_layers(fixed_geometry(cfg), dtype);
 }
 
 KvCache::KvCache(const ModelConfig& cfg, kernels::KvDtype dtype, int num_pages, int num_slots, int max_pages_per_seq)
-    : num_pages_(num_pages), num_slots_(num_slots), max_pages_per_seq_(max_pages_per_seq), dtype_(dtype),
-      kv_heads_(cfg.num_key_value_heads) {
+    : KvCache(fixed_geometry(cfg), dtype, num_pages, num_slots, max_pages_per_seq) {
   QWEN38_CHECK(cfg.head_dim == kernels::kHeadDim, "KV cache: head_dim");
+}
+
+KvCache::KvCache(std::vector<KvLayerGeometry> layers, kernels::KvDtype dtype, int num_pages, int num_slots,
+                 int max_pages_per_seq)
+    : num_pages_(num_pages), num_slots_(num_slots), max_pages_per_seq_(max_pages_per_seq), dtype_(dtype),
+      layers_(std::move(layers)) {
   QWEN38_CHECK(num_pages > 0 && num_slots > 0 && max_pages_per_seq > 0, "KV cache: sizes");
-  page_bytes_ = kernels::KvCacheDesc::page_bytes_for(dtype, kv_heads_);
-  layer_stride_ = page_bytes_ * size_t(num_pages);
-  pool_ = DeviceBuffer(layer_stride_ * size_t(std::max(1, cfg.num_attention_layers())));
+  size_t total = 0;
+  for (const KvLayerGeometry& l : layers_) {  // layer-major: all pages of a layer, then the next layer's
+    layer_offset_.push_back(total);
+    total += l.page_bytes(dtype_) * size_t(num_pages);
+  }
+  pool_ = DeviceBuffer(std::max<size_t>(total, 256));
   QWEN38_CUDA(cudaMemset(pool_.get(), 0, pool_.bytes()));
   const size_t table_bytes = size_t(num_slots) * size_t(max_pages_per_seq) * sizeof(int);
   table_dev_ = DeviceBuffer(table_bytes);
@@ -114,10 +140,27 @@ kernels::KvCacheDesc KvCache::desc() const {
   kernels::KvCacheDesc d;
   d.pool = pool_.as<uint8_t>();
   d.dtype = dtype_;
-  d.kv_heads = kv_heads_;
   d.num_pages = num_pages_;
-  d.page_bytes = page_bytes_;
-  d.layer_stride = layer_stride_;
+  if (!layers_.empty()) {
+    d.kv_heads = layers_[0].kv_heads;
+    d.page_bytes = layers_[0].page_bytes(dtype_);
+  }
+  d.layer_stride = d.page_bytes * size_t(num_pages_);
+  d.block_table = table_dev_.as<int>();
+  d.max_pages_per_seq = max_pages_per_seq_;
+  return d;
+}
+
+kernels::KvLayerDesc KvCache::layer_desc(int attn_layer) const {
+  const KvLayerGeometry& l = layers_[size_t(attn_layer)];
+  kernels::KvLayerDesc d;
+  d.pages = pool_.as<uint8_t>() + layer_offset_[size_t(attn_layer)];
+  d.dtype = int(dtype_);
+  d.kv_heads = l.kv_heads;
+  d.k_dim = l.k_dim;
+  d.v_dim = l.v_dim;
+  d.num_pages = num_pages_;
+  d.page_bytes = l.page_bytes(dtype_);
   d.block_table = table_dev_.as<int>();
   d.max_pages_per_seq = max_pages_per_seq_;
   return d;
@@ -189,6 +232,46 @@ void GdnStatePool::reset(int slot, cudaStream_t stream) {
   if (num_gdn_layers_ == 0) return;
   QWEN38_CUDA(cudaMemsetAsync(recurrent_.as<uint8_t>() + recurrent_per_slot_ * size_t(slot), 0, recurrent_per_slot_, stream));
   QWEN38_CUDA(cudaMemsetAsync(conv_.as<uint8_t>() + conv_per_slot_ * size_t(slot), 0, conv_per_slot_, stream));
+}
+
+// ---- elementwise recurrent state ----------------------------------------------------------------------
+namespace {
+// Byte layout of one slot: per layer the fp32 state vector, then the convolution's ring [taps][channels].
+size_t lay_out(const std::vector<RecurrentLayerGeometry>& layers, size_t elem, std::vector<size_t>* state,
+               std::vector<size_t>* conv) {
+  size_t at = 0;
+  for (const RecurrentLayerGeometry& l : layers) {
+    if (state) state->push_back(at);
+    at += padded(int64_t(l.width) * 4);
+    if (conv) conv->push_back(at);
+    at += padded(int64_t(l.taps) * l.channels * int64_t(elem));
+  }
+  return at;
+}
+}  // namespace
+
+size_t RecurrentStatePool::bytes_per_slot(const std::vector<RecurrentLayerGeometry>& layers, size_t conv_elem_bytes) {
+  return lay_out(layers, conv_elem_bytes, nullptr, nullptr);
+}
+
+RecurrentStatePool::RecurrentStatePool(std::vector<RecurrentLayerGeometry> layers, size_t conv_elem_bytes, int num_slots)
+    : layers_(std::move(layers)), elem_bytes_(conv_elem_bytes) {
+  slot_bytes_ = lay_out(layers_, elem_bytes_, &state_offset_, &conv_offset_);
+  pool_ = DeviceBuffer(std::max<size_t>(slot_bytes_ * size_t(num_slots), 256));
+  QWEN38_CUDA(cudaMemset(pool_.get(), 0, pool_.bytes()));
+}
+
+kernels::RecurrentStateDesc RecurrentStatePool::layer_desc(int recurrent_layer) const {
+  kernels::RecurrentStateDesc d;
+  d.state = pool_.as<uint8_t>() + state_offset_[size_t(recurrent_layer)];
+  d.conv = pool_.as<uint8_t>() + conv_offset_[size_t(recurrent_layer)];
+  d.slot_bytes = slot_bytes_;
+  return d;
+}
+
+void RecurrentStatePool::reset(int slot, cudaStream_t stream) {
+  if (slot_bytes_ == 0) return;
+  QWEN38_CUDA(cudaMemsetAsync(pool_.as<uint8_t>() + slot_bytes_ * size_t(slot), 0, slot_bytes_, stream));
 }
 
 }  // namespace qwen38
