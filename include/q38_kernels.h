@@ -402,7 +402,8 @@ typedef struct q38_mixed_attention_params {
   const float* head_mix; /* [heads][heads] or NULL */
   void* out;             /* [M][ld_out]: heads x vdim */
   int ld_out;
-  float* stats;          /* [M][heads][2] */
+  float* stats;          /* [max(1, stat_splits)][M][heads][2] */
+  int stat_splits;       /* prefill: key ranges the normalisers may be computed in */
   float* scores;         /* decode: [num_pages][heads][64] (NULL: the decode call uses the prefill kernels) */
   float* partials;       /* decode: [num_seqs][max_splits][heads][v_dim of the cache + 2] */
   int max_splits;

@@ -135,7 +135,7 @@ class RopeAppendParams(C.Structure):
 
 class MixedAttentionParams(C.Structure):
     _fields_ = [("q", C.c_void_p), ("act", C.c_int), ("heads", C.c_int), ("vdim", C.c_int), ("scale", C.c_float),
-                ("head_mix", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int), ("stats", C.c_void_p),
+                ("head_mix", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int), ("stats", C.c_void_p), ("stat_splits", C.c_int),
                 ("scores", C.c_void_p), ("partials", C.c_void_p), ("max_splits", C.c_int)]
 
 

@@ -12,8 +12,11 @@ struct DenseCall {
   q38_dense_epilogue ep;
   const q38_gemm_workspace* ws;
 };
-constexpr int kDenseUmmaTiles = 4;  // token tiles of the tcgen05 kernel
-int dense_umma_tile(int index);     // 32, 64, 128, 256 tokens
-int dense_umma(const DenseCall& c, int tile_index, cudaStream_t stream);
+struct DenseUmmaChoice {
+  int tok, cluster;  // token tile; CTAs that split one tile's k range
+};
+bool dense_umma_fits(const DenseCall& c);
+DenseUmmaChoice dense_umma_choice(int m, int n, int k);
+int dense_umma(const DenseCall& c, DenseUmmaChoice choice, cudaStream_t stream);
 
 }  // namespace q38

@@ -262,6 +262,7 @@ extern "C" int q38_mixed_attention_prefill(const q38_mixed_attention_params* p, 
   if (const int rc = check_attention(p, batch, kv)) return rc;
   if (batch->num_tokens == 0) return Q38_OK;
   if (p->act == Q38_ACT_F32) return launch_general<float>(*p, *batch, *kv, as_stream(stream));
+  if (mixed_prefill_mma_fits(*p, *kv)) return mixed_prefill_mma(*p, *batch, *kv, as_stream(stream));
   return launch_general<__nv_bfloat16>(*p, *batch, *kv, as_stream(stream));
 }
 
@@ -270,5 +271,6 @@ extern "C" int q38_mixed_attention_decode(const q38_mixed_attention_params* p, c
   if (const int rc = check_attention(p, batch, kv)) return rc;
   if (batch->num_tokens == 0) return Q38_OK;
   if (p->act == Q38_ACT_F32) return launch_general<float>(*p, *batch, *kv, as_stream(stream));
+  if (batch->num_tokens == batch->num_seqs && mixed_decode_mma_fits(*p, *kv)) return mixed_decode_mma(*p, *batch, *kv, as_stream(stream));
   return launch_general<__nv_bfloat16>(*p, *batch, *kv, as_stream(stream));
 }

@@ -44,6 +44,7 @@
 #include "common.cuh"
 #include "host_util.h"
 #include "qgemm.h"
+#include "tcgen05.cuh"
 
 namespace q38 {
 namespace {
@@ -140,44 +141,6 @@ __device__ __forceinline__ long long u_begin(const UmmaArgs& a, int cta, int gri
   return ((long long)cta * a.items / grid) * a.kg;
 }
 
-// Bounded wait that also gives up once another thread of the CTA has given up (the flag is polled only on the slow
-// path, so a wait that is already satisfied costs one try_wait).
-__device__ __forceinline__ bool wait_flag(uint64_t* bar, uint32_t parity, volatile int* abort_flag, unsigned site) {
-  if (mbar_try_wait(bar, parity)) return true;
-  for (uint32_t i = 0; i < kSpinLimit; ++i) {
-    if (mbar_try_wait(bar, parity)) return true;
-    if ((i & 255u) == 255u && *abort_flag) return false;
-  }
-  report_error(site);
-  *abort_flag = 1;
-  return false;
-}
-
-// ---- tcgen05 wrappers ---------------------------------------------------------------------------------
-__device__ __forceinline__ void tmem_alloc(uint32_t* dst_smem, uint32_t cols) {
-  asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(dst_smem)), "r"(cols)
-               : "memory");
-  asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t cols) {
-  asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(cols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-
-// Both are called by a whole, converged warp with warp-uniform arguments; one elected lane issues. Keeping the
-// issuing code warp-uniform lets the descriptors live in uniform registers, which the instruction reads directly.
-__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc,
-                                          uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p, leader;\n\t"
-      "elect.sync _|leader, 0xffffffff;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "@leader tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
 // With the A operand in tensor memory an MMA reads [128 lanes][8 columns], column c of lane r = A[r][2c], A[r][2c+1].
 // The four MMAs of one 64-wide k-group in one block, so that the election and the operand arithmetic are paid once:
 // A = tensor memory columns a_tmem + 8 ks, B = shared-memory descriptor {b_lo + 2 ks, b_hi} (32 bytes per k16 step;
@@ -210,33 +173,6 @@ __device__ __forceinline__ void tmem_st_16x128b_x8(uint32_t taddr, const uint32_
       : "memory");
 }
 __device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-  asm volatile(
-      "{\n\t.reg .pred leader;\n\t"
-      "elect.sync _|leader, 0xffffffff;\n\t"
-      "@leader tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
-      ::"r"(smem_u32(bar))
-      : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-      : "r"(taddr));
-  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-
-// K-major operand tile with the 128-byte swizzle: rows of 128 bytes, 8-row groups 1024 bytes apart.
-__device__ __forceinline__ uint64_t smem_desc_sw128(uint32_t addr) {
-  uint64_t d = uint64_t((addr & 0x3FFFFu) >> 4);
-  d |= uint64_t(1) << 16;             // leading byte offset (unused for swizzled K-major)
-  d |= uint64_t(1024 >> 4) << 32;     // stride byte offset between 8-row groups
-  d |= uint64_t(1) << 46;             // descriptor version of this architecture
-  d |= uint64_t(2) << 61;             // 128-byte swizzle
-  return d;
-}
-
 template <int BITS, int TOK, bool ATM>
 __global__ void __launch_bounds__(kThreads, 1)
 qgemm_umma_kernel(const __grid_constant__ CUtensorMap xmap, const UmmaArgs a) {

@@ -8,6 +8,7 @@ namespace qwen38 {
 namespace {
 
 constexpr int kMaxSplits = 64;
+constexpr int kStatSplits = 8;
 int up(int x, int to) { return int(align_up(x, to)); }
 
 // The tensors of one design by name and expected shape; `at` reads one as fp32.
@@ -341,7 +342,7 @@ void LayerListModel::carve(Workspace& w, const StepContext& ctx) {
   y_ = w.take<float>(T * size_t(ld_x_));
   q_ = w.take<uint8_t>(T * size_t(max_q_) * elem_);
   v_first_ = w.take<uint8_t>(T * size_t(max_v_) * elem_);
-  stats_ = w.take<float>(T * size_t(max_heads_) * 2);
+  stats_ = w.take<float>(T * size_t(max_heads_) * 2 * kStatSplits);
   if (!f32_) partials_ = w.take<float>(R * kMaxSplits * (size_t(max_attn_out_) + 2 * size_t(max_heads_)));
   rec_scratch_ = w.take<float>(2 * T * size_t(max_rec_));
   head_x_ = w.take<uint8_t>(R * size_t(ld_x_) * elem_);
@@ -387,6 +388,7 @@ void LayerListModel::attention(const StepContext& ctx, const StepBatch& b, const
   ap.out = mixer_;
   ap.ld_out = ld_mixer_;
   ap.stats = stats_;
+  ap.stat_splits = kStatSplits;
   ap.scores = scores_.as<float>();
   ap.partials = partials_;
   ap.max_splits = kMaxSplits;
