@@ -1,5 +1,5 @@
-// Dense GEMM y[m][n] = x[m][k] W^T + bias with bf16 weights: dispatcher, the fp32 kernels, and the streaming kernel for
-// small bf16 batches. Larger bf16 batches take the tcgen05 kernel (dense_umma.cu).
+// Dense GEMM y[m][n] = x[m][k] W^T + bias with bf16 weights: dispatcher and the fp32 kernel. bf16 activations take
+// the tcgen05 kernel (dense_umma.cu).
 #include <algorithm>
 
 #include "act.cuh"
@@ -68,103 +68,10 @@ int launch_simt(const DenseCall& c, cudaStream_t s) {
   return Q38_OK;
 }
 
-// ---- streaming kernel, bf16, up to 32 tokens ----------------------------------------------------------------------
-// A CTA owns 16 output columns; its eight warps interleave over the 32-wide k blocks and their sums meet in shared memory.
-// Weights go straight from global memory into mma.m16n8k16 fragments: a lane takes 16 contiguous bytes of its row, which
-// are the fragment registers of two k16 steps under a permutation of k that the activation fragments share. The first
-// weights are requested before griddepcontrol.wait.
-constexpr int kStreamWarps = 8, kStreamUnroll = 4;
-__device__ __forceinline__ uint4 ld_stream(const void* p) {
-  uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.L2::128B.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-  return v;
-}
-
-template <int NT>
-__global__ void __launch_bounds__(kStreamWarps * 32)
-dense_stream_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int m, q38_dense_weight w, q38_dense_epilogue ep) {
-  __shared__ float red[kStreamWarps][16][NT * 8 + 1];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
-  const int n0 = blockIdx.x * 16, blocks = (w.k + 31) / 32;
-  const __nv_bfloat16* wp = reinterpret_cast<const __nv_bfloat16*>(w.w) + (size_t)(n0 + g) * w.ld + t * 8;
-  const size_t row8 = (size_t)8 * w.ld;
-  uint4 a0[kStreamUnroll], a1[kStreamUnroll];
-  auto load = [&](int kb, int i) {
-    if (kb < blocks) {
-      a0[i] = ld_stream(wp + kb * 32);
-      a1[i] = ld_stream(wp + row8 + kb * 32);
-    } else {
-      a0[i] = a1[i] = make_uint4(0, 0, 0, 0);
-    }
-  };
-#pragma unroll
-  for (int i = 0; i < kStreamUnroll; ++i) load(warp + i * kStreamWarps, i);
-  float acc[NT][4] = {};
-  pdl_wait();
-  pdl_launch_dependents();
-  for (int kb = warp; kb < blocks; kb += kStreamWarps * kStreamUnroll) {
-#pragma unroll
-    for (int i = 0; i < kStreamUnroll; ++i) {
-      const int k = kb + i * kStreamWarps;
-      const uint4 c0 = a0[i], c1 = a1[i];
-      load(k + kStreamWarps * kStreamUnroll, i);
-      if (k >= blocks) continue;
-      const uint32_t f0[4] = {c0.x, c1.x, c0.y, c1.y}, f1[4] = {c0.z, c1.z, c0.w, c1.w};
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        const int tok = nt * 8 + g;
-        uint4 b = make_uint4(0, 0, 0, 0);
-        if (tok < m) b = *reinterpret_cast<const uint4*>(x + (size_t)tok * ldx + k * 32 + t * 8);
-        mma_bf16_16816(acc[nt], f0, b.x, b.y);
-        mma_bf16_16816(acc[nt], f1, b.z, b.w);
-      }
-    }
-  }
-#pragma unroll
-  for (int nt = 0; nt < NT; ++nt) {
-    red[warp][g][nt * 8 + 2 * t] = acc[nt][0];
-    red[warp][g][nt * 8 + 2 * t + 1] = acc[nt][1];
-    red[warp][g + 8][nt * 8 + 2 * t] = acc[nt][2];
-    red[warp][g + 8][nt * 8 + 2 * t + 1] = acc[nt][3];
-  }
-  __syncthreads();
-  auto value = [&](int r, int tok) {
-    float v = 0.0f;
-#pragma unroll
-    for (int i = 0; i < kStreamWarps; ++i) v += red[i][r][tok];
-    return v + (w.bias ? w.bias[n0 + r] : 0.0f);
-  };
-  if (ep.kind == Q38_DENSE_STORE || ep.kind == Q38_DENSE_STORE_F32) {
-    for (int e = threadIdx.x; e < 16 * NT * 8; e += blockDim.x) {
-      const int r = e & 15, tok = e >> 4;
-      if (tok >= m || n0 + r >= w.n) continue;
-      const float v = value(r, tok);
-      if (ep.kind == Q38_DENSE_STORE_F32) static_cast<float*>(ep.out)[(size_t)tok * ep.ldo + n0 + r] = v;
-      else static_cast<__nv_bfloat16*>(ep.out)[(size_t)tok * ep.ldo + n0 + r] = __float2bfloat16_rn(v);
-    }
-  } else {
-    for (int e = threadIdx.x; e < 8 * NT * 8; e += blockDim.x) {
-      const int r = 2 * (e & 7), tok = e >> 3;
-      if (tok >= m || n0 + r >= w.n) continue;
-      static_cast<__nv_bfloat16*>(ep.out)[(size_t)tok * ep.ldo + (n0 + r) / 2] =
-          __float2bfloat16_rn(glu_act(ep.kind, value(r, tok)) * value(r + 1, tok));
-    }
-  }
-}
-
-template <int NT>
-int launch_stream(const DenseCall& c, cudaStream_t s) {
-  (void)launch_kernel(dense_stream_kernel<NT>, dim3((c.w.n + 15) / 16), dim3(kStreamWarps * 32), 0, s,
-                      static_cast<const __nv_bfloat16*>(c.x), c.ldx, c.m, c.w, c.ep);
-  Q38_LAUNCH_OK("dense_stream_kernel");
-  return Q38_OK;
-}
-
-enum Config { kSimt, kStream, kUmma32, kUmma64, kUmma128, kUmma256, kCluster2, kCluster4, kCluster8 };
-constexpr const char* kConfigNames[] = {"simt", "stream", "umma_t32", "umma_t64", "umma_t128", "umma_t256",
+enum Config { kSimt, kUmma32, kUmma64, kUmma128, kUmma256, kCluster2, kCluster4, kCluster8 };
+constexpr const char* kConfigNames[] = {"simt", "umma_t32", "umma_t64", "umma_t128", "umma_t256",
                                         "umma_cluster2", "umma_cluster4", "umma_cluster8"};
 constexpr int kNumDenseConfigs = int(sizeof(kConfigNames) / sizeof(kConfigNames[0]));
-constexpr int kStreamTokens = 32;
 
 }  // namespace
 }  // namespace q38
@@ -189,13 +96,10 @@ extern "C" int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_
   cudaStream_t s = as_stream(stream);
   if (act == Q38_ACT_F32) return launch_simt<float>(c, s);
   const bool aligned = dense_umma_fits(c);
-  if (config < 0) config = !aligned ? kSimt : m <= 16 ? kStream : -1;
+  if (config < 0 && !aligned) config = kSimt;
   Q38_REQUIRE(config < 0 || config == kSimt || aligned, "dense_gemm: rows must start at multiples of 16 bytes");
   switch (config) {
     case kSimt: return launch_simt<__nv_bfloat16>(c, s);
-    case kStream:
-      Q38_REQUIRE(m <= kStreamTokens && ldx >= (w->k + 31) / 32 * 32, "dense_gemm: the streaming kernel takes %d tokens", kStreamTokens);
-      return m <= 8 ? launch_stream<1>(c, s) : m <= 16 ? launch_stream<2>(c, s) : launch_stream<4>(c, s);
     case kUmma32: return dense_umma(c, {32, 1}, s);
     case kUmma64: return dense_umma(c, {64, 1}, s);
     case kUmma128: return dense_umma(c, {128, 1}, s);

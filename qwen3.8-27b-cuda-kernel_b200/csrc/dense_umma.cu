@@ -1,4 +1,4 @@
-// Dense bf16 GEMM on the 5th-generation tensor cores (tcgen05.mma, accumulators in TMEM), 17 tokens and more.
+// Dense bf16 GEMM on the 5th-generation tensor cores (tcgen05.mma, accumulators in TMEM), any number of tokens.
 //
 // Orientation as in the BQ kernel: the weights are the MMA's A operand (128 output columns fill the 128 TMEM lanes), the
 // tokens its N operand (TOK = 32 ... 256). Both operands arrive by TMA (2-D tensor maps, 128-byte swizzle; rows and
@@ -180,7 +180,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       const uint32_t taddr = tmem + acc * C::kAccCols + (uint32_t(quarter * 32) << 16);
       if (CLUSTER) {
         float* part = reinterpret_cast<float*>(ring);  // [TOK][128]; every MMA of this CTA has read its stages
-        for (int c = 0; c < TOK; c += 16) {
+        for (int c = 0; c < TOK && c < tokens; c += 16) {
           uint32_t r[16];
           tmem_ld16(taddr + uint32_t(c), r);
 #pragma unroll
@@ -246,19 +246,29 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       const int n = tn * kTileN + nl, t0 = tm * TOK, tokens = min(TOK, a.m - t0);
       const float bias = a.bias && n < a.n ? a.bias[n] : 0.0f;
       const uint32_t part = smem_u32(ring);
-      for (int t = rank; t < tokens; t += a.cluster) {
-        float v = 0.0f;
-#pragma unroll 8
-        for (int c = 0; c < a.cluster; ++c) v += ld_cluster_f32(part + uint32_t((t * kTileN + nl) * 4), uint32_t(c));
-        v += bias;
-        const size_t row = (size_t)(t0 + t) * a.ldo;
-        if (a.kind == Q38_DENSE_STORE_F32) {
-          if (n < a.n) static_cast<float*>(a.out)[row + n] = v;
-        } else if (a.kind == Q38_DENSE_STORE) {
-          if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(v);
-        } else {
-          const float up = __shfl_xor_sync(0xffffffffu, v, 1);
-          if (!(lane & 1) && n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + (n >> 1)] = __float2bfloat16_rn(glu(a.kind, v, up));
+      constexpr int kU = 8;  // token rows in flight
+      for (int tb = rank; tb < tokens; tb += kU * a.cluster) {
+        float v[kU] = {};
+        for (int c = 0; c < a.cluster; ++c)
+#pragma unroll
+          for (int u = 0; u < kU; ++u) {
+            const int t = tb + u * a.cluster;
+            if (t < tokens) v[u] += ld_cluster_f32(part + uint32_t((t * kTileN + nl) * 4), uint32_t(c));
+          }
+#pragma unroll
+        for (int u = 0; u < kU; ++u) {
+          const int t = tb + u * a.cluster;
+          if (t >= tokens) break;
+          const float x = v[u] + bias;
+          const size_t row = (size_t)(t0 + t) * a.ldo;
+          if (a.kind == Q38_DENSE_STORE_F32) {
+            if (n < a.n) static_cast<float*>(a.out)[row + n] = x;
+          } else if (a.kind == Q38_DENSE_STORE) {
+            if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(x);
+          } else {
+            const float up = __shfl_xor_sync(0xffffffffu, x, 1);
+            if (!(lane & 1) && n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + (n >> 1)] = __float2bfloat16_rn(glu(a.kind, x, up));
+          }
         }
       }
     }
@@ -359,20 +369,22 @@ bool dense_umma_fits(const DenseCall& c) {
   return c.ldx % 8 == 0 && c.w.ld % 8 == 0 && reinterpret_cast<uintptr_t>(c.x) % 16 == 0 && reinterpret_cast<uintptr_t>(c.w.w) % 16 == 0;
 }
 
-// Tile and cluster size by a cost in cycles: waves x k-groups x the larger of the tensor and the issue time of a k-group,
-// plus the tile's epilogue; clusters are only used when the whole list fits the GPU at once.
+// Tile and cluster size by a cost in cycles. A CTA spends kStep cycles on a k-group (it is the transfer from L2 that bounds
+// it, not the MMA); CTAs that share an SM share its transfer rate. Clusters add their reduction and are only used when every
+// CTA of the launch is resident at once (two per SM up to 64 tokens).
 DenseUmmaChoice dense_umma_choice(int m, int n, int k) {
   const int sms = num_sms(), kg = (k + 63) / 64, tiles_n = (n + kTileN - 1) / kTileN;
-  constexpr int kTok[4] = {32, 64, 128, 256}, kStep[4] = {200, 220, 300, 540};
+  constexpr int kTok[4] = {32, 64, 128, 256}, kStep[4] = {400, 420, 560, 900}, kShared[4] = {320, 380, 560, 900};
   DenseUmmaChoice best{64, 1};
   long long best_cost = -1;
   for (int i = 0; i < 4; ++i) {
     if (i > 0 && kTok[i - 1] >= m) break;  // the next smaller tile already holds every token
     const long long items = (long long)tiles_n * ((m + kTok[i] - 1) / kTok[i]);
     for (int c = 1; c <= (kTok[i] <= 128 ? 8 : 1); c *= 2) {
-      if (c > 1 && (items * c > sms || kg < 2 * c)) break;
-      const long long waves = (items * c + sms - 1) / sms;
-      long long cost = waves * ((kg + c - 1) / c) * kStep[i] + kTok[i] * 14 + (c > 1 ? 1500 + kTok[i] * 4 : 0);
+      if (c > 1 && (items * c > (kTok[i] <= 64 ? 2 : 1) * sms || kg < 2 * c)) break;
+      const long long waves = (items * c + sms - 1) / sms, kgs = (kg + c - 1) / c;
+      const long long cost = (waves == 1 ? kgs * kStep[i] : waves * kgs * kShared[i]) + std::min(m, kTok[i]) * 14 +
+                             (c > 1 ? 1500 + std::min(m, kTok[i]) * 12 : 0);
       if (best_cost < 0 || cost < best_cost) {
         best_cost = cost;
         best = {kTok[i], c};

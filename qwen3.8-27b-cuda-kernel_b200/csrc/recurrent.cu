@@ -217,6 +217,79 @@ rglru_gates_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_state
   }
 }
 
+// Tensor-core form (bf16 activations): a CTA holds the convolved inputs of 32 tokens x one block in shared memory, as
+// bf16 terms hi + lo, and makes 64 output channels of both gates: a warp the 8 channels of one n tile, r and i side by
+// side in its registers. Weights come straight from global memory into fragments (16 contiguous bytes of a row = two k16
+// steps under a permutation of k that both operands share).
+constexpr int kMmaTokens = 32, kMmaWarps = 8, kMmaOut = kMmaWarps * 8;
+__host__ __device__ constexpr int gate_stride(int cols) { return cols % 64 == 32 ? cols : cols + 32; }
+
+template <bool DECODE>
+__global__ void __launch_bounds__(kMmaWarps * 32)
+rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_state_desc st) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int bs = p.width / p.blocks, ld = p.block_ld, us = gate_stride(ld), blk = blockIdx.y, t0 = blockIdx.x * kMmaTokens;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  __nv_bfloat16* hi = reinterpret_cast<__nv_bfloat16*>(smem);  // [32][us]
+  __nv_bfloat16* lo = hi + kMmaTokens * us;
+  const int o0 = blockIdx.z * kMmaOut + warp * 8;
+  const bool live = o0 < ld;
+  const __nv_bfloat16* wr = reinterpret_cast<const __nv_bfloat16*>(p.gate_w) + ((size_t)blk * 2 * ld + o0 + g) * ld + t * 8;
+  const __nv_bfloat16* wi = wr + (size_t)ld * ld;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int n = min(kMmaTokens, batch.num_tokens - t0);
+  for (int i = threadIdx.x; i < kMmaTokens * ld; i += blockDim.x) {
+    const int tok = i / ld, k = i % ld;
+    const float u = tok < n && k < bs ? conv_at<__nv_bfloat16>(p, batch, st.conv, st.slot_bytes, t0 + tok, blk * bs + k) : 0.0f;
+    const __nv_bfloat16 h = __float2bfloat16_rn(u);
+    hi[tok * us + k] = h;
+    lo[tok * us + k] = __float2bfloat16_rn(u - __bfloat162float(h));
+  }
+  __syncthreads();
+  if (!live) return;
+  float acc[2][2][4] = {};  // [16-token tile][r, i]
+  for (int k = 0; k < ld; k += 32) {
+    const uint4 w[2] = {*reinterpret_cast<const uint4*>(wr + k), *reinterpret_cast<const uint4*>(wi + k)};
+#pragma unroll
+    for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+      for (int term = 0; term < 2; ++term) {
+        const __nv_bfloat16* u = (term ? lo : hi) + (mt * 16 + g) * us + k + t * 8;
+        const uint4 a0 = *reinterpret_cast<const uint4*>(u), a1 = *reinterpret_cast<const uint4*>(u + 8 * us);
+        const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          mma_bf16_16816(acc[mt][q], f0, w[q].x, w[q].y);
+          mma_bf16_16816(acc[mt][q], f1, w[q].z, w[q].w);
+        }
+      }
+  }
+#pragma unroll
+  for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int tok = mt * 16 + g + 8 * (e >> 1), o = o0 + 2 * t + (e & 1);
+      if (tok >= n || o >= bs) continue;
+      const float u = __bfloat162float(hi[tok * us + o]) + __bfloat162float(lo[tok * us + o]);
+      gate_finish<__nv_bfloat16, DECODE>(p, batch, st, t0 + tok, blk * bs + o, acc[mt][0][e], acc[mt][1][e], u);
+    }
+}
+
+size_t gates_mma_smem(int block_ld) { return size_t(2) * kMmaTokens * gate_stride(block_ld) * 2; }
+
+template <bool DECODE>
+int launch_gates_mma(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, cudaStream_t s) {
+  const int bs = p.width / p.blocks;
+  const size_t smem = gates_mma_smem(p.block_ld);
+  static const cudaError_t attr = cudaFuncSetAttribute(rglru_gates_mma_kernel<DECODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+  Q38_CUDA_OK(attr);
+  (void)launch_kernel(rglru_gates_mma_kernel<DECODE>, dim3((b.num_tokens + kMmaTokens - 1) / kMmaTokens, p.blocks, (bs + kMmaOut - 1) / kMmaOut),
+                      dim3(kMmaWarps * 32), smem, s, p, b, st);
+  Q38_LAUNCH_OK("rglru_gates_mma_kernel");
+  return Q38_OK;
+}
+
 int check_common(const q38_batch_desc* b, const q38_recurrent_state_desc* st, const char* what) {
   Q38_REQUIRE(b && st && st->state && b->seq_start && b->seq_slot && b->seq_pos0 && b->tok_pos && b->tok_seq, "%s: null argument", what);
   Q38_REQUIRE(b->num_seqs > 0 && b->num_tokens >= b->num_seqs && b->max_tokens_per_seq > 0, "%s: batch sizes", what);
@@ -236,16 +309,32 @@ int launch_mingru(const q38_mingru_params& p, const q38_batch_desc& b, const q38
 }
 
 template <typename T>
-int launch_rglru(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, cudaStream_t s) {
+int launch_gates_simt(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, bool decode, cudaStream_t s) {
   const int bs = p.width / p.blocks;
   const dim3 grid((b.num_tokens + kGateTokens - 1) / kGateTokens, p.blocks, (bs + kGateThreads - 1) / kGateThreads);
   const size_t smem = size_t(kGateTokens) * p.block_ld * 4;
-  const bool decode = b.max_tokens_per_seq == 1;
+  Q38_REQUIRE(smem <= size_t(max_optin_smem()), "rglru: blocks of %d channels", bs);
+  static const cudaError_t attr0 = cudaFuncSetAttribute(rglru_gates_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+  static const cudaError_t attr1 = cudaFuncSetAttribute(rglru_gates_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+  Q38_CUDA_OK(attr0);
+  Q38_CUDA_OK(attr1);
   if (decode)
     (void)launch_kernel(rglru_gates_kernel<T, true>, grid, dim3(kGateThreads), smem, s, p, b, st);
   else
     (void)launch_kernel(rglru_gates_kernel<T, false>, grid, dim3(kGateThreads), smem, s, p, b, st);
   Q38_LAUNCH_OK("rglru_gates_kernel");
+  return Q38_OK;
+}
+
+template <typename T>
+int launch_rglru(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, cudaStream_t s) {
+  const bool decode = b.max_tokens_per_seq == 1;
+  int rc;
+  if (sizeof(T) == 2 && gates_mma_smem(p.block_ld) <= size_t(max_optin_smem()))
+    rc = decode ? launch_gates_mma<true>(p, b, st, s) : launch_gates_mma<false>(p, b, st, s);
+  else
+    rc = launch_gates_simt<T>(p, b, st, decode, s);
+  if (rc) return rc;
   if (decode) return Q38_OK;
   RgLru<T> op{p, b};
   (void)launch_kernel(scan_kernel<RgLru<T>>, dim3((p.width + kScanCh - 1) / kScanCh, b.num_seqs), dim3(kScanCh, kScanSegs), 0, s,
@@ -274,7 +363,7 @@ extern "C" int q38_rglru(const q38_rglru_params* p, const q38_batch_desc* batch,
   if (const int rc = check_common(batch, st, "rglru")) return rc;
   Q38_REQUIRE(p->width > 0 && p->blocks > 0 && p->width % p->blocks == 0 && p->taps > 0 && st->conv, "rglru: sizes");
   Q38_REQUIRE(p->ld_proj >= 2 * p->width && p->ld_out >= p->width, "rglru: leading dimensions");
-  Q38_REQUIRE(p->block_ld % 32 == 0 && p->block_ld >= p->width / p->blocks && p->block_ld <= 1024, "rglru: block_ld %d", p->block_ld);
+  Q38_REQUIRE(p->block_ld % 32 == 0 && p->block_ld >= p->width / p->blocks, "rglru: block_ld %d", p->block_ld);
   Q38_REQUIRE(batch->max_tokens_per_seq == 1 || p->scratch, "rglru: scratch needed");
   return p->act == Q38_ACT_BF16 ? launch_rglru<__nv_bfloat16>(*p, *batch, *st, as_stream(stream))
                                 : launch_rglru<float>(*p, *batch, *st, as_stream(stream));
