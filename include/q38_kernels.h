@@ -375,7 +375,7 @@ int q38_gather_norm(const float* residual, const int* rows, int first, int n, in
                     int ld_out, int act, void* stream);
 
 /* Rotary positions on the leading rot_dims of every query and key head (dimension i turns with i + rot_dims / 2 by
- * position * base^(-2 i / rot_dims)), optional blending of the values with a first layer's, and the append to the cache.
+ * position * inv_freq[i]), optional blending of the values with a first layer's, and the append to the cache.
  * proj rows: [q: heads x dim | k: kv_heads x dim | v: kv_heads x vdim]. */
 typedef struct q38_rope_append_params {
   const void* proj;
@@ -383,7 +383,7 @@ typedef struct q38_rope_append_params {
   int act;
   int heads, kv_heads, dim, vdim;
   int rot_dims;
-  double rot_base;
+  const double* inv_freq; /* [rot_dims / 2]: base^(-2 i / rot_dims) */
   void* q_out;            /* [M][heads][k_dim of the cache], zero beyond dim */
   void* v_first_out;      /* [M][kv_heads * vdim]: where to keep this layer's values, or NULL */
   const void* v_first_in; /* values to blend with, or NULL: v = (1 - *v_mix) v + *v_mix v_first */

@@ -129,7 +129,7 @@ class Norm(C.Structure):
 
 class RopeAppendParams(C.Structure):
     _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int),
-                ("dim", C.c_int), ("vdim", C.c_int), ("rot_dims", C.c_int), ("rot_base", C.c_double),
+                ("dim", C.c_int), ("vdim", C.c_int), ("rot_dims", C.c_int), ("inv_freq", C.c_void_p),
                 ("q_out", C.c_void_p), ("v_first_out", C.c_void_p), ("v_first_in", C.c_void_p), ("v_mix", C.c_void_p)]
 
 

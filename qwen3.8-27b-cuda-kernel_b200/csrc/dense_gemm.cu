@@ -109,7 +109,7 @@ extern "C" int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_
     case kCluster8: {
       const int cl = config == kCluster2 ? 2 : config == kCluster4 ? 4 : 8;
       Q38_REQUIRE((w->k + 63) / 64 >= cl, "dense_gemm: k %d is too short for a cluster of %d", w->k, cl);
-      return dense_umma(c, {m <= 32 ? 32 : m <= 64 ? 64 : 128, cl}, s);
+      return dense_umma(c, {m <= 32 ? 32 : 64, cl}, s);
     }
     default: return dense_umma(c, dense_umma_choice(m, w->n, w->k), s);
   }

@@ -31,7 +31,7 @@ struct Cfg {
   static constexpr int kXBytes = TOK * 128;
   static constexpr int kStageBytes = kWBytes + kXBytes;
   // clusters: about 100 KB, so that two CTAs share an SM; persistent: what one CTA may use
-  static constexpr int kBudget = CLUSTER && TOK <= 64 ? 104 * 1024 : 200 * 1024;
+  static constexpr int kBudget = CLUSTER ? 104 * 1024 : 200 * 1024;
   static constexpr int kStages = kBudget / kStageBytes > 8 ? 8 : kBudget / kStageBytes;
   static constexpr int kAccCols = TOK < 32 ? 32 : TOK;
   static constexpr int kAccs = CLUSTER ? 1 : 2;
@@ -357,7 +357,7 @@ int launch(const DenseCall& c, int cluster, cudaStream_t stream) {
 
 template <int TOK>
 int launch_tok(const DenseCall& c, int cluster, cudaStream_t stream) {
-  if constexpr (TOK <= 128) {
+  if constexpr (TOK <= 64) {
     if (cluster > 1) return launch<TOK, true>(c, cluster, stream);
   }
   return launch<TOK, false>(c, 1, stream);
@@ -380,11 +380,11 @@ DenseUmmaChoice dense_umma_choice(int m, int n, int k) {
   for (int i = 0; i < 4; ++i) {
     if (i > 0 && kTok[i - 1] >= m) break;  // the next smaller tile already holds every token
     const long long items = (long long)tiles_n * ((m + kTok[i] - 1) / kTok[i]);
-    for (int c = 1; c <= (kTok[i] <= 128 ? 8 : 1); c *= 2) {
-      if (c > 1 && (items * c > (kTok[i] <= 64 ? 2 : 1) * sms || kg < 2 * c)) break;
+    for (int c = 1; c <= (kTok[i] <= 64 ? 8 : 1); c *= 2) {
+      if (c > 1 && (items * c > 2 * sms || kg < 2 * c)) break;
       const long long waves = (items * c + sms - 1) / sms, kgs = (kg + c - 1) / c;
       const long long cost = (waves == 1 ? kgs * kStep[i] : waves * kgs * kShared[i]) + std::min(m, kTok[i]) * 14 +
-                             (c > 1 ? 1500 + std::min(m, kTok[i]) * 12 : 0);
+                             (c > 1 ? 1500 + std::min(m, kTok[i]) * 50 : 0);
       if (best_cost < 0 || cost < best_cost) {
         best_cost = cost;
         best = {kTok[i], c};

@@ -25,7 +25,7 @@ __device__ __forceinline__ const T* v_col(const q38_kv_layer_desc& kv, int page,
 }
 
 // ---- rotary positions, value blending, append ------------------------------------------------------------------------
-// One CTA per token. The angle position * base^(-2 i / dims) is formed and reduced in double precision, so that far
+// One CTA per token. The angle position * inv_freq[i] is formed and reduced in double precision, so that far
 // positions keep the accuracy of near ones; its sine and cosine are fp32.
 template <typename T>
 __global__ void __launch_bounds__(128) rope_append_kernel(q38_rope_append_params p, q38_batch_desc b, q38_kv_layer_desc kv) {
@@ -35,7 +35,7 @@ __global__ void __launch_bounds__(128) rope_append_kernel(q38_rope_append_params
   const int m = blockIdx.x, pos = b.tok_pos[m], slot = b.seq_slot[b.tok_seq[m]];
   const int half = p.rot_dims / 2;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const double ang = double(pos) * pow(p.rot_base, -2.0 * double(i) / double(p.rot_dims));
+    const double ang = double(pos) * p.inv_freq[i];
     const double turns = ang * 0.15915494309189535;
     const float red = float((turns - rint(turns)) * 6.283185307179586);
     float sn, cs;
@@ -247,6 +247,7 @@ extern "C" int q38_rope_append(const q38_rope_append_params* p, const q38_batch_
   Q38_REQUIRE(p->rot_dims >= 0 && p->rot_dims % 2 == 0 && p->rot_dims <= p->dim && p->rot_dims <= 4096, "rope_append: rot_dims %d", p->rot_dims);
   Q38_REQUIRE(p->ld_proj >= p->heads * p->dim + p->kv_heads * (p->dim + p->vdim), "rope_append: ld_proj");
   Q38_REQUIRE(kv->dtype == (p->act == Q38_ACT_BF16 ? Q38_KV_BF16 : Q38_KV_F32), "rope_append: cache precision");
+  Q38_REQUIRE(p->rot_dims == 0 || p->inv_freq, "rope_append: inv_freq");
   Q38_REQUIRE(!p->v_first_in || p->v_mix, "rope_append: v_mix");
   const size_t smem = size_t(std::max(1, p->rot_dims)) * 4;
   if (p->act == Q38_ACT_BF16)

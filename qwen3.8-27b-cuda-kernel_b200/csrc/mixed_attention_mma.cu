@@ -378,7 +378,8 @@ mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
     }
 }
 
-// ---- prefill: values ----------------------------------------------------------------------------------------------------------
+// ---- prefill: values, operands straight from global memory ------------------------------------------------------------------
+// For shapes whose K and V tiles do not fit into shared memory (many kv heads).
 // 16 warps; warp = (row group of 16 tokens, output head, chunk of 128 value columns). Keys in tiles of 32.
 constexpr int kValWarps = 16, kKeys = 32, kPStride = 40;
 struct ValGeom {
@@ -388,7 +389,7 @@ struct ValGeom {
   int q_in_smem;
 };
 __global__ void __launch_bounds__(kValWarps * 32, 1)
-mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, ValGeom geo, int splits) {
+mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, ValGeom geo, int splits) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t smem[];
@@ -552,6 +553,255 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   }
 }
 
+// ---- prefill: values, operands staged in shared memory --------------------------------------------------------------------------
+// The same division of labour (16 warps, keys in tiles of 32) with K and V tiles copied asynchronously: K of the next tile
+// travels while the weights are mixed and the values multiplied, V of the next one while its scores are computed. The
+// mixing runs on the tensor cores too: T [out heads x heads] against the weights [heads x (token, key)], both split into
+// bf16 hi + lo (hi hi + hi lo + lo hi, fp32 sums); a weight is stored as one word (hi, lo). The CTAs of a cluster share
+// one token tile and divide its keys; their outputs (weights are normalised over all keys) are summed through the
+// cluster's shared memory in rank order.
+struct TileGeom {
+  int row_groups, vchunks, out_heads, q_in_smem;
+  int v_heads;      // kv heads whose values a CTA needs at most
+  int head_words;   // P: words per head = 16 RG * kPStride + 4
+  int out_stride;   // W: elements per output head = 16 RG * 32 + 8
+  // byte offsets
+  int k, v, p, w, t, ml, q, bytes;
+};
+__device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t local_addr, uint32_t rank) {
+  uint32_t remote;
+  float4 v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local_addr), "r"(rank));
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(remote) : "memory");
+  return v;
+}
+__device__ __forceinline__ void cluster_barrier() {
+  __syncwarp();
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ uint32_t split_word(float x) {
+  const bf16 h = __float2bfloat16_rn(x), l = __float2bfloat16_rn(x - __bfloat162float(h));
+  return uint32_t(__bfloat16_as_ushort(h)) | uint32_t(__bfloat16_as_ushort(l)) << 16;
+}
+
+__global__ void __launch_bounds__(kValWarps * 32, 1)
+mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, TileGeom geo, int splits, int cluster) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int H = p.heads, G = kv.kv_heads, RG = geo.row_groups, TQ = 16 * RG, HO = geo.out_heads, group = H / G;
+  const int qs = tile_stride(kv.k_dim), kb_n = kv.k_dim / 32, k_steps = (H + 15) / 16, m_tiles = (HO + 15) / 16;
+  bf16* k_sm = reinterpret_cast<bf16*>(smem + geo.k);            // [G][32][qs]
+  bf16* v_sm = reinterpret_cast<bf16*>(smem + geo.v);            // [v_heads][v_dim][32]
+  uint32_t* P = reinterpret_cast<uint32_t*>(smem + geo.p);       // [H][TQ][kPStride] (+4 per head)
+  bf16* W = reinterpret_cast<bf16*>(smem + geo.w);               // [HO][TQ][32] (+8 per head)
+  uint4* T = reinterpret_cast<uint4*>(smem + geo.t);             // [m_tiles][k_steps][32 lanes][hi, lo] A fragments
+  float2* ml = reinterpret_cast<float2*>(smem + geo.ml);         // [H][TQ] (maximum, 1 / sum)
+  bf16* q_sm = reinterpret_cast<bf16*>(smem + geo.q);            // [H][TQ][qs] (when it fits)
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+  const int seq = blockIdx.z, ho0 = blockIdx.y * HO, rank = int(blockIdx.x) % cluster;
+  const int start = b.seq_start[seq], count = b.seq_start[seq + 1] - start, pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
+  const int t0 = (int(gridDim.x) / cluster - 1 - int(blockIdx.x) / cluster) * TQ;  // the longest tiles first
+  if (t0 >= count) return;  // the same for all CTAs of the cluster
+  const int tokens = min(TQ, count - t0), last = pos0 + t0 + tokens - 1;
+  const int* table = kv.block_table + (size_t)slot * kv.max_pages_per_seq;
+  const int key_tiles = last / kKeys + 1, c0 = rank * key_tiles / cluster, c1 = (rank + 1) * key_tiles / cluster;
+  const int gv0 = ho0 / group, gv1 = min(G, (ho0 + HO - 1) / group + 1);
+
+  auto copy_k = [&](int c) {
+    const int page = table[c / 2], chunks = kv.k_dim / 8, rows = kKeys * chunks;
+    for (int hd = 0; hd < G; ++hd) {
+      const bf16* src = k_page(kv, page, hd) + (size_t)(c % 2) * kKeys * kv.k_dim;
+      bf16* dst = k_sm + (size_t)hd * kKeys * qs;
+      for (int i = threadIdx.x; i < rows; i += blockDim.x) cp_async16(dst + i / chunks * qs + i % chunks * 8, src + (size_t)i * 8);
+    }
+    cp_async_commit();
+  };
+  auto copy_v = [&](int c) {
+    const int page = table[c / 2];
+    for (int hd = gv0; hd < gv1; ++hd) {
+      const bf16* src = v_page(kv, page, hd) + (size_t)(c % 2) * kKeys;
+      bf16* dst = v_sm + (size_t)(hd - gv0) * kv.v_dim * kKeys;
+      for (int i = threadIdx.x; i < kv.v_dim * 4; i += blockDim.x) cp_async16(dst + i * 8, src + (size_t)(i / 4) * kPage + i % 4 * 8);
+    }
+    cp_async_commit();
+  };
+  if (c0 < c1) copy_k(c0);
+
+  const bf16* qg = static_cast<const bf16*>(p.q) + (size_t)(start + t0) * H * kv.k_dim;
+  const size_t i0 = size_t(start - b.seq_start[0] + t0);
+  for (int e = threadIdx.x; e < H * TQ; e += blockDim.x) {
+    const int h = e % H, i = e / H;
+    float M = -INFINITY, L = 0.0f;
+    if (i < tokens)
+      for (int s = 0; s < splits; ++s) {
+        const float2 v = *reinterpret_cast<const float2*>(p.stats + (((size_t)s * b.num_tokens + i0 + i) * H + h) * 2);
+        merge_ml(M, L, v.x, v.y);
+      }
+    ml[h * TQ + i] = i < tokens ? make_float2(M, 1.0f / L) : make_float2(0.0f, 0.0f);
+  }
+  for (int e = threadIdx.x; e < m_tiles * k_steps * 32; e += blockDim.x) {
+    const int ln = e % 32, k = e / 32 % k_steps, mt = e / (32 * k_steps), r = mt * 16 + ln / 4, c = k * 16 + ln % 4 * 2;
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int f = 0; f < 4; ++f) {  // rows r, r + 8 x columns c, c + 8
+      uint32_t w[2];
+#pragma unroll
+      for (int d = 0; d < 2; ++d) {
+        const int o = r + (f & 1) * 8, h = c + (f >> 1) * 8 + d, ho = ho0 + o;
+        w[d] = split_word(o >= HO || ho >= H || h >= H ? 0.0f : p.head_mix ? p.head_mix[(size_t)ho * H + h] : float(ho == h));
+      }
+      hi[f] = __byte_perm(w[0], w[1], 0x5410);
+      lo[f] = __byte_perm(w[0], w[1], 0x7632);
+    }
+    T[2 * e] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    T[2 * e + 1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  if (geo.q_in_smem) {
+    const int chunks = kv.k_dim / 8;
+    for (int e = threadIdx.x; e < H * TQ * chunks; e += blockDim.x) {
+      const int c = e % chunks, h = e / chunks % H, i = e / (chunks * H);
+      *reinterpret_cast<uint4*>(q_sm + ((size_t)h * TQ + i) * qs + c * 8) =
+          i < tokens ? ld16(qg + ((size_t)i * H + h) * kv.k_dim + c * 8) : make_uint4(0, 0, 0, 0);
+    }
+  }
+  const float scale2 = p.scale * kLog2e;
+  const int rg = warp % RG, vc = warp / RG % geo.vchunks, ho = warp / (RG * geo.vchunks);
+  const bool live = ho < HO && ho0 + ho < H;
+  const int v0 = vc * 128, nvt = live ? min(16, (kv.v_dim - v0) / 8) : 0;
+  float acc[16][4] = {};
+  for (int c = c0; c < c1; ++c) {
+    const int j0 = c * kKeys;
+    cp_async_wait<0>();
+    __syncthreads();  // K of this tile is here; the previous tile's weights and values are done with
+    copy_v(c);
+    for (int u = warp; u < H * RG; u += kValWarps) {
+      const int h = u / RG, r = u % RG;
+      const bf16* K = k_sm + ((size_t)(h / group) * kKeys + g) * qs + t * 8;
+      float s[4][4] = {};
+      if (geo.q_in_smem) {
+        const bf16* Q = q_sm + ((size_t)h * TQ + r * 16 + g) * qs + t * 8;
+#pragma unroll 2
+        for (int kb = 0; kb < kb_n; ++kb) {
+          const uint4 a0 = ld16(Q + kb * 32), a1 = ld16(Q + 8 * qs + kb * 32);
+#pragma unroll
+          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, ld16(K + nt * 8 * qs + kb * 32));
+        }
+      } else {
+        const int ia = r * 16 + g;
+        const bf16* Q = qg + ((size_t)ia * H + h) * kv.k_dim + t * 8;
+        const uint4 zero = make_uint4(0, 0, 0, 0);
+#pragma unroll 2
+        for (int kb = 0; kb < kb_n; ++kb) {
+          const uint4 a0 = ia < tokens ? ld16(Q + kb * 32) : zero;
+          const uint4 a1 = ia + 8 < tokens ? ld16(Q + (size_t)8 * H * kv.k_dim + kb * 32) : zero;
+#pragma unroll
+          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, ld16(K + nt * 8 * qs + kb * 32));
+        }
+      }
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        const int i = r * 16 + hf * 8 + g, lim = pos0 + t0 + i;
+        const float2 st = ml[h * TQ + i];
+        uint32_t* out = P + (size_t)h * geo.head_words + i * kPStride + 2 * t;
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) {
+          const int j = j0 + nt * 8 + 2 * t;
+          const float w0 = j <= lim ? exp2f(s[nt][2 * hf] * scale2 - st.x) * st.y : 0.0f;
+          const float w1 = j + 1 <= lim ? exp2f(s[nt][2 * hf + 1] * scale2 - st.x) * st.y : 0.0f;
+          *reinterpret_cast<uint2*>(out + nt * 8) = make_uint2(split_word(w0), split_word(w1));
+        }
+      }
+    }
+    __syncthreads();
+    if (c + 1 < c1) copy_k(c + 1);
+    else cp_async_commit();  // an empty group keeps the count below the same
+    // mixing: (token, key octet) tiles of 8 columns
+    for (int n = warp; n < TQ * 4; n += kValWarps) {
+      const int i = n / 4, j = n % 4 * 8;
+      const uint32_t* col = P + i * kPStride + j + g;
+      for (int mt = 0; mt < m_tiles; ++mt) {
+        float d[4] = {};
+        for (int k = 0; k < k_steps; ++k) {
+          uint32_t w[4];
+#pragma unroll
+          for (int f = 0; f < 4; ++f) {
+            const int h = k * 16 + 2 * t + (f & 1) + (f >> 1) * 8;
+            w[f] = h < H ? col[(size_t)h * geo.head_words] : 0u;
+          }
+          const uint32_t bh0 = __byte_perm(w[0], w[1], 0x5410), bl0 = __byte_perm(w[0], w[1], 0x7632);
+          const uint32_t bh1 = __byte_perm(w[2], w[3], 0x5410), bl1 = __byte_perm(w[2], w[3], 0x7632);
+          const uint4 ah4 = T[2 * ((mt * k_steps + k) * 32 + lane)], al4 = T[2 * ((mt * k_steps + k) * 32 + lane) + 1];
+          const uint32_t ah[4] = {ah4.x, ah4.y, ah4.z, ah4.w}, al[4] = {al4.x, al4.y, al4.z, al4.w};
+          mma_bf16_16816(d, ah, bh0, bh1);
+          mma_bf16_16816(d, ah, bl0, bl1);
+          mma_bf16_16816(d, al, bh0, bh1);
+        }
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          const int o = mt * 16 + g + 8 * hf;
+          if (o < HO)
+            *reinterpret_cast<__nv_bfloat162*>(W + (size_t)o * geo.out_stride + i * kKeys + j + 2 * t) =
+                __floats2bfloat162_rn(d[2 * hf], d[2 * hf + 1]);
+        }
+      }
+    }
+    cp_async_wait<1>();
+    __syncthreads();  // V of this tile and the mixed weights are here
+    if (live) {
+      const bf16* w = W + (size_t)ho * geo.out_stride + (rg * 16 + g) * kKeys + t * 8;
+      const uint4 a0 = ld16(w), a1 = ld16(w + 8 * kKeys);
+      const bf16* V = v_sm + ((size_t)((ho0 + ho) / group - gv0) * kv.v_dim + v0 + g) * kKeys + t * 8;
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (i < nvt) mma_pair(acc[i], a0, a1, ld16(V + i * 8 * kKeys));
+    }
+  }
+  auto store = [&](int wp, int nt, int ln, float4 v) {  // the fragment of lane `ln` of warp `wp`, value tile nt
+    const int r = wp % RG, vch = wp / RG % geo.vchunks, o = wp / (RG * geo.vchunks), gg = ln >> 2, tt = ln & 3;
+    if (o >= HO || ho0 + o >= H) return;
+    const int d = vch * 128 + nt * 8 + 2 * tt;
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int i = r * 16 + hf * 8 + gg;
+      if (i >= tokens) continue;
+      bf16* out = static_cast<bf16*>(p.out) + (size_t)(start + t0 + i) * p.ld_out + (size_t)(ho0 + o) * p.vdim + d;
+      if (d < p.vdim) out[0] = __float2bfloat16_rn(hf ? v.z : v.x);
+      if (d + 1 < p.vdim) out[1] = __float2bfloat16_rn(hf ? v.w : v.y);
+    }
+  };
+  if (cluster == 1) {
+#pragma unroll
+    for (int nt = 0; nt < 16; ++nt)
+      if (nt < nvt) store(warp, nt, lane, make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]));
+    return;
+  }
+  float4* red = reinterpret_cast<float4*>(smem);  // [16 warps][4][32 lanes]
+  cp_async_wait<0>();
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    if (q * 32 >= kv.v_dim) break;  // uniform: no warp holds further columns
+    __syncthreads();
+    cluster_barrier();  // everyone is done with its tiles / with reading the previous quarter
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      red[(warp * 4 + i) * 32 + lane] = make_float4(acc[4 * q + i][0], acc[4 * q + i][1], acc[4 * q + i][2], acc[4 * q + i][3]);
+    __syncthreads();
+    cluster_barrier();
+    for (int e = rank * (kValWarps * 32) + threadIdx.x; e < kValWarps * 4 * 32; e += cluster * kValWarps * 32) {
+      float4 v = make_float4(0, 0, 0, 0);
+      for (int r = 0; r < cluster; ++r) {
+        const float4 x = ld_cluster_f32x4(smem_u32(red + e), uint32_t(r));
+        v.x += x.x, v.y += x.y, v.z += x.z, v.w += x.w;
+      }
+      const int wp = e / 128, nt = 4 * q + e / 32 % 4, vch = wp / RG % geo.vchunks;
+      if (vch * 128 + nt * 8 < kv.v_dim) store(wp, nt, e % 32, v);
+    }
+  }
+  __syncthreads();
+  cluster_barrier();  // nobody leaves while its shared memory is being read
+}
+
 // ---- host -----------------------------------------------------------------------------------------------------------------------
 size_t val_smem(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv, const ValGeom& g) {
   const size_t H = size_t(p.heads), TQ = 16 * size_t(g.row_groups), HO = size_t(g.out_heads);
@@ -571,6 +821,44 @@ bool val_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv, 
     for (int q : {1, 0}) {
       g.q_in_smem = q;
       if (val_smem(p, kv, g) <= limit) {
+        *out = g;
+        return true;
+      }
+    }
+  }
+  return false;
+}
+
+bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv, TileGeom* out) {
+  TileGeom g{};
+  const int H = p.heads, group = H / kv.kv_heads;
+  g.vchunks = (kv.v_dim + 127) / 128;
+  if (g.vchunks > kValWarps) return false;
+  for (int rg : {4, 2, 1}) {
+    if (rg > 1 && rg * g.vchunks * H > kValWarps) continue;  // few heads: more tokens per CTA instead
+    g.row_groups = rg;
+    g.out_heads = std::max(1, std::min(H, kValWarps / (rg * g.vchunks)));
+    g.v_heads = std::min(kv.kv_heads, (g.out_heads + group - 2) / group + 1);
+    const int TQ = 16 * rg;
+    g.head_words = TQ * kPStride + 4;
+    g.out_stride = TQ * kKeys + 8;
+    for (int q : {1, 0}) {
+      int at = 0;
+      auto take = [&](int bytes) {
+        const int here = at;
+        at = (at + bytes + 127) / 128 * 128;
+        return here;
+      };
+      g.k = take(kv.kv_heads * kKeys * tile_stride(kv.k_dim) * 2);
+      g.v = take(g.v_heads * kv.v_dim * kKeys * 2);
+      g.p = take(H * g.head_words * 4);
+      g.w = take(g.out_heads * g.out_stride * 2);
+      g.t = take((g.out_heads + 15) / 16 * ((H + 15) / 16) * 32 * 32);
+      g.ml = take(H * TQ * 8);
+      g.q_in_smem = q;
+      g.q = take(q ? H * TQ * tile_stride(kv.k_dim) * 2 : 0);
+      g.bytes = std::max(at, kValWarps * 4 * 32 * 16);  // the cluster's reduction reuses the space
+      if (g.bytes <= max_optin_smem()) {
         *out = g;
         return true;
       }
@@ -603,7 +891,8 @@ int launch_decode_values_v(const q38_mixed_attention_params& p, const q38_batch_
 
 bool mixed_prefill_mma_fits(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv) {
   ValGeom g;
-  return p.heads / kv.kv_heads <= kStatRows && kv.k_dim <= 256 && val_geom(p, kv, &g);
+  TileGeom t;
+  return p.heads / kv.kv_heads <= kStatRows && kv.k_dim <= 256 && (tile_geom(p, kv, &t) || val_geom(p, kv, &g));
 }
 
 int mixed_prefill_mma(const q38_mixed_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
@@ -618,14 +907,43 @@ int mixed_prefill_mma(const q38_mixed_attention_params& p, const q38_batch_desc&
   (void)launch_kernel(mixed_prefill_stats_kernel, dim3(tiles, kv.kv_heads * splits, b.num_seqs), dim3(kStatWarps * 32), smem, s, p, b,
                       kv, tile, splits);
   Q38_LAUNCH_OK("mixed_prefill_stats_kernel");
+  TileGeom tg;
+  if (tile_geom(p, kv, &tg)) {
+    static const cudaError_t attr3 = cudaFuncSetAttribute(mixed_prefill_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+    Q38_CUDA_OK(attr3);
+    const int TQ = 16 * tg.row_groups, q_tiles = (b.max_tokens_per_seq + TQ - 1) / TQ, hb = (p.heads + tg.out_heads - 1) / tg.out_heads;
+    int cluster = 1;
+    while (cluster < 8 && q_tiles * hb * b.num_seqs * cluster < 2 * num_sms()) cluster *= 2;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(q_tiles * cluster, hb, b.num_seqs);
+    cfg.blockDim = dim3(kValWarps * 32);
+    cfg.dynamicSmemBytes = size_t(tg.bytes);
+    cfg.stream = s;
+    cudaLaunchAttribute attrs[2];
+    int n = 0;
+    if (dependent_launch_allowed()) {
+      attrs[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+      attrs[n++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 1) {
+      attrs[n].id = cudaLaunchAttributeClusterDimension;
+      attrs[n].val.clusterDim.x = unsigned(cluster);
+      attrs[n].val.clusterDim.y = 1;
+      attrs[n++].val.clusterDim.z = 1;
+    }
+    cfg.attrs = attrs;
+    cfg.numAttrs = unsigned(n);
+    Q38_CUDA_OK(cudaLaunchKernelEx(&cfg, mixed_prefill_values_kernel, p, b, kv, tg, splits, cluster));
+    return Q38_OK;
+  }
   ValGeom g;
   Q38_REQUIRE(val_geom(p, kv, &g), "mixed_attention: shape does not fit");
-  static const cudaError_t attr2 = cudaFuncSetAttribute(mixed_prefill_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+  static const cudaError_t attr2 = cudaFuncSetAttribute(mixed_prefill_direct_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
   Q38_CUDA_OK(attr2);
   const int TQ = 16 * g.row_groups;
-  (void)launch_kernel(mixed_prefill_values_kernel, dim3((b.max_tokens_per_seq + TQ - 1) / TQ, (p.heads + g.out_heads - 1) / g.out_heads, b.num_seqs),
+  (void)launch_kernel(mixed_prefill_direct_kernel, dim3((b.max_tokens_per_seq + TQ - 1) / TQ, (p.heads + g.out_heads - 1) / g.out_heads, b.num_seqs),
                       dim3(kValWarps * 32), val_smem(p, kv, g), s, p, b, kv, g, splits);
-  Q38_LAUNCH_OK("mixed_prefill_values_kernel");
+  Q38_LAUNCH_OK("mixed_prefill_direct_kernel");
   return Q38_OK;
 }
 

@@ -239,12 +239,65 @@ rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_s
   pdl_wait();
   pdl_launch_dependents();
   const int n = min(kMmaTokens, batch.num_tokens - t0);
-  for (int i = threadIdx.x; i < kMmaTokens * ld; i += blockDim.x) {
-    const int tok = i / ld, k = i % ld;
-    const float u = tok < n && k < bs ? conv_at<__nv_bfloat16>(p, batch, st.conv, st.slot_bytes, t0 + tok, blk * bs + k) : 0.0f;
-    const __nv_bfloat16 h = __float2bfloat16_rn(u);
-    hi[tok * us + k] = h;
-    lo[tok * us + k] = __float2bfloat16_rn(u - __bfloat162float(h));
+  __shared__ int tok_pos[kMmaTokens], tok_pos0[kMmaTokens];
+  __shared__ const __nv_bfloat16* tok_ring[kMmaTokens];
+  if (threadIdx.x < n) {
+    const int s = batch.tok_seq[t0 + threadIdx.x] - batch.tok_seq[0];
+    tok_pos[threadIdx.x] = batch.tok_pos[t0 + threadIdx.x];
+    tok_pos0[threadIdx.x] = batch.seq_pos0[s];
+    tok_ring[threadIdx.x] = reinterpret_cast<const __nv_bfloat16*>(st.conv + (size_t)batch.seq_slot[s] * st.slot_bytes);
+  }
+  __syncthreads();
+  const __nv_bfloat16* x0 = static_cast<const __nv_bfloat16*>(p.proj) + (size_t)(batch.seq_start[0] + t0) * p.ld_proj + p.width;
+  if (bs % 8 == 0 && p.width % 8 == 0 && p.ld_proj % 8 == 0 && p.taps <= 4) {
+    // eight channels of one token at a time; all taps requested before the first is used
+    const int vecs = ld / 8;
+    for (int i = threadIdx.x; i < kMmaTokens * vecs; i += blockDim.x) {
+      const int tok = i / vecs, k = i % vecs * 8, c = blk * bs + k;
+      float u[8] = {};
+      if (tok < n && k < bs) {
+        uint4 in[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {  // j tokens back
+          in[j] = make_uint4(0, 0, 0, 0);
+          const int q = tok_pos[tok] - j;
+          if (j < p.taps && q >= 0)
+            in[j] = *reinterpret_cast<const uint4*>(q >= tok_pos0[tok] ? x0 + (ptrdiff_t)(tok - j) * p.ld_proj + c
+                                                                     : tok_ring[tok] + (size_t)(q % p.taps) * p.width + c);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) u[e] = p.conv_b[c + e];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (j < p.taps) {
+            const float* w = p.conv_w + (size_t)(p.taps - 1 - j) * p.width + c;
+            const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&in[j]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 f = __bfloat1622float2(v[e]);
+              u[2 * e] += w[2 * e] * f.x;
+              u[2 * e + 1] += w[2 * e + 1] * f.y;
+            }
+          }
+      }
+      __nv_bfloat162 h[4], l[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        h[e] = __floats2bfloat162_rn(u[2 * e], u[2 * e + 1]);
+        const float2 f = __bfloat1622float2(h[e]);
+        l[e] = __floats2bfloat162_rn(u[2 * e] - f.x, u[2 * e + 1] - f.y);
+      }
+      *reinterpret_cast<uint4*>(hi + tok * us + k) = *reinterpret_cast<const uint4*>(h);
+      *reinterpret_cast<uint4*>(lo + tok * us + k) = *reinterpret_cast<const uint4*>(l);
+    }
+  } else {
+    for (int i = threadIdx.x; i < kMmaTokens * ld; i += blockDim.x) {
+      const int tok = i / ld, k = i % ld;
+      const float u = tok < n && k < bs ? conv_at<__nv_bfloat16>(p, batch, st.conv, st.slot_bytes, t0 + tok, blk * bs + k) : 0.0f;
+      const __nv_bfloat16 h = __float2bfloat16_rn(u);
+      hi[tok * us + k] = h;
+      lo[tok * us + k] = __float2bfloat16_rn(u - __bfloat162float(h));
+    }
   }
   __syncthreads();
   if (!live) return;
@@ -282,7 +335,7 @@ template <bool DECODE>
 int launch_gates_mma(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, cudaStream_t s) {
   const int bs = p.width / p.blocks;
   const size_t smem = gates_mma_smem(p.block_ld);
-  static const cudaError_t attr = cudaFuncSetAttribute(rglru_gates_mma_kernel<DECODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+  static const cudaError_t attr = cudaFuncSetAttribute(rglru_gates_mma_kernel<DECODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
   Q38_CUDA_OK(attr);
   (void)launch_kernel(rglru_gates_mma_kernel<DECODE>, dim3((b.num_tokens + kMmaTokens - 1) / kMmaTokens, p.blocks, (bs + kMmaOut - 1) / kMmaOut),
                       dim3(kMmaWarps * 32), smem, s, p, b, st);
@@ -330,7 +383,7 @@ template <typename T>
 int launch_rglru(const q38_rglru_params& p, const q38_batch_desc& b, const q38_recurrent_state_desc& st, cudaStream_t s) {
   const bool decode = b.max_tokens_per_seq == 1;
   int rc;
-  if (sizeof(T) == 2 && gates_mma_smem(p.block_ld) <= size_t(max_optin_smem()))
+  if (sizeof(T) == 2 && gates_mma_smem(p.block_ld) <= size_t(max_optin_smem() - 1024))
     rc = decode ? launch_gates_mma<true>(p, b, st, s) : launch_gates_mma<false>(p, b, st, s);
   else
     rc = launch_gates_simt<T>(p, b, st, decode, s);

@@ -90,6 +90,7 @@ struct LayerWeightsDev {
   kernels::DenseWeight in{}, out{}, glu{}, down{};
   const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
   const float *v_mix = nullptr, *head_mix = nullptr;
+  const double* inv_freq = nullptr;
   const float *conv_w = nullptr, *conv_b = nullptr, *gate_b = nullptr, *lam = nullptr;
   const q38_bf16* gate_w = nullptr;
   int block_ld = 0;
@@ -294,6 +295,9 @@ void LayerListModel::visit_weights(DeviceArena* arena) {
     }
     if (l.mixer == MixerKind::Attention) {
       if (l.attn.value_mix) W.v_mix = put_f32(arena, mix(i, "vmix"));
+      std::vector<double> freq(size_t(l.attn.rot_dims / 2));
+      for (size_t k = 0; k < freq.size(); ++k) freq[k] = std::pow(l.attn.rot_base, -2.0 * double(k) / double(l.attn.rot_dims));
+      W.inv_freq = put(arena, freq);
       if (l.attn.head_mix) W.head_mix = put_f32(arena, mix(i, "talk"));
     }
     if (l.mixer == MixerKind::RgLru) {
@@ -371,7 +375,7 @@ void LayerListModel::attention(const StepContext& ctx, const StepBatch& b, const
   rp.dim = a.dim;
   rp.vdim = a.vdim;
   rp.rot_dims = a.rot_dims;
-  rp.rot_base = a.rot_base;
+  rp.inv_freq = W.inv_freq;
   rp.q_out = q_;
   rp.v_first_out = first_values ? v_first_ : nullptr;
   rp.v_first_in = blend ? v_first_ : nullptr;

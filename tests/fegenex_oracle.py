@@ -63,7 +63,7 @@ def mixed_head_attention(q, k, v, scale, talk):
 
 
 def blend_values(v, v_first, lam):
-    return (1.0 - lam) * v + lam * v_first
+    return (1.0 - lam) * v + lam * v_first.reshape(v.shape)  # the token's values as one vector, however cut into heads
 
 
 def min_gru(h, Wz, bz, Wx, bx, Wg, Wo, state=None):
