@@ -28,7 +28,7 @@ __device__ __forceinline__ const T* v_col(const q38_kv_layer_desc& kv, int page,
 // One CTA per token. The angle position * inv_freq[i] is formed and reduced in double precision, so that far
 // positions keep the accuracy of near ones; its sine and cosine are fp32.
 template <typename T>
-__global__ void __launch_bounds__(128) rope_append_kernel(q38_rope_append_params p, q38_batch_desc b, q38_kv_layer_desc kv) {
+__global__ void __launch_bounds__(256) rope_append_kernel(q38_rope_append_params p, q38_batch_desc b, q38_kv_layer_desc kv) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ float trig[];  // [rot_dims / 2][cos, sin]
@@ -51,23 +51,28 @@ __global__ void __launch_bounds__(128) rope_append_kernel(q38_rope_append_params
     return;
   }
   uint8_t* base = kv.pages + (size_t)page * kv.page_bytes;
-  auto turned = [&](const T* h, int d) -> float {
-    if (d >= p.dim) return 0.0f;
-    const float x = to_f32(h[d]);
-    if (d >= 2 * half) return x;
-    const int i = d < half ? d : d - half;
-    const float cs = trig[2 * i], sn = trig[2 * i + 1];
-    return d < half ? x * cs - to_f32(h[d + half]) * sn : x * cs + to_f32(h[d - half]) * sn;
+  // one warp per query or key head
+  auto turn_head = [&](const T* h, T* out) {
+    for (int d = threadIdx.x & 31; d < kv.k_dim; d += 32) {
+      float y = 0.0f;
+      if (d < p.dim) {
+        y = to_f32(h[d]);
+        if (d < 2 * half) {
+          const int i = d < half ? d : d - half;
+          const float cs = trig[2 * i], sn = trig[2 * i + 1];
+          y = d < half ? y * cs - to_f32(h[d + half]) * sn : y * cs + to_f32(h[d - half]) * sn;
+        }
+      }
+      out[d] = from_f32<T>(y);
+    }
   };
+  const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   T* q = static_cast<T*>(p.q_out) + (size_t)m * p.heads * kv.k_dim;
-  for (int i = threadIdx.x; i < p.heads * kv.k_dim; i += blockDim.x) {
-    const int h = i / kv.k_dim, d = i % kv.k_dim;
-    q[i] = from_f32<T>(turned(row + (size_t)h * p.dim, d));
-  }
   const T* krow = row + (size_t)p.heads * p.dim;
-  for (int i = threadIdx.x; i < p.kv_heads * kv.k_dim; i += blockDim.x) {
-    const int h = i / kv.k_dim, d = i % kv.k_dim;
-    reinterpret_cast<T*>(base)[((size_t)h * Q38_PAGE_TOKENS + at) * kv.k_dim + d] = from_f32<T>(turned(krow + (size_t)h * p.dim, d));
+  for (int h = warp; h < p.heads + p.kv_heads; h += warps) {
+    const bool key = h >= p.heads;
+    turn_head(row + (size_t)h * p.dim, key ? reinterpret_cast<T*>(base) + ((size_t)(h - p.heads) * Q38_PAGE_TOKENS + at) * kv.k_dim
+                                           : q + (size_t)h * kv.k_dim);
   }
   const T* vrow = krow + (size_t)p.kv_heads * p.dim;
   T* vbase = reinterpret_cast<T*>(base) + (size_t)p.kv_heads * Q38_PAGE_TOKENS * kv.k_dim;
@@ -75,17 +80,17 @@ __global__ void __launch_bounds__(128) rope_append_kernel(q38_rope_append_params
   T* first_out = static_cast<T*>(p.v_first_out);
   const float lam = first_in ? *p.v_mix : 0.0f;
   const size_t vw = (size_t)p.kv_heads * p.vdim;
-  for (int i = threadIdx.x; i < p.kv_heads * kv.v_dim; i += blockDim.x) {
-    const int h = i / kv.v_dim, d = i % kv.v_dim;
-    float v = 0.0f;
-    if (d < p.vdim) {
-      const size_t c = (size_t)h * p.vdim + d;
-      v = to_f32(vrow[c]);
-      if (first_out) first_out[(size_t)m * vw + c] = from_f32<T>(v);
-      if (first_in) v = (1.0f - lam) * v + lam * to_f32(first_in[(size_t)m * vw + c]);
+  for (int h = warp; h < p.kv_heads; h += warps)
+    for (int d = threadIdx.x & 31; d < kv.v_dim; d += 32) {
+      float v = 0.0f;
+      if (d < p.vdim) {
+        const size_t c = (size_t)h * p.vdim + d;
+        v = to_f32(vrow[c]);
+        if (first_out) first_out[(size_t)m * vw + c] = from_f32<T>(v);
+        if (first_in) v = (1.0f - lam) * v + lam * to_f32(first_in[(size_t)m * vw + c]);
+      }
+      vbase[((size_t)h * kv.v_dim + d) * Q38_PAGE_TOKENS + at] = from_f32<T>(v);
     }
-    vbase[(size_t)i * Q38_PAGE_TOKENS + at] = from_f32<T>(v);
-  }
 }
 
 // ---- general attention ---------------------------------------------------------------------------------------------------
@@ -251,9 +256,9 @@ extern "C" int q38_rope_append(const q38_rope_append_params* p, const q38_batch_
   Q38_REQUIRE(!p->v_first_in || p->v_mix, "rope_append: v_mix");
   const size_t smem = size_t(std::max(1, p->rot_dims)) * 4;
   if (p->act == Q38_ACT_BF16)
-    (void)launch_kernel(rope_append_kernel<__nv_bfloat16>, dim3(batch->num_tokens), dim3(128), smem, as_stream(stream), *p, *batch, *kv);
+    (void)launch_kernel(rope_append_kernel<__nv_bfloat16>, dim3(batch->num_tokens), dim3(256), smem, as_stream(stream), *p, *batch, *kv);
   else
-    (void)launch_kernel(rope_append_kernel<float>, dim3(batch->num_tokens), dim3(128), smem, as_stream(stream), *p, *batch, *kv);
+    (void)launch_kernel(rope_append_kernel<float>, dim3(batch->num_tokens), dim3(256), smem, as_stream(stream), *p, *batch, *kv);
   Q38_LAUNCH_OK("rope_append_kernel");
   return Q38_OK;
 }

@@ -45,6 +45,11 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // merge of two (maximum, sum) pairs in base 2
 __device__ __forceinline__ void merge_ml(float& m, float& l, float m2, float l2) {
   const float nm = fmaxf(m, m2);
@@ -124,8 +129,8 @@ mixed_decode_scores_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
         float sum = 0.0f;
         if (mx != -INFINITY) {
 #pragma unroll
-          for (int nt = 0; nt < 8; ++nt) sum += exp2f(acc[nt][2 * hf] - mx) + exp2f(acc[nt][2 * hf + 1] - mx);
-          l[hf] = (m[hf] == -INFINITY ? 0.0f : l[hf] * exp2f(m[hf] - mx)) + sum;
+          for (int nt = 0; nt < 8; ++nt) sum += ex2(acc[nt][2 * hf] - mx) + ex2(acc[nt][2 * hf + 1] - mx);
+          l[hf] = (m[hf] == -INFINITY ? 0.0f : l[hf] * ex2(m[hf] - mx)) + sum;
           m[hf] = mx;
         }
         const int rr = g + 8 * hf;
@@ -202,7 +207,7 @@ mixed_decode_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
     float2 w[GROUP] = {};
     for (int h = 0; h < H; ++h) {
       const float2 s = S[h * (kPage / 2)];
-      const float mx = mx_sm[h], e0 = exp2f(s.x - mx), e1 = exp2f(s.y - mx);
+      const float mx = mx_sm[h], e0 = ex2(s.x - mx), e1 = ex2(s.y - mx);
 #pragma unroll
       for (int o = 0; o < GROUP; ++o) {
         const float f = t_sm[h * GROUP + o];
@@ -278,19 +283,18 @@ mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
   const int head = blockIdx.y / splits, split = blockIdx.y % splits, seq = blockIdx.z;
   const int group = p.heads / kv.kv_heads;
   const int start = b.seq_start[seq], count = b.seq_start[seq + 1] - start, pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
-  const int t0 = blockIdx.x * tile_tokens;
+  const int t0 = (int(gridDim.x) - 1 - int(blockIdx.x)) * tile_tokens;  // the longest tiles first
   if (t0 >= count) return;
   const int tokens = min(tile_tokens, count - t0);
   const int last = pos0 + t0 + tokens - 1, pages = last / kPage + 1;
   const int per = (pages + splits - 1) / splits, p0 = min(pages, split * per), p1 = min(pages, p0 + per);
   const int* table = kv.block_table + (size_t)slot * kv.max_pages_per_seq;
+  const int k_row = threadIdx.x >> 4, k_chunk = threadIdx.x & 15;  // half a warp per key row
   auto stage = [&](int pg) {
-    const bf16* K = k_page(kv, table[pg], head);
-    bf16* dst = k_sm + ((pg - p0) & 1) * kPage * ks;
-    for (int i = threadIdx.x; i < kPage * chunks; i += blockDim.x) {
-      const int rr = i / chunks, c = i % chunks;
-      cp_async16(dst + rr * ks + c * 8, K + (size_t)rr * kv.k_dim + c * 8);
-    }
+    const bf16* src = k_page(kv, table[pg], head) + (size_t)k_row * kv.k_dim;
+    bf16* dst = k_sm + (((pg - p0) & 1) * kPage + k_row) * ks;
+    for (int r = k_row; r < kPage; r += kStatWarps * 2, src += kStatWarps * 2 * kv.k_dim, dst += kStatWarps * 2 * ks)
+      for (int c = k_chunk; c < chunks; c += 16) cp_async16(dst + c * 8, src + c * 8);
     cp_async_commit();
   };
   if (p0 < p1) stage(p0);
@@ -354,8 +358,8 @@ mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
         if (mx == -INFINITY) continue;
         float sum = 0.0f;
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) sum += exp2f(acc[mt][nt][2 * hf] - mx) + exp2f(acc[mt][nt][2 * hf + 1] - mx);
-        l[mt][hf] = (m[mt][hf] == -INFINITY ? 0.0f : l[mt][hf] * exp2f(m[mt][hf] - mx)) + sum;
+        for (int nt = 0; nt < 8; ++nt) sum += ex2(acc[mt][nt][2 * hf] - mx) + ex2(acc[mt][nt][2 * hf + 1] - mx);
+        l[mt][hf] = (m[mt][hf] == -INFINITY ? 0.0f : l[mt][hf] * ex2(m[mt][hf] - mx)) + sum;
         m[mt][hf] = mx;
       }
     __syncthreads();
@@ -584,11 +588,22 @@ __device__ __forceinline__ uint32_t split_word(float x) {
   return uint32_t(__bfloat16_as_ushort(h)) | uint32_t(__bfloat16_as_ushort(l)) << 16;
 }
 
+// two values as (hi, lo) words
+__device__ __forceinline__ uint2 split_words(float a, float b) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const uint32_t hw = *reinterpret_cast<const uint32_t*>(&h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - __uint_as_float(hw << 16), b - __uint_as_float(hw & 0xffff0000u));
+  const uint32_t lw = *reinterpret_cast<const uint32_t*>(&l);
+  return make_uint2(__byte_perm(hw, lw, 0x5410), __byte_perm(hw, lw, 0x7632));
+}
+
+constexpr int kMaxMixHeads = 256;
 __global__ void __launch_bounds__(kValWarps * 32, 1)
 mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, TileGeom geo, int splits, int cluster) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ uint8_t kv_of[kMaxMixHeads];  // kv head of a query head
   const int H = p.heads, G = kv.kv_heads, RG = geo.row_groups, TQ = 16 * RG, HO = geo.out_heads, group = H / G;
   const int qs = tile_stride(kv.k_dim), kb_n = kv.k_dim / 32, k_steps = (H + 15) / 16, m_tiles = (HO + 15) / 16;
   bf16* k_sm = reinterpret_cast<bf16*>(smem + geo.k);            // [G][32][qs]
@@ -608,25 +623,24 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   const int key_tiles = last / kKeys + 1, c0 = rank * key_tiles / cluster, c1 = (rank + 1) * key_tiles / cluster;
   const int gv0 = ho0 / group, gv1 = min(G, (ho0 + HO - 1) / group + 1);
 
+  // half a warp per key row, one kv head per turn; V rows of 32 keys are four 16-byte pieces
+  const int k_row = warp * 2 + (lane >> 4), k_chunk = lane & 15, k_chunks = kv.k_dim / 8;
   auto copy_k = [&](int c) {
-    const int page = table[c / 2], chunks = kv.k_dim / 8, rows = kKeys * chunks;
-    for (int hd = 0; hd < G; ++hd) {
-      const bf16* src = k_page(kv, page, hd) + (size_t)(c % 2) * kKeys * kv.k_dim;
-      bf16* dst = k_sm + (size_t)hd * kKeys * qs;
-      for (int i = threadIdx.x; i < rows; i += blockDim.x) cp_async16(dst + i / chunks * qs + i % chunks * 8, src + (size_t)i * 8);
-    }
+    const bf16* src = k_page(kv, table[c / 2], 0) + (size_t)((c % 2) * kKeys + k_row) * kv.k_dim;
+    bf16* dst = k_sm + k_row * qs;
+    for (int hd = 0; hd < G; ++hd, src += (size_t)kPage * kv.k_dim, dst += kKeys * qs)
+      for (int ch = k_chunk; ch < k_chunks; ch += 16) cp_async16(dst + ch * 8, src + ch * 8);
     cp_async_commit();
   };
   auto copy_v = [&](int c) {
-    const int page = table[c / 2];
-    for (int hd = gv0; hd < gv1; ++hd) {
-      const bf16* src = v_page(kv, page, hd) + (size_t)(c % 2) * kKeys;
-      bf16* dst = v_sm + (size_t)(hd - gv0) * kv.v_dim * kKeys;
-      for (int i = threadIdx.x; i < kv.v_dim * 4; i += blockDim.x) cp_async16(dst + i * 8, src + (size_t)(i / 4) * kPage + i % 4 * 8);
-    }
+    const int rows = (gv1 - gv0) * kv.v_dim;  // consecutive heads' rows are consecutive in the page and here
+    const bf16* src = v_page(kv, table[c / 2], gv0) + (size_t)(c % 2) * kKeys + (threadIdx.x & 3) * 8;
+    for (int r = threadIdx.x >> 2; r < rows; r += kValWarps * 8) cp_async16(v_sm + r * kKeys + (threadIdx.x & 3) * 8, src + (size_t)r * kPage);
     cp_async_commit();
   };
   if (c0 < c1) copy_k(c0);
+  const int rg_shift = RG == 4 ? 2 : RG == 2 ? 1 : 0;
+  for (int h = threadIdx.x; h < H; h += blockDim.x) kv_of[h] = uint8_t(h / group);
 
   const bf16* qg = static_cast<const bf16*>(p.q) + (size_t)(start + t0) * H * kv.k_dim;
   const size_t i0 = size_t(start - b.seq_start[0] + t0);
@@ -669,15 +683,17 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   const int rg = warp % RG, vc = warp / RG % geo.vchunks, ho = warp / (RG * geo.vchunks);
   const bool live = ho < HO && ho0 + ho < H;
   const int v0 = vc * 128, nvt = live ? min(16, (kv.v_dim - v0) / 8) : 0;
+  const bf16* V = v_sm + (live ? ((ho0 + ho) / group - gv0) * kv.v_dim + v0 + g : 0) * kKeys + t * 8;
   float acc[16][4] = {};
   for (int c = c0; c < c1; ++c) {
     const int j0 = c * kKeys;
     cp_async_wait<0>();
     __syncthreads();  // K of this tile is here; the previous tile's weights and values are done with
     copy_v(c);
-    for (int u = warp; u < H * RG; u += kValWarps) {
-      const int h = u / RG, r = u % RG;
-      const bf16* K = k_sm + ((size_t)(h / group) * kKeys + g) * qs + t * 8;
+    const bool edge = j0 + kKeys - 1 > pos0 + t0;  // some row of the tile ends inside these keys
+    for (int u = warp; u < H << rg_shift; u += kValWarps) {
+      const int h = u >> rg_shift, r = u & (RG - 1);
+      const bf16* K = k_sm + (kv_of[h] * kKeys + g) * qs + t * 8;
       float s[4][4] = {};
       if (geo.q_in_smem) {
         const bf16* Q = q_sm + ((size_t)h * TQ + r * 16 + g) * qs + t * 8;
@@ -701,15 +717,17 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
       }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int i = r * 16 + hf * 8 + g, lim = pos0 + t0 + i;
+        const int i = r * 16 + hf * 8 + g, lim = pos0 + t0 + i - j0 - 2 * t;
         const float2 st = ml[h * TQ + i];
-        uint32_t* out = P + (size_t)h * geo.head_words + i * kPStride + 2 * t;
+        uint32_t* out = P + h * geo.head_words + i * kPStride + 2 * t;
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
-          const int j = j0 + nt * 8 + 2 * t;
-          const float w0 = j <= lim ? exp2f(s[nt][2 * hf] * scale2 - st.x) * st.y : 0.0f;
-          const float w1 = j + 1 <= lim ? exp2f(s[nt][2 * hf + 1] * scale2 - st.x) * st.y : 0.0f;
-          *reinterpret_cast<uint2*>(out + nt * 8) = make_uint2(split_word(w0), split_word(w1));
+          float w0 = ex2(fmaf(s[nt][2 * hf], scale2, -st.x)) * st.y, w1 = ex2(fmaf(s[nt][2 * hf + 1], scale2, -st.x)) * st.y;
+          if (edge) {
+            if (nt * 8 > lim) w0 = 0.0f;
+            if (nt * 8 + 1 > lim) w1 = 0.0f;
+          }
+          *reinterpret_cast<uint2*>(out + nt * 8) = split_words(w0, w1);
         }
       }
     }
@@ -727,7 +745,7 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
 #pragma unroll
           for (int f = 0; f < 4; ++f) {
             const int h = k * 16 + 2 * t + (f & 1) + (f >> 1) * 8;
-            w[f] = h < H ? col[(size_t)h * geo.head_words] : 0u;
+            w[f] = h < H ? col[h * geo.head_words] : 0u;
           }
           const uint32_t bh0 = __byte_perm(w[0], w[1], 0x5410), bl0 = __byte_perm(w[0], w[1], 0x7632);
           const uint32_t bh1 = __byte_perm(w[2], w[3], 0x5410), bl1 = __byte_perm(w[2], w[3], 0x7632);
@@ -741,7 +759,7 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
         for (int hf = 0; hf < 2; ++hf) {
           const int o = mt * 16 + g + 8 * hf;
           if (o < HO)
-            *reinterpret_cast<__nv_bfloat162*>(W + (size_t)o * geo.out_stride + i * kKeys + j + 2 * t) =
+            *reinterpret_cast<__nv_bfloat162*>(W + o * geo.out_stride + i * kKeys + j + 2 * t) =
                 __floats2bfloat162_rn(d[2 * hf], d[2 * hf + 1]);
         }
       }
@@ -751,7 +769,6 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     if (live) {
       const bf16* w = W + (size_t)ho * geo.out_stride + (rg * 16 + g) * kKeys + t * 8;
       const uint4 a0 = ld16(w), a1 = ld16(w + 8 * kKeys);
-      const bf16* V = v_sm + ((size_t)((ho0 + ho) / group - gv0) * kv.v_dim + v0 + g) * kKeys + t * 8;
 #pragma unroll
       for (int i = 0; i < 16; ++i)
         if (i < nvt) mma_pair(acc[i], a0, a1, ld16(V + i * 8 * kKeys));
@@ -833,7 +850,7 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
   TileGeom g{};
   const int H = p.heads, group = H / kv.kv_heads;
   g.vchunks = (kv.v_dim + 127) / 128;
-  if (g.vchunks > kValWarps) return false;
+  if (g.vchunks > kValWarps || H > kMaxMixHeads) return false;
   for (int rg : {4, 2, 1}) {
     if (rg > 1 && rg * g.vchunks * H > kValWarps) continue;  // few heads: more tokens per CTA instead
     g.row_groups = rg;
@@ -858,7 +875,7 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
       g.q_in_smem = q;
       g.q = take(q ? H * TQ * tile_stride(kv.k_dim) * 2 : 0);
       g.bytes = std::max(at, kValWarps * 4 * 32 * 16);  // the cluster's reduction reuses the space
-      if (g.bytes <= max_optin_smem()) {
+      if (g.bytes <= max_optin_smem() - 1024) {
         *out = g;
         return true;
       }
@@ -900,7 +917,7 @@ int mixed_prefill_mma(const q38_mixed_attention_params& p, const q38_batch_desc&
   const int tiles = (b.max_tokens_per_seq + tile - 1) / tile;
   // the keys of a tile are cut over several CTAs when the tiles alone leave most of the GPU idle
   const int ctas = tiles * kv.kv_heads * b.num_seqs;
-  const int splits = std::max(1, std::min({p.stat_splits, 2 * num_sms() / ctas, 8}));
+  const int splits = std::max(1, std::min({p.stat_splits, 5 * num_sms() / ctas, 8}));
   const size_t smem = size_t(kStatRows + 2 * kPage) * size_t(tile_stride(kv.k_dim)) * 2;
   static const cudaError_t attr = cudaFuncSetAttribute(mixed_prefill_stats_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
   Q38_CUDA_OK(attr);
@@ -909,7 +926,7 @@ int mixed_prefill_mma(const q38_mixed_attention_params& p, const q38_batch_desc&
   Q38_LAUNCH_OK("mixed_prefill_stats_kernel");
   TileGeom tg;
   if (tile_geom(p, kv, &tg)) {
-    static const cudaError_t attr3 = cudaFuncSetAttribute(mixed_prefill_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
+    static const cudaError_t attr3 = cudaFuncSetAttribute(mixed_prefill_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
     Q38_CUDA_OK(attr3);
     const int TQ = 16 * tg.row_groups, q_tiles = (b.max_tokens_per_seq + TQ - 1) / TQ, hb = (p.heads + tg.out_heads - 1) / tg.out_heads;
     int cluster = 1;

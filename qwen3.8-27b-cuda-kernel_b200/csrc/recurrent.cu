@@ -151,14 +151,21 @@ __device__ __forceinline__ float conv_at(const q38_rglru_params& p, const q38_ba
   return u;
 }
 
+struct GateConst {  // of one channel: the gates' biases and log_decay * softplus(lam)
+  float rb, ib, decay;
+};
+__device__ __forceinline__ GateConst gate_const(const q38_rglru_params& p, int c) {
+  return {p.gate_b[c], p.gate_b[p.width + c], p.log_decay * softplus_f(p.lam[c])};
+}
+
 // From the gates' pre-activations to (a, b); decode batches go on to the state and the output.
 template <typename T, bool DECODE>
 __device__ __forceinline__ void gate_finish(const q38_rglru_params& p, const q38_batch_desc& b,
-                                            const q38_recurrent_state_desc& st, int i, int c, float r_pre, float i_pre,
-                                            float u) {
+                                            const q38_recurrent_state_desc& st, int i, int c, float r_pre, float i_pre, float u,
+                                            const GateConst& k) {
   const int t = b.seq_start[0] + i;
-  const float r = sigmoid_f(r_pre + p.gate_b[c]), gi = sigmoid_f(i_pre + p.gate_b[p.width + c]);
-  const float log_a = p.log_decay * r * softplus_f(p.lam[c]);
+  const float r = sigmoid_f(r_pre + k.rb), gi = sigmoid_f(i_pre + k.ib);
+  const float log_a = k.decay * r;
   const float a = expf(log_a);
   const float x = sqrtf(-expm1f(2.0f * log_a)) * gi * u;
   if (!DECODE) {
@@ -212,14 +219,14 @@ rglru_gates_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_state
 #pragma unroll
       for (int q = 0; q < kGateTokens; ++q)
         if (q == t) r = ar[q], gi = ai[q];
-      gate_finish<T, DECODE>(p, batch, st, t0 + t, blk * bs + o, r, gi, u_sm[t * p.block_ld + o]);
+      gate_finish<T, DECODE>(p, batch, st, t0 + t, blk * bs + o, r, gi, u_sm[t * p.block_ld + o], gate_const(p, blk * bs + o));
     }
   }
 }
 
 // Tensor-core form (bf16 activations): a CTA holds the convolved inputs of 32 tokens x one block in shared memory, as
-// bf16 terms hi + lo, and makes 64 output channels of both gates: a warp the 8 channels of one n tile, r and i side by
-// side in its registers. Weights come straight from global memory into fragments (16 contiguous bytes of a row = two k16
+// bf16 terms hi + lo, and makes output channels of both gates, 64 at a time: a warp the 8 channels of one n tile, r and i
+// side by side in its registers. Weights come straight from global memory into fragments (16 contiguous bytes of a row = two k16
 // steps under a permutation of k that both operands share).
 constexpr int kMmaTokens = 32, kMmaWarps = 8, kMmaOut = kMmaWarps * 8;
 __host__ __device__ constexpr int gate_stride(int cols) { return cols % 64 == 32 ? cols : cols + 32; }
@@ -232,10 +239,7 @@ rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_s
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   __nv_bfloat16* hi = reinterpret_cast<__nv_bfloat16*>(smem);  // [32][us]
   __nv_bfloat16* lo = hi + kMmaTokens * us;
-  const int o0 = blockIdx.z * kMmaOut + warp * 8;
-  const bool live = o0 < ld;
-  const __nv_bfloat16* wr = reinterpret_cast<const __nv_bfloat16*>(p.gate_w) + ((size_t)blk * 2 * ld + o0 + g) * ld + t * 8;
-  const __nv_bfloat16* wi = wr + (size_t)ld * ld;
+  const __nv_bfloat16* gw = reinterpret_cast<const __nv_bfloat16*>(p.gate_w) + ((size_t)blk * 2 * ld + g) * ld + t * 8;
   pdl_wait();
   pdl_launch_dependents();
   const int n = min(kMmaTokens, batch.num_tokens - t0);
@@ -250,45 +254,53 @@ rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_s
   __syncthreads();
   const __nv_bfloat16* x0 = static_cast<const __nv_bfloat16*>(p.proj) + (size_t)(batch.seq_start[0] + t0) * p.ld_proj + p.width;
   if (bs % 8 == 0 && p.width % 8 == 0 && p.ld_proj % 8 == 0 && p.taps <= 4) {
-    // eight channels of one token at a time; all taps requested before the first is used
+    // a thread keeps the taps of eight channels in registers and takes several tokens; all inputs of a token are
+    // requested before the first is used
     const int vecs = ld / 8;
-    for (int i = threadIdx.x; i < kMmaTokens * vecs; i += blockDim.x) {
-      const int tok = i / vecs, k = i % vecs * 8, c = blk * bs + k;
-      float u[8] = {};
-      if (tok < n && k < bs) {
+    for (int kv = threadIdx.x & 31; kv < vecs; kv += 32) {
+      const int k = kv * 8, c = blk * bs + k;
+      const bool in_block = k < bs;
+      float w[4][8], bias[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        bias[e] = in_block ? p.conv_b[c + e] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j][e] = in_block && j < p.taps ? p.conv_w[(size_t)(p.taps - 1 - j) * p.width + c + e] : 0.0f;
+      }
+      for (int tok = warp; tok < kMmaTokens; tok += kMmaWarps) {
+        float u[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) u[e] = bias[e];
         uint4 in[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {  // j tokens back
           in[j] = make_uint4(0, 0, 0, 0);
-          const int q = tok_pos[tok] - j;
-          if (j < p.taps && q >= 0)
-            in[j] = *reinterpret_cast<const uint4*>(q >= tok_pos0[tok] ? x0 + (ptrdiff_t)(tok - j) * p.ld_proj + c
-                                                                     : tok_ring[tok] + (size_t)(q % p.taps) * p.width + c);
+          if (in_block && tok < n && j < p.taps) {
+            const int q = tok_pos[tok] - j;
+            if (q >= tok_pos0[tok]) in[j] = *reinterpret_cast<const uint4*>(x0 + (ptrdiff_t)(tok - j) * p.ld_proj + c);
+            else if (q >= 0) in[j] = *reinterpret_cast<const uint4*>(tok_ring[tok] + (size_t)(q % p.taps) * p.width + c);
+          }
         }
 #pragma unroll
-        for (int e = 0; e < 8; ++e) u[e] = p.conv_b[c + e];
+        for (int j = 0; j < 4; ++j) {
+          const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&in[j]);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-          if (j < p.taps) {
-            const float* w = p.conv_w + (size_t)(p.taps - 1 - j) * p.width + c;
-            const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&in[j]);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const float2 f = __bfloat1622float2(v[e]);
-              u[2 * e] += w[2 * e] * f.x;
-              u[2 * e + 1] += w[2 * e + 1] * f.y;
-            }
+          for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(v[e]);
+            u[2 * e] += w[j][2 * e] * f.x;
+            u[2 * e + 1] += w[j][2 * e + 1] * f.y;
           }
-      }
-      __nv_bfloat162 h[4], l[4];
+        }
+        __nv_bfloat162 h[4], l[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        h[e] = __floats2bfloat162_rn(u[2 * e], u[2 * e + 1]);
-        const float2 f = __bfloat1622float2(h[e]);
-        l[e] = __floats2bfloat162_rn(u[2 * e] - f.x, u[2 * e + 1] - f.y);
+        for (int e = 0; e < 4; ++e) {
+          h[e] = __floats2bfloat162_rn(u[2 * e], u[2 * e + 1]);
+          const float2 f = __bfloat1622float2(h[e]);
+          l[e] = __floats2bfloat162_rn(u[2 * e] - f.x, u[2 * e + 1] - f.y);
+        }
+        *reinterpret_cast<uint4*>(hi + tok * us + k) = *reinterpret_cast<const uint4*>(h);
+        *reinterpret_cast<uint4*>(lo + tok * us + k) = *reinterpret_cast<const uint4*>(l);
       }
-      *reinterpret_cast<uint4*>(hi + tok * us + k) = *reinterpret_cast<const uint4*>(h);
-      *reinterpret_cast<uint4*>(lo + tok * us + k) = *reinterpret_cast<const uint4*>(l);
     }
   } else {
     for (int i = threadIdx.x; i < kMmaTokens * ld; i += blockDim.x) {
@@ -300,33 +312,44 @@ rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_s
     }
   }
   __syncthreads();
-  if (!live) return;
-  float acc[2][2][4] = {};  // [16-token tile][r, i]
-  for (int k = 0; k < ld; k += 32) {
-    const uint4 w[2] = {*reinterpret_cast<const uint4*>(wr + k), *reinterpret_cast<const uint4*>(wi + k)};
+  for (int o0 = blockIdx.z * kMmaOut + warp * 8; o0 < ld; o0 += gridDim.z * kMmaOut) {
+    const __nv_bfloat16* wr = gw + (size_t)o0 * ld;
+    const __nv_bfloat16* wi = wr + (size_t)ld * ld;
+    float acc[2][2][4] = {};  // [16-token tile][r, i]
+#pragma unroll 4
+    for (int k = 0; k < ld; k += 32) {
+      const uint4 w[2] = {*reinterpret_cast<const uint4*>(wr + k), *reinterpret_cast<const uint4*>(wi + k)};
 #pragma unroll
-    for (int mt = 0; mt < 2; ++mt)
+      for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
-      for (int term = 0; term < 2; ++term) {
-        const __nv_bfloat16* u = (term ? lo : hi) + (mt * 16 + g) * us + k + t * 8;
-        const uint4 a0 = *reinterpret_cast<const uint4*>(u), a1 = *reinterpret_cast<const uint4*>(u + 8 * us);
-        const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
+        for (int term = 0; term < 2; ++term) {
+          const __nv_bfloat16* u = (term ? lo : hi) + (mt * 16 + g) * us + k + t * 8;
+          const uint4 a0 = *reinterpret_cast<const uint4*>(u), a1 = *reinterpret_cast<const uint4*>(u + 8 * us);
+          const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          mma_bf16_16816(acc[mt][q], f0, w[q].x, w[q].y);
-          mma_bf16_16816(acc[mt][q], f1, w[q].z, w[q].w);
+          for (int q = 0; q < 2; ++q) {
+            mma_bf16_16816(acc[mt][q], f0, w[q].x, w[q].y);
+            mma_bf16_16816(acc[mt][q], f1, w[q].z, w[q].w);
+          }
         }
-      }
-  }
-#pragma unroll
-  for (int mt = 0; mt < 2; ++mt)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int tok = mt * 16 + g + 8 * (e >> 1), o = o0 + 2 * t + (e & 1);
-      if (tok >= n || o >= bs) continue;
-      const float u = __bfloat162float(hi[tok * us + o]) + __bfloat162float(lo[tok * us + o]);
-      gate_finish<__nv_bfloat16, DECODE>(p, batch, st, t0 + tok, blk * bs + o, acc[mt][0][e], acc[mt][1][e], u);
     }
+#pragma unroll
+    for (int d = 0; d < 2; ++d) {
+      const int o = o0 + 2 * t + d;
+      if (o >= bs) continue;
+      const int c = blk * bs + o;
+      const GateConst gc = gate_const(p, c);
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          const int tok = mt * 16 + g + 8 * hf;
+          if (tok >= n) continue;
+          const float u = __bfloat162float(hi[tok * us + o]) + __bfloat162float(lo[tok * us + o]);
+          gate_finish<__nv_bfloat16, DECODE>(p, batch, st, t0 + tok, c, acc[mt][0][2 * hf + d], acc[mt][1][2 * hf + d], u, gc);
+        }
+    }
+  }
 }
 
 size_t gates_mma_smem(int block_ld) { return size_t(2) * kMmaTokens * gate_stride(block_ld) * 2; }
@@ -337,7 +360,10 @@ int launch_gates_mma(const q38_rglru_params& p, const q38_batch_desc& b, const q
   const size_t smem = gates_mma_smem(p.block_ld);
   static const cudaError_t attr = cudaFuncSetAttribute(rglru_gates_mma_kernel<DECODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
   Q38_CUDA_OK(attr);
-  (void)launch_kernel(rglru_gates_mma_kernel<DECODE>, dim3((b.num_tokens + kMmaTokens - 1) / kMmaTokens, p.blocks, (bs + kMmaOut - 1) / kMmaOut),
+  // few tokens: the output channels of a block over several CTAs; many: one CTA convolves once for all of them
+  const int tiles = (b.num_tokens + kMmaTokens - 1) / kMmaTokens;
+  const int slices = std::max(1, std::min((bs + kMmaOut - 1) / kMmaOut, 2 * num_sms() / (tiles * p.blocks)));
+  (void)launch_kernel(rglru_gates_mma_kernel<DECODE>, dim3(tiles, p.blocks, slices),
                       dim3(kMmaWarps * 32), smem, s, p, b, st);
   Q38_LAUNCH_OK("rglru_gates_mma_kernel");
   return Q38_OK;

@@ -1,6 +1,8 @@
 // RMS-norm kernels of the layer-list architectures: embedding + first norm, post-norm + residual sum + next pre-norm,
 // and the final norm of the rows the output head needs. One CTA per row; the row lives in shared memory between the
 // passes, so global memory sees each operand once. Norms, the residual and its sum are fp32.
+#include <algorithm>
+
 #include "act.cuh"
 #include "host_util.h"
 
@@ -53,47 +55,82 @@ residual_norm_kernel(const float* __restrict__ y, int ldy, int width, q38_norm p
   const float* yr = y + (size_t)m * ldy;
   float* xr = residual + (size_t)m * width;
   float ss = 0.0f;
-  const bool vec = (width & 3) == 0 && (ldy & 3) == 0;
-  if (vec) {
-    for (int i = 4 * threadIdx.x; i < width; i += 4 * blockDim.x) {
-      const float4 v = *reinterpret_cast<const float4*>(yr + i);
-      *reinterpret_cast<float4*>(row + i) = v;
-      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    }
-  } else {
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-      const float v = yr[i];
-      row[i] = v;
-      ss += v * v;
-    }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = yr[i];
+    row[i] = v;
+    ss += v * v;
   }
   const float rs = inv_rms(block_sum(ss, red), width, post.eps);
   ss = 0.0f;
-  if (vec && post.gain_stride == 0) {
-    const float g = rs * post.gain[0];
-    for (int i = 4 * threadIdx.x; i < width; i += 4 * blockDim.x) {
-      const float4 v = *reinterpret_cast<const float4*>(row + i);
-      float4 x = *reinterpret_cast<const float4*>(xr + i);
-      x.x += v.x * g;
-      x.y += v.y * g;
-      x.z += v.z * g;
-      x.w += v.w * g;
-      *reinterpret_cast<float4*>(xr + i) = x;
-      *reinterpret_cast<float4*>(row + i) = x;
-      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
-    }
-  } else {
-    __syncthreads();  // the vector pass above may have filled elements another thread reads here
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-      const float x = xr[i] + row[i] * (rs * post.gain[i * post.gain_stride]);
-      xr[i] = x;
-      row[i] = x;
-      ss += x * x;
-    }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float x = xr[i] + row[i] * (rs * post.gain[i * post.gain_stride]);
+    xr[i] = x;
+    row[i] = x;
+    ss += x * x;
   }
   if (next.gain == nullptr) return;
   const float rs2 = inv_rms(block_sum(ss, red), width, next.eps);
   store_normed(row, width, rs2, next, out + (size_t)m * ld, ld);
+}
+
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+// The same with the row in registers, 16 elements per thread (rows in whole 16-byte pieces, up to 16384 elements): both
+// operands are requested at once, and the two reductions are all that is left between them and the stores.
+constexpr int kVecs = 4;
+template <typename T>
+__global__ void __launch_bounds__(1024)
+residual_norm_vec_kernel(const float* __restrict__ y, int ldy, int width, q38_norm post, float* __restrict__ residual,
+                         q38_norm next, T* __restrict__ out, int ld) {
+  pdl_wait();
+  pdl_launch_dependents();
+  __shared__ float red[33];
+  const int m = blockIdx.x;
+  const float* yr = y + (size_t)m * ldy;
+  float* xr = residual + (size_t)m * width;
+  float4 v[kVecs], x[kVecs];
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kVecs; ++i) {
+    const int c = 4 * (threadIdx.x + i * blockDim.x);
+    v[i] = x[i] = make_float4(0, 0, 0, 0);
+    if (c < width) {
+      v[i] = *reinterpret_cast<const float4*>(yr + c);
+      x[i] = *reinterpret_cast<const float4*>(xr + c);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kVecs; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  const float rs = inv_rms(block_sum(ss, red), width, post.eps);
+  ss = 0.0f;
+  auto gains = [](const q38_norm& n, int c) {
+    return n.gain_stride ? make_float4(n.gain[c], n.gain[c + 1], n.gain[c + 2], n.gain[c + 3])
+                         : make_float4(n.gain[0], n.gain[0], n.gain[0], n.gain[0]);
+  };
+#pragma unroll
+  for (int i = 0; i < kVecs; ++i) {
+    const int c = 4 * (threadIdx.x + i * blockDim.x);
+    if (c >= width) continue;
+    const float4 g = gains(post, c);
+    x[i].x += v[i].x * (rs * g.x);
+    x[i].y += v[i].y * (rs * g.y);
+    x[i].z += v[i].z * (rs * g.z);
+    x[i].w += v[i].w * (rs * g.w);
+    *reinterpret_cast<float4*>(xr + c) = x[i];
+    ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+  }
+  if (next.gain == nullptr) return;
+  const float rs2 = inv_rms(block_sum(ss, red), width, next.eps);
+#pragma unroll
+  for (int i = 0; i < kVecs; ++i) {
+    const int c = 4 * (threadIdx.x + i * blockDim.x);
+    if (c >= width) continue;
+    const float4 g = gains(next, c);
+    store4(out + (size_t)m * ld + c, make_float4(x[i].x * rs2 * g.x, x[i].y * rs2 * g.y, x[i].z * rs2 * g.z, x[i].w * rs2 * g.w));
+  }
 }
 
 template <typename T>
@@ -154,6 +191,18 @@ extern "C" int q38_residual_norm(const float* y, int ldy, int m, int width, cons
   Q38_REQUIRE(ldy >= width, "residual_norm: ldy %d", ldy);
   const size_t smem = size_t(width) * 4;
   const q38_norm nx = next ? *next : q38_norm{nullptr, 0, 0.0f};
+  if (width % 4 == 0 && ldy % 4 == 0 && (!next || ld_out % 4 == 0) && width <= 16384 &&
+      (reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(residual) | reinterpret_cast<uintptr_t>(out)) % 16 == 0) {
+    const int threads = std::max(64, std::min(1024, (width / (4 * kVecs) + 31) / 32 * 32));
+    if (act == Q38_ACT_BF16)
+      (void)launch_kernel(residual_norm_vec_kernel<__nv_bfloat16>, dim3(m), dim3(threads), 0, as_stream(stream), y, ldy, width, *post,
+                          residual, nx, static_cast<__nv_bfloat16*>(out), ld_out);
+    else
+      (void)launch_kernel(residual_norm_vec_kernel<float>, dim3(m), dim3(threads), 0, as_stream(stream), y, ldy, width, *post, residual,
+                          nx, static_cast<float*>(out), ld_out);
+    Q38_LAUNCH_OK("residual_norm_vec_kernel");
+    return Q38_OK;
+  }
   if (act == Q38_ACT_BF16)
     (void)launch_kernel(residual_norm_kernel<__nv_bfloat16>, dim3(m), dim3(kNormThreads), smem, as_stream(stream), y, ldy, width,
                         *post, residual, nx, static_cast<__nv_bfloat16*>(out), ld_out);
