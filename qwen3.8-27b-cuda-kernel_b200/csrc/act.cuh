@@ -21,6 +21,22 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
 }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
+// The A fragments of two k16 steps of mma.m16n8k16 from 16 contiguous bytes of rows g and g + 8. An MMA takes its four A
+// registers as one aligned group, and the compiler would regroup the loaded registers anew for every MMA that uses the
+// fragment; the OR with a zero it cannot see (blocks here have one layer in z) makes the group a value of its own.
+struct AFragPair {
+  uint32_t f0[4], f1[4];
+};
+__device__ __forceinline__ uint32_t pinned(uint32_t x) { return x | (blockDim.z - 1u); }
+__device__ __forceinline__ AFragPair a_fragments(const uint4& r0, const uint4& r8) {
+  return {{pinned(r0.x), pinned(r8.x), pinned(r0.y), pinned(r8.y)}, {pinned(r0.z), pinned(r8.z), pinned(r0.w), pinned(r8.w)}};
+}
+// ... against 16 contiguous bytes of a row of B
+__device__ __forceinline__ void mma_pair(float (&d)[4], const AFragPair& a, const uint4& b) {
+  mma_bf16_16816(d, a.f0, b.x, b.y);
+  mma_bf16_16816(d, a.f1, b.z, b.w);
+}
+
 // Sum over the CTA's threads (a multiple of 32, at most 1024); every thread gets the result. `red` holds 33 floats.
 __device__ __forceinline__ float block_sum(float v, float* red) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;

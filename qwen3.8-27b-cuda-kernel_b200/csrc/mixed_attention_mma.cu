@@ -32,12 +32,6 @@ __device__ __forceinline__ const bf16* v_page(const q38_kv_layer_desc& kv, int p
          (size_t)head * kv.v_dim * kPage;
 }
 __device__ __forceinline__ uint4 ld16(const bf16* p) { return *reinterpret_cast<const uint4*>(p); }
-// two k16 steps: rows g / g + 8 of A (16 bytes each) against one 16-byte row of B
-__device__ __forceinline__ void mma_pair(float (&d)[4], const uint4& a0, const uint4& a1, const uint4& b) {
-  const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
-  mma_bf16_16816(d, f0, b.x, b.y);
-  mma_bf16_16816(d, f1, b.z, b.w);
-}
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -110,9 +104,9 @@ mixed_decode_scores_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
         uint4 bf[8];
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) bf[nt] = ld16(K + (size_t)nt * 8 * kv.k_dim + kb * 32);
-        const uint4 a0 = ld16(q_sm + g * qs + kb * 32 + t * 8), a1 = ld16(q_sm + (g + 8) * qs + kb * 32 + t * 8);
+        const AFragPair a = a_fragments(ld16(q_sm + g * qs + kb * 32 + t * 8), ld16(q_sm + (g + 8) * qs + kb * 32 + t * 8));
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) mma_pair(acc[nt], a0, a1, bf[nt]);
+        for (int nt = 0; nt < 8; ++nt) mma_pair(acc[nt], a, bf[nt]);
       }
       float* out = p.scores + ((size_t)page * p.heads + head * group + h0) * kPage;
 #pragma unroll
@@ -222,7 +216,7 @@ mixed_decode_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
     const bf16* V = v_page(kv, page, head) + (size_t)(v0 + g) * kPage + t * 8;
 #pragma unroll
     for (int kb = 0; kb < 2; ++kb) {
-      const uint4 a0 = ld16(W + g * 96 + kb * 32 + t * 8), a1 = ld16(W + (g + 8) * 96 + kb * 32 + t * 8);
+      const AFragPair a = a_fragments(ld16(W + g * 96 + kb * 32 + t * 8), ld16(W + (g + 8) * 96 + kb * 32 + t * 8));
 #pragma unroll
       for (int n0 = 0; n0 < VT; n0 += 8) {
         uint4 bf[8];
@@ -231,7 +225,7 @@ mixed_decode_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
           if (n0 + i < nvt) bf[i] = ld16(V + (size_t)(n0 + i) * 8 * kPage + kb * 32);
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-          if (n0 + i < nvt) mma_pair(acc[n0 + i], a0, a1, bf[i]);
+          if (n0 + i < nvt) mma_pair(acc[n0 + i], a, bf[i]);
       }
     }
     __syncwarp();
@@ -271,12 +265,13 @@ mixed_decode_merge_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv
 
 // ---- prefill: (maximum, sum) per (token, head) -----------------------------------------------------------------------------
 constexpr int kStatWarps = 4, kStatRows = 128;
+template <int KB>
 __global__ void __launch_bounds__(kStatWarps * 32)
 mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, int tile_tokens, int splits) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t smem[];
-  const int ks = tile_stride(kv.k_dim), kb_n = kv.k_dim / 32, chunks = kv.k_dim / 8;
+  const int k_dim = KB ? KB * 32 : kv.k_dim, ks = tile_stride(k_dim), kb_n = k_dim / 32, chunks = k_dim / 8;
   bf16* q_sm = reinterpret_cast<bf16*>(smem);   // [128][ks]
   bf16* k_sm = q_sm + kStatRows * ks;           // [2][64][ks]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -326,18 +321,15 @@ mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
     const bf16* K = k_sm + ((pg - p0) & 1) * kPage * ks + g * ks + t * 8;
     const bf16* Q = q_sm + (warp * 32 + g) * ks + t * 8;
     float acc[2][8][4] = {};
-    for (int kb = 0; kb < kb_n; ++kb) {
-      uint4 a[2][2];
 #pragma unroll
-      for (int mt = 0; mt < 2; ++mt) {
-        a[mt][0] = ld16(Q + mt * 16 * ks + kb * 32);
-        a[mt][1] = ld16(Q + (mt * 16 + 8) * ks + kb * 32);
-      }
+    for (int kb = 0; kb < (KB ? KB : kb_n); ++kb) {
+      const AFragPair a[2] = {a_fragments(ld16(Q + kb * 32), ld16(Q + 8 * ks + kb * 32)),
+                              a_fragments(ld16(Q + 16 * ks + kb * 32), ld16(Q + 24 * ks + kb * 32))};
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
         const uint4 bf = ld16(K + nt * 8 * ks + kb * 32);
-        mma_pair(acc[0][nt], a[0][0], a[0][1], bf);
-        mma_pair(acc[1][nt], a[1][0], a[1][1], bf);
+        mma_pair(acc[0][nt], a[0], bf);
+        mma_pair(acc[1][nt], a[1], bf);
       }
     }
     const bool edge = (pg + 1) * kPage - 1 > pos0 + t0;
@@ -352,9 +344,17 @@ mixed_prefill_stats_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
           for (int e = 0; e < 2; ++e) {
             float& s = acc[mt][nt][2 * hf + e];
             s *= scale2;
-            if (edge && pg * kPage + nt * 8 + 2 * t + e > limit[mt][hf]) s = -INFINITY;
-            mx = fmaxf(mx, s);
           }
+        if (edge) {
+          const int lim = limit[mt][hf] - pg * kPage - 2 * t;
+#pragma unroll
+          for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+              if (nt * 8 + e > lim) acc[mt][nt][2 * hf + e] = -INFINITY;
+        }
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt) mx = fmaxf(mx, fmaxf(acc[mt][nt][2 * hf], acc[mt][nt][2 * hf + 1]));
         if (mx == -INFINITY) continue;
         float sum = 0.0f;
 #pragma unroll
@@ -461,14 +461,14 @@ mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) bf[1][nt] = ld16(K + (size_t)nt * 8 * kv.k_dim + kb * 32 + 32);
           {
-            const uint4 a0 = ld16(Q + kb * 32), a1 = ld16(Q + 8 * qs + kb * 32);
+            const AFragPair a = a_fragments(ld16(Q + kb * 32), ld16(Q + 8 * qs + kb * 32));
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, bf[0][nt]);
+            for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a, bf[0][nt]);
           }
           if (two) {
-            const uint4 a0 = ld16(Q + kb * 32 + 32), a1 = ld16(Q + 8 * qs + kb * 32 + 32);
+            const AFragPair a = a_fragments(ld16(Q + kb * 32 + 32), ld16(Q + 8 * qs + kb * 32 + 32));
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, bf[1][nt]);
+            for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a, bf[1][nt]);
           }
         }
       } else {
@@ -476,10 +476,10 @@ mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
         const bf16* Q = qg + ((size_t)ia * H + h) * kv.k_dim + t * 8;
         const uint4 zero = make_uint4(0, 0, 0, 0);
         for (int kb = 0; kb < kb_n; ++kb) {
-          const uint4 a0 = ia < tokens ? ld16(Q + kb * 32) : zero;
-          const uint4 a1 = ia + 8 < tokens ? ld16(Q + (size_t)8 * H * kv.k_dim + kb * 32) : zero;
+          const AFragPair a = a_fragments(ia < tokens ? ld16(Q + kb * 32) : zero,
+                                          ia + 8 < tokens ? ld16(Q + (size_t)8 * H * kv.k_dim + kb * 32) : zero);
 #pragma unroll
-          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, ld16(K + (size_t)nt * 8 * kv.k_dim + kb * 32));
+          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a, ld16(K + (size_t)nt * 8 * kv.k_dim + kb * 32));
         }
       }
 #pragma unroll
@@ -528,7 +528,7 @@ mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     __syncthreads();
     if (live) {
       const bf16* w = W + ((size_t)ho * TQ + rg * 16 + g) * kKeys + t * 8;
-      const uint4 a0 = ld16(w), a1 = ld16(w + 8 * kKeys);
+      const AFragPair a = a_fragments(ld16(w), ld16(w + 8 * kKeys));
       const bf16* V = v_page(kv, page, (ho0 + ho) / group) + (size_t)(v0 + g) * kPage + in_page + t * 8;
 #pragma unroll
       for (int n0 = 0; n0 < 16; n0 += 8) {
@@ -538,7 +538,7 @@ mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
           if (n0 + i < nvt) bf[i] = ld16(V + (size_t)(n0 + i) * 8 * kPage);
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-          if (n0 + i < nvt) mma_pair(acc[n0 + i], a0, a1, bf[i]);
+          if (n0 + i < nvt) mma_pair(acc[n0 + i], a, bf[i]);
       }
     }
   }
@@ -598,6 +598,8 @@ __device__ __forceinline__ uint2 split_words(float a, float b) {
 }
 
 constexpr int kMaxMixHeads = 256;
+// KB = k_dim / 32 where it is known at compile time, else 0; VT = value tiles of a warp; QS = queries in shared memory
+template <int KB, int VT, bool QS>
 __global__ void __launch_bounds__(kValWarps * 32, 1)
 mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, TileGeom geo, int splits, int cluster) {
   pdl_wait();
@@ -605,12 +607,12 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint8_t kv_of[kMaxMixHeads];  // kv head of a query head
   const int H = p.heads, G = kv.kv_heads, RG = geo.row_groups, TQ = 16 * RG, HO = geo.out_heads, group = H / G;
-  const int qs = tile_stride(kv.k_dim), kb_n = kv.k_dim / 32, k_steps = (H + 15) / 16, m_tiles = (HO + 15) / 16;
+  const int k_dim = KB ? KB * 32 : kv.k_dim, qs = tile_stride(k_dim), kb_n = k_dim / 32, k_steps = (H + 15) / 16;
   bf16* k_sm = reinterpret_cast<bf16*>(smem + geo.k);            // [G][32][qs]
   bf16* v_sm = reinterpret_cast<bf16*>(smem + geo.v);            // [v_heads][v_dim][32]
   uint32_t* P = reinterpret_cast<uint32_t*>(smem + geo.p);       // [H][TQ][kPStride] (+4 per head)
   bf16* W = reinterpret_cast<bf16*>(smem + geo.w);               // [HO][TQ][32] (+8 per head)
-  uint4* T = reinterpret_cast<uint4*>(smem + geo.t);             // [m_tiles][k_steps][32 lanes][hi, lo] A fragments
+  uint4* T = reinterpret_cast<uint4*>(smem + geo.t);             // [k_steps][32 lanes][hi, lo] A fragments
   float2* ml = reinterpret_cast<float2*>(smem + geo.ml);         // [H][TQ] (maximum, 1 / sum)
   bf16* q_sm = reinterpret_cast<bf16*>(smem + geo.q);            // [H][TQ][qs] (when it fits)
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -624,11 +626,11 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   const int gv0 = ho0 / group, gv1 = min(G, (ho0 + HO - 1) / group + 1);
 
   // half a warp per key row, one kv head per turn; V rows of 32 keys are four 16-byte pieces
-  const int k_row = warp * 2 + (lane >> 4), k_chunk = lane & 15, k_chunks = kv.k_dim / 8;
+  const int k_row = warp * 2 + (lane >> 4), k_chunk = lane & 15, k_chunks = k_dim / 8;
   auto copy_k = [&](int c) {
-    const bf16* src = k_page(kv, table[c / 2], 0) + (size_t)((c % 2) * kKeys + k_row) * kv.k_dim;
+    const bf16* src = k_page(kv, table[c / 2], 0) + (size_t)((c % 2) * kKeys + k_row) * k_dim;
     bf16* dst = k_sm + k_row * qs;
-    for (int hd = 0; hd < G; ++hd, src += (size_t)kPage * kv.k_dim, dst += kKeys * qs)
+    for (int hd = 0; hd < G; ++hd, src += (size_t)kPage * k_dim, dst += kKeys * qs)
       for (int ch = k_chunk; ch < k_chunks; ch += 16) cp_async16(dst + ch * 8, src + ch * 8);
     cp_async_commit();
   };
@@ -642,7 +644,7 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   const int rg_shift = RG == 4 ? 2 : RG == 2 ? 1 : 0;
   for (int h = threadIdx.x; h < H; h += blockDim.x) kv_of[h] = uint8_t(h / group);
 
-  const bf16* qg = static_cast<const bf16*>(p.q) + (size_t)(start + t0) * H * kv.k_dim;
+  const bf16* qg = static_cast<const bf16*>(p.q) + (size_t)(start + t0) * H * k_dim;
   const size_t i0 = size_t(start - b.seq_start[0] + t0);
   for (int e = threadIdx.x; e < H * TQ; e += blockDim.x) {
     const int h = e % H, i = e / H;
@@ -652,10 +654,10 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
         const float2 v = *reinterpret_cast<const float2*>(p.stats + (((size_t)s * b.num_tokens + i0 + i) * H + h) * 2);
         merge_ml(M, L, v.x, v.y);
       }
-    ml[h * TQ + i] = i < tokens ? make_float2(M, 1.0f / L) : make_float2(0.0f, 0.0f);
+    ml[h * TQ + i] = i < tokens ? make_float2(M, 1.0f / L) : make_float2(INFINITY, 0.0f);  // rows without a token: weight 0
   }
-  for (int e = threadIdx.x; e < m_tiles * k_steps * 32; e += blockDim.x) {
-    const int ln = e % 32, k = e / 32 % k_steps, mt = e / (32 * k_steps), r = mt * 16 + ln / 4, c = k * 16 + ln % 4 * 2;
+  for (int e = threadIdx.x; e < k_steps * 32; e += blockDim.x) {
+    const int ln = e % 32, k = e / 32, r = ln / 4, c = k * 16 + ln % 4 * 2;
     uint32_t hi[4], lo[4];
 #pragma unroll
     for (int f = 0; f < 4; ++f) {  // rows r, r + 8 x columns c, c + 8
@@ -671,20 +673,20 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     T[2 * e] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
     T[2 * e + 1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
-  if (geo.q_in_smem) {
-    const int chunks = kv.k_dim / 8;
+  if (QS) {
+    const int chunks = k_dim / 8;
     for (int e = threadIdx.x; e < H * TQ * chunks; e += blockDim.x) {
       const int c = e % chunks, h = e / chunks % H, i = e / (chunks * H);
       *reinterpret_cast<uint4*>(q_sm + ((size_t)h * TQ + i) * qs + c * 8) =
-          i < tokens ? ld16(qg + ((size_t)i * H + h) * kv.k_dim + c * 8) : make_uint4(0, 0, 0, 0);
+          i < tokens ? ld16(qg + ((size_t)i * H + h) * k_dim + c * 8) : make_uint4(0, 0, 0, 0);
     }
   }
   const float scale2 = p.scale * kLog2e;
   const int rg = warp % RG, vc = warp / RG % geo.vchunks, ho = warp / (RG * geo.vchunks);
   const bool live = ho < HO && ho0 + ho < H;
-  const int v0 = vc * 128, nvt = live ? min(16, (kv.v_dim - v0) / 8) : 0;
+  const int v0 = vc * 128, nvt = live ? min(VT, (kv.v_dim - v0) / 8) : 0;
   const bf16* V = v_sm + (live ? ((ho0 + ho) / group - gv0) * kv.v_dim + v0 + g : 0) * kKeys + t * 8;
-  float acc[16][4] = {};
+  float acc[VT][4] = {};
   for (int c = c0; c < c1; ++c) {
     const int j0 = c * kKeys;
     cp_async_wait<0>();
@@ -695,25 +697,15 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
       const int h = u >> rg_shift, r = u & (RG - 1);
       const bf16* K = k_sm + (kv_of[h] * kKeys + g) * qs + t * 8;
       float s[4][4] = {};
-      if (geo.q_in_smem) {
-        const bf16* Q = q_sm + ((size_t)h * TQ + r * 16 + g) * qs + t * 8;
-#pragma unroll 2
-        for (int kb = 0; kb < kb_n; ++kb) {
-          const uint4 a0 = ld16(Q + kb * 32), a1 = ld16(Q + 8 * qs + kb * 32);
+      // rows beyond the tile's tokens read the last one's query; their weights are zero
+      const int ia = r * 16 + g;
+      const bf16* q0 = QS ? q_sm + (h * TQ + ia) * qs + t * 8 : qg + ((size_t)min(ia, tokens - 1) * H + h) * k_dim + t * 8;
+      const bf16* q8 = QS ? q0 + 8 * qs : qg + ((size_t)min(ia + 8, tokens - 1) * H + h) * k_dim + t * 8;
+#pragma unroll (VT == 16 ? 1 : 4)
+      for (int kb = 0; kb < (KB ? KB : kb_n); ++kb) {
+        const AFragPair a = a_fragments(ld16(q0 + kb * 32), ld16(q8 + kb * 32));
 #pragma unroll
-          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, ld16(K + nt * 8 * qs + kb * 32));
-        }
-      } else {
-        const int ia = r * 16 + g;
-        const bf16* Q = qg + ((size_t)ia * H + h) * kv.k_dim + t * 8;
-        const uint4 zero = make_uint4(0, 0, 0, 0);
-#pragma unroll 2
-        for (int kb = 0; kb < kb_n; ++kb) {
-          const uint4 a0 = ia < tokens ? ld16(Q + kb * 32) : zero;
-          const uint4 a1 = ia + 8 < tokens ? ld16(Q + (size_t)8 * H * kv.k_dim + kb * 32) : zero;
-#pragma unroll
-          for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a0, a1, ld16(K + nt * 8 * qs + kb * 32));
-        }
+        for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a, ld16(K + nt * 8 * qs + kb * 32));
       }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
@@ -734,44 +726,42 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     __syncthreads();
     if (c + 1 < c1) copy_k(c + 1);
     else cp_async_commit();  // an empty group keeps the count below the same
-    // mixing: (token, key octet) tiles of 8 columns
-    for (int n = warp; n < TQ * 4; n += kValWarps) {
-      const int i = n / 4, j = n % 4 * 8;
-      const uint32_t* col = P + i * kPStride + j + g;
-      for (int mt = 0; mt < m_tiles; ++mt) {
-        float d[4] = {};
-        for (int k = 0; k < k_steps; ++k) {
-          uint32_t w[4];
+    // mixing: a warp takes the 32 keys (four column tiles) of one token row per row group; columns of heads that do not
+    // exist meet zeros of T, so any finite word serves
+    for (int i = warp; i < TQ; i += kValWarps) {
+      const uint32_t* col = P + i * kPStride + g;
+      float d[4][4] = {};
+      for (int k = 0; k < k_steps; ++k) {
+        const uint4 ah4 = T[2 * (k * 32 + lane)], al4 = T[2 * (k * 32 + lane) + 1];
+        const uint32_t ah[4] = {ah4.x, ah4.y, ah4.z, ah4.w}, al[4] = {al4.x, al4.y, al4.z, al4.w};
+        const uint32_t* c0p[4];
 #pragma unroll
-          for (int f = 0; f < 4; ++f) {
-            const int h = k * 16 + 2 * t + (f & 1) + (f >> 1) * 8;
-            w[f] = h < H ? col[h * geo.head_words] : 0u;
-          }
-          const uint32_t bh0 = __byte_perm(w[0], w[1], 0x5410), bl0 = __byte_perm(w[0], w[1], 0x7632);
-          const uint32_t bh1 = __byte_perm(w[2], w[3], 0x5410), bl1 = __byte_perm(w[2], w[3], 0x7632);
-          const uint4 ah4 = T[2 * ((mt * k_steps + k) * 32 + lane)], al4 = T[2 * ((mt * k_steps + k) * 32 + lane) + 1];
-          const uint32_t ah[4] = {ah4.x, ah4.y, ah4.z, ah4.w}, al[4] = {al4.x, al4.y, al4.z, al4.w};
-          mma_bf16_16816(d, ah, bh0, bh1);
-          mma_bf16_16816(d, ah, bl0, bl1);
-          mma_bf16_16816(d, al, bh0, bh1);
-        }
+        for (int f = 0; f < 4; ++f) c0p[f] = col + min(k * 16 + 2 * t + (f & 1) + (f >> 1) * 8, H - 1) * geo.head_words;
 #pragma unroll
-        for (int hf = 0; hf < 2; ++hf) {
-          const int o = mt * 16 + g + 8 * hf;
-          if (o < HO)
-            *reinterpret_cast<__nv_bfloat162*>(W + o * geo.out_stride + i * kKeys + j + 2 * t) =
-                __floats2bfloat162_rn(d[2 * hf], d[2 * hf + 1]);
+        for (int n = 0; n < 4; ++n) {
+          const uint32_t w0 = c0p[0][n * 8], w1 = c0p[1][n * 8], w2 = c0p[2][n * 8], w3 = c0p[3][n * 8];
+          const uint32_t bh0 = __byte_perm(w0, w1, 0x5410), bl0 = __byte_perm(w0, w1, 0x7632);
+          const uint32_t bh1 = __byte_perm(w2, w3, 0x5410), bl1 = __byte_perm(w2, w3, 0x7632);
+          mma_bf16_16816(d[n], ah, bh0, bh1);
+          mma_bf16_16816(d[n], ah, bl0, bl1);
+          mma_bf16_16816(d[n], al, bh0, bh1);
         }
       }
+      bf16* to = W + g * geo.out_stride + i * kKeys + 2 * t;
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf)
+        if (g + 8 * hf < HO)
+#pragma unroll
+          for (int n = 0; n < 4; ++n)
+            *reinterpret_cast<__nv_bfloat162*>(to + hf * 8 * geo.out_stride + n * 8) = __floats2bfloat162_rn(d[n][2 * hf], d[n][2 * hf + 1]);
     }
     cp_async_wait<1>();
     __syncthreads();  // V of this tile and the mixed weights are here
     if (live) {
       const bf16* w = W + (size_t)ho * geo.out_stride + (rg * 16 + g) * kKeys + t * 8;
-      const uint4 a0 = ld16(w), a1 = ld16(w + 8 * kKeys);
+      const AFragPair a = a_fragments(ld16(w), ld16(w + 8 * kKeys));
 #pragma unroll
-      for (int i = 0; i < 16; ++i)
-        if (i < nvt) mma_pair(acc[i], a0, a1, ld16(V + i * 8 * kKeys));
+      for (int i = 0; i < VT; ++i) mma_pair(acc[i], a, ld16(V + i * 8 * kKeys));  // tiles beyond the head are not stored
     }
   }
   auto store = [&](int wp, int nt, int ln, float4 v) {  // the fragment of lane `ln` of warp `wp`, value tile nt
@@ -789,14 +779,14 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
   };
   if (cluster == 1) {
 #pragma unroll
-    for (int nt = 0; nt < 16; ++nt)
+    for (int nt = 0; nt < VT; ++nt)
       if (nt < nvt) store(warp, nt, lane, make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]));
     return;
   }
   float4* red = reinterpret_cast<float4*>(smem);  // [16 warps][4][32 lanes]
   cp_async_wait<0>();
 #pragma unroll
-  for (int q = 0; q < 4; ++q) {
+  for (int q = 0; q < VT / 4; ++q) {
     if (q * 32 >= kv.v_dim) break;  // uniform: no warp holds further columns
     __syncthreads();
     cluster_barrier();  // everyone is done with its tiles / with reading the previous quarter
@@ -870,11 +860,12 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
       g.v = take(g.v_heads * kv.v_dim * kKeys * 2);
       g.p = take(H * g.head_words * 4);
       g.w = take(g.out_heads * g.out_stride * 2);
-      g.t = take((g.out_heads + 15) / 16 * ((H + 15) / 16) * 32 * 32);
+      g.t = take((H + 15) / 16 * 32 * 32);
       g.ml = take(H * TQ * 8);
       g.q_in_smem = q;
       g.q = take(q ? H * TQ * tile_stride(kv.k_dim) * 2 : 0);
-      g.bytes = std::max(at, kValWarps * 4 * 32 * 16);  // the cluster's reduction reuses the space
+      // the cluster's reduction reuses the space; value tiles are read in whole 128-column chunks
+      g.bytes = std::max({at, kValWarps * 4 * 32 * 16, g.v + (g.v_heads * kv.v_dim + 128) * kKeys * 2});
       if (g.bytes <= max_optin_smem() - 1024) {
         *out = g;
         return true;
@@ -882,6 +873,45 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
     }
   }
   return false;
+}
+
+template <int KB, int VT, bool QS>
+int launch_values_as(const q38_mixed_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, const TileGeom& g,
+                     int splits, cudaStream_t s) {
+  static const cudaError_t attr = cudaFuncSetAttribute(mixed_prefill_values_kernel<KB, VT, QS>,
+                                                       cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
+  Q38_CUDA_OK(attr);
+  const int TQ = 16 * g.row_groups, q_tiles = (b.max_tokens_per_seq + TQ - 1) / TQ, hb = (p.heads + g.out_heads - 1) / g.out_heads;
+  int cluster = 1;
+  while (cluster < 8 && q_tiles * hb * b.num_seqs * cluster < 2 * num_sms()) cluster *= 2;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(q_tiles * cluster, hb, b.num_seqs);
+  cfg.blockDim = dim3(kValWarps * 32);
+  cfg.dynamicSmemBytes = size_t(g.bytes);
+  cfg.stream = s;
+  cudaLaunchAttribute attrs[2];
+  int n = 0;
+  if (dependent_launch_allowed()) {
+    attrs[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attrs[n++].val.programmaticStreamSerializationAllowed = 1;
+  }
+  if (cluster > 1) {
+    attrs[n].id = cudaLaunchAttributeClusterDimension;
+    attrs[n].val.clusterDim.x = unsigned(cluster);
+    attrs[n].val.clusterDim.y = 1;
+    attrs[n++].val.clusterDim.z = 1;
+  }
+  cfg.attrs = attrs;
+  cfg.numAttrs = unsigned(n);
+  Q38_CUDA_OK(cudaLaunchKernelEx(&cfg, mixed_prefill_values_kernel<KB, VT, QS>, p, b, kv, g, splits, cluster));
+  return Q38_OK;
+}
+template <int KB>
+int launch_values(const q38_mixed_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, const TileGeom& g,
+                  int splits, cudaStream_t s) {
+  if (kv.v_dim <= 64)
+    return g.q_in_smem ? launch_values_as<KB, 8, true>(p, b, kv, g, splits, s) : launch_values_as<KB, 8, false>(p, b, kv, g, splits, s);
+  return g.q_in_smem ? launch_values_as<KB, 16, true>(p, b, kv, g, splits, s) : launch_values_as<KB, 16, false>(p, b, kv, g, splits, s);
 }
 
 template <int GROUP, int VT>
@@ -919,39 +949,19 @@ int mixed_prefill_mma(const q38_mixed_attention_params& p, const q38_batch_desc&
   const int ctas = tiles * kv.kv_heads * b.num_seqs;
   const int splits = std::max(1, std::min({p.stat_splits, 5 * num_sms() / ctas, 8}));
   const size_t smem = size_t(kStatRows + 2 * kPage) * size_t(tile_stride(kv.k_dim)) * 2;
-  static const cudaError_t attr = cudaFuncSetAttribute(mixed_prefill_stats_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
-  Q38_CUDA_OK(attr);
-  (void)launch_kernel(mixed_prefill_stats_kernel, dim3(tiles, kv.kv_heads * splits, b.num_seqs), dim3(kStatWarps * 32), smem, s, p, b,
-                      kv, tile, splits);
+  const auto stats = kv.k_dim == 64    ? &mixed_prefill_stats_kernel<2>
+                     : kv.k_dim == 128 ? &mixed_prefill_stats_kernel<4>
+                                       : &mixed_prefill_stats_kernel<0>;
+  Q38_CUDA_OK(cudaFuncSetAttribute(stats, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem()));
+  (void)launch_kernel(stats, dim3(tiles, kv.kv_heads * splits, b.num_seqs), dim3(kStatWarps * 32), smem, s, p, b, kv, tile, splits);
   Q38_LAUNCH_OK("mixed_prefill_stats_kernel");
   TileGeom tg;
   if (tile_geom(p, kv, &tg)) {
-    static const cudaError_t attr3 = cudaFuncSetAttribute(mixed_prefill_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
-    Q38_CUDA_OK(attr3);
-    const int TQ = 16 * tg.row_groups, q_tiles = (b.max_tokens_per_seq + TQ - 1) / TQ, hb = (p.heads + tg.out_heads - 1) / tg.out_heads;
-    int cluster = 1;
-    while (cluster < 8 && q_tiles * hb * b.num_seqs * cluster < 2 * num_sms()) cluster *= 2;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(q_tiles * cluster, hb, b.num_seqs);
-    cfg.blockDim = dim3(kValWarps * 32);
-    cfg.dynamicSmemBytes = size_t(tg.bytes);
-    cfg.stream = s;
-    cudaLaunchAttribute attrs[2];
-    int n = 0;
-    if (dependent_launch_allowed()) {
-      attrs[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-      attrs[n++].val.programmaticStreamSerializationAllowed = 1;
+    switch (kv.k_dim) {
+      case 64: return launch_values<2>(p, b, kv, tg, splits, s);
+      case 128: return launch_values<4>(p, b, kv, tg, splits, s);
+      default: return launch_values<0>(p, b, kv, tg, splits, s);
     }
-    if (cluster > 1) {
-      attrs[n].id = cudaLaunchAttributeClusterDimension;
-      attrs[n].val.clusterDim.x = unsigned(cluster);
-      attrs[n].val.clusterDim.y = 1;
-      attrs[n++].val.clusterDim.z = 1;
-    }
-    cfg.attrs = attrs;
-    cfg.numAttrs = unsigned(n);
-    Q38_CUDA_OK(cudaLaunchKernelEx(&cfg, mixed_prefill_values_kernel, p, b, kv, tg, splits, cluster));
-    return Q38_OK;
   }
   ValGeom g;
   Q38_REQUIRE(val_geom(p, kv, &g), "mixed_attention: shape does not fit");

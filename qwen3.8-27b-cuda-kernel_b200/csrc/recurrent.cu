@@ -324,13 +324,9 @@ rglru_gates_mma_kernel(q38_rglru_params p, q38_batch_desc batch, q38_recurrent_s
 #pragma unroll
         for (int term = 0; term < 2; ++term) {
           const __nv_bfloat16* u = (term ? lo : hi) + (mt * 16 + g) * us + k + t * 8;
-          const uint4 a0 = *reinterpret_cast<const uint4*>(u), a1 = *reinterpret_cast<const uint4*>(u + 8 * us);
-          const uint32_t f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
-#pragma unroll
-          for (int q = 0; q < 2; ++q) {
-            mma_bf16_16816(acc[mt][q], f0, w[q].x, w[q].y);
-            mma_bf16_16816(acc[mt][q], f1, w[q].z, w[q].w);
-          }
+          const AFragPair a = a_fragments(*reinterpret_cast<const uint4*>(u), *reinterpret_cast<const uint4*>(u + 8 * us));
+          mma_pair(acc[mt][0], a, w[0]);
+          mma_pair(acc[mt][1], a, w[1]);
         }
     }
 #pragma unroll
