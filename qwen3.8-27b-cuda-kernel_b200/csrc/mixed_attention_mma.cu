@@ -12,6 +12,7 @@
 // contiguous bytes of a row (8 head dimensions of a key, or 8 keys of a value column - V is stored transposed) are the
 // registers of two k16 steps under a permutation of k that both operands share.
 #include <algorithm>
+#include <type_traits>
 
 #include "act.cuh"
 #include "mixed_attention.h"
@@ -565,7 +566,8 @@ mixed_prefill_direct_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
 // one token tile and divide its keys; their outputs (weights are normalised over all keys) are summed through the
 // cluster's shared memory in rank order.
 struct TileGeom {
-  int row_groups, vchunks, out_heads, q_in_smem;
+  int tokens;       // of a tile
+  int row_groups, vchunks, out_heads, q_in_smem, heads_per_mma;
   int v_heads;      // kv heads whose values a CTA needs at most
   int head_words;   // P: words per head = 16 RG * kPStride + 4
   int out_stride;   // W: elements per output head = 16 RG * 32 + 8
@@ -598,21 +600,23 @@ __device__ __forceinline__ uint2 split_words(float a, float b) {
 }
 
 constexpr int kMaxMixHeads = 256;
-// KB = k_dim / 32 where it is known at compile time, else 0; VT = value tiles of a warp; QS = queries in shared memory
-template <int KB, int VT, bool QS>
+// KB = k_dim / 32 where it is known at compile time, else 0; VT = value tiles of a warp; QS = queries in shared memory.
+// HP = heads in the 16 rows of an MMA: 1 = 16 tokens of a head; 2 = 8 tokens of two heads of one kv head (row g + 8 is
+// the second head's token g), for models with more heads than a CTA could otherwise put out.
+template <int KB, int VT, bool QS, int HP>
 __global__ void __launch_bounds__(kValWarps * 32, 1)
 mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, TileGeom geo, int splits, int cluster) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint8_t kv_of[kMaxMixHeads];  // kv head of a query head
-  const int H = p.heads, G = kv.kv_heads, RG = geo.row_groups, TQ = 16 * RG, HO = geo.out_heads, group = H / G;
-  const int k_dim = KB ? KB * 32 : kv.k_dim, qs = tile_stride(k_dim), kb_n = k_dim / 32, k_steps = (H + 15) / 16;
+  const int H = p.heads, G = kv.kv_heads, RG = HP == 2 ? 1 : geo.row_groups, TQ = HP == 2 ? 8 : 16 * RG, HO = geo.out_heads, group = H / G;
+  const int k_dim = KB ? KB * 32 : kv.k_dim, qs = tile_stride(k_dim), kb_n = k_dim / 32, k_steps = (H + 15) / 16, m_tiles = (HO + 15) / 16;
   bf16* k_sm = reinterpret_cast<bf16*>(smem + geo.k);            // [G][32][qs]
   bf16* v_sm = reinterpret_cast<bf16*>(smem + geo.v);            // [v_heads][v_dim][32]
   uint32_t* P = reinterpret_cast<uint32_t*>(smem + geo.p);       // [H][TQ][kPStride] (+4 per head)
   bf16* W = reinterpret_cast<bf16*>(smem + geo.w);               // [HO][TQ][32] (+8 per head)
-  uint4* T = reinterpret_cast<uint4*>(smem + geo.t);             // [k_steps][32 lanes][hi, lo] A fragments
+  uint4* T = reinterpret_cast<uint4*>(smem + geo.t);             // [m_tiles][k_steps][32 lanes][hi, lo] A fragments
   float2* ml = reinterpret_cast<float2*>(smem + geo.ml);         // [H][TQ] (maximum, 1 / sum)
   bf16* q_sm = reinterpret_cast<bf16*>(smem + geo.q);            // [H][TQ][qs] (when it fits)
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -656,8 +660,8 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
       }
     ml[h * TQ + i] = i < tokens ? make_float2(M, 1.0f / L) : make_float2(INFINITY, 0.0f);  // rows without a token: weight 0
   }
-  for (int e = threadIdx.x; e < k_steps * 32; e += blockDim.x) {
-    const int ln = e % 32, k = e / 32, r = ln / 4, c = k * 16 + ln % 4 * 2;
+  for (int e = threadIdx.x; e < m_tiles * k_steps * 32; e += blockDim.x) {
+    const int ln = e % 32, k = e / 32 % k_steps, r = e / (32 * k_steps) * 16 + ln / 4, c = k * 16 + ln % 4 * 2;
     uint32_t hi[4], lo[4];
 #pragma unroll
     for (int f = 0; f < 4; ++f) {  // rows r, r + 8 x columns c, c + 8
@@ -682,36 +686,41 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     }
   }
   const float scale2 = p.scale * kLog2e;
-  const int rg = warp % RG, vc = warp / RG % geo.vchunks, ho = warp / (RG * geo.vchunks);
+  const int rg = warp % RG, vc = warp / RG % geo.vchunks, ho = warp / (RG * geo.vchunks) * HP;
   const bool live = ho < HO && ho0 + ho < H;
   const int v0 = vc * 128, nvt = live ? min(VT, (kv.v_dim - v0) / 8) : 0;
-  const bf16* V = v_sm + (live ? ((ho0 + ho) / group - gv0) * kv.v_dim + v0 + g : 0) * kKeys + t * 8;
+  const int v_row = live ? ((ho0 + ho) / group - gv0) * kv.v_dim + v0 : 0;
   float acc[VT][4] = {};
   for (int c = c0; c < c1; ++c) {
     const int j0 = c * kKeys;
+    // the accumulators take half the registers: addresses are recomputed per tile, not kept (and spilled) across tiles
+    int tid = int(threadIdx.x);
+    asm volatile("" : "+r"(tid));
+    const int lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     cp_async_wait<0>();
     __syncthreads();  // K of this tile is here; the previous tile's weights and values are done with
     copy_v(c);
     const bool edge = j0 + kKeys - 1 > pos0 + t0;  // some row of the tile ends inside these keys
-    for (int u = warp; u < H << rg_shift; u += kValWarps) {
-      const int h = u >> rg_shift, r = u & (RG - 1);
+    for (int u = warp; u < (HP == 2 ? H / 2 : H << rg_shift); u += kValWarps) {
+      const int h = HP == 2 ? 2 * u : u >> rg_shift, r = u & (RG - 1);
       const bf16* K = k_sm + (kv_of[h] * kKeys + g) * qs + t * 8;
       float s[4][4] = {};
       // rows beyond the tile's tokens read the last one's query; their weights are zero
-      const int ia = r * 16 + g;
+      const int ia = (HP == 2 ? 0 : r * 16) + g, ib = HP == 2 ? g : ia + 8, hb = HP == 2 ? h + 1 : h;
       const bf16* q0 = QS ? q_sm + (h * TQ + ia) * qs + t * 8 : qg + ((size_t)min(ia, tokens - 1) * H + h) * k_dim + t * 8;
-      const bf16* q8 = QS ? q0 + 8 * qs : qg + ((size_t)min(ia + 8, tokens - 1) * H + h) * k_dim + t * 8;
-#pragma unroll (VT == 16 ? 1 : 4)
+      const bf16* q8 = QS ? q_sm + (hb * TQ + ib) * qs + t * 8 : qg + ((size_t)min(ib, tokens - 1) * H + hb) * k_dim + t * 8;
+#pragma unroll
       for (int kb = 0; kb < (KB ? KB : kb_n); ++kb) {
         const AFragPair a = a_fragments(ld16(q0 + kb * 32), ld16(q8 + kb * 32));
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) mma_pair(s[nt], a, ld16(K + nt * 8 * qs + kb * 32));
+        if (VT == 16) asm volatile("" ::: "memory");
       }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int i = r * 16 + hf * 8 + g, lim = pos0 + t0 + i - j0 - 2 * t;
-        const float2 st = ml[h * TQ + i];
-        uint32_t* out = P + h * geo.head_words + i * kPStride + 2 * t;
+        const int i = hf ? ib : ia, hh = hf ? hb : h, lim = pos0 + t0 + i - j0 - 2 * t;
+        const float2 st = ml[hh * TQ + i];
+        uint32_t* out = P + hh * geo.head_words + i * kPStride + 2 * t;
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) {
           float w0 = ex2(fmaf(s[nt][2 * hf], scale2, -st.x)) * st.y, w1 = ex2(fmaf(s[nt][2 * hf + 1], scale2, -st.x)) * st.y;
@@ -728,11 +737,13 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     else cp_async_commit();  // an empty group keeps the count below the same
     // mixing: a warp takes the 32 keys (four column tiles) of one token row per row group; columns of heads that do not
     // exist meet zeros of T, so any finite word serves
-    for (int i = warp; i < TQ; i += kValWarps) {
+    for (int it = warp; it < TQ * m_tiles; it += kValWarps) {
+      const int i = HP == 2 ? it & 7 : it, mt = HP == 2 ? it >> 3 : 0;
       const uint32_t* col = P + i * kPStride + g;
       float d[4][4] = {};
       for (int k = 0; k < k_steps; ++k) {
-        const uint4 ah4 = T[2 * (k * 32 + lane)], al4 = T[2 * (k * 32 + lane) + 1];
+        const uint4* tf = T + 2 * ((mt * k_steps + k) * 32 + lane);
+        const uint4 ah4 = tf[0], al4 = tf[1];
         const uint32_t ah[4] = {ah4.x, ah4.y, ah4.z, ah4.w}, al[4] = {al4.x, al4.y, al4.z, al4.w};
         const uint32_t* c0p[4];
 #pragma unroll
@@ -747,10 +758,11 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
           mma_bf16_16816(d[n], al, bh0, bh1);
         }
       }
-      bf16* to = W + g * geo.out_stride + i * kKeys + 2 * t;
+      const int o = mt * 16 + g;
+      bf16* to = W + o * geo.out_stride + i * kKeys + 2 * t;
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf)
-        if (g + 8 * hf < HO)
+        if (o + 8 * hf < HO)
 #pragma unroll
           for (int n = 0; n < 4; ++n)
             *reinterpret_cast<__nv_bfloat162*>(to + hf * 8 * geo.out_stride + n * 8) = __floats2bfloat162_rn(d[n][2 * hf], d[n][2 * hf + 1]);
@@ -758,20 +770,23 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
     cp_async_wait<1>();
     __syncthreads();  // V of this tile and the mixed weights are here
     if (live) {
+      const bf16* V = v_sm + (v_row + g) * kKeys + t * 8;
       const bf16* w = W + (size_t)ho * geo.out_stride + (rg * 16 + g) * kKeys + t * 8;
-      const AFragPair a = a_fragments(ld16(w), ld16(w + 8 * kKeys));
+      const AFragPair a = a_fragments(ld16(w), ld16(w + (HP == 2 ? geo.out_stride : 8 * kKeys)));
 #pragma unroll
-      for (int i = 0; i < VT; ++i) mma_pair(acc[i], a, ld16(V + i * 8 * kKeys));  // tiles beyond the head are not stored
+      for (int i = 0; i < VT; ++i) {  // tiles beyond the head are not stored
+        mma_pair(acc[i], a, ld16(V + i * 8 * kKeys));
+        if (i % 4 == 3) asm volatile("" ::: "memory");  // no more than four loads ahead: the accumulators hold half the registers
+      }
     }
   }
   auto store = [&](int wp, int nt, int ln, float4 v) {  // the fragment of lane `ln` of warp `wp`, value tile nt
-    const int r = wp % RG, vch = wp / RG % geo.vchunks, o = wp / (RG * geo.vchunks), gg = ln >> 2, tt = ln & 3;
-    if (o >= HO || ho0 + o >= H) return;
+    const int r = wp % RG, vch = wp / RG % geo.vchunks, unit = wp / (RG * geo.vchunks), gg = ln >> 2, tt = ln & 3;
     const int d = vch * 128 + nt * 8 + 2 * tt;
 #pragma unroll
     for (int hf = 0; hf < 2; ++hf) {
-      const int i = r * 16 + hf * 8 + gg;
-      if (i >= tokens) continue;
+      const int i = HP == 2 ? gg : r * 16 + hf * 8 + gg, o = HP == 2 ? 2 * unit + hf : unit;
+      if (i >= tokens || o >= HO || ho0 + o >= H) continue;
       bf16* out = static_cast<bf16*>(p.out) + (size_t)(start + t0 + i) * p.ld_out + (size_t)(ho0 + o) * p.vdim + d;
       if (d < p.vdim) out[0] = __float2bfloat16_rn(hf ? v.z : v.x);
       if (d + 1 < p.vdim) out[1] = __float2bfloat16_rn(hf ? v.w : v.y);
@@ -783,28 +798,34 @@ mixed_prefill_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_
       if (nt < nvt) store(warp, nt, lane, make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]));
     return;
   }
-  float4* red = reinterpret_cast<float4*>(smem);  // [16 warps][4][32 lanes]
+  float4* red = reinterpret_cast<float4*>(smem);  // [16 warps][NR value tiles][32 lanes] of one round
   cp_async_wait<0>();
+  auto join = [&](auto tiles_per_round) {
+    constexpr int NR = decltype(tiles_per_round)::value;
 #pragma unroll
-  for (int q = 0; q < VT / 4; ++q) {
-    if (q * 32 >= kv.v_dim) break;  // uniform: no warp holds further columns
-    __syncthreads();
-    cluster_barrier();  // everyone is done with its tiles / with reading the previous quarter
+    for (int q = 0; q < VT / NR; ++q) {
+      if (q * NR * 8 >= kv.v_dim) break;  // uniform: no warp holds further columns
+      __syncthreads();
+      cluster_barrier();  // everyone is done with its tiles / with reading the previous round
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-      red[(warp * 4 + i) * 32 + lane] = make_float4(acc[4 * q + i][0], acc[4 * q + i][1], acc[4 * q + i][2], acc[4 * q + i][3]);
-    __syncthreads();
-    cluster_barrier();
-    for (int e = rank * (kValWarps * 32) + threadIdx.x; e < kValWarps * 4 * 32; e += cluster * kValWarps * 32) {
-      float4 v = make_float4(0, 0, 0, 0);
-      for (int r = 0; r < cluster; ++r) {
-        const float4 x = ld_cluster_f32x4(smem_u32(red + e), uint32_t(r));
-        v.x += x.x, v.y += x.y, v.z += x.z, v.w += x.w;
+      for (int i = 0; i < NR; ++i)
+        red[(warp * NR + i) * 32 + lane] = make_float4(acc[NR * q + i][0], acc[NR * q + i][1], acc[NR * q + i][2], acc[NR * q + i][3]);
+      __syncthreads();
+      cluster_barrier();
+      for (int e = rank * (kValWarps * 32) + threadIdx.x; e < kValWarps * NR * 32; e += cluster * kValWarps * 32) {
+        float4 v = make_float4(0, 0, 0, 0);
+#pragma unroll 4
+        for (int r = 0; r < cluster; ++r) {
+          const float4 x = ld_cluster_f32x4(smem_u32(red + e), uint32_t(r));
+          v.x += x.x, v.y += x.y, v.z += x.z, v.w += x.w;
+        }
+        const int wp = e / (32 * NR), nt = NR * q + e / 32 % NR, vch = wp / RG % geo.vchunks;
+        if (vch * 128 + nt * 8 < kv.v_dim) store(wp, nt, e % 32, v);
       }
-      const int wp = e / 128, nt = 4 * q + e / 32 % 4, vch = wp / RG % geo.vchunks;
-      if (vch * 128 + nt * 8 < kv.v_dim) store(wp, nt, e % 32, v);
     }
-  }
+  };
+  if (geo.bytes >= kValWarps * VT * 32 * 16) join(std::integral_constant<int, VT>{});
+  else join(std::integral_constant<int, 4>{});
   __syncthreads();
   cluster_barrier();  // nobody leaves while its shared memory is being read
 }
@@ -841,15 +862,21 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
   const int H = p.heads, group = H / kv.kv_heads;
   g.vchunks = (kv.v_dim + 127) / 128;
   if (g.vchunks > kValWarps || H > kMaxMixHeads) return false;
-  for (int rg : {4, 2, 1}) {
-    if (rg > 1 && rg * g.vchunks * H > kValWarps) continue;  // few heads: more tokens per CTA instead
+  for (int form : {8, 4, 2, 1}) {  // 8: two heads per MMA; 4, 2, 1: row groups
+    const int rg = form == 8 ? 1 : form;
+    g.heads_per_mma = form == 8 ? 2 : 1;
+    if (form == 8 && (group % 2 != 0 || H * g.vchunks <= kValWarps)) continue;  // more heads than a CTA's warps, in pairs
+    if (rg > 1 && rg * g.vchunks * H > kValWarps) continue;                     // few heads: more tokens per CTA instead
     g.row_groups = rg;
-    g.out_heads = std::max(1, std::min(H, kValWarps / (rg * g.vchunks)));
-    g.v_heads = std::min(kv.kv_heads, (g.out_heads + group - 2) / group + 1);
-    const int TQ = 16 * rg;
+    g.out_heads = std::max(1, std::min(H, g.heads_per_mma * (kValWarps / (rg * g.vchunks))));
+    const int HO = g.out_heads, TQ = form == 8 ? 8 : 16 * rg;
+    g.tokens = TQ;
+    // kv heads that HO consecutive query heads can touch (the runs start at multiples of HO)
+    g.v_heads = std::min(kv.kv_heads, HO % group == 0 ? HO / group : group % HO == 0 ? 1 : (HO + group - 2) / group + 1);
     g.head_words = TQ * kPStride + 4;
     g.out_stride = TQ * kKeys + 8;
     for (int q : {1, 0}) {
+      if (q && form == 8) continue;
       int at = 0;
       auto take = [&](int bytes) {
         const int here = at;
@@ -860,7 +887,7 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
       g.v = take(g.v_heads * kv.v_dim * kKeys * 2);
       g.p = take(H * g.head_words * 4);
       g.w = take(g.out_heads * g.out_stride * 2);
-      g.t = take((H + 15) / 16 * 32 * 32);
+      g.t = take((g.out_heads + 15) / 16 * ((H + 15) / 16) * 32 * 32);
       g.ml = take(H * TQ * 8);
       g.q_in_smem = q;
       g.q = take(q ? H * TQ * tile_stride(kv.k_dim) * 2 : 0);
@@ -875,15 +902,25 @@ bool tile_geom(const q38_mixed_attention_params& p, const q38_kv_layer_desc& kv,
   return false;
 }
 
-template <int KB, int VT, bool QS>
+template <int KB, int VT, bool QS, int HP>
 int launch_values_as(const q38_mixed_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, const TileGeom& g,
                      int splits, cudaStream_t s) {
-  static const cudaError_t attr = cudaFuncSetAttribute(mixed_prefill_values_kernel<KB, VT, QS>,
+  static const cudaError_t attr = cudaFuncSetAttribute(mixed_prefill_values_kernel<KB, VT, QS, HP>,
                                                        cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
   Q38_CUDA_OK(attr);
-  const int TQ = 16 * g.row_groups, q_tiles = (b.max_tokens_per_seq + TQ - 1) / TQ, hb = (p.heads + g.out_heads - 1) / g.out_heads;
+  const int q_tiles = (b.max_tokens_per_seq + g.tokens - 1) / g.tokens, hb = (p.heads + g.out_heads - 1) / g.out_heads;
+  // CTAs per token tile by a cost in key tiles of a context of about 2,048 keys: the longest CTA, or the average load of
+  // an SM where there are several waves; starting and joining a CTA costs about as much as five tiles.
   int cluster = 1;
-  while (cluster < 8 && q_tiles * hb * b.num_seqs * cluster < 2 * num_sms()) cluster *= 2;
+  double best = 0.0;
+  for (int c = 1; c <= 8; c *= 2) {
+    const double ctas = double(q_tiles) * hb * b.num_seqs * c, longest = 64.0 / c + 5.0;
+    const double cost = ctas <= num_sms() ? longest : std::max(longest, 1.15 * ctas * (48.0 / c + 5.0) / num_sms());
+    if (c == 1 || cost < best) {
+      best = cost;
+      cluster = c;
+    }
+  }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(q_tiles * cluster, hb, b.num_seqs);
   cfg.blockDim = dim3(kValWarps * 32);
@@ -903,15 +940,19 @@ int launch_values_as(const q38_mixed_attention_params& p, const q38_batch_desc& 
   }
   cfg.attrs = attrs;
   cfg.numAttrs = unsigned(n);
-  Q38_CUDA_OK(cudaLaunchKernelEx(&cfg, mixed_prefill_values_kernel<KB, VT, QS>, p, b, kv, g, splits, cluster));
+  Q38_CUDA_OK(cudaLaunchKernelEx(&cfg, mixed_prefill_values_kernel<KB, VT, QS, HP>, p, b, kv, g, splits, cluster));
   return Q38_OK;
 }
 template <int KB>
 int launch_values(const q38_mixed_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, const TileGeom& g,
                   int splits, cudaStream_t s) {
   if (kv.v_dim <= 64)
-    return g.q_in_smem ? launch_values_as<KB, 8, true>(p, b, kv, g, splits, s) : launch_values_as<KB, 8, false>(p, b, kv, g, splits, s);
-  return g.q_in_smem ? launch_values_as<KB, 16, true>(p, b, kv, g, splits, s) : launch_values_as<KB, 16, false>(p, b, kv, g, splits, s);
+    return g.heads_per_mma == 2 ? launch_values_as<KB, 8, false, 2>(p, b, kv, g, splits, s)
+           : g.q_in_smem        ? launch_values_as<KB, 8, true, 1>(p, b, kv, g, splits, s)
+                                : launch_values_as<KB, 8, false, 1>(p, b, kv, g, splits, s);
+  return g.heads_per_mma == 2 ? launch_values_as<KB, 16, false, 2>(p, b, kv, g, splits, s)
+         : g.q_in_smem        ? launch_values_as<KB, 16, true, 1>(p, b, kv, g, splits, s)
+                              : launch_values_as<KB, 16, false, 1>(p, b, kv, g, splits, s);
 }
 
 template <int GROUP, int VT>

@@ -161,8 +161,8 @@ def rounded(a, act):
 
 
 # heads, kv heads, dim, vdim, rotated dims
-SHAPES = [(4, 2, 40, 24, 16), (3, 3, 96, 64, 24), (8, 1, 64, 128, 64), (16, 4, 128, 128, 32), (1, 1, 24, 8, 24),
-          (6, 6, 32, 200, 8), (20, 2, 72, 136, 0), (2, 2, 256, 256, 64), (32, 8, 64, 64, 64), (5, 1, 288, 40, 10), (16, 16, 128, 128, 32),
+SHAPES = [(4, 2, 40, 24, 16), (3, 3, 80, 56, 20), (20, 1, 24, 24, 8), (8, 1, 64, 128, 64), (16, 4, 128, 128, 32), (1, 1, 24, 8, 24),
+          (6, 6, 32, 200, 8), (20, 2, 72, 136, 0), (2, 2, 256, 256, 64), (32, 8, 64, 64, 64), (5, 1, 288, 40, 10), (16, 16, 128, 128, 32), (32, 8, 128, 128, 128),
           (9, 3, 16, 300, 6)]
 
 
