@@ -6,9 +6,9 @@
 //            each split of the keys leaves (maximum, sum). values: one pass over V; a warp normalises a page's scores with the
 //            merged (maximum, sum), mixes the heads on the fly and multiplies. K and V are read once.
 //   prefill  stats: (maximum, sum) per (token, head), flash-style without values. values: a CTA holds the heads' weights of
-//            16 ... 64 tokens x 32 keys in shared memory, mixes them over the heads there, and every warp carries the output
+//            8 ... 64 tokens x 32 keys in shared memory, mixes them over the heads there, and every warp carries the output
 //            of one (head, 128 value columns, 16 tokens) in registers.
-// Operands of the value kernels and of the decode score kernel are loaded from global memory straight into fragments: 16
+// Operands of the decode kernels are loaded from global memory straight into fragments, those of prefill from staged tiles: 16
 // contiguous bytes of a row (8 head dimensions of a key, or 8 keys of a value column - V is stored transposed) are the
 // registers of two k16 steps under a permutation of k that both operands share.
 #include <algorithm>
@@ -199,7 +199,13 @@ mixed_decode_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
   for (int pg = r.p0 + warp; pg < r.p1; pg += kDecWarps) {
     const int page = table[pg];
     const float2* S = reinterpret_cast<const float2*>(p.scores + (size_t)page * H * kPage) + lane;
+    const bf16* V = v_page(kv, page, head) + (size_t)(v0 + g) * kPage + t * 8;
+    uint4 bf[8];  // the first values travel while the weights are computed
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (i < nvt) bf[i] = ld16(V + (size_t)i * 8 * kPage);
     float2 w[GROUP] = {};
+#pragma unroll 8
     for (int h = 0; h < H; ++h) {
       const float2 s = S[h * (kPage / 2)];
       const float mx = mx_sm[h], e0 = ex2(s.x - mx), e1 = ex2(s.y - mx);
@@ -214,16 +220,15 @@ mixed_decode_values_kernel(q38_mixed_attention_params p, q38_batch_desc b, q38_k
     for (int o = 0; o < GROUP; ++o)
       *reinterpret_cast<__nv_bfloat162*>(W + o * 96 + 2 * lane) = __floats2bfloat162_rn(w[o].x, w[o].y);
     __syncwarp();
-    const bf16* V = v_page(kv, page, head) + (size_t)(v0 + g) * kPage + t * 8;
 #pragma unroll
     for (int kb = 0; kb < 2; ++kb) {
       const AFragPair a = a_fragments(ld16(W + g * 96 + kb * 32 + t * 8), ld16(W + (g + 8) * 96 + kb * 32 + t * 8));
 #pragma unroll
       for (int n0 = 0; n0 < VT; n0 += 8) {
-        uint4 bf[8];
+        if (kb > 0 || n0 > 0)
 #pragma unroll
-        for (int i = 0; i < 8; ++i)
-          if (n0 + i < nvt) bf[i] = ld16(V + (size_t)(n0 + i) * 8 * kPage + kb * 32);
+          for (int i = 0; i < 8; ++i)
+            if (n0 + i < nvt) bf[i] = ld16(V + (size_t)(n0 + i) * 8 * kPage + kb * 32);
 #pragma unroll
         for (int i = 0; i < 8; ++i)
           if (n0 + i < nvt) mma_pair(acc[n0 + i], a, bf[i]);

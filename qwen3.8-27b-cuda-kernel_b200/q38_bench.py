@@ -46,7 +46,7 @@ def ints(text: str) -> list[int]:
 
 
 def random_tokens(rng, n: int, vocab: int) -> np.ndarray:
-    return rng.integers(1000, min(vocab, 150000), size=n).astype(np.int32)
+    return rng.integers(min(1000, vocab // 2), min(vocab, 150000), size=n).astype(np.int32)
 
 
 def prefill_all(runner, slot: int, tokens: np.ndarray, chunk: int, sampling) -> tuple[int, float]:
@@ -129,7 +129,7 @@ def print_ops(title: str, ops: dict) -> None:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="", help="a .q38 model file")
+    ap.add_argument("--model", default="", help="a .q38 model file, or a folder with config.json and model.safetensors")
     ap.add_argument("--synthetic", default="", choices=["", "27b"], help="no file: random BQ planes of this geometry")
     ap.add_argument("--layers", type=int, default=64, help="--synthetic: number of layers")
     ap.add_argument("--recipe", default="default")
@@ -138,7 +138,8 @@ def main(argv=None) -> int:
     ap.add_argument("--gen", type=int, default=32, help="decode steps per measurement")
     ap.add_argument("--prefill", default="512,2048,8192", help="prompt lengths of the prefill sweep ('' = skip)")
     ap.add_argument("--chunk", type=int, default=512, help="prefill chunk")
-    ap.add_argument("--kv", default="int8", choices=["int8", "bf16"])
+    ap.add_argument("--kv", default="auto", choices=["auto", "int8", "bf16"], help="auto: the architecture's own (int8 for BQ models)")
+    ap.add_argument("--compute", default="bf16", choices=["bf16", "f32"], help="f32: layer-list models in 32-bit throughout")
     ap.add_argument("--profile", action="store_true", help="per-op GPU time of a decode and a prefill step")
     ap.add_argument("--tune", default="", metavar="FILE", help="sweep the GEMM tile configurations of the 27B shapes and write a tuning table")
     ap.add_argument("--tuning", default="", metavar="FILE", help="install a tuning table before measuring")
@@ -178,7 +179,8 @@ def main(argv=None) -> int:
     max_batch = max(batches + [1])
     kv_tokens = max(max_batch * (need + 64), max(prompts + [0]) + 128)
     runner = eng.Runner(model, eng.default_runner_options(max_batch=max_batch, prefill_chunk=args.chunk,
-                                                          kv_dtype=0 if args.kv == "int8" else 1, kv_tokens=kv_tokens,
+                                                          kv_dtype={"auto": -1, "int8": 0, "bf16": 1}[args.kv], kv_tokens=kv_tokens,
+                                                          compute_dtype=int(args.compute == "f32"),
                                                           max_context=max(need, max(prompts + [0]) + 64), verbose=0))
     rng = np.random.default_rng(42)
     results["memory"] = runner.memory()
