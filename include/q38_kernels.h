@@ -325,8 +325,8 @@ typedef struct q38_kv_layer_desc {
   int max_pages_per_seq;
 } q38_kv_layer_desc;
 
-/* One recurrent layer's state: slot s at byte offset s * slot_bytes of both pointers. `state` is fp32 [width]; `conv` is
- * a ring [taps][channels] in activation precision, the input of position p in row p % taps. Positions before the
+/* One recurrent layer's state: slot s at byte offset s * slot_bytes of both pointers. `state` is fp32 [width] (retention:
+ * [heads][dim][vdim]); `conv` is a ring [taps][channels] in activation precision, the input of position p in row p % taps. Positions before the
  * sequence's start are zero and are never read, so a fresh sequence needs no clearing: at position 0 the recurrence
  * starts from zero by itself. */
 typedef struct q38_recurrent_state_desc {
@@ -346,22 +346,38 @@ typedef struct q38_dense_weight {
 #define Q38_DENSE_STORE_F32 1 /* out[m][n] fp32 */
 #define Q38_DENSE_GLU_GELU 2  /* rows of W alternate gate, up: out[m][n / 2] = gelu_tanh(gate) * up, activation precision */
 #define Q38_DENSE_GLU_SILU 3  /* the same with silu */
+#define Q38_DENSE_XIELU 4     /* out[m][n] = xielu(y), activation precision: alpha_p y^2 + y / 2 for y > 0,
+                               * alpha_n (e^y - 1 - y) + y / 2 below */
+#define Q38_DENSE_GATE_SIGMOID 5 /* out[m][n] = y * sigmoid(gate[m][n]), both in activation precision */
 typedef struct q38_dense_epilogue {
   int kind;
   void* out;
   int ldo;
+  float alpha_p, alpha_n; /* Q38_DENSE_XIELU */
+  const void* gate;       /* Q38_DENSE_GATE_SIGMOID */
+  int ld_gate;
 } q38_dense_epilogue;
 #define Q38_DENSE_AUTO (-1)
 int q38_dense_gemm_num_configs(void);
 const char* q38_dense_gemm_config_name(int config);
 int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_dense_weight* w, const q38_dense_epilogue* ep,
                    const q38_gemm_workspace* ws, void* stream, int config);
+/* Several products of one shape side by side: group g multiplies columns g * x_stride ... of x (k of them; x_stride a
+ * multiple of 8 elements) with rows g * n ... of W and writes columns g * out_stride ... of out (and of the gate). */
+typedef struct q38_dense_groups {
+  int count, x_stride, out_stride;
+} q38_dense_groups;
+int q38_dense_gemm_grouped(const void* x, int ldx, int act, int m, const q38_dense_weight* w, const q38_dense_groups* groups,
+                           const q38_dense_epilogue* ep, const q38_gemm_workspace* ws, void* stream, int config);
 
-/* RMS norm with a gain per coordinate (gain_stride 1) or one gain for all (gain_stride 0); `out` in activation precision. */
+/* RMS norm with a gain per coordinate (gain_stride 1) or one gain for all (gain_stride 0); `out` in activation precision.
+ * With groups > 1 (the stream kernels below) each of `groups` equal consecutive parts of the row has its own root mean
+ * square; 0 or 1 = the whole row. */
 typedef struct q38_norm {
   const float* gain;
   int gain_stride;
   float eps;
+  int groups;
 } q38_norm;
 /* residual = table[token] (+ positions[position] if not NULL); out = norm(residual) */
 int q38_embed_norm(const q38_bf16* table, const q38_bf16* positions, const int32_t* tokens, const int* tok_pos, int m,
@@ -373,6 +389,25 @@ int q38_residual_norm(const float* y, int ldy, int m, int width, const q38_norm*
 /* out[i] = norm(residual[rows ? rows[i] : first + i]), i < n (rows is a device array) */
 int q38_gather_norm(const float* residual, const int* rows, int first, int n, int width, const q38_norm* norm, void* out,
                     int ld_out, int act, void* stream);
+
+/* Hyper-connections: the residual is `streams` rows per token, [m][streams][width] fp32. A sublayer reads
+ * u = sum_s in[s] x_s through its pre-norm and its output y replaces all streams at once by
+ * x_t = sum_s mix[s][t] x_s + mult * out[t] * y. One stream with in = out = mix = 1 is the ordinary residual sum. */
+typedef struct q38_stream_update {
+  const float* mix; /* [streams from][streams to] */
+  const float* out; /* [streams] */
+  float mult;
+} q38_stream_update;
+#define Q38_MAX_STREAMS 16
+/* every stream = scale * table[token]; out = norm(sum_s in[s] x_s) */
+int q38_stream_embed(const q38_bf16* table, const int32_t* tokens, int m, int width, float scale, int streams,
+                     float* residual, const float* in, const q38_norm* norm, void* out, int ld_out, int act, void* stream);
+/* The update of one sublayer, then the next one's u and pre-norm (unless next is NULL), in one pass over the row. */
+int q38_stream_norm(const float* y, int ldy, int m, int width, int streams, const q38_stream_update* update, float* residual,
+                    const float* in, const q38_norm* next, void* out, int ld_out, int act, void* stream);
+/* out[i] = norm(sum of the streams of row rows ? rows[i] : first + i), i < n */
+int q38_stream_gather(const float* residual, const int* rows, int first, int n, int width, int streams, const q38_norm* norm,
+                      void* out, int ld_out, int act, void* stream);
 
 /* Rotary positions on the leading rot_dims of every query and key head (dimension i turns with i + rot_dims / 2 by
  * position * inv_freq[i]), optional blending of the values with a first layer's, and the append to the cache.
@@ -444,6 +479,60 @@ typedef struct q38_rglru_params {
   int ld_out;
 } q38_rglru_params;
 int q38_rglru(const q38_rglru_params* p, const q38_batch_desc* batch, const q38_recurrent_state_desc* st, void* stream);
+
+/* Retention: linear attention with a fixed decay per head, S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; q and k turn
+ * on their leading rot_dims dimensions as in q38_rope_append and k is multiplied by k_scale after that; every head's o is
+ * divided by its root mean square and multiplied by silu(g). proj rows: [q: heads x dim | k: heads x dim | v: heads x vdim
+ * | g: heads x vdim]. Rotated q and k, decays, the state and o are fp32 (products of fp32 factors on the tensor cores run
+ * on bf16 hi + lo terms). */
+#define Q38_RETENTION_CHUNK 64
+typedef struct q38_retention_params {
+  const void* proj;
+  int ld_proj;
+  int act;
+  int heads, dim, vdim;
+  int rot_dims;
+  const double* inv_freq;  /* [rot_dims / 2] */
+  const float* decay_pow;  /* [heads][Q38_RETENTION_CHUNK + 1]: decay^i */
+  float k_scale, eps;
+  void* qk;                /* scratch, q38_retention_qk_bytes(num_tokens, ...); runs of one token per sequence use none */
+  float* o;                /* scratch [M][heads * vdim]; likewise */
+  void* out;
+  int ld_out;
+} q38_retention_params;
+size_t q38_retention_qk_bytes(int tokens, int heads, int dim, int act);
+int q38_retention(const q38_retention_params* p, const q38_batch_desc* batch, const q38_recurrent_state_desc* st, void* stream);
+
+/* Latent attention: queries and keys meet in the latent space of the cache. The cache (kv_heads 1, v_dim 0) holds one
+ * normalised latent c of k_dim numbers per token, which is key and value at once; the heads' key and value matrices are
+ * applied to the queries before and to the outputs after (q38_dense_gemm_grouped).
+ * Append: proj rows [query latent: q_rank | kv latent: kv_rank | ...], each divided by its root mean square and multiplied
+ * by its gain; the query latent goes to q_out, the other one into the cache (zero beyond kv_rank). */
+typedef struct q38_latent_append_params {
+  const void* proj;
+  int ld_proj;
+  int act;
+  int q_rank, kv_rank;
+  const float* q_gain;  /* [q_rank] */
+  const float* kv_gain; /* [kv_rank] */
+  float eps;
+  void* q_out;
+  int ld_q;
+} q38_latent_append_params;
+int q38_latent_append(const q38_latent_append_params* p, const q38_batch_desc* batch, const q38_kv_layer_desc* kv, void* stream);
+/* Causal softmax attention of `heads` queries per token over the latents: out_h = sum_j softmax_j(scale q_h . c_j) c_j. */
+typedef struct q38_latent_attention_params {
+  const void* q;        /* [M][heads][k_dim] */
+  int act;
+  int heads;
+  float scale;
+  void* out;            /* [M][heads][k_dim] */
+  float* partials;      /* scratch for divided key ranges; q38_latent_attention_partial_floats() is always enough */
+  size_t partial_floats;
+} q38_latent_attention_params;
+size_t q38_latent_attention_partial_floats(int k_dim);
+int q38_latent_attention(const q38_latent_attention_params* p, const q38_batch_desc* batch, const q38_kv_layer_desc* kv,
+                         void* stream);
 
 /* Diagnostics. */
 const char* q38_last_error(void);           /* message of the last failed launcher call on this thread */

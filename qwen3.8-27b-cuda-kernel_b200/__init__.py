@@ -120,11 +120,37 @@ class DenseWeight(C.Structure):
 
 
 class DenseEpilogue(C.Structure):
-    _fields_ = [("kind", C.c_int), ("out", C.c_void_p), ("ldo", C.c_int)]
+    _fields_ = [("kind", C.c_int), ("out", C.c_void_p), ("ldo", C.c_int), ("alpha_p", C.c_float), ("alpha_n", C.c_float),
+                ("gate", C.c_void_p), ("ld_gate", C.c_int)]
+
+
+class DenseGroups(C.Structure):
+    _fields_ = [("count", C.c_int), ("x_stride", C.c_int), ("out_stride", C.c_int)]
 
 
 class Norm(C.Structure):
-    _fields_ = [("gain", C.c_void_p), ("gain_stride", C.c_int), ("eps", C.c_float)]
+    _fields_ = [("gain", C.c_void_p), ("gain_stride", C.c_int), ("eps", C.c_float), ("groups", C.c_int)]
+
+
+class StreamUpdate(C.Structure):
+    _fields_ = [("mix", C.c_void_p), ("out", C.c_void_p), ("mult", C.c_float)]
+
+
+class RetentionParams(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("heads", C.c_int), ("dim", C.c_int),
+                ("vdim", C.c_int), ("rot_dims", C.c_int), ("inv_freq", C.c_void_p), ("decay_pow", C.c_void_p),
+                ("k_scale", C.c_float), ("eps", C.c_float), ("qk", C.c_void_p), ("o", C.c_void_p), ("out", C.c_void_p),
+                ("ld_out", C.c_int)]
+
+
+class LatentAppendParams(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld_proj", C.c_int), ("act", C.c_int), ("q_rank", C.c_int), ("kv_rank", C.c_int),
+                ("q_gain", C.c_void_p), ("kv_gain", C.c_void_p), ("eps", C.c_float), ("q_out", C.c_void_p), ("ld_q", C.c_int)]
+
+
+class LatentAttentionParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("act", C.c_int), ("heads", C.c_int), ("scale", C.c_float), ("out", C.c_void_p),
+                ("partials", C.c_void_p), ("partial_floats", C.c_size_t)]
 
 
 class RopeAppendParams(C.Structure):
@@ -166,7 +192,8 @@ class SamplingArgs(C.Structure):
 EPI_STORE_BF16, EPI_SWIGLU, EPI_RESIDUAL, EPI_STORE_F32, EPI_ALLREDUCE_RESIDUAL = 0, 1, 2, 3, 4
 KV_INT8, KV_BF16, KV_F32 = 0, 1, 2
 ACT_BF16, ACT_F32 = 0, 1
-DENSE_STORE, DENSE_STORE_F32, DENSE_GLU_GELU, DENSE_GLU_SILU = 0, 1, 2, 3
+DENSE_STORE, DENSE_STORE_F32, DENSE_GLU_GELU, DENSE_GLU_SILU, DENSE_XIELU, DENSE_GATE_SIGMOID = 0, 1, 2, 3, 4, 5
+RETENTION_CHUNK = 64
 
 # every entry point include/q38_kernels.h declares, with its ctypes signature
 KERNEL_API = {
@@ -213,6 +240,20 @@ KERNEL_API = {
     "q38_dense_gemm_config_name": (C.c_char_p, [C.c_int]),
     "q38_dense_gemm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(DenseWeight), C.POINTER(DenseEpilogue),
                                  C.POINTER(GemmWorkspace), C.c_void_p, C.c_int]),
+    "q38_dense_gemm_grouped": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(DenseWeight), C.POINTER(DenseGroups),
+                                         C.POINTER(DenseEpilogue), C.POINTER(GemmWorkspace), C.c_void_p, C.c_int]),
+    "q38_stream_embed": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p, C.c_void_p,
+                                   C.POINTER(Norm), C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
+    "q38_stream_norm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.POINTER(StreamUpdate), C.c_void_p,
+                                  C.c_void_p, C.POINTER(Norm), C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
+    "q38_stream_gather": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.POINTER(Norm), C.c_void_p,
+                                    C.c_int, C.c_int, C.c_void_p]),
+    "q38_retention_qk_bytes": (C.c_size_t, [C.c_int, C.c_int, C.c_int, C.c_int]),
+    "q38_retention": (C.c_int, [C.POINTER(RetentionParams), C.POINTER(BatchDesc), C.POINTER(RecurrentStateDesc), C.c_void_p]),
+    "q38_latent_append": (C.c_int, [C.POINTER(LatentAppendParams), C.POINTER(BatchDesc), C.POINTER(KvLayerDesc), C.c_void_p]),
+    "q38_latent_attention_partial_floats": (C.c_size_t, [C.c_int]),
+    "q38_latent_attention": (C.c_int, [C.POINTER(LatentAttentionParams), C.POINTER(BatchDesc), C.POINTER(KvLayerDesc),
+                                       C.c_void_p]),
     "q38_embed_norm": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p,
                                  C.POINTER(Norm), C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
     "q38_residual_norm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(Norm), C.c_void_p, C.POINTER(Norm),

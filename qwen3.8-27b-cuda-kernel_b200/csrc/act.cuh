@@ -19,6 +19,10 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
   return 0.5f * x * (1.0f + tanhf(u));
 }
+// alpha_p z^2 + z / 2 above zero, alpha_n (e^z - 1 - z) + z / 2 below
+__device__ __forceinline__ float xielu_f(float z, float alpha_p, float alpha_n) {
+  return (z > 0.0f ? alpha_p * z * z : alpha_n * (expm1f(z) - z)) + 0.5f * z;
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
 // The A fragments of two k16 steps of mma.m16n8k16 from 16 contiguous bytes of rows g and g + 8. An MMA takes its four A

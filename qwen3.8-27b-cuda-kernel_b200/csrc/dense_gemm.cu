@@ -14,13 +14,15 @@ __device__ __forceinline__ float glu_act(int kind, float gate) { return kind == 
 // ---- CUDA-core kernel, fp32 arithmetic throughout -------------------------------------------------------------------
 constexpr int kST = 64, kSK = 16;
 template <typename T>
-__global__ void __launch_bounds__(256) dense_simt_kernel(const T* __restrict__ x, int ldx, int m, q38_dense_weight w, q38_dense_epilogue ep) {
+__global__ void __launch_bounds__(256) dense_simt_kernel(const T* __restrict__ x, int ldx, int m, q38_dense_weight w, q38_dense_groups groups, q38_dense_epilogue ep) {
   pdl_wait();
   pdl_launch_dependents();
   __shared__ float xs[kSK][kST + 4], wt[kSK][kST + 4];
   const int m0 = blockIdx.y * kST, n0 = blockIdx.x * kST;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-  const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(w.w);
+  const int grp = blockIdx.z, oc = grp * groups.out_stride;  // output columns of this group start at oc
+  const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(w.w) + (size_t)grp * w.n * w.ld;
+  x += (size_t)grp * groups.x_stride;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < w.k; k0 += kSK) {
     for (int i = threadIdx.x; i < kST * kSK; i += 256) {
@@ -50,11 +52,16 @@ __global__ void __launch_bounds__(256) dense_simt_kernel(const T* __restrict__ x
       const int n = n0 + 4 * tx + j;
       if (n >= w.n) continue;
       const float v = acc[i][j] + (w.bias ? w.bias[n] : 0.0f);
-      if (ep.kind == Q38_DENSE_STORE_F32) static_cast<float*>(ep.out)[(size_t)t * ep.ldo + n] = v;
-      else if (ep.kind == Q38_DENSE_STORE) static_cast<T*>(ep.out)[(size_t)t * ep.ldo + n] = from_f32<T>(v);
+      if (ep.kind == Q38_DENSE_STORE_F32) static_cast<float*>(ep.out)[(size_t)t * ep.ldo + oc + n] = v;
+      else if (ep.kind == Q38_DENSE_STORE) static_cast<T*>(ep.out)[(size_t)t * ep.ldo + oc + n] = from_f32<T>(v);
+      else if (ep.kind == Q38_DENSE_XIELU)
+        static_cast<T*>(ep.out)[(size_t)t * ep.ldo + oc + n] = from_f32<T>(xielu_f(v, ep.alpha_p, ep.alpha_n));
+      else if (ep.kind == Q38_DENSE_GATE_SIGMOID)
+        static_cast<T*>(ep.out)[(size_t)t * ep.ldo + oc + n] =
+            from_f32<T>(v * sigmoid_f(to_f32(static_cast<const T*>(ep.gate)[(size_t)t * ep.ld_gate + oc + n])));
       else if ((j & 1) && n >= 1) {
         const float gate = acc[i][j - 1] + (w.bias ? w.bias[n - 1] : 0.0f);
-        static_cast<T*>(ep.out)[(size_t)t * ep.ldo + n / 2] = from_f32<T>(glu_act(ep.kind, gate) * v);
+        static_cast<T*>(ep.out)[(size_t)t * ep.ldo + oc + n / 2] = from_f32<T>(glu_act(ep.kind, gate) * v);
       }
     }
   }
@@ -62,8 +69,8 @@ __global__ void __launch_bounds__(256) dense_simt_kernel(const T* __restrict__ x
 
 template <typename T>
 int launch_simt(const DenseCall& c, cudaStream_t s) {
-  (void)launch_kernel(dense_simt_kernel<T>, dim3((c.w.n + kST - 1) / kST, (c.m + kST - 1) / kST), dim3(256), 0, s,
-                      static_cast<const T*>(c.x), c.ldx, c.m, c.w, c.ep);
+  (void)launch_kernel(dense_simt_kernel<T>, dim3((c.w.n + kST - 1) / kST, (c.m + kST - 1) / kST, c.groups.count), dim3(256), 0, s,
+                      static_cast<const T*>(c.x), c.ldx, c.m, c.w, c.groups, c.ep);
   Q38_LAUNCH_OK("dense_simt_kernel");
   return Q38_OK;
 }
@@ -83,16 +90,29 @@ extern "C" const char* q38_dense_gemm_config_name(int c) { return c >= 0 && c < 
 
 extern "C" int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_dense_weight* w, const q38_dense_epilogue* ep,
                               const q38_gemm_workspace* ws, void* stream, int config) {
-  Q38_REQUIRE(x && w && ep && w->w && ep->out, "dense_gemm: null argument");
+  const q38_dense_groups one{1, 0, 0};
+  return q38_dense_gemm_grouped(x, ldx, act, m, w, &one, ep, ws, stream, config);
+}
+
+extern "C" int q38_dense_gemm_grouped(const void* x, int ldx, int act, int m, const q38_dense_weight* w,
+                                      const q38_dense_groups* groups, const q38_dense_epilogue* ep, const q38_gemm_workspace* ws,
+                                      void* stream, int config) {
+  Q38_REQUIRE(x && w && groups && ep && w->w && ep->out, "dense_gemm: null argument");
   if (m == 0) return Q38_OK;
-  Q38_REQUIRE(m > 0 && w->n > 0 && w->k > 0 && w->ld >= w->k && w->ld % 64 == 0 && ldx >= w->k, "dense_gemm: sizes m %d n %d k %d ld %d ldx %d",
-              m, w->n, w->k, w->ld, ldx);
-  Q38_REQUIRE(ep->kind >= Q38_DENSE_STORE && ep->kind <= Q38_DENSE_GLU_SILU, "dense_gemm: epilogue %d", ep->kind);
-  const bool glu = ep->kind >= Q38_DENSE_GLU_GELU;
+  const q38_dense_groups g = *groups;
+  Q38_REQUIRE(g.count > 0 && g.count <= 65535 && g.x_stride >= 0 && g.out_stride >= 0 && (g.count == 1 || g.x_stride >= w->k),
+              "dense_gemm: %d groups, %d columns apart", g.count, g.x_stride);
+  Q38_REQUIRE(g.count == 1 || !w->bias, "dense_gemm: grouped products take no bias");
+  Q38_REQUIRE(m > 0 && w->n > 0 && w->k > 0 && w->ld >= w->k && w->ld % 64 == 0 && ldx >= (g.count - 1) * g.x_stride + w->k,
+              "dense_gemm: sizes m %d n %d k %d ld %d ldx %d", m, w->n, w->k, w->ld, ldx);
+  Q38_REQUIRE(ep->kind >= Q38_DENSE_STORE && ep->kind <= Q38_DENSE_GATE_SIGMOID, "dense_gemm: epilogue %d", ep->kind);
+  const bool glu = dense_glu(ep->kind);
   Q38_REQUIRE(!glu || w->n % 2 == 0, "dense_gemm: gated epilogue needs an even n, got %d", w->n);
-  Q38_REQUIRE(ep->ldo >= (glu ? w->n / 2 : w->n), "dense_gemm: ldo %d", ep->ldo);
+  const int out_n = glu ? w->n / 2 : w->n, out_cols = (g.count - 1) * g.out_stride + out_n;
+  Q38_REQUIRE(ep->ldo >= out_cols && (g.count == 1 || g.out_stride >= out_n), "dense_gemm: ldo %d, groups %d apart", ep->ldo, g.out_stride);
+  Q38_REQUIRE(ep->kind != Q38_DENSE_GATE_SIGMOID || (ep->gate && ep->ld_gate >= out_cols), "dense_gemm: gate");
   Q38_REQUIRE(config < kNumDenseConfigs, "dense_gemm: config %d", config);
-  const DenseCall c{x, ldx, m, *w, *ep, ws};
+  const DenseCall c{x, ldx, m, *w, g, *ep, ws};
   cudaStream_t s = as_stream(stream);
   if (act == Q38_ACT_F32) return launch_simt<float>(c, s);
   const bool aligned = dense_umma_fits(c);
@@ -111,6 +131,6 @@ extern "C" int q38_dense_gemm(const void* x, int ldx, int act, int m, const q38_
       Q38_REQUIRE((w->k + 63) / 64 >= cl, "dense_gemm: k %d is too short for a cluster of %d", w->k, cl);
       return dense_umma(c, {m <= 32 ? 32 : 64, cl}, s);
     }
-    default: return dense_umma(c, dense_umma_choice(m, w->n, w->k), s);
+    default: return dense_umma(c, dense_umma_choice(m, w->n, w->k, g.count), s);
   }
 }

@@ -48,7 +48,28 @@ struct Args {
   void* out;
   int ldo;
   int cluster;
+  int x_stride, out_stride;  // between the groups' columns
+  int group_tiles;           // (weight tile, token tile) pairs of one group
+  float alpha_p, alpha_n;
+  const void* gate;
+  int ld_gate;
 };
+
+// Item i of the list: group, weight tile, token tile.
+struct Item {
+  int group, tn, tm;
+};
+__device__ __forceinline__ Item item_at(const Args& a, int i) {
+  const int g = a.x_stride || a.out_stride ? i / a.group_tiles : 0, r = i - g * a.group_tiles;
+  return {g, r / a.tiles_m, r % a.tiles_m};
+}
+// Epilogues of one accumulator value: output column n of its group, token t.
+__device__ __forceinline__ float unary(const Args& a, float v, int t, int col) {
+  if (a.kind == Q38_DENSE_XIELU) return xielu_f(v, a.alpha_p, a.alpha_n);
+  if (a.kind == Q38_DENSE_GATE_SIGMOID)
+    return v * sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)t * a.ld_gate + col]));
+  return v;
+}
 
 __device__ __forceinline__ float glu(int kind, float gate, float up) {
   return (kind == Q38_DENSE_GLU_SILU ? silu_f(gate) : gelu_tanh_f(gate)) * up;
@@ -108,16 +129,19 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
     if (lane == 0) {
       // weights of the first ring turn ahead of the previous kernel's end
       const int pre = min(C::kStages, k1 - k0);
+      const Item it0 = item_at(a, first);
+      const int first_row = it0.group * a.n + it0.tn * kTileN;
       if (first < a.items)
         for (int i = 0; i < pre; ++i) {
           mbar_expect_tx(&full[i], C::kStageBytes);
-          tma_load_2d(ring + i * C::kStageBytes, &wmap, (k0 + i) * 64, (first / a.tiles_m) * kTileN, &full[i]);
+          tma_load_2d(ring + i * C::kStageBytes, &wmap, (k0 + i) * 64, first_row, &full[i]);
         }
       pdl_wait();
       uint32_t it = 0;
       bool alive = true;
       for (int item = first; item < a.items && alive; item += step) {
-        const int tn = item / a.tiles_m, tm = item % a.tiles_m;
+        const Item w = item_at(a, item);
+        const int w_row = w.group * a.n + w.tn * kTileN, x_col = w.group * a.x_stride, x_row = w.tm * TOK;
         for (int k = k0; k < k1; ++k, ++it) {
           const int s = int(it % C::kStages);
           uint8_t* dst = ring + s * C::kStageBytes;
@@ -127,9 +151,9 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
               break;
             }
             mbar_expect_tx(&full[s], C::kStageBytes);
-            tma_load_2d(dst, &wmap, k * 64, tn * kTileN, &full[s]);
+            tma_load_2d(dst, &wmap, k * 64, w_row, &full[s]);
           }
-          tma_load_2d(dst + kWBytes, &xmap, k * 64, tm * TOK, &full[s]);
+          tma_load_2d(dst + kWBytes, &xmap, x_col + k * 64, x_row, &full[s]);
         }
       }
       // nothing may still be in flight towards this CTA's shared memory when it ends: wait for the stages whose
@@ -171,7 +195,8 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
     uint32_t seg = 0;
     bool alive = true;
     for (int item = first; item < a.items && alive; item += step, ++seg) {
-      const int tn = item / a.tiles_m, tm = item % a.tiles_m;
+      const Item w = item_at(a, item);
+      const int tn = w.tn, tm = w.tm, oc = w.group * a.out_stride;
       const uint32_t acc = seg % C::kAccs;
       alive = __all_sync(0xffffffffu, wait_flag(&acc_full[acc], (seg / C::kAccs) & 1, abort_flag, 0x804));
       if (!alive) break;
@@ -188,40 +213,46 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
         }
       } else {
         const float bias = a.bias && n < a.n ? a.bias[n] : 0.0f;
-        const bool odd = lane & 1;
+        const bool odd = lane & 1, glu_kind = a.kind == Q38_DENSE_GLU_GELU || a.kind == Q38_DENSE_GLU_SILU;
         for (int c = 0; c < TOK; c += 16) {
           if (c >= tokens) break;
           uint32_t r[16];
           tmem_ld16(taddr + uint32_t(c), r);
           if (a.kind == Q38_DENSE_STORE_F32) {
-            float* out = static_cast<float*>(a.out) + (size_t)(t0 + c) * a.ldo + n;
+            float* out = static_cast<float*>(a.out) + (size_t)(t0 + c) * a.ldo + oc + n;
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (c + j < tokens && n < a.n) out[(size_t)j * a.ldo] = __uint_as_float(r[j]) + bias;
           } else {
+            if (a.kind >= Q38_DENSE_XIELU) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (c + j < tokens && n < a.n) r[j] = __float_as_uint(unary(a, __uint_as_float(r[j]) + bias, t0 + c + j, oc + n));
+            }
+            const float add = a.kind >= Q38_DENSE_XIELU ? 0.0f : bias;
             // neighbouring lanes exchange: the even lane takes token j, the odd lane token j + 1, both columns n & ~1, n | 1
             uint32_t packed[8];
 #pragma unroll
             for (int j = 0; j < 16; j += 2) {
-              const float v0 = __uint_as_float(r[j]) + bias, v1 = __uint_as_float(r[j + 1]) + bias;
+              const float v0 = __uint_as_float(r[j]) + add, v1 = __uint_as_float(r[j + 1]) + add;
               const float other = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
               const float lo = odd ? other : v0, hi = odd ? v1 : other;  // columns n & ~1 and n | 1
-              if (a.kind == Q38_DENSE_STORE) {
+              if (!glu_kind) {
                 const __nv_bfloat162 p = __floats2bfloat162_rn(lo, hi);
                 packed[j / 2] = *reinterpret_cast<const uint32_t*>(&p);
               } else {
                 packed[j / 2] = uint32_t(__bfloat16_as_ushort(__float2bfloat16_rn(glu(a.kind, lo, hi))));
               }
             }
-            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
+            __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + oc;
             const int ne = n & ~1;
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               const int t = c + 2 * j + (odd ? 1 : 0);
               if (t >= tokens || ne >= a.n) continue;
               __nv_bfloat16* row = out + (size_t)(t0 + t) * a.ldo;
-              if (a.kind != Q38_DENSE_STORE) row[ne >> 1] = __ushort_as_bfloat16(uint16_t(packed[j]));
-              else if (ne + 1 < a.n && (a.ldo & 1) == 0) *reinterpret_cast<uint32_t*>(row + ne) = packed[j];
+              if (glu_kind) row[ne >> 1] = __ushort_as_bfloat16(uint16_t(packed[j]));
+              else if (ne + 1 < a.n && ((a.ldo | oc) & 1) == 0) *reinterpret_cast<uint32_t*>(row + ne) = packed[j];
               else {
                 row[ne] = __ushort_as_bfloat16(uint16_t(packed[j] & 0xffffu));
                 if (ne + 1 < a.n) row[ne + 1] = __ushort_as_bfloat16(uint16_t(packed[j] >> 16));
@@ -242,7 +273,8 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
     cluster_sync_all();  // every CTA's partial tile is in its shared memory
     if (warp >= 2 && first < a.items && *abort_flag == 0) {
       const int quarter = warp & 3, nl = quarter * 32 + lane;
-      const int tn = first / a.tiles_m, tm = first % a.tiles_m;
+      const Item w = item_at(a, first);
+      const int tn = w.tn, tm = w.tm, oc = w.group * a.out_stride;
       const int n = tn * kTileN + nl, t0 = tm * TOK, tokens = min(TOK, a.m - t0);
       const float bias = a.bias && n < a.n ? a.bias[n] : 0.0f;
       const uint32_t part = smem_u32(ring);
@@ -260,11 +292,11 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
           const int t = tb + u * a.cluster;
           if (t >= tokens) break;
           const float x = v[u] + bias;
-          const size_t row = (size_t)(t0 + t) * a.ldo;
+          const size_t row = (size_t)(t0 + t) * a.ldo + oc;
           if (a.kind == Q38_DENSE_STORE_F32) {
             if (n < a.n) static_cast<float*>(a.out)[row + n] = x;
-          } else if (a.kind == Q38_DENSE_STORE) {
-            if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(x);
+          } else if (a.kind == Q38_DENSE_STORE || a.kind >= Q38_DENSE_XIELU) {
+            if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(unary(a, x, t0 + t, oc + n));
           } else {
             const float up = __shfl_xor_sync(0xffffffffu, x, 1);
             if (!(lane & 1) && n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + (n >> 1)] = __float2bfloat16_rn(glu(a.kind, x, up));
@@ -318,19 +350,26 @@ int launch(const DenseCall& c, int cluster, cudaStream_t stream) {
                                                        cudaFuncAttributeMaxDynamicSharedMemorySize, K::kSmemBytes);
   Q38_CUDA_OK(attr);
   CUtensorMap wmap, xmap;
-  if (const int rc = encode_2d(&wmap, c.w.w, c.w.n, c.w.k, c.w.ld, kTileN)) return rc;
-  if (const int rc = encode_2d(&xmap, c.x, c.m, c.w.k, c.ldx, TOK)) return rc;
+  if (const int rc = encode_2d(&wmap, c.w.w, c.groups.count * c.w.n, c.w.k, c.w.ld, kTileN)) return rc;
+  if (const int rc = encode_2d(&xmap, c.x, c.m, (c.groups.count - 1) * c.groups.x_stride + c.w.k, c.ldx, TOK)) return rc;
   Args a{};
   a.m = c.m;
   a.n = c.w.n;
   a.kg = (c.w.k + 63) / 64;
   a.tiles_n = (c.w.n + kTileN - 1) / kTileN;
   a.tiles_m = (c.m + TOK - 1) / TOK;
-  a.items = a.tiles_n * a.tiles_m;
+  a.group_tiles = a.tiles_n * a.tiles_m;
+  a.items = c.groups.count * a.group_tiles;
+  a.x_stride = c.groups.x_stride;
+  a.out_stride = c.groups.out_stride;
   a.bias = c.w.bias;
   a.kind = c.ep.kind;
   a.out = c.ep.out;
   a.ldo = c.ep.ldo;
+  a.alpha_p = c.ep.alpha_p;
+  a.alpha_n = c.ep.alpha_n;
+  a.gate = c.ep.gate;
+  a.ld_gate = c.ep.ld_gate;
   a.cluster = CLUSTER ? cluster : 1;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(CLUSTER ? a.items * cluster : std::min(a.items, num_sms()));
@@ -366,14 +405,14 @@ int launch_tok(const DenseCall& c, int cluster, cudaStream_t stream) {
 }  // namespace
 
 bool dense_umma_fits(const DenseCall& c) {
-  return c.ldx % 8 == 0 && c.w.ld % 8 == 0 && reinterpret_cast<uintptr_t>(c.x) % 16 == 0 && reinterpret_cast<uintptr_t>(c.w.w) % 16 == 0;
+  return c.ldx % 8 == 0 && c.groups.x_stride % 8 == 0 && c.w.ld % 8 == 0 && reinterpret_cast<uintptr_t>(c.x) % 16 == 0 && reinterpret_cast<uintptr_t>(c.w.w) % 16 == 0;
 }
 
 // Tile and cluster size by a cost in cycles. A CTA spends kStep cycles on a k-group (it is the transfer from L2 that bounds
 // it, not the MMA); CTAs that share an SM share its transfer rate. Clusters add their reduction and are only used when every
 // CTA of the launch is resident at once (two per SM up to 64 tokens).
-DenseUmmaChoice dense_umma_choice(int m, int n, int k) {
-  const int sms = num_sms(), kg = (k + 63) / 64, tiles_n = (n + kTileN - 1) / kTileN;
+DenseUmmaChoice dense_umma_choice(int m, int n, int k, int groups) {
+  const int sms = num_sms(), kg = (k + 63) / 64, tiles_n = groups * ((n + kTileN - 1) / kTileN);
   constexpr int kTok[4] = {32, 64, 128, 256}, kStep[4] = {400, 420, 560, 900}, kShared[4] = {320, 380, 560, 900};
   DenseUmmaChoice best{64, 1};
   long long best_cost = -1;

@@ -296,11 +296,21 @@ using RopeAppendParams = q38_rope_append_params;
 using MixedAttentionParams = q38_mixed_attention_params;
 using MinGruParams = q38_mingru_params;
 using RgLruParams = q38_rglru_params;
+using DenseGroups = q38_dense_groups;
+using StreamUpdate = q38_stream_update;
+using RetentionParams = q38_retention_params;
+using LatentAppendParams = q38_latent_append_params;
+using LatentAttentionParams = q38_latent_attention_params;
 
 inline void dense_gemm(const void* x, int ldx, int act, int m, const DenseWeight& w, const DenseEpilogue& ep,
                        const GemmWorkspace& ws, cudaStream_t stream) {
   const q38_gemm_workspace cws{ws.partials, ws.partial_floats, ws.counters, ws.num_counters};
   detail::ok(q38_dense_gemm(x, ldx, act, m, &w, &ep, &cws, stream, Q38_DENSE_AUTO));
+}
+inline void dense_gemm_grouped(const void* x, int ldx, int act, int m, const DenseWeight& w, const DenseGroups& groups,
+                               const DenseEpilogue& ep, const GemmWorkspace& ws, cudaStream_t stream) {
+  const q38_gemm_workspace cws{ws.partials, ws.partial_floats, ws.counters, ws.num_counters};
+  detail::ok(q38_dense_gemm_grouped(x, ldx, act, m, &w, &groups, &ep, &cws, stream, Q38_DENSE_AUTO));
 }
 inline void embed_norm(const q38_bf16* table, const q38_bf16* positions, const int32_t* tokens, const int* tok_pos, int m,
                        int width, float* residual, const Norm& norm, void* out, int ld_out, int act, cudaStream_t stream) {
@@ -313,6 +323,30 @@ inline void residual_norm(const float* y, int ldy, int m, int width, const Norm&
 inline void gather_norm(const float* residual, const int* rows, int first, int n, int width, const Norm& norm, void* out,
                         int ld_out, int act, cudaStream_t stream) {
   detail::ok(q38_gather_norm(residual, rows, first, n, width, &norm, out, ld_out, act, stream));
+}
+inline void stream_embed(const q38_bf16* table, const int32_t* tokens, int m, int width, float scale, int streams,
+                         float* residual, const float* in, const Norm& norm, void* out, int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_stream_embed(table, tokens, m, width, scale, streams, residual, in, &norm, out, ld_out, act, stream));
+}
+inline void stream_norm(const float* y, int ldy, int m, int width, int streams, const StreamUpdate& update, float* residual,
+                        const float* in, const Norm* next, void* out, int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_stream_norm(y, ldy, m, width, streams, &update, residual, in, next, out, ld_out, act, stream));
+}
+inline void stream_gather(const float* residual, const int* rows, int first, int n, int width, int streams, const Norm& norm,
+                          void* out, int ld_out, int act, cudaStream_t stream) {
+  detail::ok(q38_stream_gather(residual, rows, first, n, width, streams, &norm, out, ld_out, act, stream));
+}
+inline void retention(const RetentionParams& p, const BatchDesc& batch, const RecurrentStateDesc& st, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_retention(&p, &b, &st, stream));
+}
+inline void latent_append(const LatentAppendParams& p, const BatchDesc& batch, const KvLayerDesc& kv, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_latent_append(&p, &b, &kv, stream));
+}
+inline void latent_attention(const LatentAttentionParams& p, const BatchDesc& batch, const KvLayerDesc& kv, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_latent_attention(&p, &b, &kv, stream));
 }
 inline void rope_append(const RopeAppendParams& p, const BatchDesc& batch, const KvLayerDesc& kv, cudaStream_t stream) {
   const q38_batch_desc b = batch.c();

@@ -85,8 +85,9 @@ inline int64_t align_up(int64_t a, int64_t b) { return ceil_div(a, b) * b; }
 // model configuration (reference include/qwen38/config.h; header block of docs/FORMAT.md 1.1)
 // ===================================================================================================
 // Extension: one layer of a decoder whose configuration lists its layers one by one (layer-list architectures): a
-// sequence mixer with its own sizes and an optional gated feed-forward.
-enum class MixerKind : uint8_t { Attention, MinGru, RgLru };
+// sequence mixer with its own sizes and an optional feed-forward.
+enum class MixerKind : uint8_t { Attention, MinGru, RgLru, Retention, LatentAttention };
+inline bool is_recurrent(MixerKind k) { return k == MixerKind::MinGru || k == MixerKind::RgLru || k == MixerKind::Retention; }
 struct AttentionSpec {
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
   int rot_dims = 0;          // leading dimensions of a query / key head that turn, dimension i with i + rot_dims / 2
@@ -101,10 +102,23 @@ struct RecurrentSpec {
   int blocks = 1;            // RG-LRU: block-diagonal gates
   int taps = 0;              // RG-LRU: causal convolution, current token included
 };
+struct RetentionSpec {
+  int heads = 0, dim = 0, vdim = 0;
+  int rot_dims = 0;
+  double rot_base = 10000.0;
+  std::vector<double> decay;  // per head
+};
+struct LatentAttentionSpec {
+  int heads = 0, dim = 0, vdim = 0;
+  int q_rank = 0, kv_rank = 0;  // latents the queries and the keys / values go through
+  float scale = 1.0f;
+};
 struct LayerSpec {
   MixerKind mixer = MixerKind::Attention;
   AttentionSpec attn;
   RecurrentSpec rec;
+  RetentionSpec ret;
+  LatentAttentionSpec latent;
   int ff = 0;                // feed-forward width, 0 = the layer has none
 };
 
@@ -121,7 +135,15 @@ struct ModelConfig {
   std::vector<uint8_t> is_attention;   // per layer: 1 full attention, 0 Gated DeltaNet
   std::vector<int32_t> eos_token_ids;
   bool learned_positions = false;      // a learned position table bounds the context
-  std::vector<LayerSpec> layers;       // layer-list architectures; empty for the BQ family
+  // layer-list architectures
+  std::vector<LayerSpec> layers;       // empty for the BQ family
+  float embedding_scale = 1.0f;
+  float residual_mult = 1.0f;          // factor of every sublayer's output
+  int norm_groups = 1;                 // equal parts of the row with a root mean square each
+  int streams = 0;                     // residual streams (hyper-connections); 0 = an ordinary residual sum
+  int loop_start = 0, loop_stop = 0, loop_times = 1;  // layers [start, stop) run `times` times in a row
+  // Indices of `layers` in the order they run. Every run has a cache or state of its own.
+  std::vector<int> layer_runs() const;
 
   int num_attention_layers() const;
   int num_gdn_layers() const;

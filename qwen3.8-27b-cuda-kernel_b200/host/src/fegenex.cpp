@@ -9,7 +9,7 @@ namespace {
 
 LayerListDesign fegenex_design() {
   LayerListDesign d;
-  d.glu = LayerListDesign::Glu::Gelu;
+  d.feed_forward = LayerListDesign::FeedForward::GeluGlu;
   d.norm_gain_is_scalar = true;
   d.rglru_log_decay = -8.0f;
   return d;

@@ -53,16 +53,17 @@ struct Linear {
   std::vector<std::string> weights;             // stacked along the output
   std::vector<std::string> biases;              // one per weight, "" = none
   bool interleave = false;                      // two weights whose rows alternate
+  int block = 0, block_to = 0;                  // blocks of `block` rows are spread to `block_to` rows (zero rows between)
 };
 
 struct LayerTensors {
-  Linear in, out, glu, down;
+  Linear in, out, up, down;
 };
 
 std::string mix(int i, const char* name) { return "l" + std::to_string(i) + ".mix." + name; }
 std::string at_layer(int i, const char* name) { return "l" + std::to_string(i) + "." + name; }
 
-LayerTensors names_of(const LayerSpec& l, int i) {
+LayerTensors names_of(const LayerSpec& l, int i, LayerListDesign::FeedForward ff) {
   LayerTensors t;
   auto w = [&](const char* n) { return mix(i, n); };
   switch (l.mixer) {
@@ -78,16 +79,34 @@ LayerTensors names_of(const LayerSpec& l, int i) {
       t.in = {{w("y"), w("x")}, {w("y.b"), w("x.b")}};
       t.out = {{w("o")}, {""}};
       break;
+    case MixerKind::Retention:
+      t.in = {{w("q"), w("k"), w("v"), w("g")}, {"", "", "", ""}};
+      t.out = {{w("o")}, {""}};
+      break;
+    case MixerKind::LatentAttention:
+      t.in = {{w("dq"), w("dkv"), w("g")}, {"", "", ""}};
+      t.out = {{w("o")}, {""}};
+      break;
   }
   if (l.ff) {
-    t.glu = {{at_layer(i, "mlp.gate"), at_layer(i, "mlp.up")}, {"", ""}, true};
+    if (ff == LayerListDesign::FeedForward::Xielu) t.up = {{at_layer(i, "mlp.up")}, {""}};
+    else t.up = {{at_layer(i, "mlp.gate"), at_layer(i, "mlp.up")}, {"", ""}, true};
     t.down = {{at_layer(i, "mlp.down")}, {""}};
   }
   return t;
 }
 
+struct StreamWeights {  // one sublayer's hyper-connection
+  const float *in = nullptr, *out = nullptr, *mix = nullptr;
+};
+
 struct LayerWeightsDev {
-  kernels::DenseWeight in{}, out{}, glu{}, down{};
+  kernels::DenseWeight in{}, out{}, up{}, down{};
+  float alpha_p = 0.0f, alpha_n = 0.0f;  // xIELU
+  StreamWeights hc1, hc2;
+  const float* decay_pow = nullptr;
+  const float *q_gain = nullptr, *kv_gain = nullptr;
+  kernels::DenseWeight uq{}, uk{}, uv{};  // latent attention; uk and uv hold one matrix per head
   const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
   const float *v_mix = nullptr, *head_mix = nullptr;
   const double* inv_freq = nullptr;
@@ -130,15 +149,42 @@ class LayerListModel final : public StepModel {
   template <typename T>
   const T* put(DeviceArena* arena, const std::vector<T>& v);
   kernels::DenseWeight put_linear(DeviceArena* arena, const Linear& l);
+  kernels::DenseWeight put_heads(DeviceArena* arena, const std::string& name, int heads, int n_to, bool transpose);
   const float* put_f32(DeviceArena* arena, const std::string& name);
   const q38_bf16* put_bf16(DeviceArena* arena, const std::string& name);
 
   void gemm(const StepContext& ctx, const void* x, int ldx, int m, const kernels::DenseWeight& w, int kind, void* out, int ldo) {
-    kernels::dense_gemm(x, ldx, act_, m, w, {kind, out, ldo}, gemm_ws_, ctx.stream);
+    kernels::DenseEpilogue ep{};
+    ep.kind = kind;
+    ep.out = out;
+    ep.ldo = ldo;
+    kernels::dense_gemm(x, ldx, act_, m, w, ep, gemm_ws_, ctx.stream);
   }
-  kernels::Norm norm(const float* gain) const { return {gain, design_.norm_gain_is_scalar ? 0 : 1, cfg_.rms_norm_eps}; }
+  kernels::Norm norm(const float* gain) const {
+    return {gain, design_.norm_gain_is_scalar ? 0 : 1, cfg_.rms_norm_eps, cfg_.norm_groups};
+  }
+  StreamWeights put_streams(DeviceArena* arena, int layer, const char* name);
+  // A sublayer's output (y_) joins the residual, and the next sublayer's normed input is formed (unless there is none).
+  struct Sublayer {
+    const float* pre = nullptr;   // pre-norm gain, null = nothing follows
+    const float* post = nullptr;  // post-norm gain
+    StreamWeights hc;
+  };
+  Sublayer mixer_of(int run) const {
+    const LayerWeightsDev& W = layers_[size_t(runs_[size_t(run)])];
+    return {W.norm1, W.norm1b, W.hc1};
+  }
+  Sublayer feed_forward_of(int run) const {
+    const LayerWeightsDev& W = layers_[size_t(runs_[size_t(run)])];
+    return {W.norm2, W.norm2b, W.hc2};
+  }
+  void join_residual(const StepContext& ctx, int m, const Sublayer& done, const Sublayer& next);
+  void feed_forward(const StepContext& ctx, int m, const LayerWeightsDev& W);
   void attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i, bool first_values, bool blend);
+  void latent_attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i);
   void recurrent(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int rec_i);
+  void retention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W,
+                 const kernels::RecurrentStateDesc& st);
 
   TensorReader reader_;
   ModelConfig cfg_;
@@ -146,6 +192,9 @@ class LayerListModel final : public StepModel {
   bool f32_ = false;
   int act_ = Q38_ACT_BF16;
   size_t elem_ = 2;
+  std::vector<int> runs_;  // layers in the order they run; a run's cache or state is the run's own
+  int streams_ = 1;
+  bool hyper_ = false;     // the weights have hyper-connections (otherwise one stream, plain sum)
   std::vector<KvLayerGeometry> kv_layers_;
   std::vector<RecurrentLayerGeometry> rec_layers_;
   int score_heads_ = 0;
@@ -154,7 +203,7 @@ class LayerListModel final : public StepModel {
   DeviceArena arena_;
   std::vector<LayerWeightsDev> layers_;
   const q38_bf16 *embed_ = nullptr, *pos_ = nullptr;
-  const float* final_norm_ = nullptr;
+  const float *final_norm_ = nullptr, *ones_ = nullptr;
   kernels::DenseWeight head_{};
   std::unique_ptr<RecurrentStatePool> state_;
   DeviceBuffer scores_;
@@ -172,6 +221,16 @@ class LayerListModel final : public StepModel {
   float* stats_ = nullptr;
   float* partials_ = nullptr;
   float* rec_scratch_ = nullptr;
+  uint8_t* qk_ = nullptr;      // retention: rotated queries and keys of a prefill step
+  float* rec_o_ = nullptr;     // retention: outputs before their norm
+  uint8_t* q_latent_ = nullptr;    // latent attention: normed query latents
+  uint8_t* q_heads_ = nullptr;     // ... queries per head
+  uint8_t* q_absorbed_ = nullptr;  // ... and in the space of the cached latents
+  uint8_t* o_latent_ = nullptr;
+  float* latent_partials_ = nullptr;
+  size_t latent_partial_floats_ = 0;
+  int ld_q_latent_ = 0, ld_q_heads_ = 0, max_absorbed_ = 0, max_latent_k_ = 0, max_rec_o_ = 0;
+  size_t qk_bytes_per_token_ = 0;
   uint8_t* head_x_ = nullptr;
   kernels::GemmWorkspace gemm_ws_;
 };
@@ -181,8 +240,14 @@ LayerListModel::LayerListModel(const ModelFile& f, const RunnerOptions& o, const
   act_ = f32_ ? Q38_ACT_F32 : Q38_ACT_BF16;
   elem_ = f32_ ? 4 : 2;
   ld_x_ = up(cfg_.hidden_size, 64);
+  runs_ = cfg_.layer_runs();
+  hyper_ = cfg_.streams > 1 || (cfg_.streams == 1 && cfg_.num_layers > 0 && f.has_tensor(at_layer(0, "hc1.in")));
+  streams_ = std::max(1, cfg_.streams);
+  QWEN38_CHECK(!design_.post_norms || (streams_ == 1 && cfg_.norm_groups == 1 && cfg_.embedding_scale == 1.0f && cfg_.residual_mult == 1.0f),
+               "post-norms go with one plain residual");
   int v_first = 0;
-  for (const LayerSpec& l : cfg_.layers) {
+  for (const int run : runs_) {
+    const LayerSpec& l = cfg_.layers[size_t(run)];
     if (l.mixer == MixerKind::Attention) {
       const AttentionSpec& a = l.attn;
       const KvLayerGeometry g{a.kv_heads, up(a.dim, 32), up(a.vdim, 8)};
@@ -197,6 +262,25 @@ LayerListModel::LayerListModel(const ModelFile& f, const RunnerOptions& o, const
         QWEN38_CHECK(v_first == 0 || v_first == a.kv_heads * a.vdim, "layers that blend values need value heads of one total size");
         v_first = a.kv_heads * a.vdim;
       }
+    } else if (l.mixer == MixerKind::LatentAttention) {
+      const LatentAttentionSpec& a = l.latent;
+      const KvLayerGeometry g{1, up(a.kv_rank, 32), 0};
+      kv_layers_.push_back(g);
+      ld_proj_ = std::max(ld_proj_, up(a.q_rank + a.kv_rank + a.heads * a.vdim, 64));
+      ld_mixer_ = std::max(ld_mixer_, up(a.heads * a.vdim, 64));
+      ld_q_latent_ = std::max(ld_q_latent_, up(a.q_rank, 64));
+      ld_q_heads_ = std::max(ld_q_heads_, up(a.heads * up(a.dim, 8), 64));
+      max_absorbed_ = std::max(max_absorbed_, a.heads * g.k_dim);
+      max_latent_k_ = std::max(max_latent_k_, g.k_dim);
+    } else if (l.mixer == MixerKind::Retention) {
+      const RetentionSpec& r = l.ret;
+      RecurrentLayerGeometry g;
+      g.width = r.heads * r.dim * r.vdim;
+      rec_layers_.push_back(g);
+      ld_proj_ = std::max(ld_proj_, up(2 * r.heads * (r.dim + r.vdim), 64));
+      ld_mixer_ = std::max(ld_mixer_, up(r.heads * r.vdim, 64));
+      max_rec_o_ = std::max(max_rec_o_, r.heads * r.vdim);
+      qk_bytes_per_token_ = std::max(qk_bytes_per_token_, q38_retention_qk_bytes(1, r.heads, r.dim, act_));
     } else {
       RecurrentLayerGeometry g;
       g.width = l.rec.width;
@@ -250,7 +334,7 @@ kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear
   for (size_t i = 0; i < l.weights.size(); ++i) {
     const TensorInfo& t = reader_.file().tensor(l.weights[i]);
     QWEN38_CHECK(t.shape.size() == 2 && (i == 0 || int(t.shape[1]) == d.k), l.weights[i], ": shape");
-    d.n += int(t.shape[0]);
+    d.n += l.block ? int(t.shape[0]) / l.block * l.block_to : int(t.shape[0]);
     d.k = int(t.shape[1]);
     bias = bias || !l.biases[i].empty();
   }
@@ -262,7 +346,7 @@ kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear
     for (size_t i = 0; i < l.weights.size(); ++i) {
       const TensorInfo& t = reader_.file().tensor(l.weights[i]);
       for (int64_t r = 0; r < t.shape[0]; ++r) {
-        const int64_t to = l.interleave ? 2 * r + int64_t(i) : row0 + r;
+        const int64_t to = l.interleave ? 2 * r + int64_t(i) : l.block ? r / l.block * l.block_to + r % l.block : row0 + r;
         reader_.copy_bf16(t, r * t.shape[1], t.shape[1], w.data() + to * d.ld);
         if (!l.biases[i].empty()) b[size_t(to)] = reader_.at(reader_.file().tensor(l.biases[i]), r);
       }
@@ -274,6 +358,36 @@ kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear
   return d;
 }
 
+// One matrix [n_to][k] per head, rows padded to 64 columns: `name` holds the heads' rows one after the other,
+// [heads * rows][cols]; with `transpose` a head's matrix is [cols][rows].
+kernels::DenseWeight LayerListModel::put_heads(DeviceArena* arena, const std::string& name, int heads, int n_to, bool transpose) {
+  const TensorInfo& t = reader_.file().tensor(name);
+  const int rows = int(t.shape[0]) / heads, cols = int(t.shape[1]);
+  kernels::DenseWeight d{};
+  d.n = n_to;
+  d.k = transpose ? rows : cols;
+  d.ld = up(d.k, 64);
+  std::vector<q38_bf16> w(size_t(up(heads * d.n, 16)) * size_t(d.ld), 0);
+  if (arena) {
+    std::vector<q38_bf16> line(size_t(cols), 0);
+    for (int h = 0; h < heads; ++h)
+      for (int r = 0; r < rows; ++r) {
+        reader_.copy_bf16(t, (int64_t(h) * rows + r) * cols, cols, line.data());
+        for (int c = 0; c < cols; ++c)
+          w[transpose ? (size_t(h) * d.n + size_t(c)) * d.ld + size_t(r) : (size_t(h) * d.n + size_t(r)) * d.ld + size_t(c)] = line[size_t(c)];
+      }
+  }
+  d.w = put(arena, w);
+  return d;
+}
+
+StreamWeights LayerListModel::put_streams(DeviceArena* arena, int layer, const char* name) {
+  const std::string p = at_layer(layer, name);
+  if (hyper_) return {put_f32(arena, p + ".in"), put_f32(arena, p + ".out"), put_f32(arena, p + ".mix")};
+  const float* one = put(arena, std::vector<float>{1.0f});
+  return {one, one, one};
+}
+
 void LayerListModel::visit_weights(DeviceArena* arena) {
   weight_bytes_ = arena ? weight_bytes_ : 0;
   layers_.assign(cfg_.layers.size(), {});
@@ -282,16 +396,42 @@ void LayerListModel::visit_weights(DeviceArena* arena) {
   for (int i = 0; i < cfg_.num_layers; ++i) {
     const LayerSpec& l = cfg_.layers[size_t(i)];
     LayerWeightsDev& W = layers_[size_t(i)];
-    const LayerTensors names = names_of(l, i);
+    const LayerTensors names = names_of(l, i, design_.feed_forward);
     W.in = put_linear(arena, names.in);
     W.out = put_linear(arena, names.out);
     W.norm1 = put_f32(arena, at_layer(i, "norm1"));
-    W.norm1b = put_f32(arena, at_layer(i, "norm1b"));
+    if (design_.post_norms) W.norm1b = put_f32(arena, at_layer(i, "norm1b"));
+    else W.hc1 = put_streams(arena, i, "hc1");
     if (l.ff) {
       W.norm2 = put_f32(arena, at_layer(i, "norm2"));
-      W.norm2b = put_f32(arena, at_layer(i, "norm2b"));
-      W.glu = put_linear(arena, names.glu);
+      if (design_.post_norms) W.norm2b = put_f32(arena, at_layer(i, "norm2b"));
+      else W.hc2 = put_streams(arena, i, "hc2");
+      W.up = put_linear(arena, names.up);
       W.down = put_linear(arena, names.down);
+      if (design_.feed_forward == LayerListDesign::FeedForward::Xielu) {
+        const TensorInfo& t = reader_.file().tensor(at_layer(i, "mlp.act"));
+        auto softplus = [](double x) { return std::max(x, 0.0) + std::log1p(std::exp(-std::abs(x))); };
+        W.alpha_p = float(softplus(reader_.at(t, 0)));
+        W.alpha_n = float(0.5 + softplus(reader_.at(t, 1)));
+      }
+    }
+    if (l.mixer == MixerKind::Retention) {
+      const RetentionSpec& r = l.ret;
+      std::vector<double> freq(size_t(r.rot_dims / 2));
+      for (size_t k = 0; k < freq.size(); ++k) freq[k] = std::pow(r.rot_base, -2.0 * double(k) / double(r.rot_dims));
+      W.inv_freq = put(arena, freq);
+      std::vector<float> pow_table;
+      for (const double d : r.decay)
+        for (int k = 0; k <= Q38_RETENTION_CHUNK; ++k) pow_table.push_back(float(std::pow(d, double(k))));
+      W.decay_pow = put(arena, pow_table);
+    }
+    if (l.mixer == MixerKind::LatentAttention) {
+      const LatentAttentionSpec& a = l.latent;
+      W.q_gain = put_f32(arena, mix(i, "dq.norm"));
+      W.kv_gain = put_f32(arena, mix(i, "dkv.norm"));
+      W.uq = put_linear(arena, {{mix(i, "uq")}, {""}, false, a.dim, up(a.dim, 8)});
+      W.uk = put_heads(arena, mix(i, "uk"), a.heads, up(a.kv_rank, 32), true);
+      W.uv = put_heads(arena, mix(i, "uv"), a.heads, a.vdim, false);
     }
     if (l.mixer == MixerKind::Attention) {
       if (l.attn.value_mix) W.v_mix = put_f32(arena, mix(i, "vmix"));
@@ -326,6 +466,7 @@ void LayerListModel::visit_weights(DeviceArena* arena) {
     }
   }
   final_norm_ = put_f32(arena, "final.norm");
+  ones_ = put(arena, std::vector<float>(size_t(streams_), 1.0f));
   head_ = put_linear(arena, {{"head"}, {""}});
 }
 
@@ -338,7 +479,7 @@ void LayerListModel::load_weights() {
 void LayerListModel::carve(Workspace& w, const StepContext& ctx) {
   const size_t T = size_t(ctx.max_tokens), R = size_t(ctx.max_rows);
   const size_t gemm_partials = f32_ ? 0 : size_t(2) * size_t(ctx.num_sms) * 128 * 256;
-  residual_ = w.take<float>(T * size_t(cfg_.hidden_size));
+  residual_ = w.take<float>(T * size_t(streams_) * size_t(cfg_.hidden_size));
   x_ = w.take<uint8_t>(T * size_t(ld_x_) * elem_);
   proj_ = w.take<uint8_t>(T * size_t(ld_proj_) * elem_);
   mixer_ = w.take<uint8_t>(T * size_t(ld_mixer_) * elem_);
@@ -349,6 +490,14 @@ void LayerListModel::carve(Workspace& w, const StepContext& ctx) {
   stats_ = w.take<float>(T * size_t(max_heads_) * 2 * kStatSplits);
   if (!f32_) partials_ = w.take<float>(R * kMaxSplits * (size_t(max_attn_out_) + 2 * size_t(max_heads_)));
   rec_scratch_ = w.take<float>(2 * T * size_t(max_rec_));
+  qk_ = w.take<uint8_t>(T * qk_bytes_per_token_);
+  rec_o_ = w.take<float>(T * size_t(max_rec_o_));
+  q_latent_ = w.take<uint8_t>(T * size_t(ld_q_latent_) * elem_);
+  q_heads_ = w.take<uint8_t>(T * size_t(ld_q_heads_) * elem_);
+  q_absorbed_ = w.take<uint8_t>(T * size_t(max_absorbed_) * elem_);
+  o_latent_ = w.take<uint8_t>(T * size_t(max_absorbed_) * elem_);
+  latent_partial_floats_ = f32_ || !max_latent_k_ ? 0 : q38_latent_attention_partial_floats(max_latent_k_);
+  latent_partials_ = w.take<float>(latent_partial_floats_);
   head_x_ = w.take<uint8_t>(R * size_t(ld_x_) * elem_);
   gemm_ws_.partials = w.take<float>(gemm_partials);
   gemm_ws_.partial_floats = gemm_partials;
@@ -401,8 +550,78 @@ void LayerListModel::attention(const StepContext& ctx, const StepBatch& b, const
   ctx.mark(b.decode ? "mix.attn_decode" : "mix.attn_prefill");
 }
 
+void LayerListModel::latent_attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i) {
+  const LatentAttentionSpec& a = l.latent;
+  const kernels::KvLayerDesc kv = ctx.kv->layer_desc(attn_i);
+  const int dim_ld = up(a.dim, 8);
+  kernels::LatentAppendParams lp{};
+  lp.proj = proj_;
+  lp.ld_proj = ld_proj_;
+  lp.act = act_;
+  lp.q_rank = a.q_rank;
+  lp.kv_rank = a.kv_rank;
+  lp.q_gain = W.q_gain;
+  lp.kv_gain = W.kv_gain;
+  lp.eps = cfg_.rms_norm_eps;
+  lp.q_out = q_latent_;
+  lp.ld_q = ld_q_latent_;
+  kernels::latent_append(lp, b.all, kv, ctx.stream);
+  ctx.mark("mix.latent_append");
+  gemm(ctx, q_latent_, ld_q_latent_, b.m, W.uq, Q38_DENSE_STORE, q_heads_, ld_q_heads_);
+  ctx.mark("gemm.latent_uq");
+  kernels::DenseEpilogue ep{};
+  ep.kind = Q38_DENSE_STORE;
+  ep.out = q_absorbed_;
+  ep.ldo = a.heads * kv.k_dim;
+  kernels::dense_gemm_grouped(q_heads_, ld_q_heads_, act_, b.m, W.uk, {a.heads, dim_ld, kv.k_dim}, ep, gemm_ws_, ctx.stream);
+  ctx.mark("gemm.latent_uk");
+  kernels::LatentAttentionParams ap{};
+  ap.q = q_absorbed_;
+  ap.act = act_;
+  ap.heads = a.heads;
+  ap.scale = a.scale;
+  ap.out = o_latent_;
+  ap.partials = latent_partials_;
+  ap.partial_floats = latent_partial_floats_;
+  if (b.decode || b.mixed) kernels::latent_attention(ap, b.single_part, kv, ctx.stream);
+  if (!b.decode) kernels::latent_attention(ap, b.chunk_part, kv, ctx.stream);
+  ctx.mark(b.decode ? "mix.latent_decode" : "mix.latent_prefill");
+  ep.kind = Q38_DENSE_GATE_SIGMOID;
+  ep.out = mixer_;
+  ep.ldo = ld_mixer_;
+  ep.gate = proj_ + size_t(a.q_rank + a.kv_rank) * elem_;
+  ep.ld_gate = ld_proj_;
+  kernels::dense_gemm_grouped(o_latent_, a.heads * kv.k_dim, act_, b.m, W.uv, {a.heads, kv.k_dim, a.vdim}, ep, gemm_ws_, ctx.stream);
+  ctx.mark("gemm.latent_uv");
+}
+
+void LayerListModel::retention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W,
+                               const kernels::RecurrentStateDesc& st) {
+  const RetentionSpec& r = l.ret;
+  kernels::RetentionParams p{};
+  p.proj = proj_;
+  p.ld_proj = ld_proj_;
+  p.act = act_;
+  p.heads = r.heads;
+  p.dim = r.dim;
+  p.vdim = r.vdim;
+  p.rot_dims = r.rot_dims;
+  p.inv_freq = W.inv_freq;
+  p.decay_pow = W.decay_pow;
+  p.k_scale = float(1.0 / std::sqrt(double(r.dim)));
+  p.eps = cfg_.rms_norm_eps;
+  p.qk = qk_;
+  p.o = rec_o_;
+  p.out = mixer_;
+  p.ld_out = ld_mixer_;
+  if (b.decode || b.mixed) kernels::retention(p, b.single_part, st, ctx.stream);
+  if (!b.decode) kernels::retention(p, b.chunk_part, st, ctx.stream);
+  ctx.mark("mix.retention");
+}
+
 void LayerListModel::recurrent(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int rec_i) {
   const kernels::RecurrentStateDesc st = state_->layer_desc(rec_i);
+  if (l.mixer == MixerKind::Retention) return retention(ctx, b, l, W, st);
   if (l.mixer == MixerKind::MinGru) {
     const kernels::MinGruParams p{proj_, ld_proj_, act_, l.rec.width, mixer_, ld_mixer_};
     if (b.decode || b.mixed) kernels::mingru(p, b.single_part, st, ctx.stream);
@@ -432,47 +651,79 @@ void LayerListModel::recurrent(const StepContext& ctx, const StepBatch& b, const
   ctx.mark("mix.rglru");
 }
 
+void LayerListModel::join_residual(const StepContext& ctx, int m, const Sublayer& done, const Sublayer& next) {
+  const kernels::Norm pre = norm(next.pre);
+  const kernels::Norm* then = next.pre ? &pre : nullptr;
+  if (design_.post_norms)
+    kernels::residual_norm(y_, ld_x_, m, cfg_.hidden_size, norm(done.post), residual_, then, x_, ld_x_, act_, ctx.stream);
+  else
+    kernels::stream_norm(y_, ld_x_, m, cfg_.hidden_size, streams_, {done.hc.mix, done.hc.out, cfg_.residual_mult}, residual_,
+                         next.hc.in, then, x_, ld_x_, act_, ctx.stream);
+  ctx.mark("residual_norm");
+}
+
+void LayerListModel::feed_forward(const StepContext& ctx, int m, const LayerWeightsDev& W) {
+  kernels::DenseEpilogue ep{};
+  ep.out = ff_;
+  ep.ldo = ld_ff_;
+  ep.alpha_p = W.alpha_p;
+  ep.alpha_n = W.alpha_n;
+  switch (design_.feed_forward) {
+    case LayerListDesign::FeedForward::GeluGlu: ep.kind = Q38_DENSE_GLU_GELU; break;
+    case LayerListDesign::FeedForward::SiluGlu: ep.kind = Q38_DENSE_GLU_SILU; break;
+    case LayerListDesign::FeedForward::Xielu: ep.kind = Q38_DENSE_XIELU; break;
+  }
+  kernels::dense_gemm(x_, ld_x_, act_, m, W.up, ep, gemm_ws_, ctx.stream);
+  ctx.mark(design_.feed_forward == LayerListDesign::FeedForward::Xielu ? "gemm.mlp_up" : "gemm.mlp_gate_up");
+  gemm(ctx, ff_, ld_ff_, m, W.down, Q38_DENSE_STORE_F32, y_, ld_x_);
+  ctx.mark("gemm.mlp_down");
+}
+
 void LayerListModel::forward(const StepContext& ctx, const StepBatch& b) {
-  const int m = b.m, H = cfg_.hidden_size, n = cfg_.num_layers;
-  cudaStream_t s = ctx.stream;
-  const int glu = design_.glu == LayerListDesign::Glu::Gelu ? Q38_DENSE_GLU_GELU : Q38_DENSE_GLU_SILU;
-  kernels::embed_norm(embed_, pos_, b.tokens, b.all.tok_pos, m, H, residual_, norm(n ? layers_[0].norm1 : final_norm_), x_, ld_x_,
-                      act_, s);
+  constexpr const char* kIn[] = {"gemm.attn_qkv", "gemm.mingru_in", "gemm.rglru_in", "gemm.retention_in", "gemm.latent_in"};
+  constexpr const char* kOut[] = {"gemm.attn_o", "gemm.mingru_out", "gemm.rglru_out", "gemm.retention_out", "gemm.latent_o"};
+  const int m = b.m, H = cfg_.hidden_size, n = int(runs_.size());
+  const Sublayer nothing;
+  if (design_.post_norms) {
+    kernels::embed_norm(embed_, pos_, b.tokens, b.all.tok_pos, m, H, residual_, norm(n ? mixer_of(0).pre : final_norm_), x_, ld_x_, act_,
+                        ctx.stream);
+  } else {
+    kernels::stream_embed(embed_, b.tokens, m, H, cfg_.embedding_scale, streams_, residual_, n ? mixer_of(0).hc.in : ones_,
+                          norm(n ? mixer_of(0).pre : final_norm_), x_, ld_x_, act_, ctx.stream);
+  }
   ctx.mark("embed");
   int attn_i = 0, rec_i = 0;
   bool have_values = false;
   for (int i = 0; i < n; ++i) {
-    const LayerSpec& l = cfg_.layers[size_t(i)];
-    const LayerWeightsDev& W = layers_[size_t(i)];
-    // the pre-norm that follows this layer; the last layer's successor is the final norm, taken over the sampled rows only
-    const kernels::Norm next_layer = norm(i + 1 < n ? layers_[size_t(i + 1)].norm1 : nullptr);
-    const kernels::Norm* after = i + 1 < n ? &next_layer : nullptr;
+    const LayerSpec& l = cfg_.layers[size_t(runs_[size_t(i)])];
+    const LayerWeightsDev& W = layers_[size_t(runs_[size_t(i)])];
+    // what follows this run; the last one's successor is the final norm, taken over the sampled rows only
+    const Sublayer next = i + 1 < n ? mixer_of(i + 1) : nothing;
     gemm(ctx, x_, ld_x_, m, W.in, Q38_DENSE_STORE, proj_, ld_proj_);
-    ctx.mark(l.mixer == MixerKind::Attention ? "gemm.attn_qkv" : l.mixer == MixerKind::MinGru ? "gemm.mingru_in" : "gemm.rglru_in");
+    ctx.mark(kIn[int(l.mixer)]);
     if (l.mixer == MixerKind::Attention) {
       attention(ctx, b, l, W, attn_i++, l.attn.value_mix && !have_values, l.attn.value_mix && have_values);
       have_values = have_values || l.attn.value_mix;
+    } else if (l.mixer == MixerKind::LatentAttention) {
+      latent_attention(ctx, b, l, W, attn_i++);
     } else {
       recurrent(ctx, b, l, W, rec_i++);
     }
     gemm(ctx, mixer_, ld_mixer_, m, W.out, Q38_DENSE_STORE_F32, y_, ld_x_);
-    ctx.mark(l.mixer == MixerKind::Attention ? "gemm.attn_o" : l.mixer == MixerKind::MinGru ? "gemm.mingru_out" : "gemm.rglru_out");
-    const kernels::Norm norm2 = norm(W.norm2);
-    kernels::residual_norm(y_, ld_x_, m, H, norm(W.norm1b), residual_, l.ff ? &norm2 : after, x_, ld_x_, act_, s);
-    ctx.mark("residual_norm");
+    ctx.mark(kOut[int(l.mixer)]);
+    join_residual(ctx, m, mixer_of(i), l.ff ? feed_forward_of(i) : next);
     if (!l.ff) continue;
-    gemm(ctx, x_, ld_x_, m, W.glu, glu, ff_, ld_ff_);
-    ctx.mark("gemm.mlp_gate_up");
-    gemm(ctx, ff_, ld_ff_, m, W.down, Q38_DENSE_STORE_F32, y_, ld_x_);
-    ctx.mark("gemm.mlp_down");
-    kernels::residual_norm(y_, ld_x_, m, H, norm(W.norm2b), residual_, after, x_, ld_x_, act_, s);
-    ctx.mark("residual_norm");
+    feed_forward(ctx, m, W);
+    join_residual(ctx, m, feed_forward_of(i), next);
   }
 }
 
 void LayerListModel::head(const StepContext& ctx, const HeadRows& rows, float* logits) {
-  kernels::gather_norm(residual_, rows.rows, rows.first, rows.count, cfg_.hidden_size, norm(final_norm_), head_x_, ld_x_, act_,
-                       ctx.stream);
+  if (design_.post_norms)
+    kernels::gather_norm(residual_, rows.rows, rows.first, rows.count, cfg_.hidden_size, norm(final_norm_), head_x_, ld_x_, act_, ctx.stream);
+  else
+    kernels::stream_gather(residual_, rows.rows, rows.first, rows.count, cfg_.hidden_size, streams_, norm(final_norm_), head_x_, ld_x_,
+                           act_, ctx.stream);
   gemm(ctx, head_x_, ld_x_, rows.count, head_, Q38_DENSE_STORE_F32, logits, cfg_.vocab_size);
   ctx.mark("gemm.lm_head");
 }
@@ -499,12 +750,24 @@ void check_layer_list_tensors(const ModelFile& file, const LayerListDesign& desi
       r.require(mix(i, name), {n, k});
       if (bias) r.require(mix(i, (std::string(name) + ".b").c_str()), {n});
     };
+    const int64_t S = c.streams;
+    auto streams = [&](const char* name) {
+      if (S == 0 || (S == 1 && !file.has_tensor(at_layer(0, "hc1.in")))) return;
+      const std::string p = at_layer(i, name);
+      r.require(p + ".in", {S});
+      r.require(p + ".out", {S});
+      r.require(p + ".mix", {S, S});
+    };
+    const bool xielu = design.feed_forward == LayerListDesign::FeedForward::Xielu;
     r.require(at_layer(i, "norm1"), gain);
-    r.require(at_layer(i, "norm1b"), gain);
+    if (design.post_norms) r.require(at_layer(i, "norm1b"), gain);
+    streams("hc1");
     if (l.ff) {
       r.require(at_layer(i, "norm2"), gain);
-      r.require(at_layer(i, "norm2b"), gain);
-      r.require(at_layer(i, "mlp.gate"), {l.ff, W});
+      if (design.post_norms) r.require(at_layer(i, "norm2b"), gain);
+      streams("hc2");
+      if (xielu) r.require(at_layer(i, "mlp.act"), {2});
+      else r.require(at_layer(i, "mlp.gate"), {l.ff, W});
       r.require(at_layer(i, "mlp.up"), {l.ff, W});
       r.require(at_layer(i, "mlp.down"), {W, l.ff});
     }
@@ -521,6 +784,24 @@ void check_layer_list_tensors(const ModelFile& file, const LayerListDesign& desi
       linear("x", l.rec.width, W, true);
       linear("g", l.rec.width, W, false);
       linear("o", W, l.rec.width, false);
+    } else if (l.mixer == MixerKind::Retention) {
+      const RetentionSpec& t = l.ret;
+      linear("q", int64_t(t.heads) * t.dim, W, false);
+      linear("k", int64_t(t.heads) * t.dim, W, false);
+      linear("v", int64_t(t.heads) * t.vdim, W, false);
+      linear("g", int64_t(t.heads) * t.vdim, W, false);
+      linear("o", W, int64_t(t.heads) * t.vdim, false);
+    } else if (l.mixer == MixerKind::LatentAttention) {
+      const LatentAttentionSpec& a = l.latent;
+      linear("dq", a.q_rank, W, false);
+      r.require(mix(i, "dq.norm"), {a.q_rank});
+      linear("uq", int64_t(a.heads) * a.dim, a.q_rank, false);
+      linear("dkv", a.kv_rank, W, false);
+      r.require(mix(i, "dkv.norm"), {a.kv_rank});
+      linear("uk", int64_t(a.heads) * a.dim, a.kv_rank, false);
+      linear("uv", int64_t(a.heads) * a.vdim, a.kv_rank, false);
+      linear("g", int64_t(a.heads) * a.vdim, W, false);
+      linear("o", W, int64_t(a.heads) * a.vdim, false);
     } else {
       const int64_t w = l.rec.width, nb = l.rec.blocks, bs = w / nb;
       linear("y", w, W, true);

@@ -1,5 +1,6 @@
 // A decoder that runs the layers its configuration lists: per layer a sequence mixer (attention with mixed heads, minGRU,
-// RG-LRU), optionally a gated feed-forward, each between a pre-norm and a post-norm whose output joins the residual.
+// RG-LRU, retention, latent attention) and optionally a feed-forward. A sublayer stands between a pre-norm and a post-norm
+// whose output joins the residual, or behind a pre-norm only, with one or several residual streams.
 // Dense bf16 weights; activations bf16 or fp32. A design provides names and conventions (LayerListDesign); everything
 // below - weights, cache, state, step - is shared by the designs.
 #pragma once
@@ -9,9 +10,10 @@
 namespace qwen38 {
 
 struct LayerListDesign {
-  enum class Glu { Gelu, Silu };
-  Glu glu = Glu::Gelu;
+  enum class FeedForward { GeluGlu, SiluGlu, Xielu };
+  FeedForward feed_forward = FeedForward::GeluGlu;
   bool norm_gain_is_scalar = true;
+  bool post_norms = true;
   float rglru_log_decay = -8.0f;
 };
 

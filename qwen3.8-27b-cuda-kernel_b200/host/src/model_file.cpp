@@ -68,6 +68,15 @@ int ModelConfig::gdn_index(int layer) const {
   return idx;
 }
 
+std::vector<int> ModelConfig::layer_runs() const {
+  std::vector<int> runs;
+  for (int i = 0; i < loop_start; ++i) runs.push_back(i);
+  for (int pass = 0; pass < loop_times; ++pass)
+    for (int i = loop_start; i < loop_stop; ++i) runs.push_back(i);
+  for (int i = loop_stop; i < num_layers; ++i) runs.push_back(i);
+  return runs;
+}
+
 void ModelConfig::validate() const {
   if (!layers.empty()) {  // a layer-list architecture: its reader has checked the sizes of every layer
     QWEN38_CHECK(int(layers.size()) == num_layers && hidden_size > 0 && vocab_size > 0, "layer list");
@@ -95,10 +104,19 @@ void ModelConfig::validate() const {
 std::string ModelConfig::summary() const {
   std::ostringstream os;
   if (!layers.empty()) {
-    int kinds[3] = {0, 0, 0};
+    constexpr const char* kNames[] = {"attention", "minGRU", "RG-LRU", "retention", "latent attention"};
+    int kinds[5] = {};
     for (const LayerSpec& l : layers) ++kinds[int(l.mixer)];
-    os << architecture << ": hidden " << hidden_size << ", layers " << num_layers << " (" << kinds[0] << " attention / "
-       << kinds[1] << " minGRU / " << kinds[2] << " RG-LRU), vocab " << vocab_size;
+    os << architecture << ": hidden " << hidden_size << ", layers " << num_layers << " (";
+    const char* between = "";
+    const int first = kinds[3] + kinds[4] ? 3 : 0, last = kinds[3] + kinds[4] ? 5 : 3;  // the kinds one design combines
+    for (int k = first; k < last; ++k) {
+      os << between << kinds[k] << " " << kNames[k];
+      between = " / ";
+    }
+    os << ")";
+    if (loop_times > 1) os << ", layers " << loop_start << ".." << loop_stop - 1 << " run " << loop_times << " times";
+    os << ", vocab " << vocab_size;
     return os.str();
   }
   os << "hidden " << hidden_size << ", layers " << num_layers << " (" << num_attention_layers() << " attention / "

@@ -126,7 +126,7 @@ def main(argv=None) -> int:
     model = eng.Model(a.model)
     options = eng.default_runner_options(
         max_batch=a.slots, prefill_chunk=1024, kv_tokens=a.max_tokens + 64 * a.slots, kv_dtype=-1, verbose=0,
-        max_context=max(64, model.max_positions), compute_dtype=eng.COMPUTE_F32 if a.dtype == "float32" else eng.COMPUTE_BF16)
+        max_context=max(64, min(model.max_positions, a.max_tokens)), compute_dtype=eng.COMPUTE_F32 if a.dtype == "float32" else eng.COMPUTE_BF16)
     try:
         runner = eng.Runner(model, options)
     except eng.EngineError as e:
