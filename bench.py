@@ -355,8 +355,9 @@ def main():
     ap.add_argument("--trace-slice", type=int, default=64,
                     help="requests of the trace that the default run serves after the decode measurement (0 = none)")
     ap.add_argument("--designs", default="", metavar="SIZES",
-                    help="instead: Fegenex beside the Qwen3.8 hybrid of equal size (sizes: small, medium; comma-separated), "
-                         "prefill and decode throughput and per-op rooflines as one JSON line")
+                    help="instead: the layer-list designs beside the Qwen3.8 hybrid of equal size (sizes: small, medium; "
+                         "comma-separated), prefill and decode throughput and per-op rooflines as one JSON line")
+    ap.add_argument("--design-models", default="fegenex,nololix,qwen38", metavar="NAMES", help="models of --designs")
     ap.add_argument("--no-tp8", action="store_true",
                     help="with 8 GPUs: leave out the tensor-parallel measurement of one 262,144-token request (tp8_262k)")
     ap.add_argument("--skip-prefill", action="store_true",
@@ -416,7 +417,8 @@ def main():
         from q38b200 import design_bench, engine, synth
         peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else \
             {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
-        res = design_bench.run(engine, synth, [x for x in args.designs.split(",") if x], peaks, weight_bytes_by_role, log)
+        res = design_bench.run(engine, synth, [x for x in args.designs.split(",") if x], peaks, weight_bytes_by_role, log,
+                               models=[x for x in args.design_models.split(",") if x])
         print(json.dumps({"metric": "designs", "data": "synthetic", "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops")},
                           "context": design_bench.CONTEXT, "sizes": res}))
         return

@@ -534,6 +534,28 @@ size_t q38_latent_attention_partial_floats(int k_dim);
 int q38_latent_attention(const q38_latent_attention_params* p, const q38_batch_desc* batch, const q38_kv_layer_desc* kv,
                          void* stream);
 
+/* Attention over packed keys and values (bf16, prefill steps): the contexts (positions 0 ... pos0 + count - 1) of the batch's
+ * sequences one after the other, each rounded up to whole pages of 64 rows; `rows` is their sum.
+ * Gather: the cached latents [rows][k_dim], zero behind a context's end. */
+int q38_latent_gather(const q38_batch_desc* batch, const q38_kv_layer_desc* kv, int max_context, int rows, void* out,
+                      void* stream);
+/* Causal softmax attention, head h of a query, key or value at column h * its stride, zero-padded to a multiple of 16; the
+ * output is multiplied by sigmoid(gate) unless gate is NULL. */
+typedef struct q38_packed_attention_params {
+  const void* q; /* [M][ld_q] */
+  int ld_q, q_stride;
+  const void *k, *v; /* [rows][ld_kv] */
+  int ld_kv, k_stride, v_stride;
+  int heads, dim, vdim;
+  float scale;
+  const void* gate; /* [M][ld_gate]: heads x vdim, or NULL */
+  int ld_gate;
+  void* out; /* [M][ld_out]: heads x vdim */
+  int ld_out;
+} q38_packed_attention_params;
+int q38_packed_attention_fits(int dim, int vdim);
+int q38_packed_attention(const q38_packed_attention_params* p, const q38_batch_desc* batch, void* stream);
+
 /* Diagnostics. */
 const char* q38_last_error(void);           /* message of the last failed launcher call on this thread */
 /* Programmatic dependent launch (on by default): every launcher allows its kernel to be scheduled while the

@@ -177,6 +177,13 @@ class RgLruParams(C.Structure):
                 ("scratch", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int)]
 
 
+class PackedAttentionParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("ld_q", C.c_int), ("q_stride", C.c_int), ("k", C.c_void_p), ("v", C.c_void_p),
+                ("ld_kv", C.c_int), ("k_stride", C.c_int), ("v_stride", C.c_int), ("heads", C.c_int), ("dim", C.c_int),
+                ("vdim", C.c_int), ("scale", C.c_float), ("gate", C.c_void_p), ("ld_gate", C.c_int), ("out", C.c_void_p),
+                ("ld_out", C.c_int)]
+
+
 class SamplingParamsDev(C.Structure):
     _fields_ = [("temperature", C.c_float), ("top_k", C.c_int), ("top_p", C.c_float), ("min_p", C.c_float),
                 ("presence_penalty", C.c_float), ("repetition_penalty", C.c_float), ("seed", C.c_uint64)]
@@ -254,6 +261,9 @@ KERNEL_API = {
     "q38_latent_attention_partial_floats": (C.c_size_t, [C.c_int]),
     "q38_latent_attention": (C.c_int, [C.POINTER(LatentAttentionParams), C.POINTER(BatchDesc), C.POINTER(KvLayerDesc),
                                        C.c_void_p]),
+    "q38_latent_gather": (C.c_int, [C.POINTER(BatchDesc), C.POINTER(KvLayerDesc), C.c_int, C.c_int, C.c_void_p, C.c_void_p]),
+    "q38_packed_attention_fits": (C.c_int, [C.c_int, C.c_int]),
+    "q38_packed_attention": (C.c_int, [C.POINTER(PackedAttentionParams), C.POINTER(BatchDesc), C.c_void_p]),
     "q38_embed_norm": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p,
                                  C.POINTER(Norm), C.c_void_p, C.c_int, C.c_int, C.c_void_p]),
     "q38_residual_norm": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.POINTER(Norm), C.c_void_p, C.POINTER(Norm),

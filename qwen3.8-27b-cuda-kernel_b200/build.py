@@ -39,7 +39,7 @@ HOST_FLAGS = ["-std=c++20", "-O2", "-fPIC", "-I", str(ROOT / "include"), "-I", s
 FAMILIES = {
     "bq": {"cu": {"attention", "gdn", "qgemm", "qgemm_stream", "qgemm_umma"}, "host": {"bq_model"}},
     "layer_list": {"cu": {"dense_gemm", "dense_umma", "mixed_attention", "mixed_attention_mma", "recurrent", "row_norm",
-                          "stream_norm", "retention", "latent_attention"},
+                          "stream_norm", "retention", "latent_attention", "packed_attention"},
                    "host": {"layer_list_model", "fegenex", "nololix"}},
 }
 ARCHITECTURE_FAMILY = {"Qwen3.8": "bq", "Fegenex": "layer_list", "Nololix": "layer_list"}

@@ -63,12 +63,14 @@ __device__ __forceinline__ Item item_at(const Args& a, int i) {
   const int g = a.x_stride || a.out_stride ? i / a.group_tiles : 0, r = i - g * a.group_tiles;
   return {g, r / a.tiles_m, r % a.tiles_m};
 }
-// Epilogues of one accumulator value: output column n of its group, token t.
-__device__ __forceinline__ float unary(const Args& a, float v, int t, int col) {
-  if (a.kind == Q38_DENSE_XIELU) return xielu_f(v, a.alpha_p, a.alpha_n);
-  if (a.kind == Q38_DENSE_GATE_SIGMOID)
-    return v * sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)t * a.ld_gate + col]));
-  return v;
+// xIELU on the fast exponential: the result is stored in bf16, and what 1 - e^z loses near zero is far below z / 2.
+__device__ __forceinline__ float xielu_fast(const Args& a, float z) {
+  const float n = fminf(z, 0.0f);
+  return (z > 0.0f ? a.alpha_p * z * z : a.alpha_n * (__expf(n) - 1.0f - n)) + 0.5f * z;
+}
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float gate_at(const Args& a, int t, int col) {
+  return __bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)t * a.ld_gate + col]);
 }
 
 __device__ __forceinline__ float glu(int kind, float gate, float up) {
@@ -214,21 +216,32 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       } else {
         const float bias = a.bias && n < a.n ? a.bias[n] : 0.0f;
         const bool odd = lane & 1, glu_kind = a.kind == Q38_DENSE_GLU_GELU || a.kind == Q38_DENSE_GLU_SILU;
+        const bool gated = a.kind == Q38_DENSE_GATE_SIGMOID;
+        const int gate_col = oc + min(n, a.n - 1);
+        float gate[16];  // of the chunk that comes next
+        auto request_gate = [&](int c) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) gate[j] = gate_at(a, t0 + min(c + j, tokens - 1), gate_col);
+        };
+        if (gated) request_gate(0);
         for (int c = 0; c < TOK; c += 16) {
           if (c >= tokens) break;
           uint32_t r[16];
           tmem_ld16(taddr + uint32_t(c), r);
+          if (a.kind == Q38_DENSE_XIELU) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(xielu_fast(a, __uint_as_float(r[j]) + bias));
+          } else if (gated) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) r[j] = __float_as_uint((__uint_as_float(r[j]) + bias) * sigmoid_fast(gate[j]));
+            if (c + 16 < tokens) request_gate(c + 16);
+          }
           if (a.kind == Q38_DENSE_STORE_F32) {
             float* out = static_cast<float*>(a.out) + (size_t)(t0 + c) * a.ldo + oc + n;
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (c + j < tokens && n < a.n) out[(size_t)j * a.ldo] = __uint_as_float(r[j]) + bias;
           } else {
-            if (a.kind >= Q38_DENSE_XIELU) {
-#pragma unroll
-              for (int j = 0; j < 16; ++j)
-                if (c + j < tokens && n < a.n) r[j] = __float_as_uint(unary(a, __uint_as_float(r[j]) + bias, t0 + c + j, oc + n));
-            }
             const float add = a.kind >= Q38_DENSE_XIELU ? 0.0f : bias;
             // neighbouring lanes exchange: the even lane takes token j, the odd lane token j + 1, both columns n & ~1, n | 1
             uint32_t packed[8];
@@ -280,7 +293,10 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       const uint32_t part = smem_u32(ring);
       constexpr int kU = 8;  // token rows in flight
       for (int tb = rank; tb < tokens; tb += kU * a.cluster) {
-        float v[kU] = {};
+        float v[kU] = {}, gate[kU];
+        if (a.kind == Q38_DENSE_GATE_SIGMOID)
+#pragma unroll
+          for (int u = 0; u < kU; ++u) gate[u] = gate_at(a, t0 + min(tb + u * a.cluster, tokens - 1), oc + min(n, a.n - 1));
         for (int c = 0; c < a.cluster; ++c)
 #pragma unroll
           for (int u = 0; u < kU; ++u) {
@@ -291,12 +307,14 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
         for (int u = 0; u < kU; ++u) {
           const int t = tb + u * a.cluster;
           if (t >= tokens) break;
-          const float x = v[u] + bias;
+          float x = v[u] + bias;
+          if (a.kind == Q38_DENSE_XIELU) x = xielu_fast(a, x);
+          else if (a.kind == Q38_DENSE_GATE_SIGMOID) x *= sigmoid_fast(gate[u]);
           const size_t row = (size_t)(t0 + t) * a.ldo + oc;
           if (a.kind == Q38_DENSE_STORE_F32) {
             if (n < a.n) static_cast<float*>(a.out)[row + n] = x;
           } else if (a.kind == Q38_DENSE_STORE || a.kind >= Q38_DENSE_XIELU) {
-            if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(unary(a, x, t0 + t, oc + n));
+            if (n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + n] = __float2bfloat16_rn(x);
           } else {
             const float up = __shfl_xor_sync(0xffffffffu, x, 1);
             if (!(lane & 1) && n < a.n) static_cast<__nv_bfloat16*>(a.out)[row + (n >> 1)] = __float2bfloat16_rn(glu(a.kind, x, up));

@@ -1,9 +1,10 @@
-"""Throughput of the Fegenex design beside the framework's closest existing model (the Qwen3.8 hybrid) at equal size.
+"""Throughput of the layer-list designs (Fegenex, Nololix) beside each other and the Qwen3.8 hybrid at equal size.
 
-    python bench.py --designs small,medium
+    python bench.py --designs small,medium [--design-models nololix,qwen38]
 
-Both models get the same width, feed-forward, vocabulary, number of layers (two attention layers in six) and attention
-width; weights are random, the Qwen3.8 planes in the default recipe. Measured per size: the CUDA-graph decode step at
+All models get the same width, feed-forward, vocabulary, number of layers (two attention layers in six) and attention
+width; weights are random, the Qwen3.8 planes in the default recipe. The closest model of Nololix is the Qwen3.8 hybrid: its
+Gated DeltaNet keeps the same matrix state per head as the retention layers here. Measured per size: the CUDA-graph decode step at
 several batch sizes (device work of the step, replayed), prefill steps of 512 and 2048 tokens, and the per-op device times
 of both (eager, CUDA events between the ops) with the fraction of the measured roofline each op reaches: bytes for decode,
 FLOPs for the products and the attention of prefill.
@@ -39,7 +40,44 @@ def fegenex_config(s: dict) -> dict:
             "layers": [{"type": t, "mixer": kinds[t], "mlp": mlp} for t in order]}
 
 
-def tensor_shapes(cfg: dict) -> dict[str, tuple]:
+def nololix_config(s: dict) -> dict:
+    W, mlp = s["width"], {"kind": "dense", "ff": s["ff"]}
+    H = W // 128
+    kinds = {
+        "retention": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(5 + 5 * h / H) for h in range(H)],
+                      "rot": {"base": 10000.0, "dims": 128}},
+        "latent_attention": {"heads": s["heads"], "dim": s["dim"], "vdim": s["vdim"], "q_rank": 3 * W // 8, "kv_rank": 512,
+                             "scale": s["dim"] ** -0.5},
+    }
+    order = ["retention", "retention", "latent_attention"] * (LAYERS // 3)
+    return {"architecture": "Nololix", "width": W, "vocab": VOCAB, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6, "groups": 8},
+            "streams": 2, "residual_mult": 0.5, "loop": None,
+            "layers": [{"type": t, "mixer": kinds[t], "mlp": mlp} for t in order]}
+
+
+def nololix_shapes(cfg: dict) -> dict[str, tuple]:
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+    t = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        x, H = p + "mix.", m["heads"]
+        for q in "12":
+            t[f"{p}norm{q}"] = (W,)
+            t[f"{p}hc{q}.in"], t[f"{p}hc{q}.out"], t[f"{p}hc{q}.mix"] = (S,), (S,), (S, S)
+        if layer["type"] == "retention":
+            for n, d in (("q", m["dim"]), ("k", m["dim"]), ("v", m["vdim"]), ("g", m["vdim"])):
+                t[x + n] = (H * d, W)
+        else:
+            for n, rank in (("dq", m["q_rank"]), ("dkv", m["kv_rank"])):
+                t[x + n], t[x + n + ".norm"] = (rank, W), (rank,)
+            t[x + "uq"], t[x + "uk"] = (H * m["dim"], m["q_rank"]), (H * m["dim"], m["kv_rank"])
+            t[x + "uv"], t[x + "g"] = (H * m["vdim"], m["kv_rank"]), (H * m["vdim"], W)
+        t[x + "o"] = (W, H * m["vdim"])
+        t[p + "mlp.up"], t[p + "mlp.down"], t[p + "mlp.act"] = (layer["mlp"]["ff"], W), (W, layer["mlp"]["ff"]), (2,)
+    return t
+
+
+def fegenex_shapes(cfg: dict) -> dict[str, tuple]:
     W, V = cfg["width"], cfg["vocab"]
     t = {"embed": (V, W), "pos": (cfg["max_positions"], W), "final.norm": (), "head": (V, W)}
     for i, layer in enumerate(cfg["layers"]):
@@ -68,12 +106,11 @@ def tensor_shapes(cfg: dict) -> dict[str, tuple]:
     return t
 
 
-def write_random_folder(folder: Path, cfg: dict, seed: int = 5) -> Path:
+def write_random_folder(folder: Path, cfg: dict, shapes: dict, seed: int = 5) -> Path:
     """Gaussian weights scaled by fan-in, cut from one random block (timing does not depend on their values)."""
     folder.mkdir(parents=True, exist_ok=True)
     (folder / "config.json").write_text(json.dumps(cfg))
     block = np.random.default_rng(seed).standard_normal(1 << 22, dtype=np.float32)
-    shapes = tensor_shapes(cfg)
     head, at = {}, 0
     for name, shape in shapes.items():
         n = int(np.prod(shape)) * 2
@@ -91,16 +128,52 @@ def write_random_folder(folder: Path, cfg: dict, seed: int = 5) -> Path:
     return folder
 
 
-def fegenex_costs(cfg: dict):
+def _costs():
     """op -> (decode bytes(batch, context), prefill FLOPs(tokens, first position)); None where bytes bound prefill too."""
-    W, V = cfg["width"], cfg["vocab"]
     cost: dict[str, list] = {}
 
     def add(op, by, fl=None):
         cost.setdefault(op, []).append((by, fl))
 
-    def gemm(op, n, k):
-        add(op, lambda b, c, n=n, k=k: 2 * n * k + b * (n + k) * 2, lambda m, p, n=n, k=k: 2.0 * m * n * k)
+    def gemm(op, n, k, count=1):
+        add(op, lambda b, c: count * (2 * n * k + b * (n + k) * 2), lambda m, p: 2.0 * m * n * k * count)
+    return cost, add, gemm
+
+
+def nololix_costs(cfg: dict):
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+    cost, add, gemm = _costs()
+    gemm("gemm.lm_head", V, W)
+    for layer in cfg["layers"]:
+        m, ff = layer["mixer"], layer["mlp"]["ff"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "retention":
+            gemm("gemm.retention_in", 2 * H * (d + dv), W)
+            gemm("gemm.retention_out", W, H * dv)
+            row = 2 * H * (2 * d + 3 * dv)
+            add("mix.retention", lambda b, c, H=H, d=d, dv=dv, row=row: b * (8 * H * d * dv + row), ("bytes", lambda n, p, row=row: n * row))
+        else:
+            qr, r = m["q_rank"], m["kv_rank"]
+            gemm("gemm.latent_in", qr + r + H * dv, W)
+            gemm("gemm.latent_uq", H * d, qr)
+            gemm("gemm.latent_uk", r, d, H)
+            add("gemm.latent_kv", lambda b, c: 0, lambda n, p, r=r, H=H, d=d, dv=dv: 2.0 * (n + p) * r * H * (d + dv))
+            gemm("gemm.latent_uv", dv, r, H)
+            gemm("gemm.latent_o", W, H * dv)
+            # prefill: the FLOPs of the heads' own dimensions, however the kernel arranges the products
+            add("mix.latent", lambda b, c, r=r, H=H: b * (c * r * 2 + 4 * H * r),
+                lambda n, p, H=H, d=d, dv=dv: 2.0 * H * (d + dv) * n * (p + (n + 1) / 2))
+            add("mix.latent_append", lambda b, c, qr=qr, r=r: b * 4 * (qr + r))
+        gemm("gemm.mlp_up", ff, W)
+        gemm("gemm.mlp_down", W, ff)
+        for _ in range(2):
+            add("residual_norm", lambda b, c: b * W * (4 + 8 * S + 2), ("bytes", lambda n, p: n * W * (4 + 8 * S + 2)))
+    return cost
+
+
+def fegenex_costs(cfg: dict):
+    W, V = cfg["width"], cfg["vocab"]
+    cost, add, gemm = _costs()
     gemm("gemm.lm_head", V, W)
     for layer in cfg["layers"]:
         m, t = layer["mixer"], layer["type"]
@@ -218,23 +291,30 @@ def measure(eng, path: Path, cost: dict, peaks: dict, seed: int = 3) -> dict:
     return out
 
 
-def run(eng, synth, sizes: list[str], peaks: dict, by_role, log, recipe: str = "default") -> dict:
+DESIGNS = {"fegenex": (fegenex_config, fegenex_shapes, fegenex_costs), "nololix": (nololix_config, nololix_shapes, nololix_costs)}
+
+
+def run(eng, synth, sizes: list[str], peaks: dict, by_role, log, recipe: str = "default", models=("fegenex", "nololix", "qwen38")) -> dict:
     result = {}
     for name in sizes:
         s = SIZES[name]
         tmp = Path(tempfile.mkdtemp(prefix="design_bench_"))
+        result[name] = {}
         try:
-            cfg = fegenex_config(s)
-            log(f"design bench {name}: Fegenex")
-            result[name] = {"fegenex": measure(eng, write_random_folder(tmp / "fegenex", cfg), fegenex_costs(cfg), peaks)}
-            W = s["width"]
-            types = ["linear_attention", "linear_attention", "full_attention"] * (LAYERS // 3)
-            qcfg = synth.model_config(hidden=W, vocab=VOCAB, layers=LAYERS, intermediate=s["ff"], nq=s["heads"] * s["dim"] // 256,
-                                      nkv=s["kv_heads"] * s["dim"] // 256, lk=W // 256, lv=W // 128, layer_types=types)
-            log(f"design bench {name}: Qwen3.8 hybrid of the same size")
-            path = tmp / "qwen.q38"
-            synth.write_random_planes_q38(path, qcfg, recipe=recipe)
-            result[name]["qwen38"] = measure(eng, path, qwen_costs(qcfg, recipe, by_role), peaks)
+            for model in models:
+                log(f"design bench {name}: {model}")
+                if model in DESIGNS:
+                    config, shapes, costs = DESIGNS[model]
+                    cfg = config(s)
+                    result[name][model] = measure(eng, write_random_folder(tmp / model, cfg, shapes(cfg)), costs(cfg), peaks)
+                    continue
+                W = s["width"]
+                types = ["linear_attention", "linear_attention", "full_attention"] * (LAYERS // 3)
+                qcfg = synth.model_config(hidden=W, vocab=VOCAB, layers=LAYERS, intermediate=s["ff"], nq=s["heads"] * s["dim"] // 256,
+                                          nkv=s["kv_heads"] * s["dim"] // 256, lk=W // 256, lv=W // 128, layer_types=types)
+                path = tmp / "qwen.q38"
+                synth.write_random_planes_q38(path, qcfg, recipe=recipe)
+                result[name][model] = measure(eng, path, qwen_costs(qcfg, recipe, by_role), peaks)
         finally:
             shutil.rmtree(tmp, ignore_errors=True)
     return result

@@ -348,6 +348,15 @@ inline void latent_attention(const LatentAttentionParams& p, const BatchDesc& ba
   const q38_batch_desc b = batch.c();
   detail::ok(q38_latent_attention(&p, &b, &kv, stream));
 }
+using PackedAttentionParams = q38_packed_attention_params;
+inline void latent_gather(const BatchDesc& batch, const KvLayerDesc& kv, int max_context, int rows, void* out, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_latent_gather(&b, &kv, max_context, rows, out, stream));
+}
+inline void packed_attention(const PackedAttentionParams& p, const BatchDesc& batch, cudaStream_t stream) {
+  const q38_batch_desc b = batch.c();
+  detail::ok(q38_packed_attention(&p, &b, stream));
+}
 inline void rope_append(const RopeAppendParams& p, const BatchDesc& batch, const KvLayerDesc& kv, cudaStream_t stream) {
   const q38_batch_desc b = batch.c();
   detail::ok(q38_rope_append(&p, &b, &kv, stream));

@@ -53,7 +53,8 @@ struct Linear {
   std::vector<std::string> weights;             // stacked along the output
   std::vector<std::string> biases;              // one per weight, "" = none
   bool interleave = false;                      // two weights whose rows alternate
-  int block = 0, block_to = 0;                  // blocks of `block` rows are spread to `block_to` rows (zero rows between)
+  // rows in heads (one size per weight): every head is padded with zero rows to a multiple of 16
+  std::vector<int> heads_of = {};
 };
 
 struct LayerTensors {
@@ -107,6 +108,7 @@ struct LayerWeightsDev {
   const float* decay_pow = nullptr;
   const float *q_gain = nullptr, *kv_gain = nullptr;
   kernels::DenseWeight uq{}, uk{}, uv{};  // latent attention; uk and uv hold one matrix per head
+  kernels::DenseWeight ukv{};             // ... and all heads' keys, then values, from a latent (heads padded to 16)
   const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
   const float *v_mix = nullptr, *head_mix = nullptr;
   const double* inv_freq = nullptr;
@@ -181,6 +183,8 @@ class LayerListModel final : public StepModel {
   void join_residual(const StepContext& ctx, int m, const Sublayer& done, const Sublayer& next);
   void feed_forward(const StepContext& ctx, int m, const LayerWeightsDev& W);
   void attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i, bool first_values, bool blend);
+  bool packs(const LatentAttentionSpec& a) const { return !f32_ && q38_packed_attention_fits(a.dim, a.vdim) != 0; }
+  bool packing_pays(const LatentAttentionSpec& a, const StepBatch& b) const;
   void latent_attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i);
   void recurrent(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int rec_i);
   void retention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W,
@@ -228,6 +232,10 @@ class LayerListModel final : public StepModel {
   uint8_t* q_absorbed_ = nullptr;  // ... and in the space of the cached latents
   uint8_t* o_latent_ = nullptr;
   float* latent_partials_ = nullptr;
+  uint8_t* packed_latents_ = nullptr;  // latents of a prefill step's contexts ...
+  uint8_t* packed_kv_ = nullptr;       // ... and the heads' keys and values made from them
+  int64_t packed_rows_ = 0;            // room for
+  int ld_packed_ = 0, max_context_ = 0;
   size_t latent_partial_floats_ = 0;
   int ld_q_latent_ = 0, ld_q_heads_ = 0, max_absorbed_ = 0, max_latent_k_ = 0, max_rec_o_ = 0;
   size_t qk_bytes_per_token_ = 0;
@@ -237,6 +245,7 @@ class LayerListModel final : public StepModel {
 
 LayerListModel::LayerListModel(const ModelFile& f, const RunnerOptions& o, const LayerListDesign& d)
     : reader_(f), cfg_(f.config()), design_(d), f32_(o.compute == ComputeDtype::F32) {
+  max_context_ = o.max_context;
   act_ = f32_ ? Q38_ACT_F32 : Q38_ACT_BF16;
   elem_ = f32_ ? 4 : 2;
   ld_x_ = up(cfg_.hidden_size, 64);
@@ -269,7 +278,8 @@ LayerListModel::LayerListModel(const ModelFile& f, const RunnerOptions& o, const
       ld_proj_ = std::max(ld_proj_, up(a.q_rank + a.kv_rank + a.heads * a.vdim, 64));
       ld_mixer_ = std::max(ld_mixer_, up(a.heads * a.vdim, 64));
       ld_q_latent_ = std::max(ld_q_latent_, up(a.q_rank, 64));
-      ld_q_heads_ = std::max(ld_q_heads_, up(a.heads * up(a.dim, 8), 64));
+      ld_q_heads_ = std::max(ld_q_heads_, up(a.heads * up(a.dim, 16), 64));
+      if (packs(a)) ld_packed_ = std::max(ld_packed_, up(a.heads * (up(a.dim, 16) + up(a.vdim, 16)), 64));
       max_absorbed_ = std::max(max_absorbed_, a.heads * g.k_dim);
       max_latent_k_ = std::max(max_latent_k_, g.k_dim);
     } else if (l.mixer == MixerKind::Retention) {
@@ -334,7 +344,7 @@ kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear
   for (size_t i = 0; i < l.weights.size(); ++i) {
     const TensorInfo& t = reader_.file().tensor(l.weights[i]);
     QWEN38_CHECK(t.shape.size() == 2 && (i == 0 || int(t.shape[1]) == d.k), l.weights[i], ": shape");
-    d.n += l.block ? int(t.shape[0]) / l.block * l.block_to : int(t.shape[0]);
+    d.n += l.heads_of.empty() ? int(t.shape[0]) : int(t.shape[0]) / l.heads_of[i] * up(l.heads_of[i], 16);
     d.k = int(t.shape[1]);
     bias = bias || !l.biases[i].empty();
   }
@@ -346,11 +356,12 @@ kernels::DenseWeight LayerListModel::put_linear(DeviceArena* arena, const Linear
     for (size_t i = 0; i < l.weights.size(); ++i) {
       const TensorInfo& t = reader_.file().tensor(l.weights[i]);
       for (int64_t r = 0; r < t.shape[0]; ++r) {
-        const int64_t to = l.interleave ? 2 * r + int64_t(i) : l.block ? r / l.block * l.block_to + r % l.block : row0 + r;
+        const int64_t in_head = l.heads_of.empty() ? r : r / l.heads_of[i] * up(l.heads_of[i], 16) + r % l.heads_of[i];
+        const int64_t to = l.interleave ? 2 * r + int64_t(i) : row0 + in_head;
         reader_.copy_bf16(t, r * t.shape[1], t.shape[1], w.data() + to * d.ld);
         if (!l.biases[i].empty()) b[size_t(to)] = reader_.at(reader_.file().tensor(l.biases[i]), r);
       }
-      row0 += int(t.shape[0]);
+      row0 += l.heads_of.empty() ? int(t.shape[0]) : int(t.shape[0]) / l.heads_of[i] * up(l.heads_of[i], 16);
     }
   }
   d.w = put(arena, w);
@@ -429,9 +440,10 @@ void LayerListModel::visit_weights(DeviceArena* arena) {
       const LatentAttentionSpec& a = l.latent;
       W.q_gain = put_f32(arena, mix(i, "dq.norm"));
       W.kv_gain = put_f32(arena, mix(i, "dkv.norm"));
-      W.uq = put_linear(arena, {{mix(i, "uq")}, {""}, false, a.dim, up(a.dim, 8)});
+      W.uq = put_linear(arena, {{mix(i, "uq")}, {""}, false, {a.dim}});
       W.uk = put_heads(arena, mix(i, "uk"), a.heads, up(a.kv_rank, 32), true);
       W.uv = put_heads(arena, mix(i, "uv"), a.heads, a.vdim, false);
+      if (packs(a)) W.ukv = put_linear(arena, {{mix(i, "uk"), mix(i, "uv")}, {"", ""}, false, {a.dim, a.vdim}});
     }
     if (l.mixer == MixerKind::Attention) {
       if (l.attn.value_mix) W.v_mix = put_f32(arena, mix(i, "vmix"));
@@ -498,6 +510,14 @@ void LayerListModel::carve(Workspace& w, const StepContext& ctx) {
   o_latent_ = w.take<uint8_t>(T * size_t(max_absorbed_) * elem_);
   latent_partial_floats_ = f32_ || !max_latent_k_ ? 0 : q38_latent_attention_partial_floats(max_latent_k_);
   latent_partials_ = w.take<float>(latent_partial_floats_);
+  if (ld_packed_) {
+    // several chunks' worth of context, at most 1 GiB, no more than all slots can hold; longer contexts stay in latent form
+    const int64_t bytes = (int64_t(ld_packed_) + max_latent_k_) * 2;
+    packed_rows_ = std::min<int64_t>(std::max<int64_t>(8 * int64_t(T), 16384), (int64_t(1) << 30) / bytes);
+    packed_rows_ = std::min<int64_t>(packed_rows_, int64_t(R) * up(max_context_, 64)) / 64 * 64;
+    packed_latents_ = w.take<uint8_t>(size_t(packed_rows_) * size_t(max_latent_k_) * 2);
+    packed_kv_ = w.take<uint8_t>(size_t(packed_rows_) * size_t(ld_packed_) * 2);
+  }
   head_x_ = w.take<uint8_t>(R * size_t(ld_x_) * elem_);
   gemm_ws_.partials = w.take<float>(gemm_partials);
   gemm_ws_.partial_floats = gemm_partials;
@@ -550,10 +570,20 @@ void LayerListModel::attention(const StepContext& ctx, const StepBatch& b, const
   ctx.mark(b.decode ? "mix.attn_decode" : "mix.attn_prefill");
 }
 
+// In the latent space a (query, key) pair costs 2 kv_rank multiplications per head (half of them twice, for the weights'
+// second term), with keys and values of their own dim + vdim; those have to be made from every latent of the contexts first,
+// by a product that runs at a few times the attention kernels' rate.
+bool LayerListModel::packing_pays(const LatentAttentionSpec& a, const StepBatch& b) const {
+  if (b.decode || !packs(a) || b.chunk_packed_rows > packed_rows_ || b.chunk_part.num_seqs == 0) return false;
+  const double per_seq = double(b.chunk_part.num_tokens) / b.chunk_part.num_seqs, own = a.dim + a.vdim;
+  return per_seq * 1.5 * (2.0 * a.kv_rank - own) > 0.5 * a.kv_rank * own;
+}
+
 void LayerListModel::latent_attention(const StepContext& ctx, const StepBatch& b, const LayerSpec& l, const LayerWeightsDev& W, int attn_i) {
   const LatentAttentionSpec& a = l.latent;
   const kernels::KvLayerDesc kv = ctx.kv->layer_desc(attn_i);
-  const int dim_ld = up(a.dim, 8);
+  const int k_ld = up(a.dim, 16), v_ld = up(a.vdim, 16);
+  const uint8_t* gate = proj_ + size_t(a.q_rank + a.kv_rank) * elem_;
   kernels::LatentAppendParams lp{};
   lp.proj = proj_;
   lp.ld_proj = ld_proj_;
@@ -569,11 +599,42 @@ void LayerListModel::latent_attention(const StepContext& ctx, const StepBatch& b
   ctx.mark("mix.latent_append");
   gemm(ctx, q_latent_, ld_q_latent_, b.m, W.uq, Q38_DENSE_STORE, q_heads_, ld_q_heads_);
   ctx.mark("gemm.latent_uq");
+  int first = 0;  // rows from here on are served in the latent space
+  if (packing_pays(a, b)) {
+    first = b.chunk_part.num_tokens;
+    const int rows = int(b.chunk_packed_rows);
+    kernels::latent_gather(b.chunk_part, kv, b.chunk_longest_context, rows, packed_latents_, ctx.stream);
+    gemm(ctx, packed_latents_, kv.k_dim, rows, W.ukv, Q38_DENSE_STORE, packed_kv_, ld_packed_);
+    ctx.mark("gemm.latent_kv");
+    kernels::PackedAttentionParams pp{};
+    pp.q = q_heads_;
+    pp.ld_q = ld_q_heads_;
+    pp.q_stride = k_ld;
+    pp.k = packed_kv_;
+    pp.v = packed_kv_ + size_t(a.heads) * size_t(k_ld) * 2;
+    pp.ld_kv = ld_packed_;
+    pp.k_stride = k_ld;
+    pp.v_stride = v_ld;
+    pp.heads = a.heads;
+    pp.dim = a.dim;
+    pp.vdim = a.vdim;
+    pp.scale = a.scale;
+    pp.gate = gate;
+    pp.ld_gate = ld_proj_;
+    pp.out = mixer_;
+    pp.ld_out = ld_mixer_;
+    kernels::packed_attention(pp, b.chunk_part, ctx.stream);
+    ctx.mark("mix.latent_prefill");
+  }
+  const int rows = b.m - first;
+  if (rows == 0) return;
+  const auto row = [&](uint8_t* base, int ld) { return base + size_t(first) * size_t(ld) * elem_; };
+  const int ld_k = a.heads * kv.k_dim;
   kernels::DenseEpilogue ep{};
   ep.kind = Q38_DENSE_STORE;
-  ep.out = q_absorbed_;
-  ep.ldo = a.heads * kv.k_dim;
-  kernels::dense_gemm_grouped(q_heads_, ld_q_heads_, act_, b.m, W.uk, {a.heads, dim_ld, kv.k_dim}, ep, gemm_ws_, ctx.stream);
+  ep.out = row(q_absorbed_, ld_k);
+  ep.ldo = ld_k;
+  kernels::dense_gemm_grouped(row(q_heads_, ld_q_heads_), ld_q_heads_, act_, rows, W.uk, {a.heads, k_ld, kv.k_dim}, ep, gemm_ws_, ctx.stream);
   ctx.mark("gemm.latent_uk");
   kernels::LatentAttentionParams ap{};
   ap.q = q_absorbed_;
@@ -584,14 +645,14 @@ void LayerListModel::latent_attention(const StepContext& ctx, const StepBatch& b
   ap.partials = latent_partials_;
   ap.partial_floats = latent_partial_floats_;
   if (b.decode || b.mixed) kernels::latent_attention(ap, b.single_part, kv, ctx.stream);
-  if (!b.decode) kernels::latent_attention(ap, b.chunk_part, kv, ctx.stream);
+  if (!b.decode && first == 0) kernels::latent_attention(ap, b.chunk_part, kv, ctx.stream);
   ctx.mark(b.decode ? "mix.latent_decode" : "mix.latent_prefill");
   ep.kind = Q38_DENSE_GATE_SIGMOID;
-  ep.out = mixer_;
+  ep.out = row(mixer_, ld_mixer_);
   ep.ldo = ld_mixer_;
-  ep.gate = proj_ + size_t(a.q_rank + a.kv_rank) * elem_;
+  ep.gate = gate + size_t(first) * size_t(ld_proj_) * elem_;
   ep.ld_gate = ld_proj_;
-  kernels::dense_gemm_grouped(o_latent_, a.heads * kv.k_dim, act_, b.m, W.uv, {a.heads, kv.k_dim, a.vdim}, ep, gemm_ws_, ctx.stream);
+  kernels::dense_gemm_grouped(row(o_latent_, ld_k), ld_k, act_, rows, W.uv, {a.heads, kv.k_dim, a.vdim}, ep, gemm_ws_, ctx.stream);
   ctx.mark("gemm.latent_uv");
 }
 

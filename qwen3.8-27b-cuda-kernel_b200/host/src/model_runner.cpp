@@ -332,6 +332,12 @@ void ModelRunner::Impl::forward(int m, const kernels::BatchDesc& batch, bool dec
   b.all = batch;
   b.chunk_part = b.mixed ? sub_batch(0, 0, multi_seqs, multi_tokens, batch.max_tokens_per_seq) : batch;
   b.single_part = b.mixed ? sub_batch(multi_seqs, multi_tokens, single_seqs, single_seqs, 1) : batch;
+  if (!decode)
+    for (int i = 0; i < b.chunk_part.num_seqs; ++i) {
+      const int context = hmeta<int>(meta.seq_pos0)[i] + hmeta<int>(meta.seq_count)[i];
+      b.chunk_longest_context = std::max(b.chunk_longest_context, context);
+      b.chunk_packed_rows += align_up(context, kernels::kPageTokens);
+    }
   ctx.profiling = profiling;
   mark("start");
   model->forward(ctx, b);

@@ -41,6 +41,9 @@ struct StepBatch {
   int m = 0;
   bool decode = false, mixed = false;
   kernels::BatchDesc all, chunk_part, single_part;
+  // prefill steps: the longest context of a sequence of chunk_part, and the sum of all of them in whole pages (tokens)
+  int chunk_longest_context = 0;
+  int64_t chunk_packed_rows = 0;
 };
 
 // Token rows of the last forward() whose logits are wanted: `count` rows from `first`, or, with `rows` (device), those.

@@ -346,6 +346,62 @@ def test_latent_attention_against_the_plain_one(heads, rank, act):
             assert err < (8e-3 if act == pkg.ACT_BF16 else 1e-5), (s, err)
 
 
+@pytest.mark.parametrize("heads,dim,vdim,rank", [(3, 20, 24, 44), (2, 128, 128, 96), (1, 72, 200, 64), (5, 16, 7, 32), (2, 192, 64, 160), (1, 256, 33, 24)])
+def test_packed_attention_against_the_plain_one(heads, dim, vdim, rank):
+    """Latents of two sequences gathered from shuffled pages, keys and values that stand out at tile borders and far back; a
+    run that starts in the middle of a page, one of two tokens, and an output gate."""
+    H = heads
+    rng = np.random.default_rng(heads + dim)
+    K, act = pkg.kernels(), pkg.ACT_BF16
+    cache = LatentCache(rank, 4, 4, act)
+    rows = [(2, 0, 200), (1, 63, 2), (3, 130, 90)]
+    contexts = [200, 65, 220]
+    packed = sum(up(c, 64) for c in contexts)
+    b = Batch(rows)
+    lat = torch.full((packed, cache.kd), float("nan"), dtype=torch.bfloat16, device="cuda")
+    pkg.check(K.q38_latent_gather(C.byref(b.desc), C.byref(cache.desc), max(contexts), packed, pkg.ptr(lat), None))
+    got, at = lat.double().cpu().numpy(), 0
+    pool, table = cache.pool.double().cpu().numpy().reshape(-1, 64, cache.kd), cache.table.cpu().numpy()
+    for (slot, _, _), c in zip(rows, contexts):
+        want = np.concatenate([pool[p] for p in table[slot][:up(c, 64) // 64]])
+        want[c:] = 0
+        assert np.array_equal(got[at:at + len(want)], want)
+        at += len(want)
+    ks, vs = up(dim, 16), up(vdim, 16)
+    q, k, v = [rounded(rng.standard_normal(s), act) for s in ((b.m, H, dim), (packed, H, dim), (packed, H, vdim))]
+    gate = rounded(rng.standard_normal((b.m, H * vdim)) * 2, act)
+    base, first = [0, 256, 384], [0, 200, 202]
+    for i, j in ((199, 0), (199, 63), (198, 64), (70, 3), (64, 63), (65, 66), (130, 127), (20, 20)):
+        q[i, (i + j) % H] = 2.0 * k[j, (i + j) % H]
+    q[201] = k[256]
+    q[202 + 89] = k[384 + 5]
+    q = rounded(q, act)
+    ld_kv, ld_q = H * (ks + vs) + 8, H * ks + 16
+    qd, kvd = torch.zeros((b.m, ld_q), dtype=torch.bfloat16, device="cuda"), torch.zeros((packed, ld_kv), dtype=torch.bfloat16, device="cuda")
+    for h in range(H):
+        qd[:, h * ks:h * ks + dim] = dev(q[:, h], torch.bfloat16)
+        kvd[:, h * ks:h * ks + dim] = dev(k[:, h], torch.bfloat16)
+        kvd[:, H * ks + h * vs:H * ks + h * vs + vdim] = dev(v[:, h], torch.bfloat16)
+    for gated, ld_out in ((True, H * vdim + 2), (False, H * vdim + 3)):
+        gd = torch.zeros((b.m, H * vdim + 4), dtype=torch.bfloat16, device="cuda")
+        gd[:, :H * vdim] = dev(gate, torch.bfloat16)
+        out = torch.zeros((b.m, ld_out), dtype=torch.bfloat16, device="cuda")
+        p = pkg.PackedAttentionParams(pkg.ptr(qd), ld_q, ks, pkg.ptr(kvd), kvd.data_ptr() + 2 * H * ks, ld_kv, ks, vs, H, dim, vdim, 0.4,
+                                      pkg.ptr(gd) if gated else None, H * vdim + 4, pkg.ptr(out), ld_out)
+        pkg.check(K.q38_packed_attention(C.byref(p), C.byref(b.desc), None))
+        torch.cuda.synchronize()
+        got = out.double().cpu().numpy()
+        assert np.all(got[:, H * vdim:] == 0)
+        for (slot, pos0, n), c, k0, m0 in zip(rows, contexts, base, first):
+            full = np.zeros((c, H, dim))
+            full[pos0:] = q[m0:m0 + n]
+            want = no.softmax_attention(full, k[k0:k0 + c], v[k0:k0 + c], 0.4)[pos0:].reshape(n, -1)
+            if gated:
+                want = want * no.sigmoid(gate[m0:m0 + n])
+            assert np.all(np.abs(got[m0:m0 + n, :H * vdim] - want) < 2e-3 + np.abs(want) / 200)
+    clean()
+
+
 @pytest.mark.parametrize("act", ACTS)
 @pytest.mark.parametrize("heads", [4, 24])
 def test_long_decoding_over_many_pages_with_and_without_divided_ranges(heads, act):
