@@ -3,8 +3,8 @@
 // Orientation as in the BQ kernel: the weights are the MMA's A operand (128 output columns fill the 128 TMEM lanes), the
 // tokens its N operand (TOK = 32 ... 256). Both operands arrive by TMA (2-D tensor maps, 128-byte swizzle; rows and
 // columns outside the matrices are zero-filled, so any n, k and m work) into a ring of stages of one 64-wide k-group each.
-// Warp roles (6 warps): 0 = TMA producer, 1 = MMA issuer (converged, one elected lane issues), 2-5 = epilogue, each on the
-// TMEM lane quarter its index selects.
+// Warp roles (10 warps): 0 = TMA producer, 1 = MMA issuer (converged, one elected lane issues), 2-9 = epilogue, each on the
+// TMEM lane quarter its index selects, two warps per quarter that take 16 tokens in turn.
 //   CLUSTER = false: persistent CTAs walk the (weight tile, token tile) list, tokens innermost, so that the CTAs that run
 //                    side by side share weight tiles in L2; two accumulators, the epilogue of one tile overlaps the next.
 //   CLUSTER = true:  few tiles (small batches): the CTAs of a cluster share one tile and split its k-groups; every CTA
@@ -23,7 +23,8 @@ Q38_REGISTER_ERROR_WORD();
 namespace {
 
 constexpr int kTileN = 128;
-constexpr int kThreads = 192;
+constexpr int kEpiWarps = 8;
+constexpr int kThreads = 64 + 32 * kEpiWarps;
 constexpr int kWBytes = kTileN * 128;  // [128 n][64 k] bf16
 
 template <int TOK, bool CLUSTER>
@@ -65,8 +66,8 @@ __device__ __forceinline__ Item item_at(const Args& a, int i) {
 }
 // xIELU on the fast exponential: the result is stored in bf16, and what 1 - e^z loses near zero is far below z / 2.
 __device__ __forceinline__ float xielu_fast(const Args& a, float z) {
-  const float n = fminf(z, 0.0f);
-  return (z > 0.0f ? a.alpha_p * z * z : a.alpha_n * (__expf(n) - 1.0f - n)) + 0.5f * z;
+  const float p = fmaxf(z, 0.0f), n = fminf(z, 0.0f);
+  return fmaf(a.alpha_p * p, p, a.alpha_n * (__expf(n) - 1.0f - n)) + 0.5f * z;
 }
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
 __device__ __forceinline__ float gate_at(const Args& a, int t, int col) {
@@ -109,7 +110,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
     }
     for (int i = 0; i < C::kAccs; ++i) {
       mbar_init(&acc_full[i], 1);
-      mbar_init(&acc_empty[i], 4);
+      mbar_init(&acc_empty[i], kEpiWarps);
     }
     *abort_flag = 0;
     mbar_fence_init();
@@ -193,7 +194,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
     }
   } else {
     pdl_wait();  // the output may still be read by the previous kernel
-    const int quarter = warp & 3, nl = quarter * 32 + lane;
+    const int quarter = warp & 3, nl = quarter * 32 + lane, c0 = (warp - 2) / 4 * 16;  // first token of this warp
     uint32_t seg = 0;
     bool alive = true;
     for (int item = first; item < a.items && alive; item += step, ++seg) {
@@ -207,7 +208,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       const uint32_t taddr = tmem + acc * C::kAccCols + (uint32_t(quarter * 32) << 16);
       if (CLUSTER) {
         float* part = reinterpret_cast<float*>(ring);  // [TOK][128]; every MMA of this CTA has read its stages
-        for (int c = 0; c < TOK && c < tokens; c += 16) {
+        for (int c = c0; c < TOK && c < tokens; c += 32) {
           uint32_t r[16];
           tmem_ld16(taddr + uint32_t(c), r);
 #pragma unroll
@@ -223,8 +224,8 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
 #pragma unroll
           for (int j = 0; j < 16; ++j) gate[j] = gate_at(a, t0 + min(c + j, tokens - 1), gate_col);
         };
-        if (gated) request_gate(0);
-        for (int c = 0; c < TOK; c += 16) {
+        if (gated) request_gate(c0);
+        for (int c = c0; c < TOK; c += 32) {
           if (c >= tokens) break;
           uint32_t r[16];
           tmem_ld16(taddr + uint32_t(c), r);
@@ -234,7 +235,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
           } else if (gated) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) r[j] = __float_as_uint((__uint_as_float(r[j]) + bias) * sigmoid_fast(gate[j]));
-            if (c + 16 < tokens) request_gate(c + 16);
+            if (c + 32 < tokens) request_gate(c + 32);
           }
           if (a.kind == Q38_DENSE_STORE_F32) {
             float* out = static_cast<float*>(a.out) + (size_t)(t0 + c) * a.ldo + oc + n;
@@ -292,7 +293,7 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
       const float bias = a.bias && n < a.n ? a.bias[n] : 0.0f;
       const uint32_t part = smem_u32(ring);
       constexpr int kU = 8;  // token rows in flight
-      for (int tb = rank; tb < tokens; tb += kU * a.cluster) {
+      for (int tb = rank + (warp - 2) / 4 * kU * a.cluster; tb < tokens; tb += 2 * kU * a.cluster) {
         float v[kU] = {}, gate[kU];
         if (a.kind == Q38_DENSE_GATE_SIGMOID)
 #pragma unroll

@@ -113,8 +113,8 @@ __global__ void __launch_bounds__(kGenThreads) latent_general_kernel(q38_latent_
 }
 
 // ---- tensor cores ---------------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool real) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(real ? 16 : 0) : "memory");
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool real) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(real ? 16 : 0) : "memory");
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
@@ -179,6 +179,8 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
   if (sh.p0 >= sh.p1) return;
   const int* table = kv.block_table + (size_t)b.seq_slot[seq] * kv.max_pages_per_seq;
   const int pieces = k_dim / 8;
+  // 16-byte pieces of a page dealt to the threads in order: row and column of the first, steps to the next
+  const int r0 = tid / pieces, k0 = tid - r0 * pieces, dr = kMmaThreads / pieces, dk = kMmaThreads - dr * pieces;
 
   auto load_page = [&](int pg) {
     int page = table[pg];
@@ -188,16 +190,23 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     }
     const bf16* src = reinterpret_cast<const bf16*>(kv.pages + (size_t)page * kv.page_bytes);
     bf16* dst = reinterpret_cast<bf16*>(smem + L.c) + (size_t)(pg & 1) * kPage * rs;
+    int r = r0, k = k0;
+    uint32_t to = smem_u32(dst);
     for (int i = tid; i < kPage * pieces; i += kMmaThreads) {
-      const int r = i / pieces, k = i - r * pieces;
-      cp_async16(dst + r * rs + 8 * k, src + (size_t)i * 8, true);
+      cp_async16(to + uint32_t(r * rs + 8 * k) * 2, src + (size_t)i * 8, true);
+      r += dr;
+      k += dk;
+      if (k >= pieces) {
+        k -= pieces;
+        ++r;
+      }
     }
     cp_async_commit();
   };
   const bf16* q = static_cast<const bf16*>(p.q) + ((size_t)start * H + sh.first) * k_dim;
   for (int i = tid; i < ROWS * pieces; i += kMmaThreads) {
     const int r = i / pieces, k = i - r * pieces;
-    cp_async16(reinterpret_cast<bf16*>(smem + L.q) + r * rs + 8 * k, r < sh.rows ? q + (size_t)i * 8 : q, r < sh.rows);
+    cp_async16(smem_u32(smem + L.q) + uint32_t(r * rs + 8 * k) * 2, r < sh.rows ? q + (size_t)i * 8 : q, r < sh.rows);
   }
   load_page(sh.p0);
 
@@ -227,7 +236,7 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     if (KT == 1) {  // 8 keys: two k16 steps per load
       const uint32_t k_a = c_a + ((key0 + (lane & 7)) * rs + (lane >> 3) * 8) * 2;
       float s2[4] = {};
-#pragma unroll 2
+#pragma unroll 4
       for (int k = 0; k < k_dim; k += 32) {
         uint32_t kf[4], a0[4], a1[4];
         ldmatrix_x4(kf, k_a + k * 2);
@@ -240,18 +249,26 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
       for (int e = 0; e < 4; ++e) s[0][e] += s2[e];
     } else {
       const uint32_t k_a = c_a + ((key0 + (lane & 7) + ((lane >> 4) << 3)) * rs + ((lane >> 3) & 1) * 8) * 2;
+      float s2[KT][4] = {};  // every other step: shorter chains of dependent products
 #pragma unroll 2
-      for (int k = 0; k < k_dim; k += 16) {
-        uint32_t a[4];
-        ldmatrix_x4(a, q_a + k * 2);
+      for (int k = 0; k < k_dim; k += 32) {
 #pragma unroll
-        for (int kp = 0; kp < KT / 2; ++kp) {
-          uint32_t kf[4];
-          ldmatrix_x4(kf, k_a + (kp * 16 * rs + k) * 2);
-          mma_bf16_16816(s[2 * kp], a, kf[0], kf[1]);
-          mma_bf16_16816(s[2 * kp + 1], a, kf[2], kf[3]);
+        for (int e = 0; e < 2; ++e) {
+          uint32_t a[4];
+          ldmatrix_x4(a, q_a + (k + 16 * e) * 2);
+#pragma unroll
+          for (int kp = 0; kp < KT / 2; ++kp) {
+            uint32_t kf[4];
+            ldmatrix_x4(kf, k_a + (kp * 16 * rs + k + 16 * e) * 2);
+            mma_bf16_16816(e ? s2[2 * kp] : s[2 * kp], a, kf[0], kf[1]);
+            mma_bf16_16816(e ? s2[2 * kp + 1] : s[2 * kp + 1], a, kf[2], kf[3]);
+          }
         }
       }
+#pragma unroll
+      for (int kt = 0; kt < KT; ++kt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[kt][e] += s2[kt][e];
     }
     float ma = -INFINITY, mb = -INFINITY;
 #pragma unroll
@@ -301,12 +318,14 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
         *reinterpret_cast<__nv_bfloat162*>(smem + L.p_hi + at) = hi;
         *reinterpret_cast<__nv_bfloat162*>(smem + L.p_lo + at) = __floats2bfloat162_rn(w0 - f.x, w1 - f.y);
       }
+    if (__any_sync(0xffffffffu, fa != 1.0f || fb != 1.0f)) {
 #pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      o[i][0] *= fa;
-      o[i][1] *= fa;
-      o[i][2] *= fb;
-      o[i][3] *= fb;
+      for (int i = 0; i < NT; ++i) {
+        o[i][0] *= fa;
+        o[i][1] *= fa;
+        o[i][2] *= fb;
+        o[i][3] *= fb;
+      }
     }
     __syncthreads();
     // ---- outputs: all keys of the page, this warp's columns ----

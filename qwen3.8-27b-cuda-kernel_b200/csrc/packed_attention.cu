@@ -4,7 +4,8 @@
 // when its runs are long enough to pay for it.
 //
 // One CTA per (64 query tokens, head, sequence), the longest contexts first: four warps of 16 rows each, 64 keys at a time
-// through a two-stage cp.async ring, online softmax in registers (mma.sync, fp32 scores, weights and sums). The weights of a
+// through one buffer for keys and one for values, each refilled (cp.async) while the other is used, so that several CTAs
+// share an SM; online softmax in registers (mma.sync, fp32 scores, weights and sums). The weights of a
 // tile are the A operand of the value product as they stand, as bf16 hi + lo (16 mantissa bits). The output gate is applied
 // as the rows are stored.
 #include <algorithm>
@@ -80,7 +81,7 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
   extern __shared__ __align__(16) uint8_t smem[];
   const int dk = up16(p.dim), dv = up16(p.vdim), ks = dk + 8, vs = dv + 8;  // rows an odd multiple of 16 bytes apart
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const uint32_t q_s = smem_u32(smem), k_s = q_s + uint32_t(kTile * ks) * 2, v_s = k_s + uint32_t(2 * kTile * ks) * 2;
+  const uint32_t q_s = smem_u32(smem), k_s = q_s + uint32_t(kTile * ks) * 2, v_s = k_s + uint32_t(kTile * ks) * 2;
   pdl_wait();
   pdl_launch_dependents();
   const int h = blockIdx.y, seq = blockIdx.z, i0 = (int(gridDim.x) - 1 - int(blockIdx.x)) * kTile;
@@ -92,22 +93,27 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
   const bf16* V = static_cast<const bf16*>(p.v) + row0 * p.ld_kv + (size_t)h * p.v_stride;
   const bf16* Q = static_cast<const bf16*>(p.q) + (size_t)(start + i0) * p.ld_q + (size_t)h * p.q_stride;
 
-  // a thread copies the same 16-byte columns of every row group it visits: rows tid / pieces, ...
+  // 16-byte pieces of a [64][width] tile, dealt to the threads in order
   auto rows_in = [&](uint32_t dst, int stride, const bf16* src, int ld, int width, int live) {
-    const int pieces = width / 8;
-    for (int i = tid; i < kTile * pieces; i += kThreads) {
-      const int r = i / pieces, k = i - r * pieces;
-      cp_async16(dst + uint32_t(r * stride + 8 * k) * 2, src + (size_t)(r < live ? r : 0) * ld + 8 * k, r < live);
+    const int pieces = width / 8, dr = kThreads / pieces, dk8 = kThreads - dr * pieces;
+    int row = tid / pieces, k = tid - row * pieces;
+    while (row < kTile) {
+      cp_async16(dst + uint32_t(row * stride + 8 * k) * 2, src + (size_t)(row < live ? row : 0) * ld + 8 * k, row < live);
+      row += dr;
+      k += dk8;
+      if (k >= pieces) {
+        k -= pieces;
+        ++row;
+      }
     }
   };
-  auto load = [&](int t) {
-    const uint32_t st = uint32_t(t & 1);
-    rows_in(k_s + st * kTile * ks * 2, ks, K + (size_t)t * kTile * p.ld_kv, p.ld_kv, dk, kTile);
-    rows_in(v_s + st * kTile * vs * 2, vs, V + (size_t)t * kTile * p.ld_kv, p.ld_kv, dv, kTile);
-    cp_async_commit();
-  };
+  auto load_k = [&](int t) { rows_in(k_s, ks, K + (size_t)t * kTile * p.ld_kv, p.ld_kv, dk, kTile); };
+  auto load_v = [&](int t) { rows_in(v_s, vs, V + (size_t)t * kTile * p.ld_kv, p.ld_kv, dv, kTile); };
   rows_in(q_s, ks, Q, p.ld_q, dk, tokens);
-  load(0);
+  load_k(0);
+  cp_async_commit();
+  load_v(0);
+  cp_async_commit();
 
   const int ra = 16 * warp + g, pos_a = pos0 + i0 + ra, pos_b = pos_a + 8;
   const float scale2 = p.scale * kLog2e;
@@ -118,14 +124,12 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
   const uint32_t q_a = q_s + uint32_t((16 * warp + (lane & 15)) * ks + (lane >> 4) * 8) * 2;
-  const uint32_t k_l = uint32_t(((lane & 7) + ((lane >> 4) << 3)) * ks + ((lane >> 3) & 1) * 8) * 2;
-  const uint32_t v_l = uint32_t(((lane & 7) + (((lane >> 3) & 1) << 3)) * vs + (lane >> 4) * 8) * 2;
+  const uint32_t k_a = k_s + uint32_t(((lane & 7) + ((lane >> 4) << 3)) * ks + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t v_a = v_s + uint32_t(((lane & 7) + (((lane >> 3) & 1) << 3)) * vs + (lane >> 4) * 8) * 2;
+  cp_async_wait<1>();
+  __syncthreads();  // queries and the first keys have landed
 
   for (int t = 0; t < tiles; ++t) {
-    cp_async_wait<0>();
-    __syncthreads();
-    if (t + 1 < tiles) load(t + 1);
-    const uint32_t st = uint32_t(t & 1), k_a = k_s + st * kTile * ks * 2 + k_l, v_a = v_s + st * kTile * vs * 2 + v_l;
     float s[8][4] = {};
 #pragma unroll 4
     for (int k = 0; k < dk; k += 16) {
@@ -169,14 +173,22 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
     const float fa = ex2(m_a - ma), fb = ex2(m_b - mb);
     m_a = ma;
     m_b = mb;
-    l_a *= fa;
-    l_b *= fb;
+    if (__any_sync(0xffffffffu, fa != 1.0f || fb != 1.0f)) {
+      l_a *= fa;
+      l_b *= fb;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      o[i][0] *= fa;
-      o[i][1] *= fa;
-      o[i][2] *= fb;
-      o[i][3] *= fb;
+      for (int i = 0; i < NV; ++i) {
+        o[i][0] *= fa;
+        o[i][1] *= fa;
+        o[i][2] *= fb;
+        o[i][3] *= fb;
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();  // the values have landed; everybody is done with the keys
+    if (t + 1 < tiles) {
+      load_k(t + 1);
+      cp_async_commit();
     }
 #pragma unroll
     for (int kb = 0; kb < 4; ++kb) {
@@ -201,6 +213,12 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
         mma_bf16_16816(o[2 * np], ph, v[0], v[1]);
         mma_bf16_16816(o[2 * np + 1], ph, v[2], v[3]);
       }
+    }
+    if (t + 1 < tiles) {
+      cp_async_wait<0>();
+      __syncthreads();  // the next keys have landed; everybody is done with the values
+      load_v(t + 1);
+      cp_async_commit();
     }
   }
 #pragma unroll
@@ -238,7 +256,7 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
 }
 
 size_t smem_bytes(int dim, int vdim) {
-  return size_t(kTile) * (size_t(3) * (up16(dim) + 8) + size_t(2) * (up16(vdim) + 8)) * 2;
+  return size_t(kTile) * (size_t(2) * (up16(dim) + 8) + size_t(up16(vdim) + 8)) * 2;
 }
 
 template <int NV>
