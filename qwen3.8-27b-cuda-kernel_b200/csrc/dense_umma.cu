@@ -17,6 +17,7 @@
 #include "act.cuh"
 #include "dense_gemm.h"
 #include "tcgen05.cuh"
+#include "tensor_map.h"
 
 namespace q38 {
 Q38_REGISTER_ERROR_WORD();
@@ -334,34 +335,6 @@ __global__ void __launch_bounds__(kThreads) dense_umma_kernel(const __grid_const
   }
 }
 
-using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                              const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                              CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeFn encode_fn() {
-  static EncodeFn fn = [] {
-    void* p = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess) p = nullptr;
-    return reinterpret_cast<EncodeFn>(p);
-  }();
-  return fn;
-}
-
-// [rows][cols] bf16 with rows `ld` elements apart, boxes of 64 columns x box_rows
-int encode_2d(CUtensorMap* map, const void* base, int rows, int cols, int ld, int box_rows) {
-  EncodeFn enc = encode_fn();
-  Q38_REQUIRE(enc != nullptr, "dense_gemm: cuTensorMapEncodeTiled is not available from this driver");
-  const cuuint64_t dims[2] = {cuuint64_t(cols), cuuint64_t(rows)};
-  const cuuint64_t strides[1] = {cuuint64_t(ld) * 2};
-  const cuuint32_t box[2] = {64, cuuint32_t(box_rows)};
-  const cuuint32_t estr[2] = {1, 1};
-  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  Q38_REQUIRE(r == CUDA_SUCCESS, "dense_gemm: tensor map encode failed (%d)", int(r));
-  return Q38_OK;
-}
-
 template <int TOK, bool CLUSTER>
 int launch(const DenseCall& c, int cluster, cudaStream_t stream) {
   using K = Cfg<TOK, CLUSTER>;
@@ -369,8 +342,8 @@ int launch(const DenseCall& c, int cluster, cudaStream_t stream) {
                                                        cudaFuncAttributeMaxDynamicSharedMemorySize, K::kSmemBytes);
   Q38_CUDA_OK(attr);
   CUtensorMap wmap, xmap;
-  if (const int rc = encode_2d(&wmap, c.w.w, c.groups.count * c.w.n, c.w.k, c.w.ld, kTileN)) return rc;
-  if (const int rc = encode_2d(&xmap, c.x, c.m, (c.groups.count - 1) * c.groups.x_stride + c.w.k, c.ldx, TOK)) return rc;
+  if (const int rc = encode_bf16_rows(&wmap, c.w.w, c.groups.count * c.w.n, c.w.k, c.w.ld, kTileN)) return rc;
+  if (const int rc = encode_bf16_rows(&xmap, c.x, c.m, (c.groups.count - 1) * c.groups.x_stride + c.w.k, c.ldx, TOK)) return rc;
   Args a{};
   a.m = c.m;
   a.n = c.w.n;

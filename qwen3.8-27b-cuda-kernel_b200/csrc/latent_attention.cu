@@ -1,16 +1,19 @@
 // Latent attention of the layer-list architectures: every head's queries, brought into the latent space beforehand, meet one
 // cached latent per token, which is key and value at once.
 //
-// bf16 cache: one tensor-core kernel (mma.sync, fp32 scores, weights and sums) for prompts and decoding. The heads of a token
-//   and the tokens of a run are the same thing to it - rows that share the keys: a CTA takes 16, 32 or 64 consecutive rows
-//   (token, head) of a sequence and walks its pages, a page (64 latents) at a time, through a two-stage cp.async ring; the
-//   tile serves the scores as it lies and the values transposed by ldmatrix. The softmax weights enter the second product as
+// bf16 cache: tensor-core kernels (mma.sync, fp32 scores, weights and sums) for prompts and decoding. The heads of a token and
+//   the tokens of a run are the same thing to them - rows that share the keys: a CTA takes 16, 32 or 64 consecutive rows
+//   (token, head) of a sequence and walks its pages, 64 latents at a time, through a ring of TMA loads; a page serves the
+//   scores as it lies and the values transposed by ldmatrix. What bounds this is the traffic between shared memory and the
+//   fragments, so up to 32 rows keep their queries in registers: the warps divide the latent's dimensions (and the keys)
+//   among them and add their parts of the scores through shared memory. The softmax weights enter the second product as
 //   bf16 hi + lo (16 mantissa bits). With few rows the pages are divided over CTAs and a second kernel joins the pieces.
 // fp32 cache and outsized latents: a CTA per (token, head) on the CUDA cores.
 #include <algorithm>
 
 #include "act.cuh"
 #include "host_util.h"
+#include "tensor_map.h"
 
 namespace q38 {
 Q38_REGISTER_ERROR_WORD();
@@ -113,30 +116,22 @@ __global__ void __launch_bounds__(kGenThreads) latent_general_kernel(q38_latent_
 }
 
 // ---- tensor cores ---------------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool real) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(real ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                : "r"(addr));
 }
 
-constexpr int kMmaThreads = 256, kPS = kPage + 8;
+constexpr int kPS = kPage + 8;
 __host__ __device__ constexpr int row_stride(int k_dim) { return k_dim + 8; }  // an odd multiple of 16 bytes
-struct MmaSmem {
-  int q, c, p_hi, p_lo, total;
-  __host__ __device__ MmaSmem(int rows, int k_dim) {
-    q = 0;
-    c = q + rows * row_stride(k_dim) * 2;
-    p_hi = c + 2 * kPage * row_stride(k_dim) * 2;
-    p_lo = p_hi + rows * kPS * 2;
-    total = p_lo + rows * kPS * 2;
-  }
-};
+// A page in shared memory: tiles of 64 dimensions, [tile][64 latents][128 bytes] with the 128-byte swizzle, so that the eight
+// rows of an ldmatrix phase lie in different banks.
+constexpr int kTileBytes = kPage * 128;
+__host__ __device__ constexpr int page_smem(int k_dim) { return (k_dim + 63) / 64 * kTileBytes; }
+// byte offset of the 16 bytes at dimension 8 * chunk of latent `row` (the swizzle only depends on row & 7)
+__device__ __forceinline__ uint32_t page_at(int row, int chunk) {
+  return uint32_t((chunk >> 3) * kTileBytes + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
+}
 
 // What a block of rows has to do: its rows of the sequence and its share of the pages.
 struct Share {
@@ -159,56 +154,296 @@ __device__ __forceinline__ float* piece(const q38_latent_attention_params& p, in
   return p.partials + ((block * splits + split) * block_rows + r) * size_t(k_dim + 2);
 }
 
-// RG row groups of 16 x CG = 8 / RG warps side by side; a warp scores 64 / CG keys of a page and carries NT * 8 columns of
-// the output (k_dim up to CG * NT * 8).
-template <int RG, int NT>
-__global__ void __launch_bounds__(kMmaThreads, 1)
-latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv, int splits) {
-  constexpr int CG = 8 / RG, ROWS = 16 * RG, KT = 8 / CG;  // KT: 8-key tiles of a warp's scores
-  extern __shared__ __align__(16) uint8_t smem[];
-  __shared__ float mx[ROWS][CG], sum[ROWS][CG];
-  const int k_dim = kv.k_dim, rs = row_stride(k_dim);
-  const MmaSmem L(ROWS, k_dim);
+// The ring of pages of one CTA. Thread 0 asks for the pages, every thread sees every one of them, so one barrier per stage is
+// enough. A wait that runs out makes the results meaningless; the kernel then asks for nothing more and drains.
+template <int STAGES>
+struct PageRing {
+  uint64_t* full;  // [STAGES]
+  int* issued;     // [STAGES] loads each barrier has been told about
+  uint8_t* pages;  // 1024-byte aligned
+  const int* table;
+  int k_dim, first, last;
+
+  // thread 0
+  __device__ __forceinline__ void start(const CUtensorMap* map, int num_pages) const {
+    for (int i = 0; i < STAGES; ++i) {
+      mbar_init(&full[i], 1);
+      issued[i] = 0;
+    }
+    mbar_fence_init();
+    for (int i = 0; i < STAGES && first + i < last; ++i) load(map, num_pages, first + i);
+  }
+  __device__ __forceinline__ void load(const CUtensorMap* map, int num_pages, int pg) const {
+    const int stage = (pg - first) % STAGES;
+    int page = table[pg];
+    if (page < 0 || page >= num_pages) {
+      report_error(0x902);
+      page = 0;
+    }
+    uint8_t* dst = pages + stage * page_smem(k_dim);
+    mbar_expect_tx(&full[stage], uint32_t(page_smem(k_dim)));
+    issued[stage] += 1;
+    for (int d = 0; d < k_dim; d += 64) tma_load_2d(dst + d / 64 * kTileBytes, map, d, page * kPage, &full[stage]);
+  }
+  __device__ __forceinline__ bool wait(int pg) const {  // a whole warp, the same answer in all its lanes
+    return __all_sync(0xffffffffu, mbar_wait(&full[(pg - first) % STAGES], uint32_t((pg - first) / STAGES) & 1, 0x904));
+  }
+  __device__ __forceinline__ uint32_t at(int pg) const { return smem_u32(pages) + uint32_t((pg - first) % STAGES * page_smem(k_dim)); }
+  __device__ __forceinline__ void finish(bool ok) const {  // every thread; also a barrier
+    if (__syncthreads_or(!ok) && threadIdx.x < STAGES && issued[threadIdx.x] > 0)
+      for (uint32_t i = 0; i < kSpinLimit; ++i)
+        if (mbar_try_wait(&full[threadIdx.x], uint32_t(issued[threadIdx.x] - 1) & 1)) break;
+  }
+};
+__device__ __forceinline__ uint8_t* ring_base(uint8_t* smem) { return smem + ((1024 - (smem_u32(smem) & 1023)) & 1023); }
+
+// Output column pair of a finished row: as it is stored, or into the row's piece.
+struct RowOut {
+  bf16* out;
+  float* rec;
+  float inv;
+  __device__ __forceinline__ void put(int c, float a, float b) const {
+    if (rec) *reinterpret_cast<float2*>(rec + c) = make_float2(a, b);
+    else *reinterpret_cast<__nv_bfloat162*>(out + c) = __floats2bfloat162_rn(a * inv, b * inv);
+  }
+};
+
+// Up to 32 rows (RG groups of 16). Scores: a warp takes a quarter of the dimensions (KS k16 steps, queries in registers) of
+// 256 / WARPS keys; softmax: all threads, a row by neighbouring ones; outputs: a warp takes NT * 8 columns for all rows.
+constexpr int kXS = kPage + 8;  // row stride of the parts of the scores, in floats
+template <int RG, int WARPS, int KS, int NT, int STAGES>
+__global__ void __launch_bounds__(WARPS * 32, RG * WARPS <= 8 ? 2 : 1)
+latent_few_kernel(const __grid_constant__ CUtensorMap map, q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv,
+                  int splits) {
+  constexpr int ROWS = 16 * RG, KEYS_T = kPage * ROWS / (32 * WARPS);  // keys of a row that a thread of the softmax takes
+  constexpr int ROW_T = kPage / KEYS_T;                                // threads of a row
+  constexpr int KP = 16 / WARPS;                                       // 16-key pieces of a warp's scores
+  static_assert(KEYS_T % 4 == 0 && ROW_T <= 32 && KP >= 1 && NT % 2 == 0, "shape");
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = ring_base(smem_raw);
+  __shared__ __align__(8) uint64_t full[STAGES];
+  __shared__ int issued[STAGES];
+  __shared__ float factor[ROWS], row_m[ROWS], row_l[ROWS];
+  const int k_dim = kv.k_dim;
+  float* part = reinterpret_cast<float*>(smem + STAGES * page_smem(k_dim));  // [4 quarters][ROWS][kXS]
+  bf16* p_hi = reinterpret_cast<bf16*>(part + 4 * ROWS * kXS);               // [ROWS][kPS]
+  bf16* p_lo = p_hi + ROWS * kPS;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int rg = warp / CG, cg = warp % CG;
   const int split = blockIdx.y, seq = blockIdx.z;
   pdl_wait();
   pdl_launch_dependents();
   const int start = b.seq_start[seq], count = b.seq_start[seq + 1] - start, pos0 = b.seq_pos0[seq], H = p.heads;
   const Share sh = share_of(blockIdx.x, ROWS, count, H, pos0, split, splits);
   if (sh.p0 >= sh.p1) return;
-  const int* table = kv.block_table + (size_t)b.seq_slot[seq] * kv.max_pages_per_seq;
-  const int pieces = k_dim / 8;
-  // 16-byte pieces of a page dealt to the threads in order: row and column of the first, steps to the next
-  const int r0 = tid / pieces, k0 = tid - r0 * pieces, dr = kMmaThreads / pieces, dk = kMmaThreads - dr * pieces;
+  const PageRing<STAGES> ring{full, issued, smem, kv.block_table + (size_t)b.seq_slot[seq] * kv.max_pages_per_seq, k_dim, sh.p0, sh.p1};
+  if (tid == 0) ring.start(&map, kv.num_pages);
+  __syncthreads();
 
-  auto load_page = [&](int pg) {
-    int page = table[pg];
-    if (page < 0 || page >= kv.num_pages) {
-      if (tid == 0) report_error(0x902);
-      page = 0;
+  // this warp's share of the queries: fragments of KS k16 steps, zero where there is no row or no dimension
+  const int kg = warp & 3, key0 = (warp >> 2) * 16 * KP;
+  const bf16* q = static_cast<const bf16*>(p.q) + ((size_t)start * H + sh.first) * k_dim;
+  uint32_t qf[RG][KS][4];
+#pragma unroll
+  for (int r = 0; r < RG; ++r)
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int row = 16 * r + g + 8 * (e & 1), d = (kg * KS + k) * 16 + 2 * t4 + 8 * (e >> 1);
+        qf[r][k][e] = row < sh.rows && d < k_dim ? *reinterpret_cast<const uint32_t*>(q + (size_t)row * k_dim + d) : 0u;
+      }
+  // this thread's row of the softmax
+  const int srow = tid / ROW_T, skey = tid % ROW_T * 4;  // ... and of its keys: four from skey, four from skey + 4 ROW_T, ...
+  const int spos = srow < sh.rows ? pos0 + (sh.first + srow) / H : -1;
+  const float scale2 = p.scale * kLog2e;
+  float m = -INFINITY, l = 0.0f;
+  float o[RG][NT][4];
+#pragma unroll
+  for (int r = 0; r < RG; ++r)
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[r][i][e] = 0.0f;
+  const int c0 = warp * NT * 8;
+  uint32_t k_l[KS], v_l[NT / 2];  // this lane's rows of the fragments; sixteen latents further is 2048 bytes further
+#pragma unroll
+  for (int k = 0; k < KS; ++k) k_l[k] = page_at(key0 + (lane & 7) + ((lane >> 4) << 3), 2 * (kg * KS + k) + ((lane >> 3) & 1));
+#pragma unroll
+  for (int np = 0; np < NT / 2; ++np) v_l[np] = page_at((lane & 7) + (((lane >> 3) & 1) << 3), c0 / 8 + 2 * np + (lane >> 4));
+  const uint32_t ph_a = smem_u32(p_hi) + uint32_t((lane & 15) * kPS + (lane >> 4) * 8) * 2, pl_a = ph_a + ROWS * kPS * 2;
+  bool ok = true;
+
+  for (int pg = sh.p0; pg < sh.p1; ++pg) {
+    ok = ok && ring.wait(pg);
+    const uint32_t c_a = ring.at(pg);
+    // ---- this warp's part of the scores ----
+    float s[RG][2 * KP][4] = {};
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      if ((kg * KS + k) * 16 >= k_dim) break;
+      uint32_t kf[KP][4];
+#pragma unroll
+      for (int x = 0; x < KP; ++x) ldmatrix_x4(kf[x], c_a + k_l[k] + uint32_t(x * 2048));
+#pragma unroll
+      for (int r = 0; r < RG; ++r)
+#pragma unroll
+        for (int x = 0; x < KP; ++x) {
+          mma_bf16_16816(s[r][2 * x], qf[r][k], kf[x][0], kf[x][1]);
+          mma_bf16_16816(s[r][2 * x + 1], qf[r][k], kf[x][2], kf[x][3]);
+        }
     }
-    const bf16* src = reinterpret_cast<const bf16*>(kv.pages + (size_t)page * kv.page_bytes);
-    bf16* dst = reinterpret_cast<bf16*>(smem + L.c) + (size_t)(pg & 1) * kPage * rs;
-    int r = r0, k = k0;
-    uint32_t to = smem_u32(dst);
-    for (int i = tid; i < kPage * pieces; i += kMmaThreads) {
-      cp_async16(to + uint32_t(r * rs + 8 * k) * 2, src + (size_t)i * 8, true);
-      r += dr;
-      k += dk;
-      if (k >= pieces) {
-        k -= pieces;
-        ++r;
+#pragma unroll
+    for (int r = 0; r < RG; ++r)
+#pragma unroll
+      for (int kt = 0; kt < 2 * KP; ++kt)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf)
+          *reinterpret_cast<float2*>(part + (kg * ROWS + 16 * r + g + 8 * hf) * kXS + key0 + 8 * kt + 2 * t4) =
+              make_float2(s[r][kt][2 * hf], s[r][kt][2 * hf + 1]);
+    __syncthreads();
+    // ---- softmax ----
+    {
+      float x[KEYS_T], top = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < KEYS_T; i += 4) {
+        float4 v = make_float4(0, 0, 0, 0);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float4 y = *reinterpret_cast<const float4*>(part + (k * ROWS + srow) * kXS + skey + i * ROW_T);
+          v.x += y.x;
+          v.y += y.y;
+          v.z += y.z;
+          v.w += y.w;
+        }
+        x[i] = v.x;
+        x[i + 1] = v.y;
+        x[i + 2] = v.z;
+        x[i + 3] = v.w;
+      }
+#pragma unroll
+      for (int i = 0; i < KEYS_T; ++i) {
+        x[i] = pg * kPage + skey + i / 4 * 4 * ROW_T + i % 4 <= spos ? x[i] * scale2 : -INFINITY;
+        top = fmaxf(top, x[i]);
+      }
+#pragma unroll
+      for (int d = 1; d < ROW_T; d <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, d));
+      top = fmaxf(top, m);
+      const float base = top == -INFINITY ? 0.0f : top, f = ex2(m - base);
+      m = top;
+      l *= f;
+      if (skey == 0) factor[srow] = f;
+#pragma unroll
+      for (int i = 0; i < KEYS_T; i += 4) {
+        __nv_bfloat162 hi[2], lo[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float w0 = ex2(x[i + 2 * e] - base), w1 = ex2(x[i + 2 * e + 1] - base);
+          l += w0 + w1;
+          hi[e] = __floats2bfloat162_rn(w0, w1);
+          const float2 h = __bfloat1622float2(hi[e]);
+          lo[e] = __floats2bfloat162_rn(w0 - h.x, w1 - h.y);
+        }
+        *reinterpret_cast<uint2*>(p_hi + srow * kPS + skey + i * ROW_T) = *reinterpret_cast<const uint2*>(hi);
+        *reinterpret_cast<uint2*>(p_lo + srow * kPS + skey + i * ROW_T) = *reinterpret_cast<const uint2*>(lo);
       }
     }
-    cp_async_commit();
-  };
-  const bf16* q = static_cast<const bf16*>(p.q) + ((size_t)start * H + sh.first) * k_dim;
-  for (int i = tid; i < ROWS * pieces; i += kMmaThreads) {
-    const int r = i / pieces, k = i - r * pieces;
-    cp_async16(smem_u32(smem + L.q) + uint32_t(r * rs + 8 * k) * 2, r < sh.rows ? q + (size_t)i * 8 : q, r < sh.rows);
+    __syncthreads();
+    // ---- outputs: all rows and keys, this warp's columns ----
+#pragma unroll
+    for (int r = 0; r < RG; ++r) {
+      const float fa = factor[16 * r + g], fb = factor[16 * r + g + 8];
+      if (__any_sync(0xffffffffu, fa != 1.0f || fb != 1.0f)) {
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+          o[r][i][0] *= fa;
+          o[r][i][1] *= fa;
+          o[r][i][2] *= fb;
+          o[r][i][3] *= fb;
+        }
+      }
+    }
+    if (c0 < k_dim) {
+#pragma unroll
+      for (int kb = 0; kb < kPage / 16; ++kb) {
+        uint32_t ph[RG][4], pl[RG][4], v[NT / 2][4];
+#pragma unroll
+        for (int r = 0; r < RG; ++r) {
+          ldmatrix_x4(ph[r], ph_a + uint32_t(16 * r * kPS + kb * 16) * 2);
+          ldmatrix_x4(pl[r], pl_a + uint32_t(16 * r * kPS + kb * 16) * 2);
+        }
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np)
+          if (c0 + 16 * np < k_dim) ldmatrix_x4_trans(v[np], c_a + v_l[np] + uint32_t(kb * 2048));
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int r = 0; r < RG; ++r)
+#pragma unroll
+            for (int np = 0; np < NT / 2; ++np)
+              if (c0 + 16 * np < k_dim) {
+                mma_bf16_16816(o[r][2 * np], term ? ph[r] : pl[r], v[np][0], v[np][1]);
+                mma_bf16_16816(o[r][2 * np + 1], term ? ph[r] : pl[r], v[np][2], v[np][3]);
+              }
+      }
+    }
+    if (pg + 1 < sh.p1) {
+      __syncthreads();  // everybody is done with the page, the weights and the factors
+      if (tid == 0 && ok && pg + STAGES < sh.p1) ring.load(&map, kv.num_pages, pg + STAGES);
+    }
   }
-  load_page(sh.p0);
+#pragma unroll
+  for (int d = 1; d < ROW_T; d <<= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+  if (skey == 0) {
+    row_m[srow] = m;
+    row_l[srow] = l;
+  }
+  ring.finish(ok);
+#pragma unroll
+  for (int r = 0; r < RG; ++r)
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int row = 16 * r + g + 8 * hf;
+      if (row >= sh.rows) continue;
+      RowOut to{static_cast<bf16*>(p.out) + ((size_t)start * H + sh.first + row) * k_dim, nullptr, 1.0f / row_l[row]};
+      if (splits > 1) to.rec = piece(p, k_dim, (size_t)seq * gridDim.x + blockIdx.x, split, splits, ROWS, row);
+#pragma unroll
+      for (int i = 0; i < NT; ++i)
+        if (c0 + 8 * i < k_dim) to.put(c0 + 8 * i + 2 * t4, o[r][i][2 * hf], o[r][i][2 * hf + 1]);
+      if (splits > 1 && warp == 0 && t4 == 0) *reinterpret_cast<float2*>(to.rec + k_dim) = make_float2(row_m[row], row_l[row]);
+    }
+}
+
+// 64 rows, sixteen warps: four row groups x four column groups; a warp scores 16 keys of a page for its rows (queries from
+// shared memory) and carries NT * 8 columns of their outputs.
+constexpr int kManyThreads = 512, kManyRows = 64, kCG = 4;
+template <int NT, int STAGES>
+__global__ void __launch_bounds__(kManyThreads, 1)
+latent_many_kernel(const __grid_constant__ CUtensorMap map, q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_desc kv,
+                   int splits) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = ring_base(smem_raw);
+  __shared__ __align__(8) uint64_t full[STAGES];
+  __shared__ int issued[STAGES];
+  __shared__ float mx[kManyRows][kCG], sum[kManyRows][kCG];
+  const int k_dim = kv.k_dim, rs = row_stride(k_dim);
+  bf16* q_s = reinterpret_cast<bf16*>(smem + STAGES * page_smem(k_dim));  // [64][rs]
+  bf16* p_hi = q_s + kManyRows * rs;                                      // [64][kPS]
+  bf16* p_lo = p_hi + kManyRows * kPS;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int rg = warp / kCG, cg = warp % kCG, split = blockIdx.y, seq = blockIdx.z;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int start = b.seq_start[seq], count = b.seq_start[seq + 1] - start, pos0 = b.seq_pos0[seq], H = p.heads;
+  const Share sh = share_of(blockIdx.x, kManyRows, count, H, pos0, split, splits);
+  if (sh.p0 >= sh.p1) return;
+  const PageRing<STAGES> ring{full, issued, smem, kv.block_table + (size_t)b.seq_slot[seq] * kv.max_pages_per_seq, k_dim, sh.p0, sh.p1};
+  if (tid == 0) ring.start(&map, kv.num_pages);
+  __syncthreads();
+  const uint4* q = reinterpret_cast<const uint4*>(static_cast<const bf16*>(p.q) + ((size_t)start * H + sh.first) * k_dim);
+  const int pieces = k_dim / 8;
+  for (int i = tid; i < kManyRows * pieces; i += kManyThreads)
+    *reinterpret_cast<uint4*>(q_s + i / pieces * rs + i % pieces * 8) = i < sh.rows * pieces ? q[i] : make_uint4(0, 0, 0, 0);
+  __syncthreads();
 
   const int ra = 16 * rg + g, rb = ra + 8;
   const int pos_a = ra < sh.rows ? pos0 + (sh.first + ra) / H : -1, pos_b = rb < sh.rows ? pos0 + (sh.first + rb) / H : -1;
@@ -219,65 +454,38 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
   for (int i = 0; i < NT; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
-  const uint32_t q_a = smem_u32(smem + L.q) + ((16 * rg + (lane & 15)) * rs + (lane >> 4) * 8) * 2;
-  const uint32_t ph_a = smem_u32(smem + L.p_hi) + ((16 * rg + (lane & 15)) * kPS + (lane >> 4) * 8) * 2;
-  const uint32_t pl_a = ph_a + uint32_t(L.p_lo - L.p_hi);
-  const int c0 = cg * NT * 8;  // first output column of this warp
+  const uint32_t q_a = smem_u32(q_s) + ((16 * rg + (lane & 15)) * rs + (lane >> 4) * 8) * 2;
+  const uint32_t ph_a = smem_u32(p_hi) + ((16 * rg + (lane & 15)) * kPS + (lane >> 4) * 8) * 2, pl_a = ph_a + kManyRows * kPS * 2;
+  const int c0 = cg * NT * 8, key0 = cg * 16;  // first output column and key of this warp
+  bool ok = true;
 
   for (int pg = sh.p0; pg < sh.p1; ++pg) {
-    cp_async_wait<0>();
-    __syncthreads();  // the page has landed; everybody is done with the one before
-    if (pg + 1 < sh.p1) load_page(pg + 1);
-    const uint32_t c_a = smem_u32(smem + L.c) + uint32_t((pg & 1) * kPage * rs) * 2;
-
-    // ---- scores of this warp's keys ----
-    float s[KT][4] = {};
-    const int key0 = cg * KT * 8;
-    if (KT == 1) {  // 8 keys: two k16 steps per load
-      const uint32_t k_a = c_a + ((key0 + (lane & 7)) * rs + (lane >> 3) * 8) * 2;
-      float s2[4] = {};
-#pragma unroll 4
-      for (int k = 0; k < k_dim; k += 32) {
-        uint32_t kf[4], a0[4], a1[4];
-        ldmatrix_x4(kf, k_a + k * 2);
-        ldmatrix_x4(a0, q_a + k * 2);
-        ldmatrix_x4(a1, q_a + k * 2 + 32);
-        mma_bf16_16816(s[0], a0, kf[0], kf[1]);
-        mma_bf16_16816(s2, a1, kf[2], kf[3]);
-      }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[0][e] += s2[e];
-    } else {
-      const uint32_t k_a = c_a + ((key0 + (lane & 7) + ((lane >> 4) << 3)) * rs + ((lane >> 3) & 1) * 8) * 2;
-      float s2[KT][4] = {};  // every other step: shorter chains of dependent products
+    ok = ok && ring.wait(pg);
+    const uint32_t c_a = ring.at(pg);
+    // ---- scores of this warp's keys, every other step into accumulators of its own ----
+    float s[2][4] = {}, s2[2][4] = {};
+    const int krow = key0 + (lane & 7) + ((lane >> 4) << 3), kchunk = (lane >> 3) & 1;
 #pragma unroll 2
-      for (int k = 0; k < k_dim; k += 32) {
+    for (int k = 0; k < k_dim; k += 32) {
+      uint32_t a[2][4], kf[2][4];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          uint32_t a[4];
-          ldmatrix_x4(a, q_a + (k + 16 * e) * 2);
-#pragma unroll
-          for (int kp = 0; kp < KT / 2; ++kp) {
-            uint32_t kf[4];
-            ldmatrix_x4(kf, k_a + (kp * 16 * rs + k + 16 * e) * 2);
-            mma_bf16_16816(e ? s2[2 * kp] : s[2 * kp], a, kf[0], kf[1]);
-            mma_bf16_16816(e ? s2[2 * kp + 1] : s[2 * kp + 1], a, kf[2], kf[3]);
-          }
-        }
+      for (int e = 0; e < 2; ++e) {
+        ldmatrix_x4(a[e], q_a + (k + 16 * e) * 2);
+        ldmatrix_x4(kf[e], c_a + page_at(krow, k / 8 + 2 * e + kchunk));
       }
-#pragma unroll
-      for (int kt = 0; kt < KT; ++kt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[kt][e] += s2[kt][e];
+      mma_bf16_16816(s[0], a[0], kf[0][0], kf[0][1]);
+      mma_bf16_16816(s[1], a[0], kf[0][2], kf[0][3]);
+      mma_bf16_16816(s2[0], a[1], kf[1][0], kf[1][1]);
+      mma_bf16_16816(s2[1], a[1], kf[1][2], kf[1][3]);
     }
     float ma = -INFINITY, mb = -INFINITY;
 #pragma unroll
-    for (int kt = 0; kt < KT; ++kt)
+    for (int kt = 0; kt < 2; ++kt)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int key = pg * kPage + key0 + 8 * kt + 2 * t4 + e;
-        s[kt][e] = key <= pos_a ? s[kt][e] * scale2 : -INFINITY;
-        s[kt][2 + e] = key <= pos_b ? s[kt][2 + e] * scale2 : -INFINITY;
+        s[kt][e] = key <= pos_a ? (s[kt][e] + s2[kt][e]) * scale2 : -INFINITY;
+        s[kt][2 + e] = key <= pos_b ? (s[kt][2 + e] + s2[kt][2 + e]) * scale2 : -INFINITY;
         ma = fmaxf(ma, s[kt][e]);
         mb = fmaxf(mb, s[kt][2 + e]);
       }
@@ -292,7 +500,7 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     }
     __syncthreads();
 #pragma unroll
-    for (int x = 0; x < CG; ++x) {
+    for (int x = 0; x < kCG; ++x) {
       ma = fmaxf(ma, mx[ra][x]);
       mb = fmaxf(mb, mx[rb][x]);
     }
@@ -306,7 +514,7 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     l_b *= fb;
     // ---- weights: this warp's keys into shared memory, hi + lo ----
 #pragma unroll
-    for (int kt = 0; kt < KT; ++kt)
+    for (int kt = 0; kt < 2; ++kt)
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
         const float base = hf ? base_b : base_a;
@@ -314,9 +522,9 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
         (hf ? l_b : l_a) += w0 + w1;
         const __nv_bfloat162 hi = __floats2bfloat162_rn(w0, w1);
         const float2 f = __bfloat1622float2(hi);
-        const int at = ((hf ? rb : ra) * kPS + key0 + 8 * kt + 2 * t4) * 2;
-        *reinterpret_cast<__nv_bfloat162*>(smem + L.p_hi + at) = hi;
-        *reinterpret_cast<__nv_bfloat162*>(smem + L.p_lo + at) = __floats2bfloat162_rn(w0 - f.x, w1 - f.y);
+        const int at = (hf ? rb : ra) * kPS + key0 + 8 * kt + 2 * t4;
+        *reinterpret_cast<__nv_bfloat162*>(p_hi + at) = hi;
+        *reinterpret_cast<__nv_bfloat162*>(p_lo + at) = __floats2bfloat162_rn(w0 - f.x, w1 - f.y);
       }
     if (__any_sync(0xffffffffu, fa != 1.0f || fb != 1.0f)) {
 #pragma unroll
@@ -329,22 +537,32 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     }
     __syncthreads();
     // ---- outputs: all keys of the page, this warp's columns ----
-    const uint32_t v_a = c_a + (((lane & 7) + (((lane >> 3) & 1) << 3)) * rs + c0 + (lane >> 4) * 8) * 2;
+    uint32_t v_l[NT / 2];
+#pragma unroll
+    for (int np = 0; np < NT / 2; ++np) v_l[np] = c_a + page_at((lane & 7) + (((lane >> 3) & 1) << 3), c0 / 8 + 2 * np + (lane >> 4));
 #pragma unroll
     for (int kb = 0; kb < kPage / 16; ++kb) {
       uint32_t ph[4], pl[4];
       ldmatrix_x4(ph, ph_a + kb * 32);
       ldmatrix_x4(pl, pl_a + kb * 32);
 #pragma unroll
-      for (int np = 0; np < NT / 2; ++np) {
+      for (int np = 0; np < NT / 2; np += 2) {  // four products between two that depend on one another
         if (c0 + 16 * np >= k_dim) break;
-        uint32_t v[4];
-        ldmatrix_x4_trans(v, v_a + (kb * 16 * rs + np * 16) * 2);
-        mma_bf16_16816(o[2 * np], pl, v[0], v[1]);
-        mma_bf16_16816(o[2 * np + 1], pl, v[2], v[3]);
-        mma_bf16_16816(o[2 * np], ph, v[0], v[1]);
-        mma_bf16_16816(o[2 * np + 1], ph, v[2], v[3]);
+        uint32_t v[2][4];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) ldmatrix_x4_trans(v[x], v_l[np + x] + uint32_t(kb * 2048));
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            mma_bf16_16816(o[2 * (np + x)], term ? ph : pl, v[x][0], v[x][1]);
+            mma_bf16_16816(o[2 * (np + x) + 1], term ? ph : pl, v[x][2], v[x][3]);
+          }
       }
+    }
+    if (pg + 1 < sh.p1) {
+      __syncthreads();  // everybody is done with the page, the weights and the maxima
+      if (tid == 0 && ok && pg + STAGES < sh.p1) ring.load(&map, kv.num_pages, pg + STAGES);
     }
   }
   // ---- the rows' sums over all warps ----
@@ -357,10 +575,10 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
     sum[ra][cg] = l_a;
     sum[rb][cg] = l_b;
   }
-  __syncthreads();
+  ring.finish(ok);
   l_a = l_b = 0.0f;
 #pragma unroll
-  for (int x = 0; x < CG; ++x) {
+  for (int x = 0; x < kCG; ++x) {
     l_a += sum[ra][x];
     l_b += sum[rb][x];
   }
@@ -368,20 +586,12 @@ latent_mma_kernel(q38_latent_attention_params p, q38_batch_desc b, q38_kv_layer_
   for (int hf = 0; hf < 2; ++hf) {
     const int r = hf ? rb : ra;
     if (r >= sh.rows) continue;
-    if (splits == 1) {
-      const float inv = 1.0f / (hf ? l_b : l_a);
-      bf16* out = static_cast<bf16*>(p.out) + ((size_t)start * H + sh.first + r) * k_dim + c0 + 2 * t4;
+    RowOut to{static_cast<bf16*>(p.out) + ((size_t)start * H + sh.first + r) * k_dim, nullptr, 1.0f / (hf ? l_b : l_a)};
+    if (splits > 1) to.rec = piece(p, k_dim, (size_t)seq * gridDim.x + blockIdx.x, split, splits, kManyRows, r);
 #pragma unroll
-      for (int i = 0; i < NT; ++i)
-        if (c0 + 8 * i < k_dim)
-          *reinterpret_cast<__nv_bfloat162*>(out + 8 * i) = __floats2bfloat162_rn(o[i][2 * hf] * inv, o[i][2 * hf + 1] * inv);
-    } else {
-      float* rec = piece(p, k_dim, (size_t)seq * gridDim.x + blockIdx.x, split, splits, ROWS, r);
-#pragma unroll
-      for (int i = 0; i < NT; ++i)
-        if (c0 + 8 * i < k_dim) *reinterpret_cast<float2*>(rec + c0 + 8 * i + 2 * t4) = make_float2(o[i][2 * hf], o[i][2 * hf + 1]);
-      if (cg == 0 && t4 == 0) *reinterpret_cast<float2*>(rec + k_dim) = make_float2(hf ? m_b : m_a, hf ? l_b : l_a);
-    }
+    for (int i = 0; i < NT; ++i)
+      if (c0 + 8 * i < k_dim) to.put(c0 + 8 * i + 2 * t4, o[i][2 * hf], o[i][2 * hf + 1]);
+    if (splits > 1 && cg == 0 && t4 == 0) *reinterpret_cast<float2*>(to.rec + k_dim) = make_float2(hf ? m_b : m_a, hf ? l_b : l_a);
   }
 }
 
@@ -433,38 +643,56 @@ __global__ void __launch_bounds__(128) latent_join_kernel(q38_latent_attention_p
 }
 
 constexpr int kMaxKDim = 512, kMaxSplits = 64;
-constexpr int kPieceRows = 64;  // rows of pieces per SM that the scratch holds: 64-row CTAs one per SM, 16-row CTAs four
+constexpr int kPieceRows = 64;  // rows of pieces per SM that the scratch holds
 
-template <int RG, int NT>
-int launch_mma(const q38_latent_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
-  constexpr int ROWS = 16 * RG;
-  const MmaSmem L(ROWS, kv.k_dim);
-  static const cudaError_t attr =
-      cudaFuncSetAttribute(latent_mma_kernel<RG, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - 1024);
-  Q38_CUDA_OK(attr);
-  const int blocks = (b.max_tokens_per_seq * p.heads + ROWS - 1) / ROWS;
+using MmaKernel = void (*)(CUtensorMap, q38_latent_attention_params, q38_batch_desc, q38_kv_layer_desc, int);
+// `resident`: CTAs of the kernel that share an SM
+int launch_mma(MmaKernel kernel, int threads, int block_rows, size_t smem, int resident, const q38_latent_attention_params& p,
+               const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
+  const int blocks = (b.max_tokens_per_seq * p.heads + block_rows - 1) / block_rows;
   const long long ctas = (long long)blocks * b.num_seqs;
   // Few CTAs: the pages of each over as many as there is room for (and scratch for the pieces).
-  const int resident = std::min(4 / RG, std::max(1, 220 * 1024 / (L.total + 1024 + 2 * ROWS * 8 * 4)));
   int splits = int(std::min<long long>(kMaxSplits, (long long)num_sms() * resident / ctas));
-  const size_t per_split = size_t(ctas) * ROWS * size_t(kv.k_dim + 2);
+  const size_t per_split = size_t(ctas) * block_rows * size_t(kv.k_dim + 2);
   if (!p.partials) splits = 1;
   else splits = std::max(1, std::min(splits, int(std::min<size_t>(kMaxSplits, p.partial_floats / per_split))));
-  (void)launch_kernel(latent_mma_kernel<RG, NT>, dim3(blocks, splits, b.num_seqs), dim3(kMmaThreads), size_t(L.total), s, p, b, kv, splits);
-  Q38_LAUNCH_OK("latent_mma_kernel");
+  CUtensorMap map;  // the layer's pages as one matrix of latents
+  if (const int rc = encode_bf16_rows(&map, kv.pages, (long long)kv.num_pages * kPage, kv.k_dim, kv.k_dim, kPage)) return rc;
+  (void)launch_kernel(kernel, dim3(blocks, splits, b.num_seqs), dim3(threads), smem, s, map, p, b, kv, splits);
+  Q38_LAUNCH_OK("latent attention kernel");
   if (splits > 1) {
-    (void)launch_kernel(latent_join_kernel, dim3(b.max_tokens_per_seq * p.heads, b.num_seqs), dim3(128), 0, s, p, b, kv.k_dim, blocks, ROWS, splits);
+    (void)launch_kernel(latent_join_kernel, dim3(b.max_tokens_per_seq * p.heads, b.num_seqs), dim3(128), 0, s, p, b, kv.k_dim, blocks,
+                        block_rows, splits);
     Q38_LAUNCH_OK("latent_join_kernel");
   }
   return Q38_OK;
 }
 
+constexpr int kStaticSmem = 3072;  // room left for the kernels' static shared memory
+template <int RG, int WARPS, int KS, int STAGES>
+int launch_few(const q38_latent_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
+  constexpr int NT = KS * 8 / WARPS;  // four quarters of KS * 16 dimensions over all warps
+  static const cudaError_t attr = cudaFuncSetAttribute(latent_few_kernel<RG, WARPS, KS, NT, STAGES>,
+                                                       cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - kStaticSmem);
+  Q38_CUDA_OK(attr);
+  const size_t smem = 1024 + size_t(STAGES) * page_smem(kv.k_dim) + size_t(16 * RG) * (4 * kXS * 4 + 2 * kPS * 2);
+  const int resident = smem < size_t(100) * 1024 && RG * WARPS <= 8 ? 2 : 1;
+  return launch_mma(latent_few_kernel<RG, WARPS, KS, NT, STAGES>, 32 * WARPS, 16 * RG, smem, resident, p, b, kv, s);
+}
 template <int RG>
-int launch_rows(const q38_latent_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
-  constexpr int CG = 8 / RG;
-  if (kv.k_dim <= 128) return launch_mma<RG, 16 / CG>(p, b, kv, s);
-  if (kv.k_dim <= 256) return launch_mma<RG, 32 / CG>(p, b, kv, s);
-  return launch_mma<RG, 64 / CG>(p, b, kv, s);
+int launch_few_rows(const q38_latent_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
+  // 16 rows: two CTAs per SM, which cover one another's loads where only one buffer fits
+  if (kv.k_dim <= 128) return launch_few<RG, 8, 2, 3>(p, b, kv, s);
+  if (kv.k_dim <= 256) return launch_few<RG, 8, 4, 2>(p, b, kv, s);
+  return launch_few<RG, 8, 8, RG == 1 ? 1 : 2>(p, b, kv, s);
+}
+template <int NT>
+int launch_many(const q38_latent_attention_params& p, const q38_batch_desc& b, const q38_kv_layer_desc& kv, cudaStream_t s) {
+  static const cudaError_t attr =
+      cudaFuncSetAttribute(latent_many_kernel<NT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem() - kStaticSmem);
+  Q38_CUDA_OK(attr);
+  const size_t smem = 1024 + size_t(2) * page_smem(kv.k_dim) + size_t(kManyRows) * (row_stride(kv.k_dim) + 2 * kPS) * 2;
+  return launch_mma(latent_many_kernel<NT, 2>, kManyThreads, kManyRows, smem, 1, p, b, kv, s);
 }
 
 template <typename T>
@@ -521,10 +749,11 @@ extern "C" int q38_latent_attention(const q38_latent_attention_params* p, const 
   const cudaStream_t s = as_stream(stream);
   if (p->act == Q38_ACT_F32) return launch_general<float>(*p, *batch, *kv, s);
   if (kv->k_dim > kMaxKDim || (reinterpret_cast<uintptr_t>(p->q) | reinterpret_cast<uintptr_t>(p->out) | reinterpret_cast<uintptr_t>(kv->pages)) % 16 ||
-      kv->page_bytes % 16)
+      kv->page_bytes != size_t(kPage) * kv->k_dim * 2)
     return launch_general<bf16>(*p, *batch, *kv, s);
   const int rows = batch->max_tokens_per_seq * p->heads;
-  if (rows <= 16) return launch_rows<1>(*p, *batch, *kv, s);
-  if (rows <= 32) return launch_rows<2>(*p, *batch, *kv, s);
-  return launch_rows<4>(*p, *batch, *kv, s);
+  if (rows <= 16) return launch_few_rows<1>(*p, *batch, *kv, s);
+  if (rows <= 32) return launch_few_rows<2>(*p, *batch, *kv, s);
+  return kv->k_dim <= 128 ? launch_many<4>(*p, *batch, *kv, s)
+         : kv->k_dim <= 256 ? launch_many<8>(*p, *batch, *kv, s) : launch_many<16>(*p, *batch, *kv, s);
 }

@@ -22,6 +22,9 @@ constexpr int kPage = Q38_PAGE_TOKENS, kTile = 64, kThreads = 128;
 constexpr float kLog2e = 1.4426950408889634f;
 __host__ __device__ constexpr int up16(int x) { return (x + 15) / 16 * 16; }
 
+// the value product takes 32 columns at a time
+__host__ __device__ constexpr int value_stride(int vdim) { return (vdim + 31) / 32 * 32 + 8; }
+
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -79,12 +82,12 @@ template <int NV>
 __global__ void __launch_bounds__(kThreads)
 packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int dk = up16(p.dim), dv = up16(p.vdim), ks = dk + 8, vs = dv + 8;  // rows an odd multiple of 16 bytes apart
+  const int dk = up16(p.dim), dv = up16(p.vdim), ks = dk + 8, vs = value_stride(p.vdim);  // rows an odd multiple of 16 bytes apart
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const uint32_t q_s = smem_u32(smem), k_s = q_s + uint32_t(kTile * ks) * 2, v_s = k_s + uint32_t(kTile * ks) * 2;
   pdl_wait();
   pdl_launch_dependents();
-  const int h = blockIdx.y, seq = blockIdx.z, i0 = (int(gridDim.x) - 1 - int(blockIdx.x)) * kTile;
+  const int h = blockIdx.x, seq = blockIdx.z, i0 = (int(gridDim.y) - 1 - int(blockIdx.y)) * kTile;
   const int start = b.seq_start[seq], count = b.seq_start[seq + 1] - start, pos0 = b.seq_pos0[seq];
   if (i0 >= count) return;
   const size_t row0 = size_t(packed_start(b, seq));
@@ -109,6 +112,10 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
   };
   auto load_k = [&](int t) { rows_in(k_s, ks, K + (size_t)t * kTile * p.ld_kv, p.ld_kv, dk, kTile); };
   auto load_v = [&](int t) { rows_in(v_s, vs, V + (size_t)t * kTile * p.ld_kv, p.ld_kv, dv, kTile); };
+  if (dv % 32) {  // columns no head has: their products are never stored, but must not be read from nowhere
+    for (int i = tid; i < kTile * 8; i += kThreads)
+      *reinterpret_cast<uint32_t*>(smem + (v_s - q_s) + ((i >> 3) * vs + dv + 2 * (i & 7)) * 2) = 0;
+  }
   rows_in(q_s, ks, Q, p.ld_q, dk, tokens);
   load_k(0);
   cp_async_commit();
@@ -204,14 +211,21 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
         split2(w2, w3, ph[2 * e + 1], pl[2 * e + 1]);
       }
 #pragma unroll
-      for (int np = 0; np < NV / 2; ++np) {
+      for (int np = 0; np < NV / 2; np += 2) {  // four products between two that depend on one another
         if (16 * np >= dv) break;
-        uint32_t v[4];
-        ldmatrix_x4_trans(v, v_a + uint32_t(kb * 16 * vs + np * 16) * 2);
-        mma_bf16_16816(o[2 * np], pl, v[0], v[1]);
-        mma_bf16_16816(o[2 * np + 1], pl, v[2], v[3]);
-        mma_bf16_16816(o[2 * np], ph, v[0], v[1]);
-        mma_bf16_16816(o[2 * np + 1], ph, v[2], v[3]);
+        uint32_t v[2][4];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) ldmatrix_x4_trans(v[x], v_a + uint32_t(kb * 16 * vs + (np + x) * 16) * 2);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          mma_bf16_16816(o[2 * (np + x)], pl, v[x][0], v[x][1]);
+          mma_bf16_16816(o[2 * (np + x) + 1], pl, v[x][2], v[x][3]);
+        }
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          mma_bf16_16816(o[2 * (np + x)], ph, v[x][0], v[x][1]);
+          mma_bf16_16816(o[2 * (np + x) + 1], ph, v[x][2], v[x][3]);
+        }
       }
     }
     if (t + 1 < tiles) {
@@ -256,7 +270,7 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
 }
 
 size_t smem_bytes(int dim, int vdim) {
-  return size_t(kTile) * (size_t(2) * (up16(dim) + 8) + size_t(up16(vdim) + 8)) * 2;
+  return size_t(kTile) * (size_t(2) * (up16(dim) + 8) + size_t(value_stride(vdim))) * 2;
 }
 
 template <int NV>
@@ -264,7 +278,7 @@ int launch(const q38_packed_attention_params& p, const q38_batch_desc& b, cudaSt
   static const cudaError_t attr =
       cudaFuncSetAttribute(packed_attention_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_optin_smem());
   Q38_CUDA_OK(attr);
-  (void)launch_kernel(packed_attention_kernel<NV>, dim3((b.max_tokens_per_seq + kTile - 1) / kTile, p.heads, b.num_seqs), dim3(kThreads),
+  (void)launch_kernel(packed_attention_kernel<NV>, dim3(p.heads, (b.max_tokens_per_seq + kTile - 1) / kTile, b.num_seqs), dim3(kThreads),
                       smem_bytes(p.dim, p.vdim), s, p, b);
   Q38_LAUNCH_OK("packed_attention_kernel");
   return Q38_OK;

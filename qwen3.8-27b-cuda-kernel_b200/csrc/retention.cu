@@ -3,7 +3,7 @@
 // q and k are rotated in fp32 from the projections' values and stay fp32; so do the state and o.
 //
 // Decode batches: one CTA per (head, sequence) streams the head's state through registers once, with rotation, norm and
-//   output gate in the same kernel; the first pieces of the state are requested before the previous kernel has ended.
+//   output gate in the same kernel.
 // Prefill (bf16 activations): three kernels. rope: rotated q and k as bf16 hi + lo terms (16 mantissa bits). chunk: a CTA
 //   per (32 value columns, head, sequence) walks the run in chunks of 64 tokens with the state as fp32 MMA accumulators:
 //     o_i = decay^(i+1) S^T q_i + sum_(j <= i) decay^(i-j) (q_i . k_j) v_j,   S' = decay^n S + sum_j decay^(n-1-j) k_j v_j^T,
@@ -120,7 +120,8 @@ retention_decode_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_
   __shared__ float red_ss[33];
   const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, r = tid / v4, c = tid % v4;
   const bool live = r < rows;
-  // the state was last written an earlier step ago: its first pieces may be requested before the previous kernel has ended
+  pdl_wait();
+  pdl_launch_dependents();
   float4* state = reinterpret_cast<float4*>(st.state + (size_t)b.seq_slot[seq] * st.slot_bytes) + (size_t)h * p.dim * v4 + c;
   const int rounds = (p.dim + rows - 1) / rows;
   const int start = b.seq_start[seq], pos = b.seq_pos0[seq];
@@ -133,10 +134,8 @@ retention_decode_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_
       s[i] = live && !fresh && d < p.dim ? state[(size_t)d * v4] : make_float4(0, 0, 0, 0);
     }
   };
-  load(0);
+  load(0);  // in flight while the query and the key are rotated
   const float decay = p.decay_pow[h * (kChunk + 1) + 1];
-  pdl_wait();
-  pdl_launch_dependents();
   const T* row = static_cast<const T*>(p.proj) + (size_t)start * p.ld_proj;
   for (int i = tid; i < half; i += kDecThreads) trig[i] = turn_of(pos, p.inv_freq[i]);
   float4 v = make_float4(0, 0, 0, 0), o = v;
@@ -235,6 +234,14 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   const float2 f = __bfloat1622float2(h);
   hi = *reinterpret_cast<const uint32_t*>(&h);
   lo = pack2(a - f.x, b - f.y);
+}
+
+// one 16 x 16 block against 32 columns; consecutive products are independent of one another
+__device__ __forceinline__ void mma_row(float (&d)[4][4], const uint32_t (&a)[4], const uint32_t (&b)[2][4]) {
+#pragma unroll
+  for (int np = 0; np < 2; ++np)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) mma_bf16_16816(d[2 * np + e], a, b[np][2 * e], b[np][2 * e + 1]);
 }
 
 constexpr int kMmaThreads = 256, kVT = 32;  // value columns per CTA
@@ -373,19 +380,16 @@ retention_chunk_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_s
         uint32_t qh[4], ql[4];
         ldmatrix_x4(qh, q_hi + kb * 32);
         ldmatrix_x4(ql, q_lo + kb * 32);
+        uint32_t sh[2][4], sl[2][4];
 #pragma unroll
         for (int np = 0; np < 2; ++np) {
-          uint32_t sh[4], sl[4];
           const uint32_t at = ((16 * kb + k_row) * kVS + 16 * np + k_col) * 2;
-          ldmatrix_x4_trans(sh, sh_a + at);
-          ldmatrix_x4_trans(sl, sl_a + at);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            mma_bf16_16816(o[2 * np + e], ql, sh[2 * e], sh[2 * e + 1]);
-            mma_bf16_16816(o[2 * np + e], qh, sl[2 * e], sl[2 * e + 1]);
-            mma_bf16_16816(o[2 * np + e], qh, sh[2 * e], sh[2 * e + 1]);
-          }
+          ldmatrix_x4_trans(sh[np], sh_a + at);
+          ldmatrix_x4_trans(sl[np], sl_a + at);
         }
+        mma_row(o, ql, sh);
+        mma_row(o, qh, sl);
+        mma_row(o, qh, sh);
       }
       const float fa = pw[16 * rg + g + 1], fb = pw[16 * rg + g + 9];
 #pragma unroll
@@ -396,7 +400,7 @@ retention_chunk_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_s
         o[nt][3] *= fb;
       }
       for (int jb = half; jb <= rg; jb += 2) {
-        float s[2][4] = {};
+        float s[2][4] = {}, s_lh[2][4] = {}, s_hl[2][4] = {};  // the terms apart: chains of their own
         const uint32_t k_hi = qk_a + ((16 * jb + n_row) * L.qk_stride + 2 * dp + n_col) * 2, k_lo = k_hi + dp * 2;
         for (int kb = 0; kb < dblocks; ++kb) {
           uint32_t qh[4], ql[4], kh[4], kl[4];
@@ -406,11 +410,15 @@ retention_chunk_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_s
           ldmatrix_x4(kl, k_lo + kb * 32);
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            mma_bf16_16816(s[e], ql, kh[2 * e], kh[2 * e + 1]);
-            mma_bf16_16816(s[e], qh, kl[2 * e], kl[2 * e + 1]);
+            mma_bf16_16816(s_lh[e], ql, kh[2 * e], kh[2 * e + 1]);
+            mma_bf16_16816(s_hl[e], qh, kl[2 * e], kl[2 * e + 1]);
             mma_bf16_16816(s[e], qh, kh[2 * e], kh[2 * e + 1]);
           }
         }
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) s[e][x] += s_lh[e][x] + s_hl[e][x];
         uint32_t ah[4], al[4];
 #pragma unroll
         for (int e = 0; e < 2; ++e)
@@ -421,16 +429,11 @@ retention_chunk_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_s
             const float a1 = j + 1 <= i ? s[e][2 * hf + 1] * pw[i - j - 1] : 0.0f;
             split2(a0, a1, ah[2 * e + hf], al[2 * e + hf]);
           }
+        uint32_t v[2][4];
 #pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          uint32_t v[4];
-          ldmatrix_x4_trans(v, v_a + ((16 * jb + k_row) * kVS + 16 * np + k_col) * 2);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            mma_bf16_16816(o[2 * np + e], al, v[2 * e], v[2 * e + 1]);
-            mma_bf16_16816(o[2 * np + e], ah, v[2 * e], v[2 * e + 1]);
-          }
-        }
+        for (int np = 0; np < 2; ++np) ldmatrix_x4_trans(v[np], v_a + ((16 * jb + k_row) * kVS + 16 * np + k_col) * 2);
+        mma_row(o, al, v);
+        mma_row(o, ah, v);
       }
       // the two warps of a row block swap halves: warp `half` finishes columns 16 half .. 16 half + 15
       float* mine = X + (size_t)(1 - half) * kChunk * kXS;
@@ -459,19 +462,16 @@ retention_chunk_kernel(q38_retention_params p, q38_batch_desc b, q38_recurrent_s
         const uint32_t at = qk_a + ((16 * jb + t_row) * L.qk_stride + 2 * dp + 16 * db + t_col) * 2;
         ldmatrix_x4_trans(kh, at);
         ldmatrix_x4_trans(kl, at + dp * 2);
+        uint32_t wh[2][4], wl[2][4];
 #pragma unroll
         for (int np = 0; np < 2; ++np) {
-          uint32_t wh[4], wl[4];
           const uint32_t wat = ((16 * jb + k_row) * kVS + 16 * np + k_col) * 2;
-          ldmatrix_x4_trans(wh, wh_a + wat);
-          ldmatrix_x4_trans(wl, wl_a + wat);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            mma_bf16_16816(S[i][2 * np + e], kl, wh[2 * e], wh[2 * e + 1]);
-            mma_bf16_16816(S[i][2 * np + e], kh, wl[2 * e], wl[2 * e + 1]);
-            mma_bf16_16816(S[i][2 * np + e], kh, wh[2 * e], wh[2 * e + 1]);
-          }
+          ldmatrix_x4_trans(wh[np], wh_a + wat);
+          ldmatrix_x4_trans(wl[np], wl_a + wat);
         }
+        mma_row(S[i], kl, wh);
+        mma_row(S[i], kh, wl);
+        mma_row(S[i], kh, wh);
       }
     }
     __syncthreads();  // the partial outputs are in X
