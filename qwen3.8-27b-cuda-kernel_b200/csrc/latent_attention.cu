@@ -633,6 +633,7 @@ __global__ void __launch_bounds__(128) latent_join_kernel(q38_latent_attention_p
   bf16* out = static_cast<bf16*>(p.out) + ((size_t)start * p.heads + row) * k_dim;
   for (int c = 2 * threadIdx.x; c < k_dim; c += 256) {
     float2 v = make_float2(0, 0);
+#pragma unroll 8
     for (int s = 0; s < sh.active; ++s) {
       const float2 x = *reinterpret_cast<const float2*>(piece(p, k_dim, at, s, splits, block_rows, r) + c);
       v.x += factor[s] * x.x;

@@ -604,6 +604,7 @@ void LayerListModel::latent_attention(const StepContext& ctx, const StepBatch& b
     first = b.chunk_part.num_tokens;
     const int rows = int(b.chunk_packed_rows);
     kernels::latent_gather(b.chunk_part, kv, b.chunk_longest_context, rows, packed_latents_, ctx.stream);
+    ctx.mark("mix.latent_gather");
     gemm(ctx, packed_latents_, kv.k_dim, rows, W.ukv, Q38_DENSE_STORE, packed_kv_, ld_packed_);
     ctx.mark("gemm.latent_kv");
     kernels::PackedAttentionParams pp{};

@@ -94,5 +94,5 @@ CONFIGS = {
     "latent": config(96, 200, [latent(20, 16, 8, 24, 200, ff=64), latent(2, 40, 56, 72, 128), latent(7, 12, 20, 8, 24, scale=0.5)],
                      groups=3, streams=2, loop=(0, 3, 2), scale=0.7, mult=0.6),
     "wide": config(200, 96, [latent(2, 72, 100, 120, 300, ff=136), retention(4, 40, 72, (0.99, 0.93, 0.997, 0.9999), 24, ff=88),
-                             retention(1, 16, 8, (0.9,), 16)], groups=10, streams=5, loop=(2, 3, 3), scale=12.0, mult=0.3),
+                             retention(1, 16, 8, (0.9,), 16)], groups=10, streams=5, loop=(2, 3, 3), scale=8.0, mult=0.4),
 }
