@@ -240,7 +240,9 @@ packed_attention_kernel(q38_packed_attention_params p, q38_batch_desc b) {
     l_a += __shfl_xor_sync(0xffffffffu, l_a, x);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, x);
   }
-  const bool pairs = ((p.vdim | p.ld_out | p.ld_gate) & 1) == 0;
+  // whole pairs of numbers: every row and head starts at a multiple of four bytes
+  const bool pairs = ((p.vdim | p.ld_out | (p.gate ? p.ld_gate : 0)) & 1) == 0 &&
+                     ((reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & 3) == 0;
 #pragma unroll
   for (int hf = 0; hf < 2; ++hf) {
     const int r = ra + 8 * hf;

@@ -81,7 +81,7 @@ def make_model(folder, cfg, seed=1, **kw):
     return ll.write_model(folder, cfg, tensors), no.Model(cfg, tensors)
 
 
-# Sizes that share nothing with one another: one, two, three and five streams, norms over the whole row and over parts, heads
+# Sizes that share nothing with one another: one to five streams, norms over the whole row and over parts, heads
 # of odd sizes (values the vector kernels cannot take among them), no, partial and full rotation, decays up to 1, latents on
 # either side of the tensor-core kernels' instances, layers without a feed-forward, a loop at the start, in the middle, at the
 # end, and none.
@@ -93,6 +93,8 @@ CONFIGS = {
                                  retention(2, 64, 128, (0.9, 0.999), 32, ff=36)], groups=1, streams=1, eps=1e-6),
     "latent": config(96, 200, [latent(20, 16, 8, 24, 200, ff=64), latent(2, 40, 56, 72, 128), latent(7, 12, 20, 8, 24, scale=0.5)],
                      groups=3, streams=2, loop=(0, 3, 2), scale=0.7, mult=0.6),
+    "odd": config(63, 57, [latent(3, 21, 24, 33, 100, ff=35), retention(3, 14, 11, (0.95, 0.99, 0.9), 10, ff=41), latent(5, 40, 9, 17, 75)],
+                  groups=9, streams=4, loop=(0, 2, 2), scale=2.0, mult=0.4),
     "wide": config(200, 96, [latent(2, 72, 100, 120, 300, ff=136), retention(4, 40, 72, (0.99, 0.93, 0.997, 0.9999), 24, ff=88),
                              retention(1, 16, 8, (0.9,), 16)], groups=10, streams=5, loop=(2, 3, 3), scale=8.0, mult=0.4),
 }

@@ -382,12 +382,13 @@ def test_packed_attention_against_the_plain_one(heads, dim, vdim, rank):
         qd[:, h * ks:h * ks + dim] = dev(q[:, h], torch.bfloat16)
         kvd[:, h * ks:h * ks + dim] = dev(k[:, h], torch.bfloat16)
         kvd[:, H * ks + h * vs:H * ks + h * vs + vdim] = dev(v[:, h], torch.bfloat16)
-    for gated, ld_out in ((True, H * vdim + 2), (False, H * vdim + 3)):
+    # gates that start at an odd column of their matrix too
+    for gated, ld_out, shift in ((True, H * vdim + 2, 0), (True, H * vdim + 2, 1), (False, H * vdim + 3, 0)):
         gd = torch.zeros((b.m, H * vdim + 4), dtype=torch.bfloat16, device="cuda")
-        gd[:, :H * vdim] = dev(gate, torch.bfloat16)
+        gd[:, shift:shift + H * vdim] = dev(gate, torch.bfloat16)
         out = torch.zeros((b.m, ld_out), dtype=torch.bfloat16, device="cuda")
         p = pkg.PackedAttentionParams(pkg.ptr(qd), ld_q, ks, pkg.ptr(kvd), kvd.data_ptr() + 2 * H * ks, ld_kv, ks, vs, H, dim, vdim, 0.4,
-                                      pkg.ptr(gd) if gated else None, H * vdim + 4, pkg.ptr(out), ld_out)
+                                      gd.data_ptr() + 2 * shift if gated else None, H * vdim + 4, pkg.ptr(out), ld_out)
         pkg.check(K.q38_packed_attention(C.byref(p), C.byref(b.desc), None))
         torch.cuda.synchronize()
         got = out.double().cpu().numpy()
